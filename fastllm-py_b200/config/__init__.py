@@ -5,11 +5,13 @@ from .tigitar import TigitarConfig
 from .lasonex import LasonexConfig
 from .sakusun import SakusunConfig
 from .saberax import SaberaxConfig
+from .lufozen import LufozenConfig
 from .registry import (Architecture, architecture_names, architecture_of, load_config,
                        register_architecture)
 
 __all__ = [
     "ConfigError", "read_raw_config", "EngineConfig", "canonical_dtype", "LinearRopeScaling",
-    "LlamaConfig", "TigitarConfig", "LasonexConfig", "SakusunConfig", "SaberaxConfig", "Architecture", "architecture_names", "architecture_of", "load_config",
+    "LlamaConfig", "TigitarConfig", "LasonexConfig", "SakusunConfig", "SaberaxConfig", "LufozenConfig",
+    "Architecture", "architecture_names", "architecture_of", "load_config",
     "register_architecture",
 ]

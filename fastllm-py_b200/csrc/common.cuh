@@ -80,7 +80,7 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 //   4 relu(g)^2 * u
 // A unit without a gate is f(x, 1).
 enum FlAct : int { FL_ACT_SILU = 0, FL_ACT_RELU = 1, FL_ACT_GELU_TANH = 2, FL_ACT_CLAMPED_SWISH = 3, FL_ACT_RELU_SQUARED = 4,
-                   FL_ACT_COUNT = 5 };
+                   FL_ACT_COUNT = 5, FL_ACT_NONE = -1 };
 struct FlGate {
     int act;
     float p0, p1;

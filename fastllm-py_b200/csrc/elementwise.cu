@@ -75,13 +75,33 @@ FL_API int fl_embed(const void* table, int table_dtype, long table_ld, const int
 
 // -------------------------------------------------------------------- RMSNorm
 // out = x * (mean(x^2) + eps)^-1/2 * w.  With `delta`, first x += delta (x is
-// the float residual stream and is written back unless rows are gathered).
+// the float residual stream and is written back unless rows are gathered), and
+// with `add` the row vectors add.a and add.b (float [dim], null: none) as well.
 // `rows`, when given, selects the input row of each output row.
+struct RowAdd {                  // vectors added to every row: an output bias, a vector a pass of layers starts with
+    const float *a, *b;
+};
+__device__ __forceinline__ void add_rows4(float4& v, const RowAdd add, int i) {
+    if (add.a != nullptr) {
+        const float4 o = *reinterpret_cast<const float4*>(add.a + i);
+        v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
+    }
+    if (add.b != nullptr) {
+        const float4 o = *reinterpret_cast<const float4*>(add.b + i);
+        v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
+    }
+}
+__device__ __forceinline__ void add_rows1(float& v, const RowAdd add, int i) {
+    if (add.a != nullptr) v += add.a[i];
+    if (add.b != nullptr) v += add.b[i];
+}
+static inline bool row_add_vec_ok(const RowAdd add) { return ((uintptr_t)add.a % 16) == 0 && ((uintptr_t)add.b % 16) == 0; }
+
 template <typename TX, typename TD, typename TW, typename TO, bool ADD, bool VEC>
 __global__ void rmsnorm_kernel(TX* __restrict__ x, long x_ld, const TD* __restrict__ delta,
                                long delta_ld, const TW* __restrict__ w, TO* __restrict__ out,
                                long out_ld, int dim, float eps, const int* __restrict__ rows,
-                               int write_back) {
+                               int write_back, const RowAdd add) {
     pdl_wait();
     pdl_trigger();
     __shared__ float scratch[32];
@@ -100,6 +120,7 @@ __global__ void rmsnorm_kernel(TX* __restrict__ x, long x_ld, const TD* __restri
                 float4 d;
                 load4(dr + i, d);
                 v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+                add_rows4(v, add, i);
                 if (write_back) store4(xr + i, v);
             }
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -107,6 +128,7 @@ __global__ void rmsnorm_kernel(TX* __restrict__ x, long x_ld, const TD* __restri
             float v = to_f32<TX>(xr[i]);
             if (ADD) {
                 v += to_f32<TD>(dr[i]);
+                add_rows1(v, add, i);
                 if (write_back) xr[i] = from_f32<TX>(v);
             }
             ss += v * v;
@@ -125,12 +147,16 @@ __global__ void rmsnorm_kernel(TX* __restrict__ x, long x_ld, const TD* __restri
                 float4 d;
                 load4(dr + i, d);
                 v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+                add_rows4(v, add, i);
             }
             load4(w + i, g);
             store4(o + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
         } else {
             float v = to_f32<TX>(xr[i]);
-            if (readd) v += to_f32<TD>(dr[i]);
+            if (readd) {
+                v += to_f32<TD>(dr[i]);
+                add_rows1(v, add, i);
+            }
             o[i] = from_f32<TO>(v * inv * to_f32<TW>(w[i]));
         }
     }
@@ -153,7 +179,7 @@ FL_API int fl_rmsnorm(const void* x, int x_dtype, long x_ld, const void* w, int 
     FL_DISPATCH(x_dtype, TX, FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,                      \
         return fl_launch(rmsnorm_kernel<TX, float, TW, TO, false, VEC>, dim3(n_rows), dim3(threads), 0,  \
                          stream, (TX*)x, x_ld, (const float*)nullptr, 0L, (const TW*)w, (TO*)out,       \
-                         out_ld, dim, eps, rows, 0))))
+                         out_ld, dim, eps, rows, 0, RowAdd{nullptr, nullptr}))))
     if (vec) { FL_NORM_LAUNCH(true); } else { FL_NORM_LAUNCH(false); }
 #undef FL_NORM_LAUNCH
     return 0;
@@ -167,7 +193,7 @@ template <typename TD, typename TW, typename TO, int KEEP>
 __global__ void __launch_bounds__(256) add_rmsnorm_rows_kernel(float* __restrict__ resid, long resid_ld,
                                                                const TD* __restrict__ delta, long delta_ld,
                                                                const TW* __restrict__ w, TO* __restrict__ out,
-                                                               long out_ld, int dim, float eps) {
+                                                               long out_ld, int dim, float eps, const RowAdd add) {
     pdl_wait();
     pdl_trigger();
     __shared__ float scratch[32];
@@ -185,6 +211,7 @@ __global__ void __launch_bounds__(256) add_rmsnorm_rows_kernel(float* __restrict
             load4(dr + i, d);
             load4(w + i, gain[c]);
             v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+            add_rows4(v, add, i);
             *reinterpret_cast<float4*>(xr + i) = v;
             keep[c] = v;
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -203,11 +230,12 @@ __global__ void __launch_bounds__(256) add_rmsnorm_rows_kernel(float* __restrict
 
 FL_API int fl_add_rmsnorm(float* resid, long resid_ld, const void* delta, int delta_dtype,
                           long delta_ld, const void* w, int w_dtype, void* out, int out_dtype,
-                          long out_ld, int n_rows, int dim, float eps, const int* rows,
-                          cudaStream_t stream) {
+                          long out_ld, int n_rows, int dim, float eps, const int* rows, const float* add_a,
+                          const float* add_b, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
+    const RowAdd add{add_a, add_b};
     const int write_back = rows ? 0 : 1;
-    if (write_back && dim <= 8 * 1024 && vec4_ok(dim, resid, resid_ld, 4) &&
+    if (write_back && dim <= 8 * 1024 && row_add_vec_ok(add) && vec4_ok(dim, resid, resid_ld, 4) &&
         vec4_ok(dim, delta, delta_ld, delta_dtype == FL_F32 ? 4 : 2) && vec4_ok(dim, w, 4, w_dtype == FL_F32 ? 4 : 2) &&
         vec4_ok(dim, out, out_ld, out_dtype == FL_F32 ? 4 : 2)) {
         const int chunks = (dim / 4 + 255) / 256;                      // per thread
@@ -215,21 +243,21 @@ FL_API int fl_add_rmsnorm(float* resid, long resid_ld, const void* delta, int de
     FL_DISPATCH(delta_dtype, TD, FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,                      \
         return fl_launch(add_rmsnorm_rows_kernel<TD, TW, TO, KEEP>, dim3(n_rows), dim3(256), 0, stream,   \
                          resid, resid_ld, (const TD*)delta, delta_ld, (const TW*)w, (TO*)out, out_ld, dim, \
-                         eps))))
+                         eps, add))))
         if (chunks <= 1) { FL_ROWS_LAUNCH(1); }
         else if (chunks <= 2) { FL_ROWS_LAUNCH(2); }
         else if (chunks <= 4) { FL_ROWS_LAUNCH(4); }
         else { FL_ROWS_LAUNCH(8); }
 #undef FL_ROWS_LAUNCH
     }
-    const bool vec = vec4_ok(dim, resid, resid_ld, 4) && vec4_ok(dim, delta, delta_ld, delta_dtype == FL_F32 ? 4 : 2) &&
+    const bool vec = row_add_vec_ok(add) && vec4_ok(dim, resid, resid_ld, 4) && vec4_ok(dim, delta, delta_ld, delta_dtype == FL_F32 ? 4 : 2) &&
                      vec4_ok(dim, w, 4, w_dtype == FL_F32 ? 4 : 2) && vec4_ok(dim, out, out_ld, out_dtype == FL_F32 ? 4 : 2);
     const int threads = norm_threads(dim, vec);
 #define FL_NORM_LAUNCH(VEC)                                                                          \
     FL_DISPATCH(delta_dtype, TD, FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,                  \
         return fl_launch(rmsnorm_kernel<float, TD, TW, TO, true, VEC>, dim3(n_rows), dim3(threads), 0,  \
                          stream, resid, resid_ld, (const TD*)delta, delta_ld, (const TW*)w, (TO*)out,  \
-                         out_ld, dim, eps, rows, write_back))))
+                         out_ld, dim, eps, rows, write_back, add))))
     if (vec) { FL_NORM_LAUNCH(true); } else { FL_NORM_LAUNCH(false); }
 #undef FL_NORM_LAUNCH
     return 0;
@@ -251,6 +279,33 @@ FL_API int fl_residual_add(float* resid, long resid_ld, const void* delta, int d
     if (n_rows <= 0) return 0;
     FL_DISPATCH(delta_dtype, TD, return fl_launch(add_kernel<TD>, dim3(n_rows), dim3(256), 0, stream, resid,
                                                   resid_ld, (const TD*)delta, delta_ld, dim));
+    return 0;
+}
+
+// resid[r] += add.a + add.b in every row, for whoever reads the stream before a norm that adds them could.
+template <typename T>
+__global__ void row_add_kernel(T* __restrict__ resid, long resid_ld, const RowAdd add, int dim) {
+    pdl_wait();
+    pdl_trigger();
+    T* xr = resid + (long)blockIdx.x * resid_ld;
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+        float v = to_f32<T>(xr[i]);
+        add_rows1(v, add, i);
+        xr[i] = from_f32<T>(v);
+    }
+}
+
+FL_API int fl_row_add(float* resid, long resid_ld, const float* add_a, const float* add_b, int n_rows, int dim,
+                      cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    return fl_launch(row_add_kernel<float>, dim3(n_rows), dim3(256), 0, stream, resid, resid_ld, RowAdd{add_a, add_b}, dim);
+}
+
+// x[r] += bias for a product's result that no kernel with the bias in it reads next.
+FL_API int fl_add_bias(void* x, int dtype, long x_ld, const float* bias, int n_rows, int dim, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    FL_DISPATCH(dtype, T, return fl_launch(row_add_kernel<T>, dim3(n_rows), dim3(256), 0, stream, (T*)x, x_ld,
+                                           RowAdd{bias, nullptr}, dim));
     return 0;
 }
 
@@ -328,7 +383,7 @@ template <typename TW, typename TO>
 __global__ void add_rmsnorm_partial_kernel(float* __restrict__ resid, long resid_ld,
                                            const float* __restrict__ partial, int splits,
                                            long split_stride, long ld, const TW* __restrict__ w,
-                                           TO* __restrict__ out, long out_ld, int dim, float eps) {
+                                           TO* __restrict__ out, long out_ld, int dim, float eps, const RowAdd add) {
     pdl_wait();
     pdl_trigger();
     __shared__ float scratch[32];
@@ -339,7 +394,8 @@ __global__ void add_rmsnorm_partial_kernel(float* __restrict__ resid, long resid
     float ss = 0.0f;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
         // the sum is rounded to the activation type first, as the separate reduction stores it
-        const float v = xr[i] + to_f32<TO>(from_f32<TO>(sum_splits(pr, i, splits, split_stride)));
+        float v = xr[i] + to_f32<TO>(from_f32<TO>(sum_splits(pr, i, splits, split_stride)));
+        add_rows1(v, add, i);
         xr[i] = v;
         ss += v * v;
     }
@@ -359,7 +415,7 @@ __global__ void add_rmsnorm_partial_kernel(float* __restrict__ resid, long resid
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(1024) add_rmsnorm_partial_vec_kernel(
     float* __restrict__ resid, long resid_ld, const float* __restrict__ partial, int splits, long split_stride,
-    long ld, const TW* __restrict__ w, TO* __restrict__ out, long out_ld, int dim, float eps) {
+    long ld, const TW* __restrict__ w, TO* __restrict__ out, long out_ld, int dim, float eps, const RowAdd add) {
     pdl_wait();
     pdl_trigger();
     __shared__ float scratch[32];
@@ -386,6 +442,7 @@ __global__ void __launch_bounds__(1024) add_rmsnorm_partial_vec_kernel(
             v.y += to_f32<TO>(from_f32<TO>(acc.y));
             v.z += to_f32<TO>(from_f32<TO>(acc.z));
             v.w += to_f32<TO>(from_f32<TO>(acc.w));
+            add_rows4(v, add, i);
             *reinterpret_cast<float4*>(xr + i) = v;
             keep[c] = v;
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -404,10 +461,11 @@ __global__ void __launch_bounds__(1024) add_rmsnorm_partial_vec_kernel(
 
 FL_API int fl_add_rmsnorm_partial(float* resid, long resid_ld, const float* partial, int splits,
                                   long split_stride, long ld, const void* w, int w_dtype, void* out,
-                                  int out_dtype, long out_ld, int n_rows, int dim, float eps,
-                                  cudaStream_t stream) {
+                                  int out_dtype, long out_ld, int n_rows, int dim, float eps, const float* add_a,
+                                  const float* add_b, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    const bool vec = vec4_ok(dim, resid, resid_ld, 4) && vec4_ok(dim, partial, ld, 4) && split_stride % 4 == 0 &&
+    const RowAdd add{add_a, add_b};
+    const bool vec = row_add_vec_ok(add) && vec4_ok(dim, resid, resid_ld, 4) && vec4_ok(dim, partial, ld, 4) && split_stride % 4 == 0 &&
                      vec4_ok(dim, w, 4, w_dtype == FL_F32 ? 4 : 2) &&
                      vec4_ok(dim, out, out_ld, out_dtype == FL_F32 ? 4 : 2) && dim <= ARP_KEEP * 4 * 1024;
     if (vec) {
@@ -415,13 +473,13 @@ FL_API int fl_add_rmsnorm_partial(float* resid, long resid_ld, const float* part
         FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,
             return fl_launch(add_rmsnorm_partial_vec_kernel<TW, TO>, dim3(n_rows), dim3(vthreads), 0, stream,
                              resid, resid_ld, partial, splits, split_stride, ld, (const TW*)w, (TO*)out, out_ld,
-                             dim, eps)));
+                             dim, eps, add)));
     }
     const int threads = norm_threads(dim, false);
     FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,
         return fl_launch(add_rmsnorm_partial_kernel<TW, TO>, dim3(n_rows), dim3(threads), 0, stream, resid,
                          resid_ld, partial, splits, split_stride, ld, (const TW*)w, (TO*)out, out_ld, dim,
-                         eps)));
+                         eps, add)));
     return 0;
 }
 

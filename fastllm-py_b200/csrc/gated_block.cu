@@ -15,7 +15,8 @@
 //                    never read and written by one launch
 //   sigmoid_gate     a[t, i] *= sigmoid(g[t, i])  (an output gate inside a mixer)
 //   pair_embed       x[t] = table[id_t] * scale + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets], row
-//                    `buckets` for a request's first token; the token before a step's first is per-request state,
+//                    `buckets` for a request's first token (and, where a norm's weight is given, the row normed); the
+//                    token before a step's first is per-request state,
 //                    read and rewritten by the block of the request's first row only
 //
 // All arithmetic is float; the residual stream is float in both precisions.
@@ -278,10 +279,11 @@ __global__ void __launch_bounds__(256) pair_embed_kernel(
     float* __restrict__ out, long out_ld, int hidden, int vocab, int buckets, long mul_prev, long mul_cur, float scale,
     const int* __restrict__ tok_req, const int* __restrict__ req_start, const int* __restrict__ req_ctx,
     const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int* __restrict__ last_token,
-    int* __restrict__ status, const int* __restrict__ fed, int n_fed) {
+    int* __restrict__ status, const int* __restrict__ fed, int n_fed, const float* __restrict__ norm_w, float eps) {
     pdl_wait();
     pdl_trigger();
     __shared__ int before;
+    __shared__ float scratch[32];
     const int t = blockIdx.x;
     const int r = tok_req[t], start = req_start[r];
     const int id = fed_token(ids[t], fed, n_fed);
@@ -305,21 +307,28 @@ __global__ void __launch_bounds__(256) pair_embed_kernel(
     const long pair_row = prev < 0 ? (long)buckets : ((long)prev * mul_prev + (long)id * mul_cur) % (long)buckets;
     const TT* row = table + (long)id * table_ld;
     const TT* prow = pairs + pair_row * pairs_ld;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-        o[i] = to_f32<TT>(row[i]) * scale + to_f32<TT>(prow[i]);
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = to_f32<TT>(row[i]) * scale + to_f32<TT>(prow[i]);
+        o[i] = v;
+        ss += v * v;
+    }
+    if (norm_w == nullptr) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = o[i] * inv * norm_w[i];    // each thread its own elements
 }
 
-// pairs: [buckets + 1, hidden]; last_token: [slots] int.
+// pairs: [buckets + 1, hidden]; last_token: [slots] int; norm_w: [hidden] float, or null: the row is not normed.
 FL_API int fl_pair_embed(const void* table, long table_ld, const void* pairs, long pairs_ld, int dtype, const int* ids,
                          float* out, long out_ld, int n_tokens, int hidden, int vocab, int buckets, long mul_prev,
                          long mul_cur, float scale, const int* tok_req, const int* req_start, const int* req_ctx,
                          const int* req_qlen, const int* req_slot, int* last_token, int* status, const int* fed, int n_fed,
-                         cudaStream_t stream) {
+                         const float* norm_w, float eps, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (buckets < 1) return (int)cudaErrorInvalidValue;
     FL_DISPATCH(dtype, TT, return fl_launch(pair_embed_kernel<TT>, dim3(n_tokens), dim3(256), 0, stream, (const TT*)table,
                                             table_ld, (const TT*)pairs, pairs_ld, ids, out, out_ld, hidden, vocab, buckets,
                                             mul_prev, mul_cur, scale, tok_req, req_start, req_ctx, req_qlen, req_slot,
-                                            last_token, status, fed, n_fed));
+                                            last_token, status, fed, n_fed, norm_w, eps));
     return 0;
 }

@@ -140,6 +140,7 @@ __device__ __forceinline__ void tmem_ld_wait() {
 // clamped swish unit with its two constants.
 __device__ __forceinline__ float gated_act(float g, float u, const FlGate act) {
     if (act.act == FL_ACT_RELU) return fmaxf(g, 0.0f) * u;
+    if (act.act == FL_ACT_RELU_SQUARED) return fmaxf(g, 0.0f) * fmaxf(g, 0.0f) * u;
     if (act.act == FL_ACT_GELU_TANH) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
     if (act.act == FL_ACT_CLAMPED_SWISH) {
         g = fminf(g, act.p0);
@@ -147,6 +148,13 @@ __device__ __forceinline__ float gated_act(float g, float u, const FlGate act) {
         return __fdividef(g, 1.0f + __expf(-act.p1 * g)) * (u + 1.0f);
     }
     return __fdividef(g, 1.0f + __expf(-g)) * u;
+}
+
+// A product that is not gated may pass an activation of one argument on its way out: f(v, 1), or FL_ACT_NONE.
+template <int N> __device__ __forceinline__ void unary_act(uint32_t (&r)[N], const FlGate act) {
+    if (act.act == FL_ACT_NONE) return;
+#pragma unroll
+    for (int j = 0; j < N; ++j) r[j] = __float_as_uint(gated_act(__uint_as_float(r[j]), 1.0f, act));
 }
 
 // A barrier among the four epilogue warps only (hardware barrier 1; barrier 0 is __syncthreads).
@@ -440,6 +448,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(
                                                        cols, e, vec_ok);
                     } else {
                         OutT* st = reinterpret_cast<OutT*>(half);
+                        unary_act(r, act);
 #pragma unroll
                         for (int j = 0; j < 16; ++j) st[j * TC_BM + e] = from_f32<OutT>(__uint_as_float(r[j]));
                         epilogue_sync();
@@ -896,6 +905,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_pair_kernel(
                                                      min(cols, 128), e, vec_ok);
                     } else {
                         OutT* st = reinterpret_cast<OutT*>(half);
+                        unary_act(r, act);
 #pragma unroll
                         for (int j = 0; j < 32; ++j) st[j * 128 + e] = from_f32<OutT>(__uint_as_float(r[j]));
                         epilogue_sync();
@@ -936,7 +946,7 @@ template <int BNT, typename OutT, bool GATED = false, bool ROPE = false>
 static int launch_tc_pair(const CUtensorMap& map_w, const CUtensorMap& map_a, void* C, long ldc, int M, int N,
                           int K, int num_sms, int* status, cudaStream_t stream, int gate_rows = 0, int splits = 1,
                           int kb_per_split = 0, float* partial = nullptr, long ld_partial = 0,
-                          const TcRope* rope_args = nullptr, int wp = 0, FlGate act = FlGate{0, 0.0f, 0.0f}) {
+                          const TcRope* rope_args = nullptr, int wp = 0, FlGate act = FlGate{FL_ACT_NONE, 0.0f, 0.0f}) {
     static bool configured = false;
     auto kernel = gemm_tc_pair_kernel<BNT, OutT, GATED, ROPE>;
     TcRope rope = {};
@@ -974,11 +984,11 @@ static int launch_tc_pair(const CUtensorMap& map_w, const CUtensorMap& map_a, vo
 template <typename OutT>
 static int dispatch_tc_pair(int bnt, const CUtensorMap& map_w, const CUtensorMap& map_a, void* C, long ldc, int M,
                             int N, int K, int num_sms, int* status, cudaStream_t stream, int splits,
-                            int kb_per_split, float* partial, long ld_partial, int wp) {
+                            int kb_per_split, float* partial, long ld_partial, int wp, FlGate act) {
     switch (bnt) {
-        case 64: return launch_tc_pair<64, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp);
-        case 128: return launch_tc_pair<128, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp);
-        case 256: return launch_tc_pair<256, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp);
+        case 64: return launch_tc_pair<64, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp, act);
+        case 128: return launch_tc_pair<128, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp, act);
+        case 256: return launch_tc_pair<256, OutT>(map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, 0, splits, kb_per_split, partial, ld_partial, nullptr, wp, act);
     }
     return (int)cudaErrorInvalidValue;
 }
@@ -986,7 +996,7 @@ static int dispatch_tc_pair(int bnt, const CUtensorMap& map_w, const CUtensorMap
 // C[t, o] = sum over splits of partial[z][t][o], added in the order z = 0, 1, ...
 template <typename OutT>
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, long ld_partial, int splits,
-                                     OutT* __restrict__ C, long ldc, int M, int N) {
+                                     OutT* __restrict__ C, long ldc, int M, int N, FlGate act) {
     pdl_wait();
     pdl_trigger();
     const int o = blockIdx.x * blockDim.x + threadIdx.x;
@@ -994,23 +1004,24 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, long ld_
     if (o >= N) return;
     float acc = 0.0f;
     for (int z = 0; z < splits; ++z) acc += partial[((long)z * M + t) * ld_partial + o];
-    C[(long)t * ldc + o] = from_f32<OutT>(acc);
+    C[(long)t * ldc + o] = from_f32<OutT>(act.act == FL_ACT_NONE ? acc : gated_act(acc, 1.0f, act));
+}
+
+static int splitk_reduce(const float* partial, long ld_partial, int splits, void* C, int c_dtype, long ldc, int M, int N,
+                         cudaStream_t stream, FlGate act) {
+    if (M <= 0 || N <= 0) return 0;
+    if (splits < 1 || M > 65535) return (int)cudaErrorInvalidValue;
+    dim3 grid((N + 255) / 256, M);
+    FL_DISPATCH(c_dtype, T, return fl_launch(splitk_reduce_kernel<T>, grid, dim3(256), 0, stream, partial, ld_partial, splits,
+                                             (T*)C, ldc, M, N, act));
+    return (int)cudaErrorInvalidValue;
 }
 
 // C = the sum of `splits` slabs partial[z][M][ld_partial] (what fl_gemm_tc_partial leaves), for a
 // consumer that has no kernel of its own that adds the slabs while it reads them.
 FL_API int fl_splitk_reduce(const float* partial, long ld_partial, int splits, void* C, int c_dtype, long ldc,
                             int M, int N, cudaStream_t stream) {
-    if (M <= 0 || N <= 0) return 0;
-    if (splits < 1 || M > 65535) return (int)cudaErrorInvalidValue;
-    dim3 grid((N + 255) / 256, M);
-    if (c_dtype == FL_BF16)
-        return fl_launch(splitk_reduce_kernel<bf16>, grid, dim3(256), 0, stream, partial, ld_partial, splits,
-                         (bf16*)C, ldc, M, N);
-    if (c_dtype == FL_F32)
-        return fl_launch(splitk_reduce_kernel<float>, grid, dim3(256), 0, stream, partial, ld_partial, splits,
-                         (float*)C, ldc, M, N);
-    return (int)cudaErrorInvalidValue;
+    return splitk_reduce(partial, ld_partial, splits, C, c_dtype, ldc, M, N, stream, FlGate{FL_ACT_NONE, 0.0f, 0.0f});
 }
 
 // dst[kb][n][c] = src[n][kb * 64 + c] (zero where kb * 64 + c >= K): a weight matrix packed by k-block, so that
@@ -1090,7 +1101,7 @@ template <int BN, int STAGES, typename OutT, bool GATED = false>
 static int launch_tc(const CUtensorMap& map_w, const CUtensorMap& map_a, void* C, long ldc,
                      float* partial, long ld_partial, int M, int N, int K, int splits,
                      int kb_per_split, int* status, cudaStream_t stream, int gate_rows = 0, int feat = 64, int wp = 0,
-                     FlGate act = FlGate{0, 0.0f, 0.0f}) {
+                     FlGate act = FlGate{FL_ACT_NONE, 0.0f, 0.0f}) {
     using L = TcSmem<BN, STAGES>;
     // This kernel is launched with programmatic overlap, so CTAs of it and of its neighbours in the stream share
     // SMs; as many of them as fit an SM by shared memory must find their tensor-memory columns free at once, or an
@@ -1118,13 +1129,13 @@ static int launch_tc(const CUtensorMap& map_w, const CUtensorMap& map_a, void* C
 template <typename OutT>
 static int dispatch_tc(int bn, const CUtensorMap& map_w, const CUtensorMap& map_a, void* C, long ldc,
                        float* partial, long ld_partial, int M, int N, int K, int splits,
-                       int kb_per_split, int* status, cudaStream_t stream, int wp) {
+                       int kb_per_split, int* status, cudaStream_t stream, int wp, FlGate act) {
     switch (bn) {
-        case 16: return launch_tc<16, 6, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp);
-        case 32: return launch_tc<32, 5, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp);
-        case 64: return launch_tc<64, 4, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp);
-        case 128: return launch_tc<128, 3, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp);
-        case 256: return launch_tc<256, 4, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp);
+        case 16: return launch_tc<16, 6, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp, act);
+        case 32: return launch_tc<32, 5, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp, act);
+        case 64: return launch_tc<64, 4, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp, act);
+        case 128: return launch_tc<128, 3, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp, act);
+        case 256: return launch_tc<256, 4, OutT>(map_w, map_a, C, ldc, partial, ld_partial, M, N, K, splits, kb_per_split, status, stream, 0, 64, wp, act);
     }
     return (int)cudaErrorInvalidValue;
 }
@@ -1245,7 +1256,8 @@ FL_API void fl_gemm_tc_plan(int M, int N, int K, int num_sms, int* bn_out, int* 
 // from fl_gemm_tc_plan, or 0 to plan here).
 static int gemm_tc_impl(const void* A, long lda, const void* W, long ldw, void* C, int c_dtype, long ldc,
                         int M, int N, int K, int bn, int splits, float* workspace, long workspace_floats,
-                        int num_sms, int* status, cudaStream_t stream, int skip_reduce) {
+                        int num_sms, int* status, cudaStream_t stream, int skip_reduce,
+                        FlGate act = FlGate{FL_ACT_NONE, 0.0f, 0.0f}) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0) return (int)cudaErrorInvalidValue;
     if (bn == 0) fl_gemm_tc_plan_for(M, N, K, num_sms, skip_reduce, &bn, &splits);
@@ -1269,20 +1281,20 @@ static int gemm_tc_impl(const void* A, long lda, const void* W, long ldw, void* 
     if (paired) {                                            // each CTA of a pair loads half of the token rows
         float* part = splits > 1 ? workspace : nullptr;
         if (c_dtype == FL_BF16)
-            rc = dispatch_tc_pair<bf16>(bnt, map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, splits, kb_per_split, part, ld_partial, wp);
+            rc = dispatch_tc_pair<bf16>(bnt, map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, splits, kb_per_split, part, ld_partial, wp, act);
         else if (c_dtype == FL_F32)
-            rc = dispatch_tc_pair<float>(bnt, map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, splits, kb_per_split, part, ld_partial, wp);
+            rc = dispatch_tc_pair<float>(bnt, map_w, map_a, C, ldc, M, N, K, num_sms, status, stream, splits, kb_per_split, part, ld_partial, wp, act);
         else
             return (int)cudaErrorInvalidValue;
     } else if (c_dtype == FL_BF16) {
-        rc = dispatch_tc<bf16>(bn, map_w, map_a, C, ldc, workspace, ld_partial, M, N, K, splits, kb_per_split, status, stream, wp);
+        rc = dispatch_tc<bf16>(bn, map_w, map_a, C, ldc, workspace, ld_partial, M, N, K, splits, kb_per_split, status, stream, wp, act);
     } else if (c_dtype == FL_F32) {
-        rc = dispatch_tc<float>(bn, map_w, map_a, C, ldc, workspace, ld_partial, M, N, K, splits, kb_per_split, status, stream, wp);
+        rc = dispatch_tc<float>(bn, map_w, map_a, C, ldc, workspace, ld_partial, M, N, K, splits, kb_per_split, status, stream, wp, act);
     } else {
         return (int)cudaErrorInvalidValue;
     }
     if (rc || splits == 1 || skip_reduce) return rc;
-    return fl_splitk_reduce(workspace, ld_partial, splits, C, c_dtype, ldc, M, N, stream);
+    return splitk_reduce(workspace, ld_partial, splits, C, c_dtype, ldc, M, N, stream, act);
 }
 
 FL_API int fl_gemm_tc(const void* A, long lda, const void* W, long ldw, void* C, int c_dtype, long ldc,
@@ -1290,6 +1302,16 @@ FL_API int fl_gemm_tc(const void* A, long lda, const void* W, long ldw, void* C,
                       int num_sms, int* status, cudaStream_t stream) {
     return gemm_tc_impl(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, bn, splits, workspace, workspace_floats,
                         num_sms, status, stream, 0);
+}
+
+// C = f(A W^T, 1): the product with an activation of one argument (FlAct in common.cuh) applied on its way out, or by the
+// kernel that adds the partial sums up.
+FL_API int fl_gemm_tc_act(const void* A, long lda, const void* W, long ldw, void* C, int c_dtype, long ldc, int M, int N, int K,
+                          int bn, int splits, float* workspace, long workspace_floats, int num_sms, int* status, int act_code,
+                          float act_p0, float act_p1, cudaStream_t stream) {
+    if (act_code < 0 || act_code >= FL_ACT_COUNT) return (int)cudaErrorInvalidValue;
+    return gemm_tc_impl(A, lda, W, ldw, C, c_dtype, ldc, M, N, K, bn, splits, workspace, workspace_floats, num_sms, status,
+                        stream, 0, FlGate{act_code, act_p0, act_p1});
 }
 
 // The same, but with splits > 1 the partial sums stay in the workspace

@@ -18,7 +18,10 @@
 //                         multiples of 128 of the absolute position and tiles without a visible key are skipped, so
 //                         every sum's order depends on the token's own position only
 //
-// Scores, softmax, norms and the blend are float.
+// The attention kernels may multiply their result, channel by channel, by the sigmoid of a gate row of the same token
+// ([heads x vdim], in the activation type) before it is rounded.
+//
+// Scores, softmax, norms, gates and the blend are float.
 #include "common.cuh"
 
 #define SINK_TILE 128
@@ -212,6 +215,11 @@ FL_API int fl_head_gate(void* x, int dtype, long x_ld, const void* gate, long g_
     return 0;
 }
 
+// v times the sigmoid of gate[at] (no gate: v).
+template <typename T> __device__ __forceinline__ float sink_gated(float v, const T* gate, long at) {
+    return gate != nullptr ? v / (1.0f + expf(-to_f32<T>(gate[at]))) : v;
+}
+
 // The score of key j for a query at `pos` from the dot product.
 __device__ __forceinline__ float sink_score(float dot, float scale, float cap, const int* bucket_of, int n_dist,
                                             const float* rel, int heads, int h, int dist) {
@@ -227,7 +235,7 @@ __global__ void __launch_bounds__(SINK_TILE) sink_attention_simt_kernel(
     int page_size, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ tok_req,
     const int* __restrict__ positions, int heads, int kv_heads, int dim, int vdim, int window, int keep_first, int chunk,
     float scale, float cap, const int* __restrict__ bucket_of, int n_dist, const float* __restrict__ rel,
-    const float* __restrict__ sink) {
+    const float* __restrict__ sink, const T* __restrict__ gate, long gate_ld) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char sink_smem[];
@@ -292,8 +300,10 @@ __global__ void __launch_bounds__(SINK_TILE) sink_attention_simt_kernel(
     }
     T* dst = out + (long)t * out_ld + (long)h * vdim;
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
-        if (tid + c * SINK_TILE < vdim) dst[tid + c * SINK_TILE] = from_f32<T>(acc[c] / l);
+    for (int c = 0; c < 2; ++c) {
+        const int d = tid + c * SINK_TILE;
+        if (d < vdim) dst[d] = from_f32<T>(sink_gated<T>(acc[c] / l, gate, (long)t * gate_ld + (long)h * vdim + d));
+    }
 }
 
 // q: [n_tokens, q_ld], head h at columns [h * dim, (h + 1) * dim); out: [n_tokens, out_ld], head h at columns
@@ -303,8 +313,8 @@ FL_API int fl_sink_attention_simt(const void* q, int q_dtype, long q_ld, void* o
                                   long page_stride, int page_size, const int* block_table, int bt_stride,
                                   const int* tok_req, const int* positions, int n_tokens, int heads, int kv_heads, int dim,
                                   int vdim, int window, int keep_first, int chunk, float scale, float cap,
-                                  const int* bucket_of, int n_dist, const float* rel, const float* sink,
-                                  cudaStream_t stream) {
+                                  const int* bucket_of, int n_dist, const float* rel, const float* sink, const void* gate,
+                                  long gate_ld, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (vdim < 1 || vdim > 2 * SINK_TILE || dim < 1 || dim > 4096 || heads > 65535 || heads % kv_heads ||
         (rel != nullptr && (bucket_of == nullptr || n_dist < 1)))
@@ -314,7 +324,8 @@ FL_API int fl_sink_attention_simt(const void* q, int q_dtype, long q_ld, void* o
     FL_DISPATCH(dtype, T, FL_DISPATCH(q_dtype, TQ,
         return fl_launch(sink_attention_simt_kernel<T, TQ>, grid, dim3(SINK_TILE), smem, stream, (const TQ*)q, q_ld, (T*)out,
                          out_ld, (const T*)cache, page_stride, page_size, block_table, bt_stride, tok_req, positions, heads,
-                         kv_heads, dim, vdim, window, keep_first, chunk, scale, cap, bucket_of, n_dist, rel, sink)));
+                         kv_heads, dim, vdim, window, keep_first, chunk, scale, cap, bucket_of, n_dist, rel, sink,
+                         (const T*)gate, gate_ld)));
     return 0;
 }
 
@@ -489,7 +500,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) sink_decode_merge_kernel(const float* __restrict__ partial, int n_splits,
                                                                 const int* __restrict__ decode_tokens, T* __restrict__ out,
                                                                 long out_ld, int heads, int vdim,
-                                                                const float* __restrict__ sink) {
+                                                                const float* __restrict__ sink, const T* __restrict__ gate,
+                                                                long gate_ld) {
     pdl_wait();
     pdl_trigger();
     const int h = blockIdx.y, tid = threadIdx.x;
@@ -508,7 +520,7 @@ __global__ void __launch_bounds__(128) sink_decode_merge_kernel(const float* __r
             const float ms = base[(long)s * (vdim + 2)];
             if (ms != -CUDART_INF_F) a += base[(long)s * (vdim + 2) + 2 + d] * expf(ms - top);
         }
-        dst[d] = from_f32<T>(a / sum);
+        dst[d] = from_f32<T>(sink_gated<T>(a / sum, gate, (long)decode_tokens[blockIdx.x] * gate_ld + (long)h * vdim + d));
     }
 }
 
@@ -527,7 +539,8 @@ FL_API int fl_sink_decode(const void* q, int dtype, long q_ld, void* out, long o
                           int page_size, const int* block_table, int bt_stride, const int* tok_req, const int* positions,
                           const int* decode_tokens, int n_decode, float* partial, int n_splits, int kept_splits, int heads,
                           int kv_heads, int dim, int vdim, int window, int keep_first, int chunk, float scale, float cap,
-                          const int* bucket_of, int n_dist, const float* rel, const float* sink, cudaStream_t stream) {
+                          const int* bucket_of, int n_dist, const float* rel, const float* sink, const void* gate, long gate_ld,
+                          cudaStream_t stream) {
     if (n_decode <= 0) return 0;
     if (!fl_sink_decode_takes(heads, kv_heads, dim, vdim) || n_splits < 1 || n_splits > 65535 || kv_heads > 65535 ||
         kept_splits < 0 || kept_splits >= n_splits || (rel != nullptr && (bucket_of == nullptr || n_dist < 1)))
@@ -552,6 +565,6 @@ FL_API int fl_sink_decode(const void* q, int dtype, long q_ld, void* out, long o
     if (rc) return rc;
     FL_DISPATCH(dtype, T, return fl_launch(sink_decode_merge_kernel<T>, dim3(n_decode, heads), dim3(128), 0, stream,
                                            (const float*)partial, n_splits, decode_tokens, (T*)out, out_ld, heads, vdim,
-                                           sink));
+                                           sink, (const T*)gate, gate_ld));
     return 0;
 }

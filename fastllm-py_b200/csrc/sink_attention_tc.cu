@@ -17,7 +17,8 @@
 // cp.async into a two-stage ring while the block before is multiplied.  The bias of this head by distance is staged
 // in shared memory for the first SINK_NEAR distances; farther ones (kept tokens far behind) are looked up in global
 // memory.  The sink enters as the softmax's starting state: running maximum = sink, running sum = 1, no value.
-// Probabilities are rounded to bfloat16 only as the operand of P V.
+// Probabilities are rounded to bfloat16 only as the operand of P V.  With a gate, a row's result is multiplied channel by
+// channel by the sigmoid of its gate row before it is rounded.
 //
 // SINK_DIM and SINK_VDIM are compile-time constants, multiples of 16 up to 128.
 #include "common.cuh"
@@ -76,7 +77,8 @@ __global__ void __launch_bounds__(STC_THREADS, 3) sink_attention_tc_kernel(
     long page_stride, int page_size, int page_shift, const int* __restrict__ block_table, int bt_stride,
     const int* __restrict__ req_start, const int* __restrict__ req_ctx, const int* __restrict__ req_qlen,
     int n_requests, int include_single, int heads, int kv_heads, int window, int keep_first, int chunk, float scale, float cap,
-    const int* __restrict__ row_of, int n_dist, const float* __restrict__ rel, const float* __restrict__ sink) {
+    const int* __restrict__ row_of, int n_dist, const float* __restrict__ rel, const float* __restrict__ sink,
+    const bf16* __restrict__ gate, long gate_ld) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char stc_raw[];
@@ -276,10 +278,15 @@ __global__ void __launch_bounds__(STC_THREADS, 3) sink_attention_tc_kernel(
         if (row >= rows_here) continue;
         const float inv = 1.0f / l_run[r];
         bf16* dst = out + (long)(tok0 + row) * out_ld + (long)h * SINK_VDIM + 2 * tq;
+        const bf16* gr = gate != nullptr ? gate + (long)(tok0 + row) * gate_ld + (long)h * SINK_VDIM + 2 * tq : nullptr;
 #pragma unroll
         for (int i = 0; i < SINK_VDIM / 8; ++i) {
-            const __nv_bfloat162 v = __floats2bfloat162_rn(o_acc[i][2 * r] * inv, o_acc[i][2 * r + 1] * inv);
-            *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = v;
+            float a = o_acc[i][2 * r] * inv, b = o_acc[i][2 * r + 1] * inv;
+            if (gr != nullptr) {
+                a = a / (1.0f + expf(-__bfloat162float(gr[i * 8])));
+                b = b / (1.0f + expf(-__bfloat162float(gr[i * 8 + 1])));
+            }
+            *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(a, b);
         }
     }
 }
@@ -296,7 +303,8 @@ FL_API int fl_sink_attention_tc(const void* q, long q_ld, void* out, long out_ld
                                 const int* req_ctx, const int* req_qlen, int n_requests, int n_tokens,
                                 int include_single, int heads,
                                 int kv_heads, int window, int keep_first, int chunk, float scale, float cap, const int* row_of,
-                                int n_dist, const float* rel, const float* sink, cudaStream_t stream) {
+                                int n_dist, const float* rel, const float* sink, const void* gate, long gate_ld,
+                                cudaStream_t stream) {
     if (n_requests <= 0 || n_tokens <= 0) return 0;
     if (heads > 65535 || heads % kv_heads || (rel != nullptr && (row_of == nullptr || n_dist < 1)))
         return (int)cudaErrorInvalidValue;
@@ -319,5 +327,5 @@ FL_API int fl_sink_attention_tc(const void* q, long q_ld, void* out, long out_ld
     return fl_launch(sink_attention_tc_kernel, grid, dim3(STC_THREADS), smem, stream, (const bf16*)q, q_ld, (bf16*)out,
                      out_ld, (const bf16*)cache, page_stride, page_size, page_shift, block_table, bt_stride, req_start,
                      req_ctx, req_qlen, n_requests, include_single, heads, kv_heads, window, keep_first, chunk, scale, cap, row_of, n_dist, rel,
-                     sink);
+                     sink, (const bf16*)gate, gate_ld);
 }

@@ -22,6 +22,8 @@ def _lib():
         lib.fl_gemm_tc.restype = c_int
         lib.fl_gemm_tc_partial.argtypes = lib.fl_gemm_tc.argtypes
         lib.fl_gemm_tc_partial.restype = c_int
+        lib.fl_gemm_tc_act.argtypes = lib.fl_gemm_tc.argtypes[:-1] + [c_int, ctypes.c_float, ctypes.c_float, c_void_p]
+        lib.fl_gemm_tc_act.restype = c_int
         lib.fl_gemm_tc_plan.argtypes = [c_int, c_int, c_int, c_int, ctypes.POINTER(c_int),
                                         ctypes.POINTER(c_int)]
         lib.fl_gemm_tc_plan.restype = None
@@ -196,20 +198,22 @@ def _remember(key, launch) -> None:
 
 
 def gemm(a: torch.Tensor, w, out: torch.Tensor, bn: int = 0, splits: int = 0,
-         defer: bool = False, side: bool = False):
+         defer: bool = False, side: bool = False, activation: str | None = None, params=(0.0, 0.0)):
     """out[M, N] = a[M, K] @ w[N, K]^T; a and w bfloat16 (row pitch a multiple of 8
     elements, base 16-byte aligned; w may be a PackedWeight), out bfloat16 or float32.
 
     With `defer`, a product whose K is split returns a Partial instead of
     writing `out`: its consumer adds the slabs while it reads them.  With `side`
     the slabs lie in the second scratch buffer, where later products of the
-    first buffer do not overwrite them."""
+    first buffer do not overwrite them.  `activation` (`ops.ACTIVATIONS`, of one
+    argument: f(v, 1)) is applied to the product on its way out; such a product
+    is not deferred."""
     # A product asked for again with the same operands in the same places (a layer's buffers do not move
     # from step to step) is launched from what the first call worked out: the checks, the plan and the
     # argument conversions below cost more host time than the driver's launch.
     _forget_if_scratch_moved(a.device)
     key = (a.data_ptr(), a.shape, a.stride(0), a.dtype, w.data_ptr(), w.shape, out.data_ptr(), out.shape,
-           out.stride(0), out.dtype, bn, splits, defer, side)
+           out.stride(0), out.dtype, bn, splits, defer, side, activation, tuple(params))
     known = _launches.get(key)
     serial_key = ("serial", a.device, "side") if side else ("serial", a.device)
     if known is not None:
@@ -222,6 +226,8 @@ def gemm(a: torch.Tensor, w, out: torch.Tensor, bn: int = 0, splits: int = 0,
         return partial
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise ops.KernelError("tensor-core gemm takes bfloat16 operands")
+    if activation is not None and defer:
+        raise ops.KernelError("tensor-core gemm: a product with an activation cannot be left as partial sums")
     m, k = a.shape
     n = w.shape[0]
     if w.shape[1] != k or out.shape[0] != m or out.shape[1] != n:
@@ -247,6 +253,9 @@ def gemm(a: torch.Tensor, w, out: torch.Tensor, bn: int = 0, splits: int = 0,
         _state[serial_key] = _state.get(serial_key, 0) + 1    # earlier Partials are now stale
     args = (ops._ptr(a), lda, w_ptr, ldw, ops._ptr(out), ops.dtype_code(out), ldc,
             m, n, k, bn, splits, ops._ptr(ws), ws_floats, sms, ops._ptr(status_word(a.device)))
+    if activation is not None:
+        fn = _lib().fl_gemm_tc_act
+        args += (ops.activation_code(activation), float(params[0]), float(params[1]))
     kernels = 2 if (splits > 1 and not deferred) else 1
     ops._check(fn(*args, ops._stream()), "gemm_tcgen05", kernels)
     partial = Partial(ws, splits, m, n, -(-n // 4) * 4, a.device, side) if deferred else None
@@ -360,5 +369,6 @@ class TensorCoreLinear:
             weight = padded[:, :k]
         self.weight = weight
 
-    def forward(self, a: torch.Tensor, out: torch.Tensor, defer: bool = False, side: bool = False):
-        return gemm(a, self.weight, out, defer=defer, side=side)
+    def forward(self, a: torch.Tensor, out: torch.Tensor, defer: bool = False, side: bool = False,
+                activation: str | None = None, params=(0.0, 0.0)):
+        return gemm(a, self.weight, out, defer=defer, side=side, activation=activation, params=params)

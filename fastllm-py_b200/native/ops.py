@@ -129,27 +129,60 @@ def rmsnorm(x, weight, out, eps, rows=None):
            "rmsnorm")
 
 
-def add_rmsnorm(resid, delta, weight, out, eps, rows=None):
-    """resid += delta (float32, written back unless rows are gathered); out = rmsnorm(resid) * weight."""
+def _row_vectors(vectors, width, what):
+    """The pointers of up to two float32 row vectors [width] that a kernel adds to every row."""
+    if len(vectors) > 2:
+        raise KernelError(f"{what}: at most two row vectors can be added at once")
+    for v in vectors:
+        if v.dtype != torch.float32 or v.numel() != width or not v.is_contiguous():
+            raise KernelError(f"{what}: a row vector is float32 and as wide as the stream")
+    _require_cuda(*vectors)
+    ptrs = [_ptr(v) for v in vectors] + [None, None]
+    return ptrs[0], ptrs[1]
+
+
+def add_rmsnorm(resid, delta, weight, out, eps, rows=None, vectors=()):
+    """resid += delta + the row vectors in `vectors` (float32, written back unless rows are gathered);
+    out = rmsnorm(resid) * weight."""
     _require_cuda(resid, delta, weight, out, rows)
     if resid.dtype != torch.float32:
         raise KernelError("add_rmsnorm: the residual stream must be float32")
+    vec_a, vec_b = _row_vectors(vectors, resid.shape[1], "add_rmsnorm")
     fn = _fn("elementwise", "fl_add_rmsnorm", [c_void_p, c_long, c_void_p, c_int, c_long, c_void_p,
                                                c_int, c_void_p, c_int, c_long, c_int, c_int, c_float,
-                                               c_void_p, c_void_p])
+                                               c_void_p, c_void_p, c_void_p, c_void_p])
     _check(fn(_ptr(resid), _ld(resid), _ptr(delta), dtype_code(delta), _ld(delta), _ptr(weight),
               dtype_code(weight), _ptr(out), dtype_code(out), _ld(out), out.shape[0], resid.shape[1],
-              float(eps), _ptr(rows), _stream()), "add_rmsnorm")
+              float(eps), _ptr(rows), vec_a, vec_b, _stream()), "add_rmsnorm")
 
 
-def add_rmsnorm_partial(resid, partial, weight, out, eps):
-    """resid += (split-K partial sums, added in slab order); out = rmsnorm(resid) * weight."""
+def add_bias(x, bias):
+    """x += bias (a float32 row vector), in every row, for x of either dtype."""
+    _require_cuda(x, bias)
+    if bias.dtype != torch.float32 or bias.numel() != x.shape[1]:
+        raise KernelError("add_bias: the bias is float32 and as wide as x")
+    fn = _fn("elementwise", "fl_add_bias", [c_void_p, c_int, c_long, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), dtype_code(x), _ld(x), _ptr(bias), x.shape[0], x.shape[1], _stream()), "add_bias")
+
+
+def row_add(resid, vectors):
+    """resid += every one of `vectors` (one or two float32 row vectors), in every row."""
+    _require_cuda(resid)
+    if resid.dtype != torch.float32:
+        raise KernelError("row_add: the residual stream must be float32")
+    vec_a, vec_b = _row_vectors(vectors, resid.shape[1], "row_add")
+    fn = _fn("elementwise", "fl_row_add", [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(resid), _ld(resid), vec_a, vec_b, resid.shape[0], resid.shape[1], _stream()), "row_add")
+
+
+def add_rmsnorm_partial(resid, partial, weight, out, eps, vectors=()):
+    """resid += (split-K partial sums, added in slab order) + the row vectors; out = rmsnorm(resid) * weight."""
     partial.check()
     # (the same operands in the same places, as in every layer of every step of a size: launched from
     # what the first such call converted; see gemm_tc.gemm)
     key = ("add_rmsnorm_partial", resid.data_ptr(), resid.shape, resid.stride(0), partial.data.data_ptr(),
            partial.splits, partial.split_stride, partial.ld, weight.data_ptr(), weight.dtype, out.data_ptr(),
-           out.shape, out.stride(0), out.dtype, eps)
+           out.shape, out.stride(0), out.dtype, eps, tuple(v.data_ptr() for v in vectors))
     known = _launches.get(key)
     if known is not None:
         _check(known[0](*known[1], _stream()), "add_rmsnorm_partial")
@@ -157,10 +190,10 @@ def add_rmsnorm_partial(resid, partial, weight, out, eps):
     _require_cuda(resid, weight, out)
     fn = _fn("elementwise", "fl_add_rmsnorm_partial", [c_void_p, c_long, c_void_p, c_int, c_long, c_long,
                                                        c_void_p, c_int, c_void_p, c_int, c_long, c_int,
-                                                       c_int, c_float, c_void_p])
+                                                       c_int, c_float, c_void_p, c_void_p, c_void_p])
     args = (_ptr(resid), _ld(resid), _ptr(partial.data), partial.splits, partial.split_stride,
             partial.ld, _ptr(weight), dtype_code(weight), _ptr(out), dtype_code(out), _ld(out),
-            out.shape[0], resid.shape[1], float(eps))
+            out.shape[0], resid.shape[1], float(eps), *_row_vectors(vectors, resid.shape[1], "add_rmsnorm_partial"))
     _check(fn(*args, _stream()), "add_rmsnorm_partial")
     if len(_launches) > 8192:
         _launches.clear()
@@ -652,21 +685,25 @@ def sigmoid_gate(a, g):
     _check(fn(_ptr(a), _ld(a), _ptr(g), _ld(g), dtype_code(a), a.shape[0], a.shape[1], _stream()), "sigmoid_gate")
 
 
-def pair_embed(table, pairs, out, step, last_token, buckets, mul_prev, mul_cur, scale):
+def pair_embed(table, pairs, out, step, last_token, buckets, mul_prev, mul_cur, scale, norm_w=None, eps=0.0):
     """out[t] = table[id_t] * scale + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets] (row `buckets` for a
-    request's first token).  `last_token` ([slots] int32) keeps each request's last token between steps."""
-    _require_cuda(table, pairs, out, last_token)
+    request's first token).  `last_token` ([slots] int32) keeps each request's last token between steps.  With `norm_w`
+    (float32 [hidden]) the row is then divided by its root mean square and multiplied by it."""
+    _require_cuda(table, pairs, out, last_token, norm_w)
+    if norm_w is not None and norm_w.dtype != torch.float32:
+        raise KernelError("pair_embed: the norm's weight is float32")
     fed = getattr(step, "token_feed", None)
     if out.dtype != torch.float32 or table.dtype != pairs.dtype or last_token.dtype != torch.int32:
         raise KernelError("pair_embed: out float32, both tables of one dtype, last_token int32")
     fn = _fn("gated_block", "fl_pair_embed", [c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_void_p, c_long, c_int,
                                               c_int, c_int, c_int, c_long, c_long, c_float, c_void_p, c_void_p, c_void_p,
-                                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+                                              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float,
+                                              c_void_p])
     _check(fn(_ptr(table), _ld(table), _ptr(pairs), _ld(pairs), dtype_code(table), _ptr(step.token_ids), _ptr(out), _ld(out),
               step.token_ids.numel(), table.shape[1], table.shape[0], int(buckets), int(mul_prev), int(mul_cur),
               float(scale), _ptr(step.tok_req), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen),
               _ptr(step.req_slot), _ptr(last_token), _ptr(step.status), _ptr(fed), 0 if fed is None else fed.numel(),
-              _stream()), "pair_embed")
+              _ptr(norm_w), float(eps), _stream()), "pair_embed")
 
 
 # ------------------------------------------------- attention with soft cap, distance bias, kept first tokens, sink
@@ -690,23 +727,31 @@ def sink_prep(proj, bias, q_w, k_w, eps, q_out, heads, kv_heads, dim, vdim, v_mo
               _stream()), "sink_prep")
 
 
+def _check_gate(gate, out):
+    if gate is not None and (gate.dtype != out.dtype or gate.shape != out.shape):
+        raise KernelError("attention: the output gate has the output's shape and dtype")
+
+
 def sink_attention_simt(q, out, cache, block_table, tok_req, positions, heads, kv_heads, dim, vdim, window, keep_first,
-                        scale, cap, bucket_of, rel, sink, page_size, chunk=None):
+                        scale, cap, bucket_of, rel, sink, page_size, chunk=None, gate=None):
     """Attention of every token over its request's visible keys (the last `window` and the first `keep_first`), scores
     capped (`cap` None or 0: not), biased by `rel[bucket_of[distance]]` and with `sink` in the denominator (each may be
     None).  With `chunk` a query sees only keys at or after the last multiple of `chunk` at or below its own position.
+    With `gate` ([N, heads * vdim], typed like `out`) the result is multiplied by its sigmoid, channel by channel.
     CUDA cores, any sizes, both number formats."""
-    _require_cuda(q, out, cache, block_table, tok_req, positions, bucket_of, rel, sink)
+    _require_cuda(q, out, cache, block_table, tok_req, positions, bucket_of, rel, sink, gate)
+    _check_gate(gate, out)
     if vdim > 256:
         raise KernelError(f"sink_attention: value size {vdim} is beyond the kernel's limit of 256")
     fn = _fn("sink_attention", "fl_sink_attention_simt",
              [c_void_p, c_int, c_long, c_void_p, c_long, c_void_p, c_int, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p,
               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
-              c_void_p])
+              c_void_p, c_long, c_void_p])
     _check(fn(_ptr(q), dtype_code(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), dtype_code(cache), cache.stride(0), page_size,
               _ptr(block_table), block_table.stride(0), _ptr(tok_req), _ptr(positions), q.shape[0], heads, kv_heads, dim,
               vdim, int(window or 0), int(keep_first or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(bucket_of),
-              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _stream()), "sink_attention_simt")
+              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _ptr(gate), 0 if gate is None else _ld(gate),
+              _stream()), "sink_attention_simt")
 
 
 def sink_tc_takes(dtype, dim: int, vdim: int) -> bool:
@@ -719,21 +764,23 @@ def sink_tc_library(dim: int, vdim: int):
 
 
 def sink_attention_tc(q, out, cache, block_table, step, heads, kv_heads, dim, vdim, window, keep_first, scale, cap,
-                      bucket_of, rel, sink, page_size, include_single=True, chunk=None):
+                      bucket_of, rel, sink, page_size, include_single=True, chunk=None, gate=None):
     """`sink_attention_simt` on tensor cores: q, cache and out bfloat16; one build per (dim, vdim); 64 rows of a
     request and one head per block, single tokens as tiles of one row (left out with include_single=False)."""
-    _require_cuda(q, out, cache, block_table, bucket_of, rel, sink)
+    _require_cuda(q, out, cache, block_table, bucket_of, rel, sink, gate)
+    _check_gate(gate, out)
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("sink_attention_tc: q, cache and out must be bfloat16")
     name, defines = sink_tc_library(dim, vdim)
     fn = _fn(name, "fl_sink_attention_tc", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_int,
                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                            c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p], defines)
+                                            c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long,
+                                            c_void_p], defines)
     _check(fn(_ptr(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), cache.stride(0), page_size, _ptr(block_table),
               block_table.stride(0), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), step.n_requests,
               q.shape[0], int(include_single), heads, kv_heads, int(window or 0), int(keep_first or 0), int(chunk or 0),
               float(scale), float(cap or 0.0), _ptr(bucket_of), 0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink),
-              _stream()), "sink_attention_tc")
+              _ptr(gate), 0 if gate is None else _ld(gate), _stream()), "sink_attention_tc")
 
 
 SINK_SPLIT = 128                 # keys of one split of the single-token kernel
@@ -755,11 +802,12 @@ def sink_decode_splits(window, keep_first: int, longest: int, chunk=None):
 
 
 def sink_decode(q, out, cache, block_table, tok_req, positions, decode_tokens, partial, n_splits, kept_splits, heads,
-                kv_heads, dim, vdim, window, keep_first, scale, cap, bucket_of, rel, sink, page_size, chunk=None):
+                kv_heads, dim, vdim, window, keep_first, scale, cap, bucket_of, rel, sink, page_size, chunk=None, gate=None):
     """Sink attention for the rows `decode_tokens` of q (each the single token of its request): the keys split over
     blocks of 128, every query head of a key/value head served by the block that reads its rows, then a merge with
     the sink.  partial: float32, decode tokens * heads * n_splits * (vdim + 2)."""
-    _require_cuda(q, out, cache, block_table, tok_req, positions, decode_tokens, partial, bucket_of, rel, sink)
+    _require_cuda(q, out, cache, block_table, tok_req, positions, decode_tokens, partial, bucket_of, rel, sink, gate)
+    _check_gate(gate, out)
     n = decode_tokens.numel()
     if partial.dtype != torch.float32 or partial.numel() < n * heads * n_splits * (vdim + 2):
         raise KernelError("sink_decode: the buffer for the splits' results is too small")
@@ -768,12 +816,13 @@ def sink_decode(q, out, cache, block_table, tok_req, positions, decode_tokens, p
     fn = _fn("sink_attention", "fl_sink_decode",
              [c_void_p, c_int, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p,
               c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-              c_void_p, c_int, c_void_p, c_void_p, c_void_p])
+              c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p])
     _check(fn(_ptr(q), dtype_code(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), cache.stride(0), page_size,
               _ptr(block_table), block_table.stride(0), _ptr(tok_req), _ptr(positions), _ptr(decode_tokens), n,
               _ptr(partial), int(n_splits), int(kept_splits), heads, kv_heads, dim, vdim, int(window or 0),
               int(keep_first or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(bucket_of),
-              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _stream()), "sink_decode", 2)
+              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _ptr(gate), 0 if gate is None else _ld(gate),
+              _stream()), "sink_decode", 2)
 
 
 def head_prep(proj, bias, q_w, k_w, norm_mode, eps, rot, interleaved, cos, sin, positions, temp, v_from_k, q_out, heads,
@@ -810,6 +859,109 @@ def head_gate(x, gate, heads, vdim):
         raise KernelError("head_gate: x and the gate share a dtype")
     fn = _fn("sink_attention", "fl_head_gate", [c_void_p, c_int, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(x), dtype_code(x), _ld(x), _ptr(gate), _ld(gate), x.shape[0], heads, vdim, _stream()), "head_gate")
+
+
+def conv_head_prep(proj, bias, conv_w, tail, q_w, k_w, norm_mode, eps, rot, interleaved, cos, sin, step, temp, v_scale, q_out,
+                   heads, kv_heads, dim, vdim, slots, cache, page_size):
+    """`head_prep` behind a short causal convolution on every channel of q | k | v (`conv_w` [taps, channels] float32, the
+    last row the current token's; None: no convolution), which takes the rows before the step's first from `tail`
+    ([slots, >= (taps - 1) * channels] float32: each request's last inputs, moved on here).  Values are multiplied by
+    `v_scale`.  The biases are part of the convolution's input."""
+    _require_cuda(proj, bias, conv_w, tail, q_w, k_w, cos, sin, q_out, slots, cache)
+    channels = (heads + kv_heads) * dim + kv_heads * vdim
+    taps = 1 if conv_w is None else conv_w.shape[0]
+    if cache.dtype != proj.dtype or q_out.dtype != proj.dtype or not cache.is_contiguous():
+        raise KernelError("conv_head_prep: queries and cache have the activations' dtype, and the cache is contiguous")
+    for v in (bias, conv_w, tail, q_w, k_w, cos, sin):
+        if v is not None and v.dtype != torch.float32:
+            raise KernelError("conv_head_prep: biases, taps, kept rows, norm weights and the rotation's tables are float32")
+    if conv_w is not None and (conv_w.shape[1] != channels or not conv_w.is_contiguous() or
+                               (taps > 1 and (tail is None or tail.shape[1] < (taps - 1) * channels))):
+        raise KernelError("conv_head_prep: the taps and the kept rows must cover every channel")
+    if rot and cos.shape[1] != rot // 2:
+        raise KernelError("conv_head_prep: the rotation's tables do not fit the rotated dimensions")
+    coef, every = temp if temp is not None else (0.0, 0)
+    several = step.n_decode_tokens != step.n_requests
+    fn = _fn("conv_head", "fl_conv_head_prep",
+             [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_void_p, c_long, c_void_p, c_void_p, c_int, c_float, c_int,
+              c_int, c_void_p, c_void_p, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+              c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_void_p])
+    _check(fn(_ptr(proj), dtype_code(proj), _ld(proj), _ptr(bias), _ptr(conv_w), taps, _ptr(tail),
+              0 if tail is None else tail.stride(0), _ptr(q_w), _ptr(k_w), int(norm_mode), float(eps), int(rot or 0),
+              int(bool(interleaved)), _ptr(cos) if rot else None, _ptr(sin) if rot else None, float(coef), int(every),
+              float(v_scale), _ptr(step.positions), _ptr(step.tok_req), _ptr(step.req_start), _ptr(step.req_ctx),
+              _ptr(step.req_qlen), _ptr(step.req_slot), _ptr(slots), _ptr(q_out), _ld(q_out), proj.shape[0], step.n_requests,
+              int(several), heads, kv_heads, dim, vdim, _ptr(cache), cache.stride(0), page_size, _stream()),
+           "conv_head_prep", 2 if taps > 1 and several else 1)
+
+
+# ------------------------------------------------------- state-space recurrence
+
+def _ssd_channels(heads, vdim, state, groups):
+    return heads * vdim + 2 * groups * state
+
+
+def ssd_prep(proj, conv_w, conv_b, dt_bias, neg_a, tail, step, work, heads, vdim, state, groups):
+    """proj columns z | x | B | C | dt: convolution (`conv_w` [taps, channels], `conv_b`), silu, dt = softplus(dt + dt_bias)
+    and decay = exp(neg_a dt) (`neg_a` float64 [heads]) of every token into the float32 columns x | B | C | dt | decay of
+    `work`.  `tail`: each request's last taps - 1 inputs ([slots, ...] float32, left as they are)."""
+    _require_cuda(proj, conv_w, conv_b, dt_bias, neg_a, tail, work)
+    taps, channels = conv_w.shape
+    if neg_a.dtype != torch.float64 or channels != _ssd_channels(heads, vdim, state, groups) or not conv_w.is_contiguous() or \
+            any(v.dtype != torch.float32 for v in (conv_w, conv_b, dt_bias, work)) or (taps > 1 and tail.dtype != torch.float32):
+        raise KernelError("ssd_prep: float32 parameters (neg_a float64), taps for every channel")
+    fn = _fn("ssd", "fl_ssd_prep", [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long,
+                                    c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int,
+                                    c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(proj), dtype_code(proj), _ld(proj), _ptr(conv_w), _ptr(conv_b), taps, _ptr(dt_bias), _ptr(neg_a), _ptr(tail),
+              0 if tail is None else tail.stride(0), _ptr(step.tok_req), _ptr(step.positions), _ptr(step.req_start),
+              _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), _ptr(work), _ld(work), proj.shape[0], heads, vdim,
+              state, groups, _stream()), "ssd_prep")
+
+
+def ssd_scan(work, skip, y, state_rows, step, heads, vdim, state, groups):
+    """Per request and head S <- decay S + dt B x^T, y = S^T C + skip x over the step's tokens (`work` as ssd_prep leaves
+    it); y float32 [N, heads * vdim]; state rows [heads, vdim, state] float32 are read (unless the request starts) and
+    written."""
+    _require_cuda(work, skip, y, state_rows)
+    if any(v.dtype != torch.float32 for v in (work, skip, y, state_rows)):
+        raise KernelError("ssd_scan: all operands are float32")
+    fn = _fn("ssd", "fl_ssd_scan", [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(work), _ld(work), _ptr(skip), _ptr(y), _ld(y), _ptr(state_rows), state_rows.stride(0), _ptr(step.req_start),
+              _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests, heads, vdim, state, groups,
+              _stream()), "ssd_scan")
+
+
+def ssd_step(proj, conv_w, conv_b, dt_bias, neg_a, skip, y, state_rows, tail_off, step, heads, vdim, state, groups):
+    """ssd_prep and ssd_scan in one kernel for a step in which every request brings one token.  State rows: S, and from
+    `tail_off` on the convolution's kept inputs (left as they are)."""
+    _require_cuda(proj, conv_w, conv_b, dt_bias, neg_a, skip, y, state_rows)
+    taps, channels = conv_w.shape
+    if step.n_tokens != step.n_requests or neg_a.dtype != torch.float64 or channels != _ssd_channels(heads, vdim, state, groups) \
+            or any(v.dtype != torch.float32 for v in (conv_w, conv_b, dt_bias, skip, y, state_rows)) or not conv_w.is_contiguous():
+        raise KernelError("ssd_step: one token a request; float32 parameters (neg_a float64)")
+    fn = _fn("ssd", "fl_ssd_step", [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                    c_long, c_void_p, c_long, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                    c_void_p])
+    _check(fn(_ptr(proj), dtype_code(proj), _ld(proj), _ptr(conv_w), _ptr(conv_b), taps, _ptr(dt_bias), _ptr(neg_a), _ptr(skip),
+              _ptr(y), _ld(y), _ptr(state_rows), state_rows.stride(0), int(tail_off), _ptr(step.req_ctx), _ptr(step.req_slot),
+              step.n_requests, heads, vdim, state, groups, _stream()), "ssd_step")
+
+
+def ssd_norm(y, proj, weight, out, parts, eps, tail, taps, channels, step):
+    """out = (y * silu(z)) normed in `parts` equal parts, times `weight` (float32), z the first columns of `proj`; and the
+    convolution's kept inputs of every request of the step moved on (`tail` [slots, ...] float32, None with one tap)."""
+    _require_cuda(y, proj, weight, out, tail)
+    if y.dtype != torch.float32 or weight.dtype != torch.float32 or out.dtype != proj.dtype:
+        raise KernelError("ssd_norm: y and weight are float32, out has the activations' dtype")
+    fn = _fn("ssd", "fl_ssd_norm", [c_void_p, c_long, c_void_p, c_int, c_long, c_void_p, c_void_p, c_long, c_int, c_int, c_int,
+                                    c_float, c_void_p, c_long, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                    c_void_p])
+    _check(fn(_ptr(y), _ld(y), _ptr(proj), dtype_code(proj), _ld(proj), _ptr(weight), _ptr(out), _ld(out), out.shape[0],
+              y.shape[1], int(parts), float(eps), _ptr(tail), 0 if tail is None else tail.stride(0), int(taps), int(channels),
+              _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests, _stream()),
+           "ssd_norm")
 
 
 # ----------------------------------------------- layer norm, mixes, activation

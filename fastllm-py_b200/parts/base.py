@@ -36,6 +36,7 @@ What a part may declare beside its interface (all optional; absent means "no"):
   takes_extra = True       norm: `apply` adds `stream.extra` (a second tensor) along with a pending tensor; such a
                            norm also has `apply_pair(stream, other, out, out_other)`: its own norm and that of
                            `other` (same kind, size and eps) of the one row in one pass
+  takes_vectors = True     norm: `apply` adds `stream.vectors` (row vectors) along with a pending sum
   takes_fed_tokens = True  embedding: understands a token id -1 - r as "row r of `step.token_feed`"
                            (without it the scheduler never launches a step ahead of the host)
 """
@@ -108,6 +109,20 @@ class ResidualStream:
                                      # side leaves two); a norm with `takes_extra` adds both while it reads
         self.pending_scale = 1.0     # the pending sum is multiplied by this as it is added (a layer that scales its
                                      # sublayers' results); a norm with `takes_scale` does so while it reads
+        self.vectors = ()            # float32 row vectors [hidden] not yet added, each to every row (a product's output
+                                     # bias, the vector that a pass of layers starts with)
+
+    def add_vector(self, vector):
+        """Every row is to be increased by `vector`, at the latest when the next norm reads the stream."""
+        if len(self.vectors) == 2:
+            self._add_vectors()
+        self.vectors = self.vectors + (vector,)
+
+    def _add_vectors(self):
+        """x += the row vectors, for whoever cannot take them itself."""
+        from ..native import ops
+        ops.row_add(self.x, self.vectors)
+        self.vectors = ()
 
     def _add_scaled(self):
         """x += pending_scale * pending (a tensor), for whoever cannot take the scale itself."""
@@ -118,6 +133,8 @@ class ResidualStream:
     def settle(self):
         """x takes in whatever is still pending (for a block whose sublayers read x itself)."""
         from ..native import ops
+        if self.vectors:
+            self._add_vectors()
         if self.pending is not None and not isinstance(self.pending, torch.Tensor):
             self.pending = self.pending.reduce_into(self.spill())
         if self.pending is not None and self.pending_scale != 1.0:
@@ -135,6 +152,9 @@ class ResidualStream:
     def norm_into(self, norm, out, rows=None):
         """`norm.apply(self, out, rows)`, with a pending sum that the norm can take."""
         pending = self.pending
+        if self.vectors and (pending is None or self.pending_scale != 1.0 or self.pending_norm is not None or
+                             self.extra is not None or not getattr(norm, "takes_vectors", False)):
+            self._add_vectors()
         if pending is not None and not isinstance(pending, torch.Tensor):
             both = getattr(norm, "takes_partial", False) and \
                 (self.pending_scale == 1.0 or getattr(norm, "takes_scale", False)) and \
@@ -204,3 +224,70 @@ class Workspace:
             self._views.clear()
         view = self._views[(name, cols, dtype, n)] = buf[:n, :cols]
         return view
+
+
+class ProjectedMixer(Part):
+    """A mixer between two matrix products: one stacked product of the input, a core that turns a token's columns of it
+    (with a cache or state) into the operand of the second, and that second product.
+
+    A subclass names the matrices (`in_slots`, stacked in this order; `out_slot`), their widths (`in_cols`, `out_cols`,
+    `hidden`), the other tensors (`core_shapes`, `load_core`) and the core itself:
+
+        core(proj, y, step, cache)    proj [N, in_cols] -> y [N, out_cols]
+
+    Two such mixers that read the same input can share both products (`side_by_side_sum`): the parent sets `joint` before
+    the tensors are loaded, holds the matrices itself and calls the cores.  `result_scale` is a factor on the mixer's
+    result that the core applies where it costs nothing (before y is rounded)."""
+    joint = False
+    result_scale = 1.0
+    in_slots: tuple = ()
+    out_slot = "o"
+    in_cols = out_cols = hidden = 0
+    workspace_name = "mixer"
+    honours_partial_side = True          # with `partial_side` set, the last product's partial sums go to the second scratch
+    partial_side = False
+    proj = o = None
+
+    def in_rows(self) -> dict:
+        """slot -> rows of its matrix."""
+        raise NotImplementedError
+
+    def core_shapes(self) -> dict:
+        return {}
+
+    def product_shapes(self) -> dict:
+        shapes = {slot: (rows, self.hidden) for slot, rows in self.in_rows().items()}
+        shapes[self.out_slot] = (self.hidden, self.out_cols)
+        return shapes
+
+    def weight_shapes(self):
+        return self.core_shapes() if self.joint else {**self.product_shapes(), **self.core_shapes()}
+
+    def load_core(self, tensors) -> None:
+        pass
+
+    def load(self, tensors):
+        from .linear import Linear
+        if not self.joint:
+            mats = [tensors[slot] for slot in self.in_slots]
+            if len({m.dtype for m in mats}) != 1:
+                raise ValueError(f"{self.workspace_name}: the stacked matrices must be stored in one dtype")
+            self.proj = Linear(mats)
+            self.o = Linear([tensors[self.out_slot]])
+        self.load_core(tensors)
+
+    def reserve(self, limits):
+        if self.proj is not None:
+            self.proj.reserve(self.ctx.dtype, limits.max_tokens)
+            self.o.reserve(self.ctx.dtype, limits.max_tokens, side=self.partial_side)
+
+    def core(self, proj, y, step, cache) -> None:
+        raise NotImplementedError
+
+    def forward(self, h, out, step, cache):
+        n, dt, ws = h.shape[0], self.ctx.dtype, step.workspace
+        proj = ws.rows(self.workspace_name + "_proj", n, self.in_cols, dt)
+        self.proj.forward(h, proj)
+        y = ws.rows(self.workspace_name + "_y", n, self.out_cols, dt)
+        self.core(proj, y, step, cache)
+        return self.o.forward(y, out, defer=True, side=self.partial_side)

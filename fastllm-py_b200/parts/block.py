@@ -2,7 +2,8 @@
 
 "prenorm" is the Llama layer (fastllm_py/model.py:464-470):
     x = x + mixer(norm_mixer(x));  x = x + feed_forward(norm_ff(x))
-The sums are left pending on the residual stream and folded into the next norm.  With `residual_scale`
+The sums are left pending on the residual stream and folded into the next norm, and with them a bias of the mixer's
+last product (`out_bias` of a mixer that says it `defers_out_bias`).  With `residual_scale`
 m both sums are multiplied by m as they are added, and the layer may have no feed-forward.
 
 "sandwich" norms each sublayer on both sides:
@@ -38,6 +39,8 @@ class PreNormBlock(Part):
             self.norm_ff = build_part("norm", layer_spec.norms["feed_forward"], ctx)
         self.hidden = self.norm_mixer.size
         self.scale = float(layer_spec.params.get("residual_scale", 1.0))
+        if self.scale == 1.0 and hasattr(self.mixer, "defers_out_bias"):
+            self.mixer.defers_out_bias = True
 
     def children(self):
         parts = [self.mixer, self.norm_mixer]
@@ -55,6 +58,8 @@ class PreNormBlock(Part):
         stream.norm_into(self.norm_mixer, h)
         left = self.mixer.forward(h, delta, step, cache)
         stream.pending, stream.pending_scale = (delta if left is None else left), self.scale
+        if getattr(self.mixer, "defers_out_bias", False) and self.mixer.out_bias is not None:
+            stream.add_vector(self.mixer.out_bias)
         if self.feed_forward is None:
             return
         stream.norm_into(self.norm_ff, h)

@@ -27,7 +27,14 @@ class Decoder:
         self.blocks = [part_class("block", layer.block)(layer, ctx) for layer in plan.layers]
         self.final_norm = build_part("norm", plan.final_norm, ctx)
         self.head = build_part("head", plan.head, ctx)
+        self.vectors = build_part("vectors", plan.vectors, ctx) if plan.vectors is not None else None
         self.order = list(plan.order)
+        # cache id of each run and, for a mixer with several needs, their names
+        self._views_of = []
+        for i, run in enumerate(self.order):
+            mixer = self.blocks[run.layer].mixer
+            names = tuple(mixer.cache_needs()) if hasattr(mixer, "cache_needs") else ()
+            self._views_of.append((i if run.cache is None else run.cache, names))
         self.observer = None
         for i, run in enumerate(self.order):
             need = self.blocks[run.layer].mixer.cache_need()
@@ -52,6 +59,8 @@ class Decoder:
                 visit(c)
 
         visit(self.embedding)
+        if self.vectors is not None:
+            visit(self.vectors)
         for b in self.blocks:
             visit(b)
         visit(self.final_norm)
@@ -186,17 +195,20 @@ class Decoder:
         else:
             self.embedding.forward(step, stream.x)
         for i, run in enumerate(self.order):
-            cache_id = i if run.cache is None else run.cache
+            cache_id, names = self._views_of[i]
             block = self.blocks[run.layer]
-            cache = step.cache_view(cache_id, run.cache is None)
-            if hasattr(block.mixer, "cache_needs"):            # several caches or states: the views by name
-                cache = {name: step.cache_view((cache_id, name), run.cache is None) for name in block.mixer.cache_needs()}
+            if names:                                          # several caches or states: the views by name
+                cache = {name: step.cache_view((cache_id, name), run.cache is None) for name in names}
+            else:
+                cache = step.cache_view(cache_id, run.cache is None)
+            if run.vector is not None:
+                stream.add_vector(self.vectors.row(run.vector))
             if hasattr(block, "state_need"):
                 block.forward(stream, step, cache, step.cache_view(("block", i), True))
             else:
                 block.forward(stream, step, cache)
             if self.observer is not None:                      # (a debugging aid: sees the stream after every run,
-                self.observer(i, stream)                       # with the run's last sum still pending)
+                self.observer(i, stream)                       # with the run's last sum (and bias) still pending)
         m = step.n_wanted
         logits = ws.rows("logits", m, self.vocab, torch.float32, initial=64)
         if m > 0:

@@ -21,18 +21,19 @@ import torch
 
 from ..cache.needs import FixedState
 from ..native import ops
-from .base import Part
-from .linear import Linear
+from .base import ProjectedMixer
 from .registry import register_part
 
 
 @register_part("mixer", "gated_linear_attention")
-class GatedLinearAttention(Part):
+class GatedLinearAttention(ProjectedMixer):
     """params: hidden_size, heads, dim, vdim, tau, norm_eps, q_scale (None: dim^-1/2).  tensors: q, k [heads * dim, hidden],
     v, g [heads * vdim, hidden], a1 [rank, hidden], a2 [heads * dim, rank], a2_bias [heads * dim], norm [vdim],
     o [hidden, heads * vdim]; `rank` is a1's row count, a parameter too."""
     category = "mixer"
     native_libraries = ("gla",)
+    in_slots = ("q", "k", "v", "g", "a1")
+    workspace_name = "gla"
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -46,44 +47,31 @@ class GatedLinearAttention(Part):
         if self.dim > 256:
             raise ValueError(f"gated_linear_attention: dim {self.dim} is beyond the scan kernel's limit of 256")
         self.hd, self.hv = self.heads * self.dim, self.heads * self.vdim
-        self.proj_cols = 2 * self.hd + 2 * self.hv + self.rank          # q | k | v | gate | low
-        self.proj = self.o = None
+        self.in_cols, self.out_cols = 2 * self.hd + 2 * self.hv + self.rank, self.hv     # q | k | v | gate | low
 
     def cache_need(self):
         return FixedState((self.heads * self.vdim * self.dim,), "float32")
 
-    def weight_shapes(self):
-        w = self.hidden
-        return {"q": (self.hd, w), "k": (self.hd, w), "v": (self.hv, w), "g": (self.hv, w), "a1": (self.rank, w),
-                "a2": (self.hd, self.rank), "a2_bias": (self.hd,), "norm": (self.vdim,), "o": (w, self.hv)}
+    def in_rows(self):
+        return {"q": self.hd, "k": self.hd, "v": self.hv, "g": self.hv, "a1": self.rank}
 
-    def load(self, tensors):
-        mats = [tensors[s] for s in ("q", "k", "v", "g", "a1")]
-        if len({m.dtype for m in mats}) != 1:
-            raise ValueError("gated_linear_attention: the projections must be stored in one dtype")
-        self.proj = Linear(mats)
-        self.o = Linear([tensors["o"]])
+    def core_shapes(self):
+        return {"a2": (self.hd, self.rank), "a2_bias": (self.hd,), "norm": (self.vdim,)}
+
+    def load_core(self, tensors):
         self.a2 = tensors["a2"].float().t().contiguous()               # [rank, heads * dim]: the kernel reads along heads * dim
         self.a2_bias = tensors["a2_bias"].float().contiguous()
         self.norm_w = tensors["norm"].contiguous()
+        if self.result_scale != 1.0:
+            self.norm_w = (self.norm_w.double() * self.result_scale).float()
 
-    def reserve(self, limits):
-        for lin in (self.proj, self.o):
-            if lin is not None:
-                lin.reserve(self.ctx.dtype, limits.max_tokens)
-
-    def forward(self, h, out, step, cache):
-        n = h.shape[0]
-        dt = self.ctx.dtype
+    def core(self, proj, y, step, cache):
+        n = proj.shape[0]
         ws = step.workspace
-        proj = ws.rows("gla_proj", n, self.proj_cols, dt)
-        self.proj.forward(h, proj)
         work = ws.rows("gla_work", n, 3 * self.hd + self.hv, torch.float32)
         ops.gla_prep(proj, self.a2, self.a2_bias, work, self.heads, self.dim, self.vdim, self.rank, self.q_scale, self.tau)
         o = ws.rows("gla_o", n, self.hv, torch.float32)
         ops.gla_scan(work, o, cache.tensor, step, self.heads, self.dim, self.vdim,
-                     fixed_order=dt == torch.float32)     # the 32-bit path: cuts and batches agree bit for bit
-        y = ws.rows("gla_y", n, self.hv, dt)
+                     fixed_order=self.ctx.dtype == torch.float32)     # the 32-bit path: cuts and batches agree bit for bit
         ops.gla_gated_norm(o, proj[:, 2 * self.hd + self.hv:2 * self.hd + 2 * self.hv], self.norm_w, y, self.heads,
                            self.vdim, self.norm_eps)
-        return self.o.forward(y, out, defer=True)

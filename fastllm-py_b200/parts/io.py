@@ -15,7 +15,9 @@ from .registry import register_part
 
 @register_part("embedding", "table")
 class Embedding(Part):
-    """params: vocab_size, hidden_size, scale (1: none).  tensors: weight [vocab, hidden]."""
+    """params: vocab_size, hidden_size, scale (1: none), norm_eps (None: the rows are not normed), norm_offset (0).
+    tensors: weight [vocab, hidden]; with norm_eps norm [hidden]: the residual stream starts as the row divided by its
+    root mean square times (norm_offset + norm)."""
     category = "embedding"
     takes_fed_tokens = True              # an id -1 - r is taken from row r of step.token_feed
 
@@ -24,16 +26,25 @@ class Embedding(Part):
         self.vocab = int(spec.params["vocab_size"])
         self.hidden = int(spec.params["hidden_size"])
         self.scale = float(spec.params.get("scale", 1.0))
-        self.table = None
+        self.norm_eps = spec.params.get("norm_eps")
+        self.norm_offset = float(spec.params.get("norm_offset", 0.0))
+        self.table = self.norm_w = None
 
     def weight_shapes(self):
-        return {"weight": (self.vocab, self.hidden)}
+        shapes = {"weight": (self.vocab, self.hidden)}
+        if self.norm_eps is not None:
+            shapes["norm"] = (self.hidden,)
+        return shapes
 
     def load(self, tensors):
         self.table = tensors["weight"]
+        if self.norm_eps is not None:
+            self.norm_w = (tensors["norm"].double() + self.norm_offset).float().contiguous()
 
     def forward(self, step, out):
         ops.embed(self.table, step.token_ids, out, step.status, getattr(step, "token_feed", None), self.scale)
+        if self.norm_w is not None:
+            ops.rmsnorm(out, self.norm_w, out, self.norm_eps)       # in place: a thread rewrites what it read
 
 
 @register_part("embedding", "table_pairs")
@@ -41,8 +52,8 @@ class PairEmbedding(Embedding):
     """x = table[id] * scale + pairs[(previous id * mul_prev + id * mul_cur) mod buckets]: a second, hashed table
     indexed by the token and the one before it; a sequence's first token takes the table's last row (`buckets`).
     The token before a step's first one is per-request state (one int32 per request slot).
-    params: vocab_size, hidden_size, scale, buckets, mul_prev, mul_cur.  tensors: weight [vocab, hidden],
-    pairs [buckets + 1, hidden]."""
+    params: vocab_size, hidden_size, scale, norm_eps, norm_offset (as above; the sum is normed), buckets, mul_prev,
+    mul_cur.  tensors: weight [vocab, hidden], pairs [buckets + 1, hidden], norm."""
     native_libraries = ("gated_block",)
 
     def __init__(self, spec, ctx):
@@ -55,21 +66,44 @@ class PairEmbedding(Embedding):
         self.pairs = None
 
     def weight_shapes(self):
-        return {"weight": (self.vocab, self.hidden), "pairs": (self.buckets + 1, self.hidden)}
+        return {**super().weight_shapes(), "pairs": (self.buckets + 1, self.hidden)}
 
     def state_need(self):
         from ..cache.needs import FixedState
         return FixedState((1,), "int32")
 
     def load(self, tensors):
-        self.table = tensors["weight"]
+        super().load(tensors)
         self.pairs = tensors["pairs"]
         if self.pairs.dtype != self.table.dtype:
             raise ValueError("table_pairs: both tables must be stored in one dtype")
 
     def forward(self, step, out, state):
         ops.pair_embed(self.table, self.pairs, out, step, state.tensor, self.buckets, self.mul_prev, self.mul_cur,
-                       self.scale)
+                       self.scale, self.norm_w, self.norm_eps or 0.0)
+
+
+@register_part("vectors", "table")
+class VectorTable(Part):
+    """Vectors [n, hidden] that runs of layers start with: added to every row of the residual stream.
+    params: count, hidden_size.  tensors: rows [count, hidden]."""
+    category = "vectors"
+
+    def __init__(self, spec, ctx):
+        super().__init__(spec, ctx)
+        self.count = int(spec.params["count"])
+        self.hidden = int(spec.params["hidden_size"])
+        self.table = None
+
+    def weight_shapes(self):
+        return {"rows": (self.count, self.hidden)}
+
+    def load(self, tensors):
+        # one allocation a row: every row starts on an aligned address, whatever the width
+        self.table = [row.contiguous().clone() for row in tensors["rows"].float()]
+
+    def row(self, i):
+        return self.table[i]
 
 
 @register_part("head", "linear")

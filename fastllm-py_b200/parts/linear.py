@@ -70,6 +70,15 @@ class Linear:
         ops.gemm_simt(a, self.weight, out)
         return None
 
+    def forward_activated(self, a: torch.Tensor, out: torch.Tensor, activation: str, params=(0.0, 0.0)) -> None:
+        """out = f(a @ W^T, 1) for an activation of one argument (`native.ops.ACTIVATIONS`): in the tensor-core
+        product's epilogue, else by a kernel of its own."""
+        if a.dtype == torch.bfloat16 and self.dtype == torch.bfloat16:
+            self._tensor_core().forward(a, out, activation=activation, params=params)
+            return
+        self.forward(a, out)
+        ops.activation(out, out, activation, params)
+
     def _tensor_core(self):
         if self._tc is None:
             from ..native.gemm_tc import TensorCoreLinear

@@ -66,7 +66,7 @@ class SwiGLU(Part):
 @register_part("feed_forward", "mlp")
 class PlainMLP(Part):
     """A feed-forward without a gate: down(act(up(h))), no biases; act is the gated units' f(x, 1)
-    (`native.ops.ACTIVATIONS`: "relu_squared" is relu(x)^2).
+    (`native.ops.ACTIVATIONS`: "relu_squared" is relu(x)^2), applied in the up product's epilogue.
     params: hidden_size, intermediate_size, activation ("relu_squared"), activation_params ((0, 0)).
     tensors: up [I, hidden], down [hidden, I]."""
     category = "feed_forward"
@@ -96,6 +96,5 @@ class PlainMLP(Part):
     def forward(self, h, out, step):
         n = h.shape[0]
         act = step.workspace.rows("mlp_act", n, self.inter, self.ctx.dtype)
-        self.up.forward(h, act)
-        ops.activation(act, act, self.activation, self.activation_params)
+        self.up.forward_activated(h, act, self.activation, self.activation_params)
         return self.down.forward(act, out, defer=True)

@@ -1,5 +1,5 @@
 """RMSNorm: x * (mean(x^2) + eps)^-1/2 * w, eps inside the root, the weight
-multiplies (no "+1").  fastllm_py/kernels/ops.py:19-27; the fused
+multiplies (a weight stored around zero is a parameter).  fastllm_py/kernels/ops.py:19-27; the fused
 residual-add form is fastllm_py/graph_decode.py:300-324."""
 from __future__ import annotations
 
@@ -12,8 +12,11 @@ from .registry import register_part
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
-    """params: size, eps.  tensors: weight [size]."""
+    """params: size, eps, offset (0), gain (1).  tensors: weight [size].  The weight that multiplies is
+    (offset + stored) * gain: offset 1 for weights stored around zero; a gain on a norm whose result only a matrix
+    product reads is a gain on that product."""
     category = "norm"
+    takes_vectors = True                 # row vectors are added while the row is read
     takes_partial = True                 # split-K partial sums are added while the row is read
     takes_post_norm = True               # a pending sum that passes another RMSNorm first: one kernel does both
     takes_extra = True                   # two tensors pending: both are added while the row is read
@@ -22,6 +25,8 @@ class RMSNorm(Part):
         super().__init__(spec, ctx)
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
+        self.offset = float(spec.params.get("offset", 0.0))
+        self.gain = float(spec.params.get("gain", 1.0))
         self.weight = None
 
     def weight_shapes(self):
@@ -29,9 +34,11 @@ class RMSNorm(Part):
 
     def load(self, tensors):
         self.weight = tensors["weight"].contiguous()
+        if self.offset != 0.0 or self.gain != 1.0:       # formed in double and rounded once, float32 whatever is stored
+            self.weight = ((self.weight.double() + self.offset) * self.gain).float().contiguous()
 
     def apply(self, stream, out, rows=None):
-        """Norm the residual stream into `out`, adding the pending sum first.
+        """Norm the residual stream into `out`, adding the pending sum (and row vectors beside it) first.
         With `rows` (int32 indices) only those rows are normed, into out[0..m), and the
         pending sum (a tensor then: `ResidualStream.norm_into` sees to it) stays pending."""
         post = getattr(stream, "pending_norm", None)
@@ -54,12 +61,12 @@ class RMSNorm(Part):
             if not isinstance(stream.pending, torch.Tensor):         # split-K partial sums
                 if rows is not None:
                     raise RuntimeError("a gathered norm cannot take partial sums")
-                ops.add_rmsnorm_partial(stream.x, stream.pending, self.weight, out, self.eps)
-                stream.pending = None
+                ops.add_rmsnorm_partial(stream.x, stream.pending, self.weight, out, self.eps, stream.vectors)
+                stream.pending, stream.vectors = None, ()
                 return
-            ops.add_rmsnorm(stream.x, stream.pending, self.weight, out, self.eps, rows)
+            ops.add_rmsnorm(stream.x, stream.pending, self.weight, out, self.eps, rows, stream.vectors)
             if rows is None:
-                stream.pending = None
+                stream.pending, stream.vectors = None, ()
         else:
             ops.rmsnorm(stream.x, self.weight, out, self.eps, rows)
 

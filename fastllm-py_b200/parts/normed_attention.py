@@ -10,9 +10,13 @@ share, "unit" after the rotation without a weight.  The rotation (a `position` p
     s_ij = q_i . k_j * scale;    p_ij = exp(s_ij) / ([exp(sink_head) +] sum over visible j' of exp(s_ij'))
     visible: j <= i, and with `window` w: i - j < w; with `chunk` c: floor(i / c) = floor(j / c)
 
-The sink is one learned number per head in the denominator, without key or value.  With `values_from_keys` there
-is no W_v: a token's value is its key as projected, before norm and rotation.  With `head_gate` head h's result is
-multiplied by sigmoid(W_g h)_h, one number per head and token (W_g rides in the stacked product).
+The sink is one learned number per head in the denominator, without key or value; `sink` "unit" is a sink whose number
+is 0 (one more unit in the denominator).  With `values_from_keys` there is no W_v: a token's value is its key as
+projected, before norm and rotation.  With `head_gate` head h's result is multiplied by sigmoid(W_g h)_h, one number per
+head and token; with `channel_gate` the concatenated heads by sigmoid(W_g h), one per channel (in the attention kernels,
+before they round).  W_g rides in the stacked product.  With `taps` every channel of q, k and v passes a causal
+convolution over time, directly after the projection and its bias; a request's last taps - 1 projected rows are state
+beside its cache.  With `out_bias` the output projection has a bias, which a block that can adds with the pending sum.
 
 The attention itself is the sink-attention kernels' (CUDA cores in 32-bit; tensor cores for prompt portions and
 split keys for single tokens in bfloat16), which take the chunk beside the window.
@@ -21,26 +25,27 @@ from __future__ import annotations
 
 import torch
 
-from ..cache.needs import PagedKeysValues
+from ..cache.needs import FixedState, PagedKeysValues
 from ..native import ops, scratch
-from .base import Part
-from .linear import Linear
+from .base import ProjectedMixer
 from .registry import build_part, register_part
 
 
 @register_part("mixer", "normed_attention")
-class NormedAttention(Part):
+class NormedAttention(ProjectedMixer):
     """params: hidden_size, heads, kv_heads, dim, vdim, scale, norm_eps, qk_norm (None | "weighted" | "unit"),
     position (PartSpec | None), pairing ("half" | "interleaved"), q_temp (None | (coef, every)), window (None | int),
-    chunk (None | int), sink (bool), biases (bool), values_from_keys (bool), head_gate (bool).
+    chunk (None | int), sink (False | True | "unit"), biases (bool), out_bias (bool), taps (None: no convolution),
+    values_from_keys (bool), head_gate (bool), channel_gate (bool).
     tensors: q [heads * dim, hidden], k [kv_heads * dim, hidden], o [hidden, heads * vdim]; v [kv_heads * vdim, hidden]
-    unless values_from_keys; with biases q_bias, k_bias (and v_bias); for "weighted" q_norm, k_norm [dim]; with sink
-    sink [heads]; with head_gate gate [heads, hidden]."""
+    unless values_from_keys; with biases q_bias, k_bias (and v_bias); with out_bias o_bias [hidden]; for "weighted"
+    q_norm, k_norm [dim]; with taps q_conv, k_conv, v_conv [channels, taps]; with sink True sink [heads]; with a gate
+    gate [heads, hidden] or [heads * vdim, hidden]."""
     category = "mixer"
-    native_libraries = ("sink_attention",)
     SCRATCH = "sink attention splits"
-    honours_partial_side = True          # with `partial_side` set, the last product's partial sums go to the second scratch
-    partial_side = False
+    workspace_name = "normed_attention"
+    out_bias = None                      # float32 [hidden] where the output projection has one
+    defers_out_bias = False              # set by a block that adds `out_bias` itself, with the pending sum
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -55,67 +60,104 @@ class NormedAttention(Part):
         self.q_temp = tuple(p["q_temp"]) if p.get("q_temp") else None
         self.window = int(p["window"]) if p.get("window") else None
         self.chunk = int(p["chunk"]) if p.get("chunk") else None
-        self.has_sink = bool(p.get("sink", False))
+        self.sink_kind = p.get("sink", False)
         self.biases = bool(p.get("biases", False))
+        self.has_out_bias = bool(p.get("out_bias", False))
+        self.taps = int(p["taps"]) if p.get("taps") is not None else None
+        self.back = self.taps - 1 if self.taps else 0         # rows of a sequence that the convolution keeps
         self.v_from_k = bool(p.get("values_from_keys", False))
         self.gated = bool(p.get("head_gate", False))
+        self.channel_gated = bool(p.get("channel_gate", False))
         if self.heads % self.kv_heads:
             raise ValueError(f"normed_attention: {self.heads} heads are not a multiple of {self.kv_heads} kv heads")
         if self.qk_norm not in (None, "weighted", "unit"):
             raise ValueError(f"normed_attention: qk_norm {self.qk_norm!r} is none of None, 'weighted', 'unit'")
         if self.pairing not in ("half", "interleaved"):
             raise ValueError(f"normed_attention: pairing {self.pairing!r} is neither 'half' nor 'interleaved'")
+        if self.sink_kind not in (False, True, "unit"):
+            raise ValueError(f"normed_attention: sink {self.sink_kind!r} is none of False, True, 'unit'")
         if self.v_from_k and self.vdim != self.dim:
             raise ValueError("normed_attention: keys that serve as values have the values' size")
         if self.vdim > 256:
             raise ValueError(f"normed_attention: value size {self.vdim} is beyond the kernels' limit of 256")
+        if self.v_from_k and self.taps:
+            raise ValueError("normed_attention: a convolution does not go with keys that serve as values")
+        if self.gated and self.channel_gated:
+            raise ValueError("normed_attention: a gate per head or one per channel, not both")
         self.position = build_part("position", p["position"], ctx) if p.get("position") else None
         if self.position is not None and self.position.rot_dim > self.dim:
             raise ValueError("normed_attention: the position encoding turns more dimensions than a head has")
         self.q_cols, self.k_cols = self.heads * self.dim, self.kv_heads * self.dim
         self.v_cols = 0 if self.v_from_k else self.kv_heads * self.vdim
-        self.gate_cols = self.heads if self.gated else 0
-        self.proj = self.o = self.bias = self.q_w = self.k_w = self.sink = None
+        self.channels = self.q_cols + self.k_cols + self.v_cols
+        self.gate_cols = self.heads if self.gated else self.heads * self.vdim if self.channel_gated else 0
+        self.in_cols, self.out_cols = self.channels + self.gate_cols, self.heads * self.vdim
+        self.in_slots = ("q", "k") + (() if self.v_from_k else ("v",)) + (("gate",) if self.gate_cols else ())
+        self.bias = self.q_w = self.k_w = self.sink = self.conv_w = None
+
+    @property
+    def native_libraries(self):
+        return ("sink_attention", "conv_head") if self._conv_prep() else ("sink_attention",)
+
+    def _conv_prep(self) -> bool:
+        """Whether the preparation with a convolution (or a factor on the values) serves this part."""
+        return (self.taps is not None or self.joint) and not self.v_from_k
 
     def children(self):
         return [self.position] if self.position is not None else []
 
-    def cache_need(self):
+    def _cache(self):
         # behind a chunk's start nothing is seen again: at most `chunk` tokens back, like a window of that size
         reach = min(x for x in (self.window, self.chunk) if x) if (self.window or self.chunk) else None
         return PagedKeysValues(self.kv_heads, self.dim, self.vdim, reach, 0)
 
-    def weight_shapes(self):
-        shapes = {"q": (self.q_cols, self.hidden), "k": (self.k_cols, self.hidden), "o": (self.hidden, self.heads * self.vdim)}
-        if not self.v_from_k:
-            shapes["v"] = (self.v_cols, self.hidden)
+    def cache_need(self):
+        return self._cache() if self.back == 0 else None
+
+    def cache_needs(self) -> dict:
+        """With a convolution: the keys and values, and the last projected rows."""
+        if self.back == 0:
+            return {}
+        return {"kv": self._cache(), "conv": FixedState((self.back * self.channels,), "float32")}
+
+    def in_rows(self):
+        rows = {"q": self.q_cols, "k": self.k_cols, "v": self.v_cols, "gate": self.gate_cols}
+        return {slot: rows[slot] for slot in self.in_slots}
+
+    def core_shapes(self):
+        shapes = {}
+        cols = {"q": self.q_cols, "k": self.k_cols, **({} if self.v_from_k else {"v": self.v_cols})}
         if self.biases:
-            shapes.update({"q_bias": (self.q_cols,), "k_bias": (self.k_cols,)})
-            if not self.v_from_k:
-                shapes["v_bias"] = (self.v_cols,)
+            shapes.update({f"{s}_bias": (n,) for s, n in cols.items()})
+        if self.has_out_bias:
+            shapes["o_bias"] = (self.hidden,)
         if self.qk_norm == "weighted":
             shapes.update({"q_norm": (self.dim,), "k_norm": (self.dim,)})
-        if self.has_sink:
+        if self.taps:
+            shapes.update({f"{s}_conv": (n, self.taps) for s, n in cols.items()})
+        if self.sink_kind is True:
             shapes["sink"] = (self.heads,)
-        if self.gated:
-            shapes["gate"] = (self.heads, self.hidden)
         return shapes
 
-    def load(self, tensors):
-        names = ["q", "k"] + ([] if self.v_from_k else ["v"]) + (["gate"] if self.gated else [])
-        mats = [tensors[s] for s in names]
-        if len({m.dtype for m in mats}) != 1:
-            raise ValueError("normed_attention: the projections must be stored in one dtype")
-        self.proj = Linear(mats)
-        self.o = Linear([tensors["o"]])
+    def load_core(self, tensors):
+        cols = ["q", "k"] + ([] if self.v_from_k else ["v"])
+        if self.joint and (self.has_out_bias or self.v_from_k):
+            raise ValueError("normed_attention: an output bias, or keys as values, do not go with shared products")
+        if self.result_scale != 1.0 and not self._conv_prep():
+            raise ValueError("normed_attention: a factor on the result needs values of their own")
         if self.biases:
-            parts = [tensors["q_bias"], tensors["k_bias"]] + ([] if self.v_from_k else [tensors["v_bias"]])
-            self.bias = torch.cat([t.float() for t in parts]).contiguous()
+            self.bias = torch.cat([tensors[f"{s}_bias"].float() for s in cols]).contiguous()
+        if self.has_out_bias:
+            self.out_bias = tensors["o_bias"].float().clone()
         if self.qk_norm == "weighted":
             self.q_w = tensors["q_norm"].float().contiguous()
             self.k_w = tensors["k_norm"].float().contiguous()
-        if self.has_sink:
+        if self.taps:                                         # [taps, channels]: the kernel reads along the channels
+            self.conv_w = torch.cat([tensors[f"{s}_conv"].float() for s in cols]).t().contiguous()
+        if self.sink_kind is True:
             self.sink = tensors["sink"].float().contiguous()
+        elif self.sink_kind == "unit":
+            self.sink = torch.zeros(self.heads, dtype=torch.float32, device=self.ctx.device)
 
     def _tc(self) -> bool:
         return self.ctx.device.type == "cuda" and ops.sink_tc_takes(self.ctx.dtype, self.dim, self.vdim)
@@ -126,10 +168,7 @@ class NormedAttention(Part):
         return [ops.sink_tc_library(self.dim, self.vdim)] if self._tc() else []
 
     def reserve(self, limits):
-        if self.proj is not None:
-            self.proj.reserve(self.ctx.dtype, limits.max_tokens)
-        if self.o is not None:
-            self.o.reserve(self.ctx.dtype, limits.max_tokens, side=self.partial_side)
+        super().reserve(limits)
         if self._tc():
             from ..native.build import load_library
             load_library(*ops.sink_tc_library(self.dim, self.vdim))        # built now, not inside the first step
@@ -163,24 +202,31 @@ class NormedAttention(Part):
     def _partials(self, n_tokens: int, n_splits: int):
         return scratch.get(self.ctx.device, self.SCRATCH, n_tokens * self.heads * n_splits * (self.vdim + 2))
 
-    def forward(self, h, out, step, cache):
-        n = h.shape[0]
-        dt = self.ctx.dtype
-        ws = step.workspace
-        cols = self.q_cols + self.k_cols + self.v_cols + self.gate_cols
-        proj = ws.rows("normed_attention_proj", n, cols, dt)
-        self.proj.forward(h, proj)
-        q = ws.rows("normed_attention_q", n, self.q_cols, dt)
-        if self.position is not None:
-            cos, sin = self.position.tables()
-            rot = self.position.rot_dim
+    def _prepare(self, proj, q, step, cache, tail):
+        """Queries to `q`, keys and values to the tokens' cache rows."""
+        cos, sin = self.position.tables() if self.position is not None else (None, None)
+        rot = self.position.rot_dim if self.position is not None else 0
+        mode = {None: 0, "weighted": 1, "unit": 2}[self.qk_norm]
+        interleaved = self.pairing == "interleaved"
+        if self._conv_prep():
+            ops.conv_head_prep(proj, self.bias, self.conv_w, tail, self.q_w, self.k_w, mode, self.norm_eps, rot, interleaved, cos,
+                               sin, step, self.q_temp, self.result_scale, q, self.heads, self.kv_heads, self.dim, self.vdim,
+                               cache.slots, cache.tensor, cache.page_size)
         else:
-            cos = sin = None
-            rot = 0
-        ops.head_prep(proj, self.bias, self.q_w, self.k_w, {None: 0, "weighted": 1, "unit": 2}[self.qk_norm], self.norm_eps,
-                      rot, self.pairing == "interleaved", cos, sin, step.positions, self.q_temp, self.v_from_k, q,
-                      self.heads, self.kv_heads, self.dim, self.vdim, cache.slots, cache.tensor, cache.page_size)
-        ctx = ws.rows("normed_attention_ctx", n, self.heads * self.vdim, dt)
+            ops.head_prep(proj, self.bias, self.q_w, self.k_w, mode, self.norm_eps, rot, interleaved, cos, sin, step.positions,
+                          self.q_temp, self.v_from_k, q, self.heads, self.kv_heads, self.dim, self.vdim, cache.slots,
+                          cache.tensor, cache.page_size)
+
+    def core(self, proj, ctx, step, cache):
+        n = proj.shape[0]
+        dt = self.ctx.dtype
+        tail = None
+        if self.back:
+            tail, cache = cache["conv"].tensor, cache["kv"]
+        q = step.workspace.rows("normed_attention_q", n, self.q_cols, dt)
+        self._prepare(proj, q, step, cache, tail)
+        gate = proj[:, self.channels:self.channels + self.gate_cols] if self.gate_cols else None
+        channel_gate = gate if self.channel_gated else None
         tc = self._tc()
         # (where only the CUDA-core kernel serves prompt rows, a mixed step gives it every row)
         single = step.n_decode_tokens if self._splits_single_tokens() and (tc or step.n_decode_tokens == n) else 0
@@ -191,17 +237,25 @@ class NormedAttention(Part):
             ops.sink_decode(q, ctx, cache.tensor, cache.block_table, step.tok_req, step.positions, step.decode_tokens,
                             self._partials(single, n_splits), n_splits, kept_splits, self.heads, self.kv_heads,
                             self.dim, self.vdim, self.window, 0, self.scale, None, None, None, self.sink, cache.page_size,
-                            chunk=self.chunk)
+                            chunk=self.chunk, gate=channel_gate)
         if single == n:
             pass
         elif tc:
             ops.sink_attention_tc(q, ctx, cache.tensor, cache.block_table, step, self.heads, self.kv_heads, self.dim,
                                   self.vdim, self.window, 0, self.scale, None, None, None, self.sink, cache.page_size,
-                                  include_single=not single, chunk=self.chunk)
+                                  include_single=not single, chunk=self.chunk, gate=channel_gate)
         else:
             ops.sink_attention_simt(q, ctx, cache.tensor, cache.block_table, step.tok_req, step.positions, self.heads,
                                     self.kv_heads, self.dim, self.vdim, self.window, 0, self.scale, None, None, None,
-                                    self.sink, cache.page_size, chunk=self.chunk)
+                                    self.sink, cache.page_size, chunk=self.chunk, gate=channel_gate)
         if self.gated:
-            ops.head_gate(ctx, proj[:, self.q_cols + self.k_cols + self.v_cols:], self.heads, self.vdim)
-        return self.o.forward(ctx, out, defer=True, side=self.partial_side)
+            ops.head_gate(ctx, gate, self.heads, self.vdim)
+
+    def forward(self, h, out, step, cache):
+        left = super().forward(h, out, step, cache)
+        if self.out_bias is None or self.defers_out_bias:
+            return left
+        if left is not None:
+            left.reduce_into(out)
+        ops.add_bias(out, self.out_bias)
+        return None

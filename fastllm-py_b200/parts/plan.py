@@ -45,9 +45,11 @@ class LayerRun:
     `layer` indexes ModelPlan.layers; a layer may be named in several runs.
     `cache` names the cache (or state) this run uses: by default a cache of its
     own; the number of an earlier run to read that run's cache instead, in which
-    case this run writes nothing to it."""
+    case this run writes nothing to it.  `vector`: the row of ModelPlan.vectors that is
+    added to the residual stream before this run (None: none)."""
     layer: int
     cache: int | None = None
+    vector: int | None = None
 
 
 @dataclass
@@ -60,6 +62,7 @@ class ModelPlan:
     order: list
     final_norm: PartSpec
     head: PartSpec
+    vectors: PartSpec | None = None      # a table [n, hidden] of vectors that runs start with (LayerRun.vector)
     ignorable: tuple = ()      # fnmatch patterns of checkpoint names that may be present and are not used
 
     def validate(self):
@@ -67,6 +70,8 @@ class ModelPlan:
         for i, run in enumerate(self.order):
             if not 0 <= run.layer < n:
                 raise ValueError(f"order[{i}] names layer {run.layer}, plan has {n} layers")
+            if run.vector is not None and self.vectors is None:
+                raise ValueError(f"order[{i}] starts with vector {run.vector}, but the plan has no vectors")
             if run.cache is not None:
                 if not 0 <= run.cache < i:
                     raise ValueError(f"order[{i}] reads the cache of run {run.cache}, "
@@ -90,6 +95,8 @@ class ModelPlan:
                     visit(v)
 
         visit(self.embedding)
+        if self.vectors is not None:
+            visit(self.vectors)
         for layer in self.layers:
             for name in layer.tensors.values():
                 if name not in seen:
