@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--workload decode|serve|67b|tables|hybrid|lasonex|sakusun|saberax]
+                    [--workload decode|serve|67b|tables|hybrid|lasonex|sakusun|saberax|lufozen]
 
 The default run is the DeepSeek-LLM-7B sized model (30 layers, hidden 4096,
 32 heads, head size 128, feed-forward 11008, vocabulary 102400) with random
@@ -48,6 +48,8 @@ Two more workloads, each printing one line of its own:
                      input convolution) at the same two widths, beside the Tigitar hybrid and the dense decoder
   --workload saberax the Saberax design (attention beside a gated recurrence or gated linear attention in pre-norm layers,
                      chunked attention, experts without a gate) beside the Lasonex design and the dense decoder
+  --workload lufozen the Lufozen design (attention behind a short convolution, gated linear attention, attention beside a
+                     state-space recurrence, layers that run twice) beside the Saberax design and the dense decoder
   --workload 67b     deepseek-llm-67b size (95 layers, hidden 8192, 64 heads over 8 key/value
              heads; 135 GB of weights on the one GPU): a 2048-token prompt step and decode
              steps at batch 1, 8 and 16 with 4000-token contexts, with their roofline fractions.
@@ -1104,6 +1106,151 @@ def run_saberax(args, warmup):
     return 0
 
 
+LUFOZEN_SIZES = {
+    # pre-norm layers at the widths of HYBRID_SIZES: six layers of which two run twice, so eight runs, as many as the other
+    # designs have layers.  The unit without a gate is as large as their gated ones.  The Saberax design (attention beside a
+    # recurrent mixer in pre-norm layers) and the dense Llama-style decoder of the same width and depth are timed beside it
+    "w2048": dict(width=2048, vocab=32256, attention=dict(heads=16, kv_heads=4, dim=128, vdim=128, conv=4),
+                  linear=dict(heads=16, dim=64, vdim=128, tau=16.0),
+                  state_space=dict(heads=64, vdim=64, state=128, groups=2, conv=4), ff=8192, runs=8),
+    "w4096": dict(width=4096, vocab=32256, attention=dict(heads=32, kv_heads=8, dim=128, vdim=128, conv=4),
+                  linear=dict(heads=32, dim=64, vdim=128, tau=16.0),
+                  state_space=dict(heads=128, vdim=64, state=128, groups=4, conv=4), ff=16384, runs=4),
+}
+
+
+def lufozen_config(size):
+    from fastllm_py_b200.config.lufozen import (AttentionConfig, DenseConfig, GatedLinearAttentionConfig, LoopConfig,
+                                                LufozenConfig, LufozenLayerConfig, PairConfig, RotationConfig, StateSpaceConfig)
+
+    z = LUFOZEN_SIZES[size]
+    a, g, r = z["attention"], z["linear"], z["state_space"]
+    sizes = (a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["dim"] ** -0.5)
+    rot = RotationConfig(500000.0, a["dim"], (8.0, 8192.0, 1.0, 4.0))
+    lone = ("attention", AttentionConfig(*sizes, rot, a["conv"]))
+    pair = ("parallel", PairConfig(AttentionConfig(*sizes, rot),
+                                   StateSpaceConfig(r["heads"], r["vdim"], r["state"], r["groups"], r["conv"], r["groups"]), 0.6, 0.5))
+    linear = ("gla", GatedLinearAttentionConfig(g["heads"], g["dim"], g["vdim"], g["tau"]))
+    if z["runs"] == 8:
+        kinds, loop = [lone, pair, linear, pair, lone, linear], LoopConfig(1, 3, 2)
+    else:
+        kinds, loop = [lone, pair, linear], LoopConfig(1, 2, 2)
+    layers = tuple(LufozenLayerConfig(*k, DenseConfig(z["ff"])) for k in kinds)
+    return LufozenConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, embedding_scale=16.0, bigram_buckets=65521,
+                         bigram_mul_prev=31, bigram_mul_cur=7, logit_scale=0.5, loop=loop, layers=layers)
+
+
+def _lufozen_layer_sizes(layer, w):
+    """(weight elements a token's mixer products touch, state floats per request, [attention config], [(dim, vdim of a
+    recurrence's state per head, heads)])."""
+    from fastllm_py_b200.config.lufozen import AttentionConfig, GatedLinearAttentionConfig
+
+    def attention(m):
+        lone = m.conv is not None
+        return w * (m.heads * m.dim + m.kv_heads * (m.dim + m.vdim) + m.heads * m.vdim * (2 if lone else 1))
+
+    m = layer.mixer
+    if isinstance(m, AttentionConfig):
+        return attention(m), (m.conv - 1) * (m.heads * m.dim + m.kv_heads * (m.dim + m.vdim)), [m], []
+    if isinstance(m, GatedLinearAttentionConfig):
+        weights = w * (2 * m.heads * m.dim + 3 * m.heads * m.vdim + m.rank) + m.heads * m.dim * m.rank
+        return weights, m.heads * m.dim * m.vdim, [], [(m.dim, m.vdim, m.heads)]
+    r = m.right
+    inner, channels = r.heads * r.vdim, r.heads * r.vdim + 2 * r.groups * r.state
+    weights = attention(m.left) + w * (2 * inner + channels + r.heads)
+    return weights, inner * r.state + (r.conv - 1) * channels, [m.left], [(r.state, r.vdim, r.heads)]
+
+
+def lufozen_decode_bytes(cfg, batch, context):
+    """Bytes a decode step has to move: every run's weights in bfloat16 (a layer that runs twice is read twice), every
+    request's states read and written in float, and the cache rows that the attentions see."""
+    w, total = cfg.width, 0
+    for i, _ in cfg.running_order():
+        layer = cfg.layers[i]
+        weights, state, attentions, _ = _lufozen_layer_sizes(layer, w)
+        total += 2 * weights + batch * 2 * 4 * state
+        for m in attentions:
+            total += batch * context * m.kv_heads * (m.dim + m.vdim) * 2
+        if layer.mlp is not None:
+            total += 2 * 2 * w * layer.mlp.ff
+    return total + 2 * w * cfg.vocab + 2 * batch * w * 2
+
+
+def lufozen_prefill_flops(cfg, tokens):
+    """Matrix-product FLOPs of a prompt step (projections, feed-forwards, attention, head) and 4 per state element and token
+    of the two recurrences."""
+    w, total = cfg.width, 0
+    for i, _ in cfg.running_order():
+        layer = cfg.layers[i]
+        weights, _, attentions, states = _lufozen_layer_sizes(layer, w)
+        total += 2 * tokens * weights
+        for dim, vdim, heads in states:
+            total += tokens * heads * 4 * dim * vdim
+        for m in attentions:
+            total += 2 * m.heads * (tokens * (tokens + 1) // 2) * (m.dim + m.vdim)
+        if layer.mlp is not None:
+            total += 2 * tokens * 2 * w * layer.mlp.ff
+    return total + 2 * w * cfg.vocab
+
+
+def run_lufozen(args, warmup):
+    """The Lufozen design beside the Saberax design (the closest model: attention beside a recurrent mixer in pre-norm layers)
+    and the dense decoder of equal width and number of layer runs, one JSON line: prompt steps of 512 and 2048 tokens and
+    decode steps at batch 1 and 8 over 2048-token contexts, with each model's fraction of its own roofline (measured tensor
+    peak for prompts, measured copy bandwidth for decode steps)."""
+    from fastllm_py_b200 import LlamaConfig, Model
+
+    pk = peaks()
+    steps = max(8, min(args.steps, 32))
+    out = {}
+    sampler = ClockSampler().start()
+    sampler.__enter__()
+    for size in (args.size.split(",") if args.size else list(LUFOZEN_SIZES)):
+        z, hz = LUFOZEN_SIZES[size], HYBRID_SIZES[size]
+        llama = LlamaConfig(architecture="LlamaForCausalLM", rope_scaling=None, tie_word_embeddings=False,
+                            num_layers=z["runs"], hidden_size=z["width"], vocab_size=z["vocab"], rope_theta=10000.0,
+                            rms_norm_eps=1e-6, max_position_embeddings=4096, **hz["llama"])
+        models = [("lufozen", lufozen_config(size), lufozen_prefill_flops, lufozen_decode_bytes),
+                  ("saberax", saberax_config(size), saberax_prefill_flops, saberax_decode_bytes),
+                  ("dense", llama, prefill_flops, decode_bytes)]
+        res = {}
+        for name, cfg, flops_of, bytes_of in models:
+            if args.only and name not in args.only.split(","):
+                continue
+            model = Model.from_config(cfg, seed=0, dtype="bfloat16", page_size=16, max_tokens=8 * (CONTEXT + 256),
+                                      max_requests=8, max_batched_tokens=2048, max_model_len=4096,
+                                      cuda_graph=not args.no_graph)
+            r = {"prompt_step": {}, "decode": {}}
+            for t in (512, 2048):
+                ms, _ = time_prefill(model, t, 8, 3)
+                r["prompt_step"][str(t)] = {"ms": round(ms, 3), "value": round(t * 1000.0 / ms, 1),
+                                            "frac": round(flops_of(cfg, t) / (ms * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
+            for b in (1, 8):
+                v, ms, launches, _ = time_decode(model, b, steps, warmup, CONTEXT)
+                ctx = CONTEXT + warmup + (steps + 1) / 2
+                r["decode"][f"{b}x{CONTEXT}"] = {"ms_per_step": round(ms, 3), "value": round(v, 1),
+                                                 "launches_per_step": launches // steps,
+                                                 "frac": round(bytes_of(cfg, b, ctx) / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+            res[name] = r
+            del model
+            import gc
+
+            import torch
+            gc.collect()
+            torch.cuda.empty_cache()
+        out[size] = res
+    sampler.__exit__()
+    print(json.dumps({
+        "metric": "prompt and decode steps of the Lufozen design beside the Saberax design and the dense decoder "
+                  "of equal size, bf16",
+        "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours", "steps": steps, "warmup": warmup,
+        "config": {"sizes": {k: dict(LUFOZEN_SIZES[k]) for k in out}, "page_size": 16,
+                   "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"],
+                   "cuda_graph": not args.no_graph},
+        "sizes": out, "clocks": sampler.summary()}))
+    return 0
+
+
 def reference_cpu_path(ref_root, layers=1, context=256, decode_tokens=8):
     """fastllm-py's own NumPy model code (its CPU device, float32) timed at DeepSeek-LLM-7B layer
     sizes: `layers` of the 30 layers, one sequence (that path has no batch), a `context`-token
@@ -1240,11 +1387,11 @@ def main():
                     help="run fewer layers of the same sizes (the line names both numbers)")
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and the prefill")
     ap.add_argument("--no-graph", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "67b", "tables", "hybrid", "lasonex", "sakusun", "saberax"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "67b", "tables", "hybrid", "lasonex", "sakusun", "saberax", "lufozen"],
                     help="decode: the headline line (DeepSeek-LLM-7B size); serve: continuous batching at "
                          "deepseek-coder-1.3b size; 67b: prompt and decode steps at deepseek-llm-67b size")
-    ap.add_argument("--size", default="", help="hybrid, lasonex, sakusun, saberax: which sizes (w2048,w4096; default both)")
-    ap.add_argument("--only", default="", help="lasonex, sakusun, saberax: which of the models timed side by side (the design itself, hybrid or lasonex, dense)")
+    ap.add_argument("--size", default="", help="hybrid, lasonex, sakusun, saberax, lufozen: which sizes (w2048,w4096; default both)")
+    ap.add_argument("--only", default="", help="lasonex, sakusun, saberax, lufozen: which of the models timed side by side (the design itself, hybrid, lasonex or saberax, dense)")
     ap.add_argument("--requests", type=int, default=128, help="serve: how many requests")
     ap.add_argument("--rate", type=float, default=16.0, help="serve: mean arrivals a second")
     ap.add_argument("--reference-cpu", action="store_true",
@@ -1269,6 +1416,8 @@ def main():
         return run_sakusun(args, warmup)
     if args.workload == "saberax":
         return run_saberax(args, warmup)
+    if args.workload == "lufozen":
+        return run_lufozen(args, warmup)
     if args.workload == "hybrid":
         return run_hybrid(args, warmup)
     args.layers = args.layers or MODEL_7B["num_layers"]

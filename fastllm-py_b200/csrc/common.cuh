@@ -124,8 +124,8 @@ static inline bool fl_pdl_enabled() {
 }
 
 template <typename... KArgs, typename... Args>
-static inline int fl_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
-                            cudaStream_t stream, Args... args) {
+static inline int fl_launch_as(bool overlap, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                               cudaStream_t stream, Args... args) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
@@ -135,6 +135,20 @@ static inline int fl_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
-    cfg.numAttrs = fl_pdl_enabled() ? 1 : 0;
+    cfg.numAttrs = overlap && fl_pdl_enabled() ? 1 : 0;
     return (int)cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+}
+
+template <typename... KArgs, typename... Args>
+static inline int fl_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                            cudaStream_t stream, Args... args) {
+    return fl_launch_as(true, kernel, grid, block, smem, stream, args...);
+}
+
+// In plain stream order, for long kernels of no more CTAs than SMs: brought in while the predecessor still runs, several
+// of their CTAs end up on the first SMs that have room, and the kernel takes as long as the fullest SM.
+template <typename... KArgs, typename... Args>
+static inline int fl_launch_spread(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                                   cudaStream_t stream, Args... args) {
+    return fl_launch_as(false, kernel, grid, block, smem, stream, args...);
 }

@@ -11,9 +11,8 @@
 //
 // A request's last taps - 1 rows u (bias included) are its state, [taps - 1][channels] float, oldest first.
 //
-//   conv_head_prep   one warp a head and `run` consecutive tokens: a lane holds the pairs that rotate together in
-//                    registers, and of each channel a window of the last taps - 1 inputs, so that a row is read once.  A
-//                    request that brings a single token has its state moved on here, by the lane that owns the channel
+//   conv_head_prep   one warp a head and a few consecutive tokens: a lane holds the pairs that rotate together in
+//                    registers, for these tokens and the taps - 1 rows before them.  A request that brings a single token has its state moved on here, by the lane that owns the channel
 //   conv_head_tail   the new state of requests that bring several tokens (after every reader of the old one)
 //
 // All arithmetic is float; every sum's order depends on the channel alone.
@@ -21,28 +20,146 @@
 
 #define CH_WARPS 4               // warps of a block: neighbouring heads of the same tokens
 
-// Two neighbouring channels at once where they lie on an even column.
-__device__ __forceinline__ float2 ch_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
-__device__ __forceinline__ float2 ch_pair(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
-__device__ __forceinline__ void ch_put_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-__device__ __forceinline__ void ch_put_pair(bf16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+// N consecutive elements (N 1, 2 or a multiple of 4) from or to an address that is aligned for it.
+template <int N> __device__ __forceinline__ void ch_get(const float* p, float* v) {
+    if constexpr (N == 1) {
+        v[0] = p[0];
+    } else if constexpr (N == 2) {
+        const float2 q = *reinterpret_cast<const float2*>(p);
+        v[0] = q.x; v[1] = q.y;
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+            const float4 q = *reinterpret_cast<const float4*>(p + i);
+            v[i] = q.x; v[i + 1] = q.y; v[i + 2] = q.z; v[i + 3] = q.w;
+        }
+    }
+}
+template <int N> __device__ __forceinline__ void ch_get(const bf16* p, float* v) {
+    if constexpr (N == 1) {
+        v[0] = __bfloat162float(p[0]);
+    } else if constexpr (N == 2) {
+        const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        v[0] = q.x; v[1] = q.y;
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+            const uint2 raw = *reinterpret_cast<const uint2*>(p + i);
+            const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            v[i] = a.x; v[i + 1] = a.y; v[i + 2] = b.x; v[i + 3] = b.y;
+        }
+    }
+}
+template <int N> __device__ __forceinline__ void ch_put(float* p, const float* v) {
+    if constexpr (N == 1) {
+        p[0] = v[0];
+    } else if constexpr (N == 2) {
+        *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    }
+}
+template <int N> __device__ __forceinline__ void ch_put(bf16* p, const float* v) {
+    if constexpr (N == 1) {
+        p[0] = __float2bfloat16_rn(v[0]);
+    } else if constexpr (N == 2) {
+        *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v[i], v[i + 1]), b = __floats2bfloat162_rn(v[i + 2], v[i + 3]);
+            uint2 q;
+            q.x = *reinterpret_cast<const uint32_t*>(&a);
+            q.y = *reinterpret_cast<const uint32_t*>(&b);
+            *reinterpret_cast<uint2*>(p + i) = q;
+        }
+    }
+}
+
+// How a lane's 2 PPL elements lie in a head, pair after pair: CH_RUN: consecutive channels from `first` on (pairs of
+// neighbours); CH_HALVES: PPL channels from `first` on paired with those `half` further; CH_ANY: pairs found one by one.
+enum { CH_RUN = 0, CH_HALVES = 1, CH_ANY = 2 };
+template <int PPL> struct ChLane {
+    int mode, size, turn, half, slot0;                                // slot0: the lane's first pair
+    bool side;
+    __device__ __forceinline__ int channel(int e) const {             // of element e; -1 where there is none
+        const int s = slot0 + (e >> 1);
+        int c;
+        if (side) c = 2 * s + (e & 1);
+        else if (s < half) c = s + (e & 1) * half;
+        else c = turn + 2 * (s - half) + (e & 1);
+        return c < size ? c : -1;
+    }
+    template <typename T> __device__ __forceinline__ void get(const T* p, float* v, float missing = 0.0f) const {
+        if (mode == CH_RUN) {
+            if (2 * slot0 < size) { ch_get<2 * PPL>(p + 2 * slot0, v); return; }
+        } else if (mode == CH_HALVES) {
+            if (slot0 < half) {
+                float a[PPL], b[PPL];
+                ch_get<PPL>(p + slot0, a);
+                ch_get<PPL>(p + half + slot0, b);
+#pragma unroll
+                for (int i = 0; i < PPL; ++i) { v[2 * i] = a[i]; v[2 * i + 1] = b[i]; }
+                return;
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < 2 * PPL; ++e) {
+                const int c = channel(e);
+                v[e] = c >= 0 ? to_f32<T>(p[c]) : missing;
+            }
+            return;
+        }
+#pragma unroll
+        for (int e = 0; e < 2 * PPL; ++e) v[e] = missing;
+    }
+    template <typename T> __device__ __forceinline__ void put(T* p, const float* v) const {
+        if (mode == CH_RUN) {
+            if (2 * slot0 < size) ch_put<2 * PPL>(p + 2 * slot0, v);
+        } else if (mode == CH_HALVES) {
+            if (slot0 < half) {
+                float a[PPL], b[PPL];
+#pragma unroll
+                for (int i = 0; i < PPL; ++i) { a[i] = v[2 * i]; b[i] = v[2 * i + 1]; }
+                ch_put<PPL>(p + slot0, a);
+                ch_put<PPL>(p + half + slot0, b);
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < 2 * PPL; ++e) {
+                const int c = channel(e);
+                if (c >= 0) p[c] = from_f32<T>(v[e]);
+            }
+        }
+    }
+};
+
+template <typename T> __device__ __forceinline__ float ch_rms(float ss, int dim, float eps) {
+    const float x = ss / (float)dim + eps;
+    if constexpr (sizeof(T) == 2) return rsqrtf(x);                   // (two units in the last place of float)
+    else return 1.0f / sqrtf(x);
+}
 
 struct ChRows {                  // the step's tables
     const int *positions, *tok_req, *req_start, *req_ctx, *req_qlen, *req_slot, *slots;
 };
 
-// PPL: pairs a lane holds (head sizes up to 64 PPL); TAPS: the window's length, the layer's taps rounded up; 0: any number
-// of taps, every earlier input read again for every token.
-template <typename T, int PPL, int TAPS>
+// PPL: pairs a lane holds (head sizes up to 64 PPL); TAPS: the layer's taps rounded up (1: one tap or no convolution), 0:
+// any number, every earlier input read again for every token; RUN: consecutive tokens of a warp, whose rows (and the
+// TAPS - 1 before them) are all asked for at once.
+template <typename T, int PPL, int TAPS, int RUN>
 __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
     const T* __restrict__ proj, long ld, const float* __restrict__ bias, const float* __restrict__ conv_w, int taps,
     float* __restrict__ tail, long tail_stride, const float* __restrict__ q_w, const float* __restrict__ k_w, int norm_mode,
     float eps, int rot, int interleaved, const float* __restrict__ cos_t, const float* __restrict__ sin_t, float temp_coef,
     int temp_every, float v_scale, const ChRows rows, T* __restrict__ q_out, long q_ld, int heads, int kv_heads, int dim,
-    int vdim, T* __restrict__ cache, long page_stride, int page_size, int n_tokens, int run, int pairs_ok) {
+    int vdim, T* __restrict__ cache, long page_stride, int page_size, int page_shift, int n_tokens, int aligned) {
     pdl_wait();
     pdl_trigger();
-    constexpr int WIN = TAPS > 1 ? TAPS - 1 : 1;
+    constexpr int HIST = TAPS > 1 ? TAPS - 1 : 0;                     // rows before the run that its tokens may need
+    constexpr int KEPT = TAPS > 0 ? TAPS : 1, E = 2 * PPL;
     const int lane = threadIdx.x & 31;
     const int unit = blockIdx.y * CH_WARPS + (threadIdx.x >> 5);
     if (unit >= heads + 2 * kv_heads) return;
@@ -53,203 +170,194 @@ __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
     const int channels = (heads + kv_heads) * dim + kv_heads * vdim;
     const int turn = is_v ? 0 : rot, half = turn / 2;
     const bool side = interleaved || turn == 0;                       // a pair's two channels are neighbours
+    ChLane<PPL> at;
+    at.size = size; at.turn = turn; at.half = half; at.slot0 = PPL * lane; at.side = side;
+    at.mode = aligned && side && size % E == 0 ? CH_RUN : aligned && !side && turn == size && half % PPL == 0 ? CH_HALVES : CH_ANY;
+    const int t0 = blockIdx.x * RUN;
 
-    int ca[PPL], cb[PPL];                                             // the pair's channels within the head (-1: none)
-    constexpr int KEPT = TAPS > 0 ? TAPS : 1;
-    float ba[PPL], bb[PPL], ga[PPL], gb[PPL], wa[PPL][KEPT], wb[PPL][KEPT];
-    const float* gain = is_v || norm_mode != 1 ? nullptr : (is_q ? q_w : k_w);
+    // everything that does not depend on something else is asked for first
+    float x[HIST + RUN][E];                                           // as projected, without the bias
+    {
+        const T* row = proj + (long)(t0 - HIST) * ld + col0;
 #pragma unroll
-    for (int p = 0; p < PPL; ++p) {
-        const int s = lane + 32 * p;
-        if (side) {
-            ca[p] = 2 * s;
-            cb[p] = 2 * s + 1;
-        } else if (s < half) {
-            ca[p] = s;
-            cb[p] = s + half;
-        } else {
-            ca[p] = turn + 2 * (s - half);
-            cb[p] = ca[p] + 1;
+        for (int i = 0; i < HIST + RUN; ++i, row += ld) {
+            const int t = t0 + i - HIST;
+            if (t >= 0 && t < n_tokens) at.get(row, x[i]);
+            else
+#pragma unroll
+                for (int e = 0; e < E; ++e) x[i][e] = 0.0f;
         }
-        if (ca[p] >= size) ca[p] = -1;
-        if (cb[p] >= size) cb[p] = -1;
-        const int a = col0 + max(ca[p], 0), b = col0 + max(cb[p], 0);
-        ba[p] = bias != nullptr && ca[p] >= 0 ? bias[a] : 0.0f;
-        bb[p] = bias != nullptr && cb[p] >= 0 ? bias[b] : 0.0f;
-        ga[p] = gain != nullptr && ca[p] >= 0 ? gain[max(ca[p], 0)] : 1.0f;
-        gb[p] = gain != nullptr && cb[p] >= 0 ? gain[max(cb[p], 0)] : 1.0f;
-        if (TAPS > 0 && conv_w != nullptr) {
+    }
+    // what the step's tables say of the run's tokens, a token a lane
+    int l_pos = 0, l_slot = 0, l_local = 0, l_row = 0, l_single = 0;  // local: tokens of the request in this step before it
+    if (lane < RUN && t0 + lane < n_tokens) {
+        l_pos = rows.positions[t0 + lane];
+        l_slot = rows.slots[t0 + lane];
+        if (TAPS != 1) {
+            const int r = rows.tok_req[t0 + lane];
+            l_local = t0 + lane - rows.req_start[r];
+            l_row = rows.req_slot[r];
+            l_single = rows.req_qlen[r] == 1;
+        }
+    }
+    float b[E], gain[E], w[KEPT][E];
+    const float* gain_p = is_v || norm_mode != 1 ? nullptr : (is_q ? q_w : k_w);
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) {                          // tap j of the window is tap j - (TAPS - taps) of w
-                const int k = j - (TAPS - taps);
-                wa[p][j] = k >= 0 && ca[p] >= 0 ? conv_w[(long)k * channels + a] : 0.0f;
-                wb[p][j] = k >= 0 && cb[p] >= 0 ? conv_w[(long)k * channels + b] : 0.0f;
+    for (int e = 0; e < E; ++e) { b[e] = 0.0f; gain[e] = 1.0f; }
+    if (bias != nullptr) at.get(bias + col0, b);
+    if (gain_p != nullptr) at.get(gain_p, gain, 1.0f);
+    if (TAPS > 0 && conv_w != nullptr) {
+#pragma unroll
+        for (int j = 0; j < KEPT; ++j) {                              // tap j of the window is tap j - (KEPT - taps) of w
+            const int k = j - (KEPT - taps);
+            if (k >= 0) at.get(conv_w + (long)k * channels + col0, w[j]);
+            else
+#pragma unroll
+                for (int e = 0; e < E; ++e) w[j][e] = 0.0f;
+        }
+    }
+    int pos[RUN];
+    float cosv[RUN][PPL], sinv[RUN][PPL];
+#pragma unroll
+    for (int u = 0; u < RUN; ++u) {
+        pos[u] = __shfl_sync(0xffffffffu, l_pos, u);
+        const long line = (long)pos[u] * half + at.slot0;
+        if (at.slot0 + PPL <= half && half % PPL == 0) {
+            ch_get<PPL>(cos_t + line, cosv[u]);
+            ch_get<PPL>(sin_t + line, sinv[u]);
+        } else {
+#pragma unroll
+            for (int p = 0; p < PPL; ++p) {
+                cosv[u][p] = at.slot0 + p < half ? cos_t[line + p] : 1.0f;
+                sinv[u][p] = at.slot0 + p < half ? sin_t[line + p] : 0.0f;
             }
         }
     }
-    const bool vec = pairs_ok && side;
-    auto load_u = [&](int t, int p, float& a, float& b) {
-        const T* row = proj + (long)t * ld + col0;
-        if (vec) {
-            a = b = 0.0f;
-            if (ca[p] >= 0) {
-                const float2 v = ch_pair(row + ca[p]);                // (sizes are even where vec holds: both exist)
-                a = v.x + ba[p];
-                b = v.y + bb[p];
-            }
-        } else {
-            a = ca[p] >= 0 ? to_f32<T>(row[ca[p]]) + ba[p] : 0.0f;
-            b = cb[p] >= 0 ? to_f32<T>(row[cb[p]]) + bb[p] : 0.0f;
-        }
-    };
 
-    float xa[WIN][PPL], xb[WIN][PPL];                                 // inputs of the positions before, oldest first
-    const int t0 = blockIdx.x * run, t1 = min(n_tokens, t0 + run);
-    int known = -1;                                                   // the request the window belongs to
-    for (int t = t0; t < t1; ++t) {
-        const int r = rows.tok_req[t];
-        const int pos = rows.positions[t];
-        float ya[PPL], yb[PPL];
 #pragma unroll
-        for (int p = 0; p < PPL; ++p) load_u(t, p, ya[p], yb[p]);
+    for (int u = 0; u < RUN; ++u) {
+        const int t = t0 + u;
+        const int slot = __shfl_sync(0xffffffffu, l_slot, u);
+        float y[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) y[e] = x[HIST + u][e] + b[e];
         if constexpr (TAPS > 1) {
-            float* mine = tail + (long)rows.req_slot[r] * tail_stride + col0;
-            if (r != known) {
-                known = r;
-                const int ctx = rows.req_ctx[r];
+            // input `back` positions behind: from the step's rows, from the kept rows, or zero before the sequence's start
+            const int local = __shfl_sync(0xffffffffu, l_local, u), state_row = __shfl_sync(0xffffffffu, l_row, u);
+            const int single = __shfl_sync(0xffffffffu, l_single, u);
+            float* mine = tail + (long)state_row * tail_stride + col0;
+            float h[HIST][E];                                         // oldest first
 #pragma unroll
-                for (int k = 0; k < WIN; ++k) {
-                    const int back = WIN - k, at = pos - back;        // window entry k holds position pos - WIN + k
+            for (int j = 0; j < HIST; ++j) {
 #pragma unroll
-                    for (int p = 0; p < PPL; ++p) {
-                        xa[k][p] = xb[k][p] = 0.0f;
-                        if (at < 0 || back > taps - 1) continue;
-                        if (at >= ctx) {
-                            load_u(t - back, p, xa[k][p], xb[k][p]);
-                        } else {
-                            const float* kept = mine + (long)(at - ctx + taps - 1) * channels;
-                            if (ca[p] >= 0) xa[k][p] = kept[ca[p]];
-                            if (cb[p] >= 0) xb[k][p] = kept[cb[p]];
-                        }
+                for (int e = 0; e < E; ++e) h[j][e] = x[u + j][e] + b[e];
+            }
+            if (local < HIST && t < n_tokens) {                       // the same for the whole warp
+#pragma unroll
+                for (int j = 0; j < HIST; ++j) {
+                    const int back = HIST - j;
+                    if (local >= back) continue;
+                    if (pos[u] >= back && back <= taps - 1) {
+                        at.get(mine + (long)(local - back + taps - 1) * channels, h[j]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < E; ++e) h[j][e] = 0.0f;
                     }
                 }
             }
-            const bool single = rows.req_qlen[r] == 1;
+            float keep[E];
 #pragma unroll
-            for (int p = 0; p < PPL; ++p) {
-                const float na = ya[p], nb = yb[p];
-                float sa = 0.0f, sb = 0.0f;
+            for (int e = 0; e < E; ++e) {
+                keep[e] = y[e];
+                float sum = 0.0f;
 #pragma unroll
-                for (int j = 0; j < WIN; ++j) {
-                    sa = fmaf(wa[p][j], xa[j][p], sa);
-                    sb = fmaf(wb[p][j], xb[j][p], sb);
-                }
-                ya[p] = fmaf(wa[p][TAPS - 1], na, sa);
-                yb[p] = fmaf(wb[p][TAPS - 1], nb, sb);
+                for (int j = 0; j < HIST; ++j) sum = fmaf(w[j][e], h[j][e], sum);
+                y[e] = fmaf(w[TAPS - 1][e], y[e], sum);
+            }
+            if (single && t < n_tokens) {                             // the request's new state: the last taps - 1 inputs
 #pragma unroll
-                for (int j = 0; j + 1 < WIN; ++j) {
-                    xa[j][p] = xa[j + 1][p];
-                    xb[j][p] = xb[j + 1][p];
-                }
-                xa[WIN - 1][p] = na;
-                xb[WIN - 1][p] = nb;
-                if (single) {                                         // the window is the request's new state
-#pragma unroll
-                    for (int j = 0; j < WIN; ++j) {
-                        const int k = j - (TAPS - taps);
-                        if (k < 0) continue;
-                        if (ca[p] >= 0) mine[(long)k * channels + ca[p]] = xa[j][p];
-                        if (cb[p] >= 0) mine[(long)k * channels + cb[p]] = xb[j][p];
-                    }
+                for (int j = 0; j < HIST; ++j) {
+                    const int k = j - (TAPS - taps);
+                    if (k >= 0) at.put(mine + (long)k * channels, j + 1 < HIST ? h[j + 1 < HIST ? j + 1 : j] : keep);
                 }
             }
         }
         if constexpr (TAPS == 0) {
-            const int ctx = rows.req_ctx[r];
-            float* mine = tail + (long)rows.req_slot[r] * tail_stride + col0;
-            const bool single = rows.req_qlen[r] == 1;
+            const int local = __shfl_sync(0xffffffffu, l_local, u), state_row = __shfl_sync(0xffffffffu, l_row, u);
+            const int single = __shfl_sync(0xffffffffu, l_single, u);
+            float* mine = tail + (long)state_row * tail_stride + col0;
+            float keep[E], sum[E], wj[E], h[E];
 #pragma unroll
-            for (int p = 0; p < PPL; ++p) {
-                const float na = ya[p], nb = yb[p];
-                const int a = max(ca[p], 0), b = max(cb[p], 0);
-                float sa = 0.0f, sb = 0.0f;
-                for (int j = 0; j < taps - 1; ++j) {                  // oldest first
-                    const int back = taps - 1 - j, at = pos - back;
-                    if (at < 0) continue;
-                    float ua, ub;
-                    if (at >= ctx) {
-                        load_u(t - back, p, ua, ub);
-                    } else {
-                        const float* kept = mine + (long)(at - ctx + taps - 1) * channels;
-                        ua = kept[a];
-                        ub = kept[b];
-                    }
-                    sa = fmaf(conv_w[(long)j * channels + col0 + a], ua, sa);
-                    sb = fmaf(conv_w[(long)j * channels + col0 + b], ub, sb);
+            for (int e = 0; e < E; ++e) { keep[e] = y[e]; sum[e] = 0.0f; }
+            for (int j = 0; j < taps - 1 && t < n_tokens; ++j) {      // oldest first
+                const int back = taps - 1 - j;
+                if (pos[u] < back) continue;
+                at.get(conv_w + (long)j * channels + col0, wj);
+                if (local >= back) {
+                    at.get(proj + (long)(t - back) * ld + col0, h);
+#pragma unroll
+                    for (int e = 0; e < E; ++e) h[e] += b[e];
+                } else {
+                    at.get(mine + (long)(local - back + taps - 1) * channels, h);
                 }
-                ya[p] = ca[p] >= 0 ? fmaf(conv_w[(long)(taps - 1) * channels + col0 + a], na, sa) : 0.0f;
-                yb[p] = cb[p] >= 0 ? fmaf(conv_w[(long)(taps - 1) * channels + col0 + b], nb, sb) : 0.0f;
-                if (single) {
-                    for (int k = 0; k < taps - 1; ++k) {
-                        if (ca[p] >= 0) mine[(long)k * channels + a] = k + 1 < taps - 1 ? mine[(long)(k + 1) * channels + a] : na;
-                        if (cb[p] >= 0) mine[(long)k * channels + b] = k + 1 < taps - 1 ? mine[(long)(k + 1) * channels + b] : nb;
-                    }
+#pragma unroll
+                for (int e = 0; e < E; ++e) sum[e] = fmaf(wj[e], h[e], sum[e]);
+            }
+            at.get(conv_w + (long)(taps - 1) * channels + col0, wj);
+#pragma unroll
+            for (int e = 0; e < E; ++e) y[e] = fmaf(wj[e], y[e], sum[e]);
+            if (single && t < n_tokens) {
+                for (int k = 0; k + 1 < taps - 1; ++k) {
+                    at.get(mine + (long)(k + 1) * channels, h);
+                    at.put(mine + (long)k * channels, h);
                 }
+                at.put(mine + (long)(taps - 2) * channels, keep);
             }
         }
         if constexpr (TAPS == 1) {
             if (conv_w != nullptr) {
 #pragma unroll
-                for (int p = 0; p < PPL; ++p) { ya[p] *= wa[p][0]; yb[p] *= wb[p][0]; }
+                for (int e = 0; e < E; ++e) y[e] *= w[0][e];
             }
         }
-        const int slot = rows.slots[t];
-        const long page = slot / page_size;
-        T* dst;
-        if (is_q) dst = q_out + (long)t * q_ld + (long)unit * dim;
-        else dst = cache + page * page_stride + ((long)g * page_size + (slot - (int)page * page_size)) * (dim + vdim) + (is_v ? dim : 0);
         if (is_v) {
 #pragma unroll
-            for (int p = 0; p < PPL; ++p) { ya[p] *= v_scale; yb[p] *= v_scale; }
+            for (int e = 0; e < E; ++e) y[e] *= v_scale;
         } else {
             if (norm_mode == 1) {
                 float ss = 0.0f;
 #pragma unroll
-                for (int p = 0; p < PPL; ++p) ss += ya[p] * ya[p] + yb[p] * yb[p];
-                const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+                for (int e = 0; e < E; ++e) ss = fmaf(y[e], y[e], ss);
+                const float inv = ch_rms<T>(warp_sum(ss), dim, eps);
 #pragma unroll
-                for (int p = 0; p < PPL; ++p) { ya[p] = ya[p] * inv * ga[p]; yb[p] = yb[p] * inv * gb[p]; }
+                for (int e = 0; e < E; ++e) y[e] = y[e] * inv * gain[e];
             }
 #pragma unroll
             for (int p = 0; p < PPL; ++p) {
-                const int i = lane + 32 * p;
-                if (i < half) {
-                    const float c = cos_t[(long)pos * half + i], sn = sin_t[(long)pos * half + i];
-                    const float a = ya[p], b = yb[p];
-                    ya[p] = a * c - b * sn;
-                    yb[p] = b * c + a * sn;
-                }
+                const float a = y[2 * p], c = y[2 * p + 1];           // (no rotation: cos 1, sin 0)
+                y[2 * p] = a * cosv[u][p] - c * sinv[u][p];
+                y[2 * p + 1] = c * cosv[u][p] + a * sinv[u][p];
             }
             float f = 1.0f;
             if (norm_mode == 2) {
                 float ss = 0.0f;
 #pragma unroll
-                for (int p = 0; p < PPL; ++p) ss += ya[p] * ya[p] + yb[p] * yb[p];
-                f = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+                for (int e = 0; e < E; ++e) ss = fmaf(y[e], y[e], ss);
+                f = ch_rms<T>(warp_sum(ss), dim, eps);
             }
-            if (is_q && temp_every > 0) f *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f);
+            if (is_q && temp_every > 0) f *= 1.0f + temp_coef * logf((float)((pos[u] + 1) / temp_every) + 1.0f);
 #pragma unroll
-            for (int p = 0; p < PPL; ++p) { ya[p] *= f; yb[p] *= f; }
+            for (int e = 0; e < E; ++e) y[e] *= f;
         }
-#pragma unroll
-        for (int p = 0; p < PPL; ++p) {
-            if (vec) {
-                if (ca[p] >= 0) ch_put_pair(dst + ca[p], ya[p], yb[p]);
-            } else {
-                if (ca[p] >= 0) dst[ca[p]] = from_f32<T>(ya[p]);
-                if (cb[p] >= 0) dst[cb[p]] = from_f32<T>(yb[p]);
-            }
+        if (t >= n_tokens) continue;
+        T* dst;
+        if (is_q) {
+            dst = q_out + (long)t * q_ld + (long)unit * dim;
+        } else {
+            const int page = page_shift >= 0 ? slot >> page_shift : slot / page_size;
+            dst = cache + (long)page * page_stride + ((long)g * page_size + (slot - page * page_size)) * (dim + vdim) + (is_v ? dim : 0);
         }
+        at.put(dst, y);
     }
 }
 
@@ -294,24 +402,29 @@ FL_API int fl_conv_head_prep(const void* proj, int dtype, long ld, const float* 
         return (int)cudaErrorInvalidValue;
     const ChRows rows{positions, tok_req, req_start, req_ctx, req_qlen, req_slot, slots};
     const size_t elem = dtype == FL_F32 ? 4 : 2;
-    // two neighbouring channels move as one where every head starts on an even element of an aligned row
-    const int pairs_ok = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0 && q_ld % 2 == 0 && page_stride % 2 == 0 &&
-                         ((uintptr_t)proj % (2 * elem)) == 0 && ((uintptr_t)q_out % (2 * elem)) == 0 && ((uintptr_t)cache % (2 * elem)) == 0;
-    const int run = n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : 1;
-    dim3 grid((n_tokens + run - 1) / run, (units + CH_WARPS - 1) / CH_WARPS);
+    // several channels move as one where every head starts on a multiple of four elements of an aligned row
+    const int aligned = dim % 4 == 0 && vdim % 4 == 0 && ld % 4 == 0 && q_ld % 4 == 0 && page_stride % 4 == 0 &&
+                        ((uintptr_t)proj % (4 * elem)) == 0 && ((uintptr_t)q_out % (4 * elem)) == 0 && ((uintptr_t)cache % (4 * elem)) == 0 &&
+                        ((uintptr_t)bias % 16) == 0 && ((uintptr_t)conv_w % 16) == 0 && ((uintptr_t)q_w % 16) == 0 &&
+                        ((uintptr_t)k_w % 16) == 0 && ((uintptr_t)tail % 16) == 0 && tail_stride % 4 == 0;
+    int page_shift = -1;
+    if ((page_size & (page_size - 1)) == 0)
+        for (page_shift = 0; (1 << page_shift) < page_size;) ++page_shift;
     int rc = 0;
-#define FL_CH(PPL, TAPS)                                                                                                \
-    FL_DISPATCH(dtype, T, rc = fl_launch(conv_head_prep_kernel<T, PPL, TAPS>, grid, dim3(32 * CH_WARPS), 0, stream,      \
-                                         (const T*)proj, ld, bias, conv_w, taps, tail, tail_stride, q_w, k_w, norm_mode, \
-                                         eps, rot, interleaved, cos_t, sin_t, temp_coef, temp_every, v_scale, rows,     \
-                                         (T*)q_out, q_ld, heads, kv_heads, dim, vdim, (T*)cache, page_stride,          \
-                                         page_size, n_tokens, run, pairs_ok))
-#define FL_CH_TAPS(PPL)                                                                                                 \
-    { if (taps == 1) { FL_CH(PPL, 1); } else if (taps <= 4) { FL_CH(PPL, 4); } else { FL_CH(PPL, 0); } }
-    if (widest <= 64) FL_CH_TAPS(1)
-    else if (widest <= 128) FL_CH_TAPS(2)
-    else if (widest <= 256) FL_CH_TAPS(4)
-    else FL_CH_TAPS(8)
+#define FL_CH(PPL, TAPS, RUN)                                                                                            \
+    FL_DISPATCH(dtype, T, rc = fl_launch(conv_head_prep_kernel<T, PPL, TAPS, RUN>,                                        \
+                                         dim3((n_tokens + RUN - 1) / RUN, (units + CH_WARPS - 1) / CH_WARPS),            \
+                                         dim3(32 * CH_WARPS), 0, stream, (const T*)proj, ld, bias, conv_w, taps, tail,   \
+                                         tail_stride, q_w, k_w, norm_mode, eps, rot, interleaved, cos_t, sin_t,          \
+                                         temp_coef, temp_every, v_scale, rows, (T*)q_out, q_ld, heads, kv_heads, dim,    \
+                                         vdim, (T*)cache, page_stride, page_size, page_shift, n_tokens, aligned))
+#define FL_CH_TAPS(PPL, RUN)                                                                                             \
+    { if (taps == 1) { FL_CH(PPL, 1, RUN); } else if (taps <= 4) { FL_CH(PPL, 4, RUN); } else { FL_CH(PPL, 0, 1); } }
+    const bool many = n_tokens >= 256;
+    if (widest <= 64) { if (many) FL_CH_TAPS(1, 4) else FL_CH_TAPS(1, 1) }
+    else if (widest <= 128) { if (many) FL_CH_TAPS(2, 4) else FL_CH_TAPS(2, 1) }
+    else if (widest <= 256) FL_CH_TAPS(4, 1)
+    else FL_CH_TAPS(8, 1)
 #undef FL_CH_TAPS
 #undef FL_CH
     if (rc || taps == 1 || !several) return rc;

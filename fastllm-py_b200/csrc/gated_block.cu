@@ -273,7 +273,7 @@ __device__ __forceinline__ int fed_token(int id, const int* fed, int n_fed) {
     return (id < 0 && fed != nullptr && -1 - id < n_fed) ? fed[-1 - id] : id;
 }
 
-template <typename TT>
+template <typename TT, int V>
 __global__ void __launch_bounds__(256) pair_embed_kernel(
     const TT* __restrict__ table, long table_ld, const TT* __restrict__ pairs, long pairs_ld, const int* __restrict__ ids,
     float* __restrict__ out, long out_ld, int hidden, int vocab, int buckets, long mul_prev, long mul_cur, float scale,
@@ -308,14 +308,25 @@ __global__ void __launch_bounds__(256) pair_embed_kernel(
     const TT* row = table + (long)id * table_ld;
     const TT* prow = pairs + pair_row * pairs_ld;
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        const float v = to_f32<TT>(row[i]) * scale + to_f32<TT>(prow[i]);
-        o[i] = v;
-        ss += v * v;
+    for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {
+        ConvRow<V> v = td_load<TT, V>(row + i);
+        const ConvRow<V> p = td_load<TT, V>(prow + i);
+#pragma unroll
+        for (int c = 0; c < V; ++c) {
+            v.v[c] = v.v[c] * scale + p.v[c];
+            ss += v.v[c] * v.v[c];
+        }
+        conv_store<float, V>(o + i, v);
     }
     if (norm_w == nullptr) return;
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = o[i] * inv * norm_w[i];    // each thread its own elements
+    for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {                         // each thread its own elements
+        ConvRow<V> v = conv_load<V>(o + i);
+        const ConvRow<V> w = conv_load<V>(norm_w + i);
+#pragma unroll
+        for (int c = 0; c < V; ++c) v.v[c] = v.v[c] * inv * w.v[c];
+        conv_store<float, V>(o + i, v);
+    }
 }
 
 // pairs: [buckets + 1, hidden]; last_token: [slots] int; norm_w: [hidden] float, or null: the row is not normed.
@@ -326,9 +337,13 @@ FL_API int fl_pair_embed(const void* table, long table_ld, const void* pairs, lo
                          const float* norm_w, float eps, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (buckets < 1) return (int)cudaErrorInvalidValue;
-    FL_DISPATCH(dtype, TT, return fl_launch(pair_embed_kernel<TT>, dim3(n_tokens), dim3(256), 0, stream, (const TT*)table,
-                                            table_ld, (const TT*)pairs, pairs_ld, ids, out, out_ld, hidden, vocab, buckets,
-                                            mul_prev, mul_cur, scale, tok_req, req_start, req_ctx, req_qlen, req_slot,
-                                            last_token, status, fed, n_fed, norm_w, eps));
+    FL_DISPATCH(dtype, TT, {
+        const bool vec = hidden % 4 == 0 && fl_rows_take_vectors(table, table_ld, sizeof(TT)) && fl_rows_take_vectors(out, out_ld, 4) &&
+                         fl_rows_take_vectors(pairs, pairs_ld, sizeof(TT)) && fl_rows_take_vectors(norm_w, 4, 4);
+        auto kernel = vec ? pair_embed_kernel<TT, 4> : pair_embed_kernel<TT, 1>;
+        return fl_launch(kernel, dim3(n_tokens), dim3(256), 0, stream, (const TT*)table, table_ld, (const TT*)pairs, pairs_ld,
+                         ids, out, out_ld, hidden, vocab, buckets, mul_prev, mul_cur, scale, tok_req, req_start, req_ctx,
+                         req_qlen, req_slot, last_token, status, fed, n_fed, norm_w, eps);
+    });
     return 0;
 }

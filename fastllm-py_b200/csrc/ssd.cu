@@ -11,20 +11,16 @@
 // request starts (context 0).
 //
 //   ssd_prep     convolution, silu, dt and decay of every token in one float work row x | B | C | dt | a
-//   ssd_scan     per (request, head, 32 or 16 value columns): the recurrence over the request's tokens in order.  A thread
-//                holds four columns of S in its registers, R rows of each; tokens come through four stages of shared memory
-//                (cp.async), and a staged B or C value serves four columns
+//   ssd_scan     the recurrence over each request's tokens in order (state_scan.cuh, one decay per token)
 //   ssd_step     steps of single tokens: convolution, recurrence and read-out of a request's head in one kernel
 //   ssd_norm     per (token, part): gate, norm, weight; and, in blocks of their own, the convolution's new state per request
 //                (after every reader of the old one)
 //
 // All arithmetic is float (dt and the decay, two numbers a head and token, in double and rounded once: the decay is
 // multiplied up over thousands of tokens).  Every sum's order depends on the sizes alone.
-#include "common.cuh"
+#include "state_scan.cuh"
 
-#define SSD_CPT 4                // value columns of a thread
-#define SSD_STAGES 4
-#define SSD_CHUNK 16             // tokens of a stage
+#define SSD_CPT 4                // value columns of a thread of the single-token kernel
 
 __device__ __forceinline__ float ssd_silu(float v) { return v / (1.0f + expf(-v)); }
 
@@ -140,15 +136,6 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(
     }
 }
 
-__device__ __forceinline__ void ssd_cp4(void* smem, const void* gmem) {
-    const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s), "l"(gmem));
-}
-__device__ __forceinline__ void ssd_cp16(void* smem, const void* gmem) {
-    const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem));
-}
-
 // The four column sums of a group of LANES lanes, each lane holding its rows' part of all four.  After the exchange a
 // lane holds the sum of column `mine` (two lanes' worth of steps carry halves, so five shuffles do for sixteen lanes).
 template <int LANES>
@@ -175,108 +162,6 @@ __device__ __forceinline__ void ssd_update(float (&S)[SSD_CPT][R], float (&acc)[
         for (int k = 0; k < SSD_CPT; ++k) {
             S[k][4 * i4 + e] = fmaf(decay, S[k][4 * i4 + e], b[e] * xd[k]);
             acc[k] = fmaf(S[k][4 * i4 + e], c[e], acc[k]);
-        }
-}
-
-// LANES lanes share SSD_CPT columns of S; a lane holds R rows of each: the groups of four rows lane + LANES i, so that the
-// lanes read consecutive 16 bytes of a staged row.  state <= LANES R (rows beyond it stay zero).
-template <int R, int LANES, int COLS>
-__global__ void __launch_bounds__(COLS / SSD_CPT * LANES) ssd_scan_kernel(
-    const float* __restrict__ work, long w_ld, const float* __restrict__ skip, float* __restrict__ y, long y_ld,
-    float* __restrict__ state, long state_stride, const int* __restrict__ req_start, const int* __restrict__ req_ctx,
-    const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int heads, int vdim, int n, int groups, int vec4) {
-    pdl_wait();
-    pdl_trigger();
-    constexpr int DP = R * LANES, TOKEN = 2 * DP + COLS + 4;          // floats of a staged token: B | C | x | dt, decay
-    extern __shared__ __align__(16) float ssd_s[];
-    const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
-    const int tid = threadIdx.x, lane = tid & (LANES - 1), cg = tid / LANES * SSD_CPT;
-    const int start = req_start[r], qlen = req_qlen[r];
-    const bool fresh = req_ctx[r] == 0;
-    const int inner = heads * vdim, gn = groups * n, g = h / (heads / groups);
-    const int cols = min(COLS, vdim - col0);
-    for (int i = tid; i < SSD_STAGES * SSD_CHUNK * TOKEN; i += blockDim.x) ssd_s[i] = 0.0f;      // the padding stays zero
-    float* srow = state + (long)req_slot[r] * state_stride + ((long)h * vdim + col0 + cg) * n;
-    float S[SSD_CPT][R];
-#pragma unroll
-    for (int k = 0; k < SSD_CPT; ++k)
-#pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int d = 4 * (lane + LANES * (i / 4)) + (i & 3);
-            S[k][i] = (!fresh && cg + k < cols && d < n) ? srow[(long)k * n + d] : 0.0f;
-        }
-    const float skip_h = skip[h];
-    __syncthreads();
-    auto load = [&](int stage, int c0) {
-        float* dst = ssd_s + stage * SSD_CHUNK * TOKEN;
-        const int here = min(SSD_CHUNK, qlen - c0);
-        const float* base = work + (long)(start + c0) * w_ld;
-        if (vec4) {
-            const int n4 = n / 4, c4 = cols / 4, per = 2 * n4 + c4;
-            for (int i = tid; i < here * per; i += blockDim.x) {
-                const int tt = i / per, e = i - tt * per;
-                const float* row = base + (long)tt * w_ld;
-                float* to = dst + tt * TOKEN;
-                if (e < n4) ssd_cp16(to + 4 * e, row + inner + g * n + 4 * e);
-                else if (e < 2 * n4) ssd_cp16(to + DP + 4 * (e - n4), row + inner + gn + g * n + 4 * (e - n4));
-                else ssd_cp16(to + 2 * DP + 4 * (e - 2 * n4), row + h * vdim + col0 + 4 * (e - 2 * n4));
-            }
-        } else {
-            const int per = 2 * n + cols;
-            for (int i = tid; i < here * per; i += blockDim.x) {
-                const int tt = i / per, e = i - tt * per;
-                const float* row = base + (long)tt * w_ld;
-                float* to = dst + tt * TOKEN;
-                if (e < n) ssd_cp4(to + e, row + inner + g * n + e);
-                else if (e < 2 * n) ssd_cp4(to + DP + (e - n), row + inner + gn + g * n + (e - n));
-                else ssd_cp4(to + 2 * DP + (e - 2 * n), row + h * vdim + col0 + (e - 2 * n));
-            }
-        }
-        for (int i = tid; i < 2 * here; i += blockDim.x)
-            ssd_cp4(dst + (i >> 1) * TOKEN + 2 * DP + COLS + (i & 1), base + (long)(i >> 1) * w_ld + inner + 2 * gn + (i & 1) * heads + h);
-        asm volatile("cp.async.commit_group;");
-    };
-    // one group of copies per chunk, empty ones beyond the end: waiting for all but the last STAGES - 1 means this one landed
-#pragma unroll
-    for (int p = 0; p < SSD_STAGES - 1; ++p) {
-        if (p * SSD_CHUNK < qlen) load(p, p * SSD_CHUNK); else asm volatile("cp.async.commit_group;");
-    }
-    int stage = 0;
-    float* yp = y + (long)start * y_ld + (long)h * vdim + col0 + cg;
-    for (int c0 = 0; c0 < qlen; c0 += SSD_CHUNK, stage = (stage + 1) % SSD_STAGES) {
-        const int here = min(SSD_CHUNK, qlen - c0), ahead = c0 + (SSD_STAGES - 1) * SSD_CHUNK;
-        // (the stage copied into now was walked in the last round, behind that round's closing barrier)
-        if (ahead < qlen) load((stage + SSD_STAGES - 1) % SSD_STAGES, ahead); else asm volatile("cp.async.commit_group;");
-        asm volatile("cp.async.wait_group %0;" ::"n"(SSD_STAGES - 1));
-        __syncthreads();                                              // this chunk has landed
-        const float* tok = ssd_s + stage * SSD_CHUNK * TOKEN;
-#pragma unroll 4
-        for (int tt = 0; tt < here; ++tt, tok += TOKEN, yp += y_ld) {
-            const float4 xv = *reinterpret_cast<const float4*>(tok + 2 * DP + cg);
-            const float dt = tok[2 * DP + COLS], decay = tok[2 * DP + COLS + 1];
-            const float x[SSD_CPT] = {xv.x, xv.y, xv.z, xv.w};
-            const float xd[SSD_CPT] = {xv.x * dt, xv.y * dt, xv.z * dt, xv.w * dt};
-            float acc[SSD_CPT] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-            for (int i = 0; i < R / 4; ++i) {
-                const float4 b4 = reinterpret_cast<const float4*>(tok)[lane + LANES * i];
-                const float4 c4 = reinterpret_cast<const float4*>(tok + DP)[lane + LANES * i];
-                const float b[4] = {b4.x, b4.y, b4.z, b4.w}, c[4] = {c4.x, c4.y, c4.z, c4.w};
-                ssd_update<R>(S, acc, b, c, xd, decay, i);
-            }
-            int mine;
-            const float sum = ssd_sum4<LANES>(acc, lane, mine);
-            const float xm = mine == 0 ? x[0] : mine == 1 ? x[1] : mine == 2 ? x[2] : x[3];
-            if ((lane & (LANES / 4 - 1)) == 0 && cg + mine < cols) yp[mine] = fmaf(skip_h, xm, sum);
-        }
-        __syncthreads();                                              // the stage is copied into again in the next round
-    }
-#pragma unroll
-    for (int k = 0; k < SSD_CPT; ++k)
-#pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int d = 4 * (lane + LANES * (i / 4)) + (i & 3);
-            if (cg + k < cols && d < n) srow[(long)k * n + d] = S[k][i];
         }
 }
 
@@ -373,31 +258,39 @@ __global__ void __launch_bounds__(COLS / SSD_CPT * LANES) ssd_step_kernel(
         y[(long)r * y_ld + (long)h * vdim + col0 + cg + mine] = fmaf(skip[h], xm, sum);
 }
 
-// Blocks [0, n_tokens) of x: token t, part blockIdx.y.  Blocks behind them: request blockIdx.x - n_tokens, its
-// convolution state (the y blocks share the channels out).
+// Blocks [0, n_tokens) of x: token t, part blockIdx.y.  Behind them `share` blocks of x a request, which with blockIdx.y
+// share its convolution channels out, one a thread: the new state (up to three
+// entries are read before the first is written, so that the loads run side by side).
 template <typename T, int V>
 __global__ void __launch_bounds__(512) ssd_norm_kernel(
     const float* __restrict__ y, long y_ld, const T* __restrict__ proj, long ld, const float* __restrict__ weight,
     T* __restrict__ out, long out_ld, int n_tokens, int inner, int part, float eps, float* __restrict__ tail, long tail_stride,
-    int taps, int channels, const int* __restrict__ req_start, const int* __restrict__ req_ctx,
+    int share, int taps, int channels, const int* __restrict__ req_start, const int* __restrict__ req_ctx,
     const int* __restrict__ req_qlen, const int* __restrict__ req_slot) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) float ssd_row[];                  // [part]
     __shared__ float scratch[32];
     if ((int)blockIdx.x >= n_tokens) {
-        const int r = blockIdx.x - n_tokens;
-        const int start = req_start[r], ctx = req_ctx[r], qlen = req_qlen[r];
-        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
-            float* mine = tail + (long)req_slot[r] * tail_stride + c;
-            // entry j takes the input of position end - (taps - 1) + j; entries that stay move down: upwards in place is safe
-            for (int j = 0; j < taps - 1; ++j) {
-                const int at = ctx + qlen - (taps - 1) + j;
-                float u = 0.0f;
-                if (at >= ctx) u = to_f32<T>(proj[(long)(start + at - ctx) * ld + inner + c]);
-                else if (at >= 0) u = mine[(long)(j + qlen) * channels];
-                mine[(long)j * channels] = u;
-            }
+        const int r = (blockIdx.x - n_tokens) / share, slice = (blockIdx.x - n_tokens) % share;
+        const int c = (slice * gridDim.y + blockIdx.y) * blockDim.x + threadIdx.x;
+        if (c >= channels) return;
+        const int start = req_start[r], ctx = req_ctx[r], qlen = req_qlen[r], back = taps - 1;
+        float* mine = tail + (long)req_slot[r] * tail_stride + c;
+        auto entry = [&](int j) {                                     // entry j takes the input of position end - back + j
+            const int at = ctx + qlen - back + j;
+            if (at >= ctx) return to_f32<T>(proj[(long)(start + at - ctx) * ld + inner + c]);
+            return at >= 0 ? mine[(long)(j + qlen) * channels] : 0.0f;
+        };
+        if (back <= 3) {
+            float u[3];
+#pragma unroll
+            for (int j = 0; j < 3; ++j) u[j] = j < back ? entry(j) : 0.0f;
+#pragma unroll
+            for (int j = 0; j < 3; ++j)
+                if (j < back) mine[(long)j * channels] = u[j];
+        } else {
+            for (int j = 0; j < back; ++j) mine[(long)j * channels] = entry(j);      // (entries that stay move down)
         }
         return;
     }
@@ -456,48 +349,21 @@ FL_API int fl_ssd_prep(const void* proj, int dtype, long ld, const float* conv_w
     return 0;
 }
 
-template <int R, int LANES, int COLS>
-static int ssd_scan_launch(int n_requests, int heads, int vdim, cudaStream_t stream, const float* work, long w_ld,
-                           const float* skip, float* y, long y_ld, float* state, long state_stride, const int* req_start,
-                           const int* req_ctx, const int* req_qlen, const int* req_slot, int n, int groups, int vec4) {
-    const size_t smem = (size_t)SSD_STAGES * SSD_CHUNK * (2 * R * LANES + COLS + 4) * sizeof(float);
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(ssd_scan_kernel<R, LANES, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return (int)e;
-        configured = true;
-    }
-    return fl_launch(ssd_scan_kernel<R, LANES, COLS>, dim3(n_requests, heads, (vdim + COLS - 1) / COLS), dim3(COLS / SSD_CPT * LANES),
-                     smem, stream, work, w_ld, skip, y, y_ld, state, state_stride, req_start, req_ctx, req_qlen, req_slot,
-                     heads, vdim, n, groups, vec4);
-}
-
 static inline bool ssd_takes(int n_requests, int heads, int vdim, int n, int groups) {
     return n >= 1 && n <= 256 && vdim >= 1 && heads >= 1 && heads <= 65535 && (vdim + 15) / 16 <= 65535 && groups >= 1 &&
            heads % groups == 0;
 }
 
+// work: what fl_ssd_prep leaves.  single_tokens: every request of the step brings one token.
 FL_API int fl_ssd_scan(const float* work, long w_ld, const float* skip, float* y, long y_ld, float* state, long state_stride,
                        const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot, int n_requests,
-                       int heads, int vdim, int n, int groups, cudaStream_t stream) {
+                       int heads, int vdim, int n, int groups, int single_tokens, int sms, cudaStream_t stream) {
     if (n_requests <= 0) return 0;
     if (!ssd_takes(n_requests, heads, vdim, n, groups)) return (int)cudaErrorInvalidValue;
-    // 16-byte copies where every source address is a multiple of 16 bytes
-    const int vec4 = vdim % 4 == 0 && n % 4 == 0 && w_ld % 4 == 0 && ((uintptr_t)work % 16) == 0;
-#define FL_SSD_SCAN(R, L, C)                                                                                             \
-    return ssd_scan_launch<R, L, C>(n_requests, heads, vdim, stream, work, w_ld, skip, y, y_ld, state, state_stride,     \
-                                    req_start, req_ctx, req_qlen, req_slot, n, groups, vec4)
-    if (vdim <= 16) {
-        if (n <= 32) FL_SSD_SCAN(4, 8, 16);
-        if (n <= 64) FL_SSD_SCAN(4, 16, 16);
-        if (n <= 128) FL_SSD_SCAN(8, 16, 16);
-        FL_SSD_SCAN(16, 16, 16);
-    }
-    if (n <= 32) FL_SSD_SCAN(4, 8, 32);
-    if (n <= 64) FL_SSD_SCAN(4, 16, 32);
-    if (n <= 128) FL_SSD_SCAN(8, 16, 32);
-    FL_SSD_SCAN(16, 16, 32);
-#undef FL_SSD_SCAN
+    const int inner = heads * vdim, gn = groups * n;
+    const ScanToken at{inner, inner + gn, n, heads / groups, 0, 0, inner + 2 * gn, inner + 2 * gn + heads};
+    return state_scan<true>(work, w_ld, at, skip, y, y_ld, state, state_stride, req_start, req_ctx, req_qlen, req_slot, n_requests,
+                            heads, n, vdim, single_tokens, sms, stream);
 }
 
 // Steps of single tokens only: row r of proj is request r's.
@@ -543,7 +409,8 @@ FL_API int fl_ssd_norm(const float* y, long y_ld, const void* proj, int dtype, l
                      ssd_aligned(weight, 4, 4);
     int threads = 32;
     while (threads < 512 && threads * (vec ? 8 : 2) < part) threads *= 2;
-    dim3 grid(n_tokens + (taps > 1 ? n_requests : 0), parts);
+    const int share = (channels + threads * parts - 1) / (threads * parts);
+    dim3 grid(n_tokens + (taps > 1 ? n_requests * share : 0), parts);
     FL_DISPATCH(dtype, T, {
         auto kernel = vec ? ssd_norm_kernel<T, 4> : ssd_norm_kernel<T, 1>;
         if (smem > 48 * 1024) {
@@ -551,7 +418,7 @@ FL_API int fl_ssd_norm(const float* y, long y_ld, const void* proj, int dtype, l
             if (e != cudaSuccess) return (int)e;
         }
         return fl_launch(kernel, grid, dim3(threads), smem, stream, y, y_ld, (const T*)proj, ld, weight, (T*)out, out_ld,
-                         n_tokens, inner, part, eps, tail, tail_stride, taps, channels, req_start, req_ctx, req_qlen, req_slot);
+                         n_tokens, inner, part, eps, tail, tail_stride, share, taps, channels, req_start, req_ctx, req_qlen, req_slot);
     });
     return 0;
 }
