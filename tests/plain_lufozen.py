@@ -115,7 +115,7 @@ def gated_attention(h, t, m, eps, alter=()):
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q, k, v = (h @ t[s].T + t[s + ".b"] for s in ("q", "k", "v"))
-    if "no_conv" not in alter:
+    if "q.conv" in t and "no_conv" not in alter:
         q, k, v = short_conv(q, t["q.conv"]), short_conv(k, t["k.conv"]), short_conv(v, t["v.conv"])
     q = rms(q.view(T, H, d), eps) * t["q.norm"]
     k = rms(k.view(T, G, d), eps) * t["k.norm"]

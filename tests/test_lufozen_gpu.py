@@ -1,0 +1,364 @@
+"""Lufozen in the engine against the plain implementation (tests/plain_lufozen.py).
+
+Small configurations with weights of their own (tests/lufozen_tiny.py).  The 32-bit engine is
+held to 2e-4 of the largest logit against the float64 oracle and, cut against cut, to bitwise
+equality (every kernel of that path sums in an order that depends on the token's own place
+only); the bfloat16 engine's error, position by position, to a fraction of the logits' spread.
+Every engine runs with the cache's check mode on (pages that go back are overwritten) and with
+fewer state slots than requests, so pages and slots are used again.
+"""
+import numpy as np
+import pytest
+import torch
+
+import lufozen_tiny as lt
+import plain_lufozen as plain
+import replay
+
+pytestmark = pytest.mark.gpu
+
+BANDS = (8.0, 64, 1.0, 4.0)
+# every size differs from model to model, and some are the degenerate values: one head, heads == kv_heads, groups of three
+# and twelve query heads, one state group and as many groups as heads, one norm part and as many as heads, one tap, nine
+# taps, no convolution, no rotation, part of the dimensions rotated, no token pairs, no loop, a loop over all layers, over
+# one layer, run once, layers without feed-forward in every place, widths that are multiples of neither 8 nor 32
+MODELS = {
+    "mix": dict(layers=[(lt.linear(2, 8, 12, 8.0), None),
+                        (lt.attention(4, 2, 16, 24, conv=4, rot=8, scaling=BANDS), lt.dense(48)),
+                        (lt.pair(lt.left(4, 2, 16, 12, rot=16), lt.right(4, 8, 12, 2, 4, 2)), lt.dense(30)),
+                        (lt.attention(6, 2, 12, 8, conv=2, rot=12), None)],
+                kw=dict(vocab=97, width=40, loop=(1, 3, 2)), page=8, rank=6),
+    "odd": dict(layers=[(lt.attention(3, 3, 10, 7, conv=1, rot=10, base=500.0), None),
+                        (lt.pair(lt.left(12, 1, 6, 5, rot=None), lt.right(3, 5, 7, 3, 6, 1), -0.5, 1.3), lt.dense(11)),
+                        (lt.linear(1, 13, 35, 2.0), lt.dense(30)),
+                        (lt.attention(1, 1, 14, 40, conv=None, rot=6), lt.dense(9)),
+                        (lt.pair(lt.left(2, 2, 9, 3, rot=4, scaling=(4.0, 16, 0.5, 2.0)), lt.right(6, 3, 33, 1, 1, 6), 1.0, 1.0), None),
+                        (lt.attention(2, 1, 8, 4, conv=9, rot=8), None)],
+                kw=dict(vocab=61, width=36, eps=1e-6, loop=(0, 6, 2), buckets=None, scale=1.0, logit_scale=1.5), page=16, rank=3),
+    # sizes that the tensor-core kernels take in bfloat16 (multiples of 16 throughout)
+    "even": dict(layers=[(lt.attention(8, 2, 32, 64, conv=4, rot=32, scaling=(8.0, 128, 1.0, 4.0)), lt.dense(128)),
+                         (lt.pair(lt.left(4, 2, 64, 32, rot=32), lt.right(6, 16, 64, 2, 4, 3), 0.5, 0.8), lt.dense(96)),
+                         (lt.linear(4, 32, 48, 16.0), lt.dense(64))],
+                 kw=dict(vocab=80, width=64, loop=(2, 3, 1), buckets=7), page=16, rank=16),
+    "single": dict(layers=[(lt.pair(lt.left(2, 1, 16, 16, rot=16), lt.right(4, 20, 70, 4, 3, 2)), lt.dense(32))],
+                   kw=dict(vocab=50, width=48, buckets=1, mul=(0, 3)), page=4, rank=4),
+}
+LENGTHS = {"mix": [1, 2, 9, 23, 40, 77], "odd": [3, 30, 64, 51], "even": [150, 70, 90], "single": [33, 5, 61]}
+
+
+@pytest.fixture(scope="module")
+def made(tmp_path_factory):
+    root = tmp_path_factory.mktemp("lufozen")
+    out = {}
+    for k, (name, m) in enumerate(MODELS.items()):
+        raw = lt.config(m["layers"], **m["kw"])
+        w = lt.weights(raw, seed=5 + k, rank=m["rank"])
+        rng = np.random.default_rng(40 + k)
+        requests = {f"q{i}": rng.integers(0, raw["vocab"], size=n).tolist() for i, n in enumerate(LENGTHS[name])}
+        want = {rid: plain.forward(raw, w, toks).float() for rid, toks in requests.items()}
+        out[name] = dict(raw=raw, weights=w, folder=lt.write(raw, w, root / name), requests=requests, want=want,
+                         page=m["page"])
+    return out
+
+
+_engines = {}
+
+
+def engine(made, name, dtype, max_tokens=None, max_requests=3, graph=False):
+    from fastllm_py_b200 import Model
+
+    key = (name, dtype, max_tokens, max_requests, graph)
+    if key not in _engines:
+        _engines[key] = Model.load(made[name]["folder"], dtype=dtype, page_size=made[name]["page"],
+                                   max_tokens=max_tokens or 512, max_requests=max_requests, max_batched_tokens=256,
+                                   max_model_len=256, cuda_graph=graph, check_cache=True)
+    return _engines[key]
+
+
+def load(folder, dtype, page=4, tokens=64, requests=2, longest=64, check=True):
+    from fastllm_py_b200 import Model
+
+    return Model.load(folder, dtype=dtype, page_size=page, max_tokens=tokens, max_requests=requests,
+                      max_batched_tokens=max(64, longest), max_model_len=longest, cuda_graph=False, check_cache=check).engine
+
+
+def cuts(requests, live):
+    return {"whole": replay.whole(requests), "tail": replay.tail_decode(requests, 12),
+            "portions": replay.portions(requests), "small": replay.portions(requests, (2, 3, 2, 5, 2)),
+            "mixed": replay.mixed(requests, live=live, seed=3, prefill_sizes=(9, 2, 17, 5), decode_tail=6)}
+
+
+def worst(got, want):
+    return max(float((got[(rid, p)] - want[rid][p]).abs().max()) for (rid, p) in got)
+
+
+@pytest.mark.parametrize("name", list(MODELS))
+def test_every_cut_in_32_bit_equals_the_oracle_and_the_other_cuts(made, name):
+    m = made[name]
+    top = max(float(v.abs().max()) for v in m["want"].values())
+    results = {}
+    for cut, steps in cuts(m["requests"], live=3).items():
+        pool = replay.peak_tokens(steps, m["page"]) + (0 if cut == "mixed" else m["page"])
+        eng = engine(made, name, "float32", pool).engine
+        got = replay.run_in_process(eng, steps)
+        assert len(got) == sum(len(t) for t in m["requests"].values())
+        assert worst(got, m["want"]) <= 2e-4 * max(1.0, top), cut
+        results[cut] = got
+        assert not eng.cache.live
+    for cut, got in results.items():
+        for key, row in got.items():
+            assert torch.equal(row, results["whole"][key]), (cut, key)
+
+
+@pytest.mark.parametrize("name", list(MODELS))
+def test_every_cut_in_bfloat16_stays_near_the_oracle(made, name):
+    m = made[name]
+    spread = float(torch.cat([v.flatten() for v in m["want"].values()]).std())
+    for cut, steps in cuts(m["requests"], live=3).items():
+        eng = engine(made, name, "bfloat16", replay.peak_tokens(steps, m["page"]) + m["page"]).engine
+        got = replay.run_in_process(eng, steps)
+        errs = np.array([float((got[k] - m["want"][k[0]][k[1]]).pow(2).mean().sqrt()) for k in got]) / spread
+        assert np.median(errs) <= 0.04, (cut, np.median(errs))
+        # a sequence's first token reads one outer product out of the linear attention's state and norms it: v times the
+        # sign of q . k, which rounding turns where q . k is nearly zero
+        first = np.array([k[1] == 0 for k in got])
+        assert errs[~first].max(initial=0.0) <= 0.12 and errs[first].max() <= 0.6, (cut, errs[~first].max(initial=0.0), errs[first].max())
+
+
+SMALL = dict(width=24, vocab=50, buckets=None, scale=1.0)
+SINGLE = {
+    "attention": lt.config([(lt.attention(2, 1, 8, 40, conv=4, rot=4), None)], **SMALL),
+    "attention_wide_key": lt.config([(lt.attention(2, 2, 72, 8, conv=3, rot=72), None)], **SMALL),
+    "attention_widest": lt.config([(lt.attention(3, 1, 136, 200, conv=2, rot=30, scaling=BANDS), None)], **SMALL),
+    "attention_key_beyond_256": lt.config([(lt.attention(1, 1, 260, 12, conv=4, rot=260), None)], **SMALL),
+    "attention_many_taps": lt.config([(lt.attention(2, 1, 12, 12, conv=7, rot=4), None)], **SMALL),
+    "attention_one_tap": lt.config([(lt.attention(2, 2, 8, 8, conv=1, rot=8), None)], **SMALL),
+    "attention_no_conv": lt.config([(lt.attention(3, 3, 8, 8, conv=None, rot=None), None)], **SMALL),
+    "linear": lt.config([(lt.linear(2, 8, 40, 4.0), None)], **SMALL),
+    "linear_wide_key": lt.config([(lt.linear(2, 72, 8, 16.0), None)], **SMALL),
+    "linear_widest_key": lt.config([(lt.linear(1, 136, 33, 64.0), None)], **SMALL),
+    "state": lt.config([(lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(6, 8, 20, 3, 4, 2)), None)], **SMALL),
+    "state_one_group": lt.config([(lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(5, 33, 48, 1, 2, 5)), None)], **SMALL),
+    "state_wide": lt.config([(lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(2, 9, 130, 2, 3, 1)), None)], **SMALL),
+    "state_many_taps": lt.config([(lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(4, 4, 6, 4, 9, 4)), None)], **SMALL),
+    "state_one_tap": lt.config([(lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(1, 50, 256, 1, 1, 1)), None)], **SMALL),
+    "left": lt.config([(lt.pair(lt.left(6, 2, 24, 40, rot=10, scaling=BANDS), lt.right(1, 4, 4, 1, 2, 1), 1.5, 0.1), None)], **SMALL),
+    "dense": lt.config([(lt.linear(1, 4, 4, 1.0), lt.dense(36))], **SMALL),
+    "pairs": lt.config([(lt.linear(1, 4, 4, 1.0), None)], width=24, vocab=50, buckets=11, mul=(1, 50)),
+    "loop": lt.config([(lt.linear(1, 4, 4, 1.0), None), (lt.attention(1, 1, 8, 8, conv=3, rot=8), None)], loop=(1, 2, 4), **SMALL),
+}
+
+
+@pytest.mark.parametrize("kind", list(SINGLE))
+def test_each_mechanism_alone(tmp_path, kind):
+    """A prompt, then single tokens, in both precisions (the bfloat16 engine's fused single-token kernels among them)."""
+    from fastllm_py_b200 import StepEntry
+
+    raw = SINGLE[kind]
+    w = lt.weights(raw, seed=17, rank=5)
+    folder = lt.write(raw, w, tmp_path / kind)
+    toks = np.random.default_rng(1).integers(0, raw["vocab"], size=45).tolist()
+    want = plain.forward(raw, w, toks).float()
+    for dtype in ("float32", "bfloat16"):
+        eng = load(folder, dtype)
+        eng.begin("a")
+        head = eng.step([StepEntry("a", toks[:20], list(range(20)))]).cpu().clone()
+        rest = [eng.step([StepEntry("a", [t], [0])]).cpu().clone() for t in toks[20:]]
+        got = torch.cat([head] + rest)
+        if dtype == "float32":
+            assert float((got - want).abs().max()) <= 2e-4 * max(1.0, float(want.abs().max()))
+        else:
+            errs = (got - want).pow(2).mean(dim=1).sqrt() / want.std()
+            assert float(errs.max()) <= 0.1, float(errs.max())
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_every_mechanism_moves_the_logits(tmp_path, dtype):
+    """The engine equals the oracle, and the oracle with one reading changed is far from both."""
+    raw = lt.config([(lt.attention(4, 2, 8, 8, conv=3, rot=8, scale=1.5), lt.dense(16)),
+                     (lt.pair(lt.left(2, 1, 8, 8, rot=8, scale=1.5), lt.right(4, 6, 5, 2, 3, 4), 0.9, 0.3), lt.dense(12)),
+                     (lt.linear(2, 4, 6, 4.0), None)], width=24, vocab=30, loop=(0, 2, 2))
+    w = lt.weights(raw, seed=1)
+    folder = lt.write(raw, w, tmp_path / "m")
+    toks = np.random.default_rng(3).integers(0, 30, size=40).tolist()
+    want = plain.forward(raw, w, toks).float()
+    got = replay.run_in_process(load(folder, dtype), replay.portions({"a": toks}, (7, 2, 11)))
+    rows = torch.stack([got[("a", p)] for p in range(len(toks))])
+
+    def err(other):                                  # mean over positions of the distance of a row, in spreads
+        return float((other - rows).pow(2).mean(dim=1).sqrt().mean() / want.std())
+
+    base = err(want)
+    assert base <= (2e-5 if dtype == "float32" else 0.03), base
+    for alter in ("no_conv", "other_pairing", "no_sink", "left_sink", "no_gate", "no_out_bias", "no_skip", "one_norm", "norm_first",
+                  "no_decay", "swapped_scales", "no_step", "no_pairs", "plain_weight"):
+        other = err(plain.forward(raw, w, toks, alter={alter}).float())
+        assert other > (100 if dtype == "float32" else 1.5) * base, (alter, other, base)
+
+
+def _loud_key(raw, at, heads, kv_heads, dim):
+    """Weights under which the vocabulary's last token, as a query, is answered by an earlier token of the one before it and
+    by nothing else: the two are the only rows of the embedding that are not zero in the first and in the second quarter
+    of the width, and the queries of every head read the first quarter as the keys read the second."""
+    w = lt.weights(raw, seed=8)
+    quarter = raw["width"] // 4
+    gen = torch.Generator().manual_seed(12)
+    w["embed"][:, :2 * quarter] = 0.0
+    w["embed"][-2:] = 0.0
+    loud = (2.0 + torch.rand(quarter, generator=gen)).to(torch.bfloat16)
+    w["embed"][-1, :quarter] = loud
+    w["embed"][-2, quarter:2 * quarter] = loud
+    block = torch.randn(dim, quarter, generator=gen)
+    q, k = torch.zeros(dim, raw["width"]), torch.zeros(dim, raw["width"])
+    q[:, :quarter], k[:, quarter:2 * quarter] = block, block
+    w[at + "q"] = q.repeat(heads, 1).to(torch.bfloat16)
+    w[at + "k"] = k.repeat(kv_heads, 1).to(torch.bfloat16)
+    w["embed.norm"] = torch.zeros(raw["width"], dtype=torch.bfloat16)
+    for s in ("q.norm", "k.norm"):
+        w[at + s] = torch.ones(dim, dtype=torch.bfloat16)
+    w["l0.norm1"] = torch.zeros(raw["width"], dtype=torch.bfloat16)
+    for s in ("q.b", "k.b"):
+        if at + s in w:
+            w[at + s] = torch.zeros_like(w[at + s])
+    for s in ("q.conv", "k.conv"):
+        if at + s in w:                              # (the current token counts most)
+            t = torch.full_like(w[at + s], 0.05)
+            t[:, -1] = 1.0
+            w[at + s] = t
+    return w
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("kind", ["attention", "left"])
+def test_a_far_key_among_hundreds_stands_out(tmp_path, dtype, kind):
+    """One early token answers a late query among 300 keys (in a prompt, and alone in a decode step, behind page borders);
+    without that token the oracle is far away."""
+    if kind == "attention":
+        mixer = lt.attention(4, 2, 32, 16, conv=3, rot=4, base=1e6, scale=0.6)
+        at, sizes = "l0.mix.", (4, 2, 32)
+    else:
+        mixer = lt.pair(lt.left(4, 1, 32, 16, rot=4, base=1e6, scale=0.6), lt.right(1, 4, 4, 1, 1, 1), 1.0, 0.05)
+        at, sizes = "l0.mix.left.", (4, 1, 32)
+    raw = lt.config([(mixer, None)], width=32, vocab=40, buckets=None, scale=1.0)
+    w = _loud_key(raw, at, *sizes)
+    folder = lt.write(raw, w, tmp_path / "far")
+    toks = np.random.default_rng(5).integers(0, 38, size=300).tolist()
+    toks[33] = 38
+    eng = load(folder, dtype, page=16, tokens=320, requests=1, longest=320)
+    for p in (40, 271, 287):                         # behind a page's border, and the last and first places of pages
+        seq = toks[:p] + [39]
+        want = plain.forward(raw, w, seq).float()
+        without = plain.forward(raw, w, seq[:33] + [0] + seq[34:]).float()
+        gap = float((without[p] - want[p]).pow(2).mean().sqrt())
+        assert gap > 0.2 * float(want.std())
+        for steps in (replay.whole({"a": seq}), replay.tail_decode({"a": seq}, 1), replay.portions({"a": seq}, (64, 30, 2))):
+            row = replay.run_in_process(eng, steps)[("a", p)]
+            err = float((row - want[p]).pow(2).mean().sqrt())
+            assert err <= (1e-4 if dtype == "float32" else 0.05) * float(want.std()) and err < 0.2 * gap
+
+
+def test_far_tokens_reach_through_both_states(tmp_path):
+    """Decays close to one: the first token still moves the last logits through the states alone, and the engine follows
+    the oracle through 150 single-token steps after a short prompt, in both precisions."""
+    raw = lt.config([(lt.linear(2, 16, 16, 64.0), lt.dense(16)),
+                     (lt.pair(lt.left(1, 1, 4, 4, rot=2), lt.right(4, 8, 16, 2, 3, 2), 0.0, 1.0), None)], width=24, vocab=40, buckets=None)
+    w = lt.weights(raw, seed=9, slow=True)
+    folder = lt.write(raw, w, tmp_path / "far")
+    toks = np.random.default_rng(4).integers(0, 40, size=160).tolist()
+    want = plain.forward(raw, w, toks).float()
+    changed = plain.forward(raw, w, [(toks[0] + 1) % 40] + toks[1:]).float()
+    eng = load(folder, "float32", page=16, tokens=256, longest=256, check=False)
+    got = replay.run_in_process(eng, replay.tail_decode({"a": toks}, 150))
+    err = worst(got, {"a": want})
+    assert err <= 2e-4 * float(want.abs().max())
+    assert float((changed[-1] - want[-1]).abs().max()) > 100 * max(err, 1e-5)
+    eng = load(folder, "bfloat16", page=16, tokens=256, longest=256, check=False)
+    got = replay.run_in_process(eng, replay.tail_decode({"a": toks}, 150))
+    errs = [float((got[("a", p)] - want[p]).pow(2).mean().sqrt() / want.std()) for p in range(160)]
+    assert max(errs[100:]) <= 0.08, max(errs[100:])                      # nothing piles up along the decode
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_the_sinks_unit_counts_where_scores_are_low(tmp_path, dtype):
+    """Early tokens with scores far below zero: nearly all of the softmax's weight goes to the added one, so a row without
+    it would be several times larger."""
+    raw = lt.config([(lt.attention(2, 1, 16, 16, conv=2, rot=None, scale=1.0), None)], width=32, vocab=40, buckets=None)
+    w = lt.weights(raw, seed=4)
+    w["l0.mix.q.b"] = torch.full((32,), 3.0, dtype=torch.bfloat16)
+    w["l0.mix.k.b"] = torch.full((16,), -3.0, dtype=torch.bfloat16)
+    for s in ("q", "k"):
+        w[f"l0.mix.{s}"] = w[f"l0.mix.{s}"] * 0.1
+        w[f"l0.mix.{s}.norm"] = torch.full((16,), 0.6, dtype=torch.bfloat16)
+        w[f"l0.mix.{s}.conv"] = torch.full_like(w[f"l0.mix.{s}.conv"], 0.5)
+    folder = lt.write(raw, w, tmp_path / "sink")
+    toks = np.random.default_rng(6).integers(0, 40, size=40).tolist()
+    want = plain.forward(raw, w, toks).float()
+    without = plain.forward(raw, w, toks, alter={"no_sink"}).float()
+    for steps in (replay.whole({"a": toks}), replay.tail_decode({"a": toks}, 39)):
+        got = replay.run_in_process(load(folder, dtype), steps)
+        for p in range(40):
+            err = float((got[("a", p)] - want[p]).pow(2).mean().sqrt())
+            assert err <= 0.1 * float((without[p] - want[p]).pow(2).mean().sqrt()), p
+
+
+def test_a_slot_used_again_starts_clean(made):
+    """Two requests one after the other in an engine with a single slot equal the same requests in
+    fresh engines, bit for bit (states, kept rows of the convolutions and the kept token among them)."""
+    m = made["mix"]
+    (ra, ta), (rb, tb) = list(m["requests"].items())[3:5]
+    eng = engine(made, "mix", "float32", 128, max_requests=1).engine
+    first = replay.run_in_process(eng, replay.portions({ra: ta}))
+    second = replay.run_in_process(eng, replay.portions({rb: tb}, (1, 1, 1, 2, 7)))
+    alone = replay.run_in_process(engine(made, "mix", "float32", 512).engine, replay.whole({rb: tb}))
+    assert all(torch.equal(second[k], alone[k]) for k in alone)
+    assert worst(first, m["want"]) <= 2e-4 * 30.0
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_greedy_generation_through_the_scheduler(made, dtype):
+    """Model.generate (scheduler, sampler, captured decode steps, tokens fed on the device) against the oracle's greedy
+    loop; where the oracle's two best logits are close the engine may take either."""
+    m = made["mix"]
+    model = engine(made, "mix", dtype, 512, max_requests=3, graph=True)
+    prompts = [m["requests"]["q2"], m["requests"]["q3"], m["requests"]["q1"], m["requests"]["q4"][:20]]
+    outs = model.generate(prompts, max_new_tokens=12)
+    assert model.generate(prompts, max_new_tokens=12, use_graph=False) == outs          # replayed steps change nothing
+    gaps = []                                                    # how far below the oracle's best each token is, in spreads
+    for prompt, new in zip(prompts, outs):
+        seq = list(prompt)
+        for tok in new:
+            logits = plain.forward(m["raw"], m["weights"], seq)[-1]
+            gaps.append(float(logits.max() - logits[tok]) / float(logits.std()))
+            seq.append(tok)
+        assert len(new) == 12
+    assert max(gaps) < (1e-3 if dtype == "float32" else 0.3), sorted(gaps)[-5:]
+
+
+def test_trace_program_on_a_folder(made, tmp_path):
+    m = made["odd"]
+    steps = replay.mixed(m["requests"], live=2, seed=1, prefill_sizes=(7, 2, 30), decode_tail=3)
+    got = replay.run_program(m["folder"], "float32", steps, tmp_path / "out", replay.peak_tokens(steps, 64),
+                             m["raw"]["vocab"], extra_args=("--max-requests", "2"))
+    top = max(float(v.abs().max()) for v in m["want"].values())
+    assert worst(got, m["want"]) <= 2e-4 * max(1.0, top)
+
+
+def test_command_line_on_a_random_weights_folder(tmp_path):
+    """bin/make_model writes a folder from a configuration, bin/generate loads it by its architecture
+    string and generates through the scheduler."""
+    import json
+    import subprocess
+    import sys
+
+    raw = lt.config([(lt.attention(2, 1, 16, 16, conv=3, rot=16), lt.dense(32)),
+                     (lt.pair(lt.left(2, 1, 16, 16), lt.right(2, 16, 16, 1, 4, 1)), None)], width=32, vocab=64, loop=(0, 2, 2))
+    (tmp_path / "config.json").write_text(json.dumps(raw))
+    made_ = subprocess.run([sys.executable, str(replay.ROOT / "bin" / "make_model"), str(tmp_path / "config.json"),
+                            str(tmp_path / "m"), "--seed", "4", "--std", "0.2"], capture_output=True, text=True)
+    assert made_.returncode == 0 and "Lufozen" in made_.stdout, made_.stderr
+    run = subprocess.run([sys.executable, str(replay.ROOT / "bin" / "generate"), str(tmp_path / "m"), "-", "9",
+                          "bfloat16", "--random-prompt", "30", "--seed", "1"], capture_output=True, text=True)
+    assert run.returncode == 0, run.stderr[-2000:]
+    lines = run.stdout.strip().splitlines()
+    assert "Lufozen: 2L width=32" in lines[0]
+    assert len([int(t) for t in lines[1].split(",")]) == 9
