@@ -81,8 +81,8 @@ template <int N> __device__ __forceinline__ void ch_put(bf16* p, const float* v)
 // How a lane's 2 PPL elements lie in a head, pair after pair: CH_RUN: consecutive channels from `first` on (pairs of
 // neighbours); CH_HALVES: PPL channels from `first` on paired with those `half` further; CH_ANY: pairs found one by one.
 enum { CH_RUN = 0, CH_HALVES = 1, CH_ANY = 2 };
-template <int PPL> struct ChLane {
-    int mode, size, turn, half, slot0;                                // slot0: the lane's first pair
+template <int PPL, int MODE> struct ChLane {
+    int size, turn, half, slot0;                                // slot0: the lane's first pair
     bool side;
     __device__ __forceinline__ int channel(int e) const {             // of element e; -1 where there is none
         const int s = slot0 + (e >> 1);
@@ -93,9 +93,9 @@ template <int PPL> struct ChLane {
         return c < size ? c : -1;
     }
     template <typename T> __device__ __forceinline__ void get(const T* p, float* v, float missing = 0.0f) const {
-        if (mode == CH_RUN) {
+        if constexpr (MODE == CH_RUN) {
             if (2 * slot0 < size) { ch_get<2 * PPL>(p + 2 * slot0, v); return; }
-        } else if (mode == CH_HALVES) {
+        } else if constexpr (MODE == CH_HALVES) {
             if (slot0 < half) {
                 float a[PPL], b[PPL];
                 ch_get<PPL>(p + slot0, a);
@@ -116,9 +116,9 @@ template <int PPL> struct ChLane {
         for (int e = 0; e < 2 * PPL; ++e) v[e] = missing;
     }
     template <typename T> __device__ __forceinline__ void put(T* p, const float* v) const {
-        if (mode == CH_RUN) {
+        if constexpr (MODE == CH_RUN) {
             if (2 * slot0 < size) ch_put<2 * PPL>(p + 2 * slot0, v);
-        } else if (mode == CH_HALVES) {
+        } else if constexpr (MODE == CH_HALVES) {
             if (slot0 < half) {
                 float a[PPL], b[PPL];
 #pragma unroll
@@ -149,36 +149,51 @@ struct ChRows {                  // the step's tables
 // PPL: pairs a lane holds (head sizes up to 64 PPL); TAPS: the layer's taps rounded up (1: one tap or no convolution), 0:
 // any number, every earlier input read again for every token; RUN: consecutive tokens of a warp, whose rows (and the
 // TAPS - 1 before them) are all asked for at once.
-template <typename T, int PPL, int TAPS, int RUN>
-__global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
-    const T* __restrict__ proj, long ld, const float* __restrict__ bias, const float* __restrict__ conv_w, int taps,
-    float* __restrict__ tail, long tail_stride, const float* __restrict__ q_w, const float* __restrict__ k_w, int norm_mode,
-    float eps, int rot, int interleaved, const float* __restrict__ cos_t, const float* __restrict__ sin_t, float temp_coef,
-    int temp_every, float v_scale, const ChRows rows, T* __restrict__ q_out, long q_ld, int heads, int kv_heads, int dim,
-    int vdim, T* __restrict__ cache, long page_stride, int page_size, int page_shift, int n_tokens, int aligned) {
-    pdl_wait();
-    pdl_trigger();
+template <typename T> struct ChArgs {
+    const T* proj;
+    long ld;
+    const float *bias, *conv_w;
+    int taps;
+    float* tail;
+    long tail_stride;
+    const float *q_w, *k_w;
+    int norm_mode;
+    float eps;
+    int rot, interleaved;
+    const float *cos_t, *sin_t;
+    float temp_coef;
+    int temp_every;
+    float v_scale;
+    ChRows rows;
+    T* q_out;
+    long q_ld;
+    int heads, kv_heads, dim, vdim;
+    T* cache;
+    long page_stride;
+    int page_size, page_shift, n_tokens, aligned;
+};
+
+template <typename T, int PPL, int TAPS, int RUN, int MODE>
+__device__ __forceinline__ void conv_head_body(const ChArgs<T>& a, const int unit, const int lane) {
     constexpr int HIST = TAPS > 1 ? TAPS - 1 : 0;                     // rows before the run that its tokens may need
     constexpr int KEPT = TAPS > 0 ? TAPS : 1, E = 2 * PPL;
-    const int lane = threadIdx.x & 31;
-    const int unit = blockIdx.y * CH_WARPS + (threadIdx.x >> 5);
-    if (unit >= heads + 2 * kv_heads) return;
+    const int heads = a.heads, kv_heads = a.kv_heads, dim = a.dim, vdim = a.vdim, taps = a.taps, n_tokens = a.n_tokens;
+    const long ld = a.ld;
     const bool is_q = unit < heads, is_v = unit >= heads + kv_heads;
     const int size = is_v ? vdim : dim;
     const int g = is_q ? 0 : (is_v ? unit - heads - kv_heads : unit - heads);
     const int col0 = is_v ? (heads + kv_heads) * dim + g * vdim : unit * dim;
     const int channels = (heads + kv_heads) * dim + kv_heads * vdim;
-    const int turn = is_v ? 0 : rot, half = turn / 2;
-    const bool side = interleaved || turn == 0;                       // a pair's two channels are neighbours
-    ChLane<PPL> at;
-    at.size = size; at.turn = turn; at.half = half; at.slot0 = PPL * lane; at.side = side;
-    at.mode = aligned && side && size % E == 0 ? CH_RUN : aligned && !side && turn == size && half % PPL == 0 ? CH_HALVES : CH_ANY;
+    const int turn = is_v ? 0 : a.rot, half = turn / 2;
+    ChLane<PPL, MODE> at;
+    at.size = size; at.turn = turn; at.half = half; at.slot0 = PPL * lane;
+    at.side = a.interleaved || turn == 0;
     const int t0 = blockIdx.x * RUN;
 
     // everything that does not depend on something else is asked for first
-    float x[HIST + RUN][E];                                           // as projected, without the bias
+    float x[HIST + RUN][E];                                           // as projected, without the a.bias
     {
-        const T* row = proj + (long)(t0 - HIST) * ld + col0;
+        const T* row = a.proj + (long)(t0 - HIST) * ld + col0;
 #pragma unroll
         for (int i = 0; i < HIST + RUN; ++i, row += ld) {
             const int t = t0 + i - HIST;
@@ -191,26 +206,26 @@ __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
     // what the step's tables say of the run's tokens, a token a lane
     int l_pos = 0, l_slot = 0, l_local = 0, l_row = 0, l_single = 0;  // local: tokens of the request in this step before it
     if (lane < RUN && t0 + lane < n_tokens) {
-        l_pos = rows.positions[t0 + lane];
-        l_slot = rows.slots[t0 + lane];
+        l_pos = a.rows.positions[t0 + lane];
+        l_slot = a.rows.slots[t0 + lane];
         if (TAPS != 1) {
-            const int r = rows.tok_req[t0 + lane];
-            l_local = t0 + lane - rows.req_start[r];
-            l_row = rows.req_slot[r];
-            l_single = rows.req_qlen[r] == 1;
+            const int r = a.rows.tok_req[t0 + lane];
+            l_local = t0 + lane - a.rows.req_start[r];
+            l_row = a.rows.req_slot[r];
+            l_single = a.rows.req_qlen[r] == 1;
         }
     }
     float b[E], gain[E], w[KEPT][E];
-    const float* gain_p = is_v || norm_mode != 1 ? nullptr : (is_q ? q_w : k_w);
+    const float* gain_p = is_v || a.norm_mode != 1 ? nullptr : (is_q ? a.q_w : a.k_w);
 #pragma unroll
     for (int e = 0; e < E; ++e) { b[e] = 0.0f; gain[e] = 1.0f; }
-    if (bias != nullptr) at.get(bias + col0, b);
+    if (a.bias != nullptr) at.get(a.bias + col0, b);
     if (gain_p != nullptr) at.get(gain_p, gain, 1.0f);
-    if (TAPS > 0 && conv_w != nullptr) {
+    if (TAPS > 0 && a.conv_w != nullptr) {
 #pragma unroll
         for (int j = 0; j < KEPT; ++j) {                              // tap j of the window is tap j - (KEPT - taps) of w
             const int k = j - (KEPT - taps);
-            if (k >= 0) at.get(conv_w + (long)k * channels + col0, w[j]);
+            if (k >= 0) at.get(a.conv_w + (long)k * channels + col0, w[j]);
             else
 #pragma unroll
                 for (int e = 0; e < E; ++e) w[j][e] = 0.0f;
@@ -223,16 +238,49 @@ __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
         pos[u] = __shfl_sync(0xffffffffu, l_pos, u);
         const long line = (long)pos[u] * half + at.slot0;
         if (at.slot0 + PPL <= half && half % PPL == 0) {
-            ch_get<PPL>(cos_t + line, cosv[u]);
-            ch_get<PPL>(sin_t + line, sinv[u]);
+            ch_get<PPL>(a.cos_t + line, cosv[u]);
+            ch_get<PPL>(a.sin_t + line, sinv[u]);
         } else {
 #pragma unroll
             for (int p = 0; p < PPL; ++p) {
-                cosv[u][p] = at.slot0 + p < half ? cos_t[line + p] : 1.0f;
-                sinv[u][p] = at.slot0 + p < half ? sin_t[line + p] : 0.0f;
+                cosv[u][p] = at.slot0 + p < half ? a.cos_t[line + p] : 1.0f;
+                sinv[u][p] = at.slot0 + p < half ? a.sin_t[line + p] : 0.0f;
             }
         }
     }
+
+    // a token's convolution with its inputs read one after another (oldest first, as everywhere), and its request's state
+    auto any_taps = [&](int t, int p, int local, float* mine, int single, float (&y)[E]) {
+        float keep[E], sum[E], wj[E], h[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) { keep[e] = y[e]; sum[e] = 0.0f; }
+#pragma unroll 1
+        for (int j = 0; j < taps - 1; ++j) {
+            const int back = taps - 1 - j;
+            if (p < back) continue;
+            at.get(a.conv_w + (long)j * channels + col0, wj);
+            if (local >= back) {
+                at.get(a.proj + (long)(t - back) * ld + col0, h);
+#pragma unroll
+                for (int e = 0; e < E; ++e) h[e] += b[e];
+            } else {
+                at.get(mine + (long)(local - back + taps - 1) * channels, h);
+            }
+#pragma unroll
+            for (int e = 0; e < E; ++e) sum[e] = fmaf(wj[e], h[e], sum[e]);
+        }
+        at.get(a.conv_w + (long)(taps - 1) * channels + col0, wj);
+#pragma unroll
+        for (int e = 0; e < E; ++e) y[e] = fmaf(wj[e], y[e], sum[e]);
+        if (single && taps > 1) {
+#pragma unroll 1
+            for (int k = 0; k + 1 < taps - 1; ++k) {
+                at.get(mine + (long)(k + 1) * channels, h);
+                at.put(mine + (long)k * channels, h);
+            }
+            at.put(mine + (long)(taps - 2) * channels, keep);
+        }
+    };
 
 #pragma unroll
     for (int u = 0; u < RUN; ++u) {
@@ -245,14 +293,17 @@ __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
             // input `back` positions behind: from the step's rows, from the kept rows, or zero before the sequence's start
             const int local = __shfl_sync(0xffffffffu, l_local, u), state_row = __shfl_sync(0xffffffffu, l_row, u);
             const int single = __shfl_sync(0xffffffffu, l_single, u);
-            float* mine = tail + (long)state_row * tail_stride + col0;
+            float* mine = a.tail + (long)state_row * a.tail_stride + col0;
             float h[HIST][E];                                         // oldest first
 #pragma unroll
             for (int j = 0; j < HIST; ++j) {
 #pragma unroll
                 for (int e = 0; e < E; ++e) h[j][e] = x[u + j][e] + b[e];
             }
-            if (local < HIST && t < n_tokens) {                       // the same for the whole warp
+            if (RUN > 1 && local < HIST) {                            // (the same for the whole warp) few tokens of a long step
+                if (t < n_tokens) any_taps(t, pos[u], local, mine, single, y);
+            } else {
+            if (RUN == 1 && local < HIST && t < n_tokens) {           // the same for the whole warp
 #pragma unroll
                 for (int j = 0; j < HIST; ++j) {
                     const int back = HIST - j;
@@ -274,91 +325,80 @@ __global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(
                 for (int j = 0; j < HIST; ++j) sum = fmaf(w[j][e], h[j][e], sum);
                 y[e] = fmaf(w[TAPS - 1][e], y[e], sum);
             }
-            if (single && t < n_tokens) {                             // the request's new state: the last taps - 1 inputs
+            if (RUN == 1 && single && t < n_tokens) {                 // the request's new state: the last taps - 1 inputs
 #pragma unroll
                 for (int j = 0; j < HIST; ++j) {
                     const int k = j - (TAPS - taps);
                     if (k >= 0) at.put(mine + (long)k * channels, j + 1 < HIST ? h[j + 1 < HIST ? j + 1 : j] : keep);
                 }
             }
+            }
         }
         if constexpr (TAPS == 0) {
             const int local = __shfl_sync(0xffffffffu, l_local, u), state_row = __shfl_sync(0xffffffffu, l_row, u);
             const int single = __shfl_sync(0xffffffffu, l_single, u);
-            float* mine = tail + (long)state_row * tail_stride + col0;
-            float keep[E], sum[E], wj[E], h[E];
-#pragma unroll
-            for (int e = 0; e < E; ++e) { keep[e] = y[e]; sum[e] = 0.0f; }
-            for (int j = 0; j < taps - 1 && t < n_tokens; ++j) {      // oldest first
-                const int back = taps - 1 - j;
-                if (pos[u] < back) continue;
-                at.get(conv_w + (long)j * channels + col0, wj);
-                if (local >= back) {
-                    at.get(proj + (long)(t - back) * ld + col0, h);
-#pragma unroll
-                    for (int e = 0; e < E; ++e) h[e] += b[e];
-                } else {
-                    at.get(mine + (long)(local - back + taps - 1) * channels, h);
-                }
-#pragma unroll
-                for (int e = 0; e < E; ++e) sum[e] = fmaf(wj[e], h[e], sum[e]);
-            }
-            at.get(conv_w + (long)(taps - 1) * channels + col0, wj);
-#pragma unroll
-            for (int e = 0; e < E; ++e) y[e] = fmaf(wj[e], y[e], sum[e]);
-            if (single && t < n_tokens) {
-                for (int k = 0; k + 1 < taps - 1; ++k) {
-                    at.get(mine + (long)(k + 1) * channels, h);
-                    at.put(mine + (long)k * channels, h);
-                }
-                at.put(mine + (long)(taps - 2) * channels, keep);
-            }
+            float* mine = a.tail + (long)state_row * a.tail_stride + col0;
+            if (t < n_tokens) any_taps(t, pos[u], local, mine, single, y);
         }
         if constexpr (TAPS == 1) {
-            if (conv_w != nullptr) {
+            if (a.conv_w != nullptr) {
 #pragma unroll
                 for (int e = 0; e < E; ++e) y[e] *= w[0][e];
             }
         }
         if (is_v) {
 #pragma unroll
-            for (int e = 0; e < E; ++e) y[e] *= v_scale;
+            for (int e = 0; e < E; ++e) y[e] *= a.v_scale;
         } else {
-            if (norm_mode == 1) {
+            if (a.norm_mode == 1) {
                 float ss = 0.0f;
 #pragma unroll
                 for (int e = 0; e < E; ++e) ss = fmaf(y[e], y[e], ss);
-                const float inv = ch_rms<T>(warp_sum(ss), dim, eps);
+                const float inv = ch_rms<T>(warp_sum(ss), dim, a.eps);
 #pragma unroll
                 for (int e = 0; e < E; ++e) y[e] = y[e] * inv * gain[e];
             }
 #pragma unroll
             for (int p = 0; p < PPL; ++p) {
-                const float a = y[2 * p], c = y[2 * p + 1];           // (no rotation: cos 1, sin 0)
-                y[2 * p] = a * cosv[u][p] - c * sinv[u][p];
-                y[2 * p + 1] = c * cosv[u][p] + a * sinv[u][p];
+                const float v = y[2 * p], c = y[2 * p + 1];           // (no rotation: cos 1, sin 0)
+                y[2 * p] = v * cosv[u][p] - c * sinv[u][p];
+                y[2 * p + 1] = c * cosv[u][p] + v * sinv[u][p];
             }
             float f = 1.0f;
-            if (norm_mode == 2) {
+            if (a.norm_mode == 2) {
                 float ss = 0.0f;
 #pragma unroll
                 for (int e = 0; e < E; ++e) ss = fmaf(y[e], y[e], ss);
-                f = ch_rms<T>(warp_sum(ss), dim, eps);
+                f = ch_rms<T>(warp_sum(ss), dim, a.eps);
             }
-            if (is_q && temp_every > 0) f *= 1.0f + temp_coef * logf((float)((pos[u] + 1) / temp_every) + 1.0f);
+            if (is_q && a.temp_every > 0) f *= 1.0f + a.temp_coef * logf((float)((pos[u] + 1) / a.temp_every) + 1.0f);
 #pragma unroll
             for (int e = 0; e < E; ++e) y[e] *= f;
         }
         if (t >= n_tokens) continue;
         T* dst;
         if (is_q) {
-            dst = q_out + (long)t * q_ld + (long)unit * dim;
+            dst = a.q_out + (long)t * a.q_ld + (long)unit * dim;
         } else {
-            const int page = page_shift >= 0 ? slot >> page_shift : slot / page_size;
-            dst = cache + (long)page * page_stride + ((long)g * page_size + (slot - page * page_size)) * (dim + vdim) + (is_v ? dim : 0);
+            const int page = a.page_shift >= 0 ? slot >> a.page_shift : slot / a.page_size;
+            dst = a.cache + (long)page * a.page_stride + ((long)g * a.page_size + (slot - page * a.page_size)) * (dim + vdim) + (is_v ? dim : 0);
         }
         at.put(dst, y);
     }
+}
+
+template <typename T, int PPL, int TAPS, int RUN>
+__global__ void __launch_bounds__(32 * CH_WARPS) conv_head_prep_kernel(const ChArgs<T> a) {
+    pdl_wait();
+    pdl_trigger();
+    const int unit = blockIdx.y * CH_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= a.heads + 2 * a.kv_heads) return;
+    const bool is_v = unit >= a.heads + a.kv_heads;
+    const int size = is_v ? a.vdim : a.dim, turn = is_v ? 0 : a.rot;
+    const bool side = a.interleaved || turn == 0;                     // a pair's two channels are neighbours
+    if (a.aligned && side && size % (2 * PPL) == 0) conv_head_body<T, PPL, TAPS, RUN, CH_RUN>(a, unit, lane);
+    else if (a.aligned && !side && turn == size && turn / 2 % PPL == 0) conv_head_body<T, PPL, TAPS, RUN, CH_HALVES>(a, unit, lane);
+    else conv_head_body<T, PPL, TAPS, RUN, CH_ANY>(a, unit, lane);
 }
 
 template <typename T>
@@ -412,12 +452,13 @@ FL_API int fl_conv_head_prep(const void* proj, int dtype, long ld, const float* 
         for (page_shift = 0; (1 << page_shift) < page_size;) ++page_shift;
     int rc = 0;
 #define FL_CH(PPL, TAPS, RUN)                                                                                            \
-    FL_DISPATCH(dtype, T, rc = fl_launch(conv_head_prep_kernel<T, PPL, TAPS, RUN>,                                        \
-                                         dim3((n_tokens + RUN - 1) / RUN, (units + CH_WARPS - 1) / CH_WARPS),            \
-                                         dim3(32 * CH_WARPS), 0, stream, (const T*)proj, ld, bias, conv_w, taps, tail,   \
-                                         tail_stride, q_w, k_w, norm_mode, eps, rot, interleaved, cos_t, sin_t,          \
-                                         temp_coef, temp_every, v_scale, rows, (T*)q_out, q_ld, heads, kv_heads, dim,    \
-                                         vdim, (T*)cache, page_stride, page_size, page_shift, n_tokens, aligned))
+    FL_DISPATCH(dtype, T, {                                                                                             \
+        const ChArgs<T> a{(const T*)proj, ld, bias, conv_w, taps, tail, tail_stride, q_w, k_w, norm_mode, eps, rot, interleaved, \
+                          cos_t, sin_t, temp_coef, temp_every, v_scale, rows, (T*)q_out, q_ld, heads, kv_heads, dim, vdim, \
+                          (T*)cache, page_stride, page_size, page_shift, n_tokens, aligned};                            \
+        rc = fl_launch(conv_head_prep_kernel<T, PPL, TAPS, RUN>, dim3((n_tokens + RUN - 1) / RUN, (units + CH_WARPS - 1) / CH_WARPS), \
+                       dim3(32 * CH_WARPS), 0, stream, a);                                                              \
+    })
 #define FL_CH_TAPS(PPL, RUN)                                                                                             \
     { if (taps == 1) { FL_CH(PPL, 1, RUN); } else if (taps <= 4) { FL_CH(PPL, 4, RUN); } else { FL_CH(PPL, 0, 1); } }
     const bool many = n_tokens >= 256;
