@@ -81,11 +81,11 @@ FL_API int fl_gla_prep(const void* proj, int dtype, long ld, const float* w2, co
 // work: what fl_gla_prep leaves.  single_tokens: every request of the step brings one token.
 FL_API int fl_gla_scan(const float* work, long w_ld, float* o, long o_ld, float* state, long state_stride,
                        const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot, int n_requests,
-                       int heads, int dim, int vdim, int single_tokens, int sms, cudaStream_t stream) {
+                       int heads, int dim, int vdim, int single_tokens, cudaStream_t stream) {
     const int hd = heads * dim;
     const ScanToken at{hd, 0, dim, 1, 2 * hd, 3 * hd, 0, 0};
     return state_scan<false>(work, w_ld, at, nullptr, o, o_ld, state, state_stride, req_start, req_ctx, req_qlen, req_slot,
-                             n_requests, heads, dim, vdim, single_tokens, sms, stream);
+                             n_requests, heads, dim, vdim, single_tokens, stream);
 }
 
 FL_API int fl_gla_gated_norm(const float* o, long o_ld, const void* gate, int dtype, long g_ld, const void* weight,

@@ -357,13 +357,13 @@ static inline bool ssd_takes(int n_requests, int heads, int vdim, int n, int gro
 // work: what fl_ssd_prep leaves.  single_tokens: every request of the step brings one token.
 FL_API int fl_ssd_scan(const float* work, long w_ld, const float* skip, float* y, long y_ld, float* state, long state_stride,
                        const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot, int n_requests,
-                       int heads, int vdim, int n, int groups, int single_tokens, int sms, cudaStream_t stream) {
+                       int heads, int vdim, int n, int groups, int single_tokens, cudaStream_t stream) {
     if (n_requests <= 0) return 0;
     if (!ssd_takes(n_requests, heads, vdim, n, groups)) return (int)cudaErrorInvalidValue;
     const int inner = heads * vdim, gn = groups * n;
     const ScanToken at{inner, inner + gn, n, heads / groups, 0, 0, inner + 2 * gn, inner + 2 * gn + heads};
     return state_scan<true>(work, w_ld, at, skip, y, y_ld, state, state_stride, req_start, req_ctx, req_qlen, req_slot, n_requests,
-                            heads, n, vdim, single_tokens, sms, stream);
+                            heads, n, vdim, single_tokens, stream);
 }
 
 // Steps of single tokens only: row r of proj is request r's.

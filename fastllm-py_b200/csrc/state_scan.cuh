@@ -7,19 +7,20 @@
 // given columns; heads may share k and q in groups.  A request's state row holds [heads][p][n] (a column of S is
 // contiguous); it is read unless the request starts (context 0) and written at the end.
 //
-// A block takes one request, one head and COLS columns of S.  LANES lanes share CPT columns; a lane holds R rows of each in
+// A block takes one request, one head and COLS columns of S.  LANES lanes share four columns; a lane holds R rows of each in
 // its registers: the groups of four rows lane + LANES i, so that the lanes read consecutive 16 bytes of a staged row
 // (n <= LANES R; rows beyond n stay zero).  Neighbouring rows are packed pairs of floats, which one instruction of the
 // float pipe works on.  Tokens come through four stages of shared memory, three chunks being copied (cp.async) while one is
-// walked; they go four at a time, so that the read-out sums of four tokens and CPT columns are added up over the lanes
+// walked; they go four at a time, so that the read-out sums of four tokens and four columns are added up over the lanes
 // together, each exchange halving what a lane still holds.  Tokens beyond the portion's end leave S as it is (decay 1,
-// nothing added).  R and LANES follow from n alone and a column's sum does not depend on CPT or COLS, so every result's
-// order of sums is fixed by the sizes: cuts and batches agree bit for bit.
+// nothing added).  R and LANES follow from n alone, so every result's order of sums is fixed by the sizes: cuts and batches
+// agree bit for bit.
 #pragma once
 
 #include "common.cuh"
 
 #define SCAN_STAGES 4
+#define SCAN_CPT 4                   // columns of S that a thread holds rows of
 
 struct ScanToken {                   // columns of a token's row, and how heads step through them
     int k0, q0, n_step, per_group;   // head h's k and q: at k0 / q0 + (h / per_group) * n_step
@@ -64,13 +65,14 @@ __device__ __forceinline__ float scan_fold(bool up, float low, float high, int o
     return (up ? high : low) + __shfl_xor_sync(0xffffffffu, up ? low : high, off);
 }
 
-template <int R, int LANES, int CPT, int COLS, bool SCALAR, int CHUNK>
-__global__ void __launch_bounds__(COLS / CPT * LANES) state_scan_kernel(
+template <int R, int LANES, int COLS, bool SCALAR, int CHUNK>
+__global__ void __launch_bounds__(COLS / SCAN_CPT * LANES, 1) state_scan_kernel(
     const float* __restrict__ rows, long ld, const ScanToken at, const float* __restrict__ skip, float* __restrict__ y,
     long y_ld, float* __restrict__ state, long state_stride, const int* __restrict__ req_start,
     const int* __restrict__ req_ctx, const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int n, int p,
     int vec4, int state_vec4) {
-    static_assert(CHUNK % 4 == 0 && R % 4 == 0 && (LANES == 8 || LANES == 16) && (CPT == 1 || CPT == 2 || CPT == 4), "");
+    constexpr int CPT = SCAN_CPT;
+    static_assert(CHUNK % 4 == 0 && R % 4 == 0 && (LANES == 8 || LANES == 16) && CPT == 4, "");
     pdl_wait();
     constexpr int DP = R * LANES, VECS = SCALAR ? 2 : 3;              // a staged token: k | q | (a) | v | (dt, decay)
     constexpr int TOKEN = VECS * DP + COLS + 4;
@@ -142,10 +144,8 @@ __global__ void __launch_bounds__(COLS / CPT * LANES) state_scan_kernel(
     }
     // the token of a group of four and the (first) column whose sum this lane is left with
     constexpr int REM = LANES / 4;                                    // lanes that share one token's sums
-    const int my_u = lane / REM;
-    const int my_k = CPT == 1 ? 0 : CPT == 2 ? (lane & (REM - 1)) / (REM / 2) : REM == 4 ? lane & 3 : 2 * (lane & 1);
-    constexpr int LEFT = CPT == 4 && REM == 2 ? 2 : 1;                // sums a lane is left with
-    const bool writes = CPT == 4 ? true : CPT == 2 ? (lane & (REM / 2 - 1)) == 0 : (lane & (REM - 1)) == 0;
+    constexpr int LEFT = 4 / REM;                                     // sums a lane is left with (1 or 2)
+    const int my_u = lane / REM, my_k = LEFT * (lane & (REM - 1));
     float* yp = y + (long)(start + my_u) * y_ld + (long)h * p + col0 + cg + my_k;
     int stage = 0;
     for (int c0 = 0; c0 < qlen; c0 += CHUNK, stage = (stage + 1) % SCAN_STAGES) {
@@ -155,54 +155,65 @@ __global__ void __launch_bounds__(COLS / CPT * LANES) state_scan_kernel(
         asm volatile("cp.async.wait_group %0;" ::"n"(SCAN_STAGES - 1));
         __syncthreads();                                              // this chunk has landed
         const float* tok = scan_s + stage * CHUNK * TOKEN;
-#pragma unroll 1
-        for (int t4 = 0; t4 < here; t4 += 4, tok += 4 * TOKEN, yp += 4 * y_ld) {
+        // four tokens from `tok` on, of which the first `left` are the portion's (whole: all of them are)
+        auto group = [&](const float* tok, float* yp, int left, bool whole) {
+            // the rows of AHEAD tokens are read into registers before the first of them is used
+            constexpr int AHEAD = VECS * R <= 16 ? 4 : VECS * R <= 32 ? 2 : 1;
             float acc[4][CPT];
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const float* tu = tok + u * TOKEN;
-                const bool real = t4 + u < here;
-                float x[CPT];
+            for (int u0 = 0; u0 < 4; u0 += AHEAD) {
+                ulonglong2 kk[AHEAD][R / 4], qq[AHEAD][R / 4], aa[AHEAD][R / 4];
+                float x[AHEAD][CPT];
+                scan_f2 a2[AHEAD] = {};
 #pragma unroll
-                for (int k = 0; k < CPT; ++k) x[k] = tu[VECS * DP + cg + k];
-                scan_f2 a2 = 0;
-                if (SCALAR) {
-                    const float2 rate = *reinterpret_cast<const float2*>(tu + VECS * DP + COLS);
-                    const float dt = real ? rate.x : 0.0f, decay = real ? rate.y : 1.0f;
-                    a2 = scan_pack(decay, decay);
+                for (int w = 0; w < AHEAD; ++w) {
+                    const float* tu = tok + (u0 + w) * TOKEN;
+                    const bool real = whole || u0 + w < left;
 #pragma unroll
-                    for (int k = 0; k < CPT; ++k) x[k] *= dt;
-                } else {
+                    for (int i = 0; i < R / 4; ++i) {
+                        kk[w][i] = reinterpret_cast<const ulonglong2*>(tu)[lane + LANES * i];
+                        qq[w][i] = reinterpret_cast<const ulonglong2*>(tu + DP)[lane + LANES * i];
+                        if (!SCALAR) {
+                            aa[w][i] = reinterpret_cast<const ulonglong2*>(tu + 2 * DP)[lane + LANES * i];
+                            if (!real) aa[w][i] = make_ulonglong2(scan_pack(1.0f, 1.0f), scan_pack(1.0f, 1.0f));
+                        }
+                    }
+                    const float4 v = *reinterpret_cast<const float4*>(tu + VECS * DP + cg);
+                    x[w][0] = v.x; x[w][1] = v.y; x[w][2] = v.z; x[w][3] = v.w;
+                    float dt = real ? 1.0f : 0.0f;
+                    if (SCALAR) {
+                        const float2 rate = *reinterpret_cast<const float2*>(tu + VECS * DP + COLS);
+                        dt = real ? rate.x : 0.0f;
+                        const float decay = real ? rate.y : 1.0f;
+                        a2[w] = scan_pack(decay, decay);
+                    }
 #pragma unroll
-                    for (int k = 0; k < CPT; ++k) x[k] = real ? x[k] : 0.0f;
+                    for (int k = 0; k < CPT; ++k) x[w][k] *= dt;
                 }
-                scan_f2 x2[CPT], sum[CPT];
 #pragma unroll
-                for (int k = 0; k < CPT; ++k) x2[k] = scan_pack(x[k], x[k]);
+                for (int w = 0; w < AHEAD; ++w) {
+                    scan_f2 x2[CPT], sum[CPT];
 #pragma unroll
-                for (int i = 0; i < R / 4; ++i) {
-                    const ulonglong2 kk = reinterpret_cast<const ulonglong2*>(tu)[lane + LANES * i];
-                    const ulonglong2 qq = reinterpret_cast<const ulonglong2*>(tu + DP)[lane + LANES * i];
-                    ulonglong2 aa = make_ulonglong2(a2, a2);
-                    if (!SCALAR) {
-                        aa = reinterpret_cast<const ulonglong2*>(tu + 2 * DP)[lane + LANES * i];
-                        if (!real) aa = make_ulonglong2(scan_pack(1.0f, 1.0f), scan_pack(1.0f, 1.0f));
+                    for (int k = 0; k < CPT; ++k) x2[k] = scan_pack(x[w][k], x[w][k]);
+#pragma unroll
+                    for (int i = 0; i < R / 4; ++i) {
+                        const scan_f2 ax = SCALAR ? a2[w] : aa[w][i].x, ay = SCALAR ? a2[w] : aa[w][i].y;
+#pragma unroll
+                        for (int k = 0; k < CPT; ++k) {
+                            S[k][2 * i] = scan_fma2(ax, S[k][2 * i], scan_mul2(kk[w][i].x, x2[k]));
+                            sum[k] = i == 0 ? scan_mul2(S[k][0], qq[w][0].x) : scan_fma2(S[k][2 * i], qq[w][i].x, sum[k]);
+                            S[k][2 * i + 1] = scan_fma2(ay, S[k][2 * i + 1], scan_mul2(kk[w][i].y, x2[k]));
+                            sum[k] = scan_fma2(S[k][2 * i + 1], qq[w][i].y, sum[k]);
+                        }
                     }
 #pragma unroll
                     for (int k = 0; k < CPT; ++k) {
-                        S[k][2 * i] = scan_fma2(aa.x, S[k][2 * i], scan_mul2(kk.x, x2[k]));
-                        sum[k] = i == 0 ? scan_mul2(S[k][0], qq.x) : scan_fma2(S[k][2 * i], qq.x, sum[k]);
-                        S[k][2 * i + 1] = scan_fma2(aa.y, S[k][2 * i + 1], scan_mul2(kk.y, x2[k]));
-                        sum[k] = scan_fma2(S[k][2 * i + 1], qq.y, sum[k]);
+                        const float2 v = scan_unpack(sum[k]);
+                        acc[u0 + w][k] = v.x + v.y;
                     }
                 }
-#pragma unroll
-                for (int k = 0; k < CPT; ++k) {
-                    const float2 v = scan_unpack(sum[k]);
-                    acc[u][k] = v.x + v.y;
-                }
             }
-            // over the lanes: first by token, then by column, then what is left plainly
+            // over the lanes: first by token, then by column
             float w[2][CPT], v[CPT];
             const bool b3 = lane & (LANES / 2), b2 = lane & (LANES / 4);
 #pragma unroll
@@ -211,23 +222,23 @@ __global__ void __launch_bounds__(COLS / CPT * LANES) state_scan_kernel(
                 for (int k = 0; k < CPT; ++k) w[u][k] = scan_fold(b3, acc[u][k], acc[u + 2][k], LANES / 2);
 #pragma unroll
             for (int k = 0; k < CPT; ++k) v[k] = scan_fold(b2, w[0][k], w[1][k], LANES / 4);
-            if constexpr (CPT == 4) {
-                const bool b1 = lane & (REM / 2);
-                v[0] = scan_fold(b1, v[0], v[2], REM / 2);
-                v[1] = scan_fold(b1, v[1], v[3], REM / 2);
-                if constexpr (REM == 4) v[0] = scan_fold(lane & 1, v[0], v[1], 1);
-            } else if constexpr (CPT == 2) {
-                v[0] = scan_fold(lane & (REM / 2), v[0], v[1], REM / 2);
-                if constexpr (REM == 4) v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
-            } else {
-#pragma unroll
-                for (int off = REM / 2; off > 0; off >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], off);
-            }
+            const bool b1 = lane & (REM / 2);
+            v[0] = scan_fold(b1, v[0], v[2], REM / 2);
+            v[1] = scan_fold(b1, v[1], v[3], REM / 2);
+            if constexpr (REM == 4) v[0] = scan_fold(lane & 1, v[0], v[1], 1);
 #pragma unroll
             for (int k = 0; k < LEFT; ++k)
-                if (writes && t4 + my_u < here && cg + my_k + k < cols)
+                if ((whole || my_u < left) && cg + my_k + k < cols)
                     yp[k] = skip != nullptr ? fmaf(skip_h, tok[my_u * TOKEN + VECS * DP + cg + my_k + k], v[k]) : v[k];
+        };
+        if (here == CHUNK) {                                          // straight-line: a group's reads overlap the sums before it
+#pragma unroll
+            for (int t4 = 0; t4 < CHUNK; t4 += 4) group(tok + t4 * TOKEN, yp + t4 * y_ld, 4, true);
+        } else {
+#pragma unroll 1
+            for (int t4 = 0; t4 < here; t4 += 4) group(tok + t4 * TOKEN, yp + t4 * y_ld, here - t4, false);
         }
+        yp += CHUNK * y_ld;
         __syncthreads();                                              // the stage is copied into again in the next round
     }
     pdl_trigger();                                                    // (not at the start: the successor's CTAs would only wait here)
@@ -250,31 +261,30 @@ __global__ void __launch_bounds__(COLS / CPT * LANES) state_scan_kernel(
         }
 }
 
-template <int R, int LANES, int CPT, int COLS, bool SCALAR>
+template <int R, int LANES, int COLS, bool SCALAR>
 static int state_scan_launch(const float* rows, long ld, const ScanToken& at, const float* skip, float* y, long y_ld, float* state,
                              long state_stride, const int* req_start, const int* req_ctx, const int* req_qlen,
                              const int* req_slot, int n_requests, int heads, int n, int p, int vec4, int state_vec4, bool overlap,
                              cudaStream_t stream) {
     constexpr int CHUNK = R * LANES <= 128 ? 16 : 8;
     constexpr size_t smem = (size_t)SCAN_STAGES * CHUNK * ((SCALAR ? 2 : 3) * R * LANES + COLS + 4) * sizeof(float);
-    auto kernel = state_scan_kernel<R, LANES, CPT, COLS, SCALAR, CHUNK>;
+    auto kernel = state_scan_kernel<R, LANES, COLS, SCALAR, CHUNK>;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return fl_launch_as(overlap, kernel, dim3(n_requests, heads, (p + COLS - 1) / COLS), dim3(COLS / CPT * LANES), smem, stream,
+    return fl_launch_as(overlap, kernel, dim3(n_requests, heads, (p + COLS - 1) / COLS), dim3(COLS / SCAN_CPT * LANES), smem, stream,
                         rows, ld, at, skip, y, y_ld, state, state_stride, req_start, req_ctx, req_qlen, req_slot, n, p, vec4,
                         state_vec4);
 }
 
-// single_tokens: every request of the step brings one token.  sms: the GPU's SMs; with few requests a thread takes fewer
-// columns, so that every SM has warps to switch between.
+// single_tokens: every request of the step brings one token.
 template <bool SCALAR>
 static int state_scan(const float* rows, long ld, const ScanToken& at, const float* skip, float* y, long y_ld, float* state,
                       long state_stride, const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot,
-                      int n_requests, int heads, int n, int p, int single_tokens, int sms, cudaStream_t stream) {
+                      int n_requests, int heads, int n, int p, int single_tokens, cudaStream_t stream) {
     if (n_requests <= 0) return 0;
     if (n < 1 || n > 256 || p < 1 || heads < 1 || heads > 65535 || (p + 15) / 16 > 65535 || at.per_group < 1)
         return (int)cudaErrorInvalidValue;
@@ -283,19 +293,13 @@ static int state_scan(const float* rows, long ld, const ScanToken& at, const flo
                      at.n_step % 4 == 0 && at.a0 % 4 == 0 && at.v0 % 4 == 0;
     const int state_vec4 = n % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0;
     const bool overlap = single_tokens != 0;         // (short kernels gain from the overlap, long ones need the SMs evenly)
-    // warps of the launch at four columns a thread, and how many of them an SM gets
-    const int lanes = n <= 32 ? 8 : 16;
-    const long warps = (long)n_requests * heads * p * lanes / (4 * 32);
-    const int cpt = warps >= 12L * sms ? 4 : warps >= 3L * sms ? 2 : 1;
-#define SCAN_GO(R, L, CPT, COLS)                                                                                           \
-    return state_scan_launch<R, L, CPT, COLS, SCALAR>(rows, ld, at, skip, y, y_ld, state, state_stride, req_start, req_ctx,    \
-                                                      req_qlen, req_slot, n_requests, heads, n, p, vec4, state_vec4, overlap, stream)
-#define SCAN_COLS(R, L)                                                                                                    \
-    {                                                                                                                      \
-        if (cpt == 1) SCAN_GO(R, L, 1, 16);                                                                                \
-        if (p <= 16) SCAN_GO(R, L, 2, 16);                                                                                 \
-        if (cpt == 2) SCAN_GO(R, L, 2, 32);                                                                                \
-        SCAN_GO(R, L, 4, 32);                                                                                              \
+#define SCAN_GO(R, L, COLS)                                                                                                 \
+    return state_scan_launch<R, L, COLS, SCALAR>(rows, ld, at, skip, y, y_ld, state, state_stride, req_start, req_ctx, req_qlen, \
+                                                 req_slot, n_requests, heads, n, p, vec4, state_vec4, overlap, stream)
+#define SCAN_COLS(R, L)                                                                                                     \
+    {                                                                                                                       \
+        if (p <= 16) SCAN_GO(R, L, 16);                                                                                     \
+        SCAN_GO(R, L, 32);                                                                                                  \
     }
     if (n <= 32) SCAN_COLS(4, 8)
     if (n <= 64) SCAN_COLS(4, 16)

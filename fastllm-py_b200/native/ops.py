@@ -927,10 +927,10 @@ def ssd_scan(work, skip, y, state_rows, step, heads, vdim, state, groups):
     if any(v.dtype != torch.float32 for v in (work, skip, y, state_rows)):
         raise KernelError("ssd_scan: all operands are float32")
     fn = _fn("ssd", "fl_ssd_scan", [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
-                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(work), _ld(work), _ptr(skip), _ptr(y), _ld(y), _ptr(state_rows), state_rows.stride(0), _ptr(step.req_start),
               _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests, heads, vdim, state, groups,
-              int(work.shape[0] == step.n_requests), _sms(work.device), _stream()), "ssd_scan")
+              int(work.shape[0] == step.n_requests), _stream()), "ssd_scan")
 
 
 def ssd_step(proj, conv_w, conv_b, dt_bias, neg_a, skip, y, state_rows, tail_off, step, heads, vdim, state, groups):
@@ -1077,13 +1077,6 @@ def gla_prep(proj, w2, b2, work, heads, dim, vdim, rank, q_scale, tau):
               vdim, rank, float(q_scale), float(tau), _stream()), "gla_prep")
 
 
-def _sms(device) -> int:
-    sms = _sm_counts.get(device)
-    if sms is None:
-        sms = _sm_counts[device] = torch.cuda.get_device_properties(device).multi_processor_count
-    return sms
-
-
 def gla_scan(work, o, state, step, heads, dim, vdim):
     """Per request and head S <- diag(alpha) S + k v^T, o = S^T q over the step's tokens; q | k | alpha | v are the
     float32 columns of `work`, `o` float32 [N, heads * vdim]; state rows [heads, vdim, dim] float32 are read (unless
@@ -1092,10 +1085,10 @@ def gla_scan(work, o, state, step, heads, dim, vdim):
     if work.dtype != torch.float32 or o.dtype != torch.float32 or state.dtype != torch.float32:
         raise KernelError("gla_scan: work, o and state must be float32")
     fn = _fn("gla", "fl_gla_scan", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
-                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(work), _ld(work), _ptr(o), _ld(o), _ptr(state), state.stride(0), _ptr(step.req_start),
               _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests, heads, dim, vdim,
-              int(work.shape[0] == step.n_requests), _sms(work.device), _stream()), "gla_scan")
+              int(work.shape[0] == step.n_requests), _stream()), "gla_scan")
 
 
 def gla_gated_norm(o, gate, weight, out, heads, vdim, eps):

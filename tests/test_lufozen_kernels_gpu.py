@@ -138,7 +138,7 @@ def test_convolved_head_preparation_over_steps(dtype, sizes, taps, rot, pairing,
 
 @pytest.mark.parametrize("sizes", [(2, 12, 20), (1, 64, 128), (3, 40, 33), (2, 100, 16), (1, 250, 70)])
 def test_scan_with_a_decay_per_row_over_steps(sizes):
-    """Bit for bit the same whatever the cut; few and many requests at once (a thread takes one, two or four columns)."""
+    """Bit for bit the same whatever the cut; few and many requests at once."""
     from fastllm_py_b200.native import ops
 
     H, d, dv = sizes
