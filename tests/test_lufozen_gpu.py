@@ -362,3 +362,59 @@ def test_command_line_on_a_random_weights_folder(tmp_path):
     lines = run.stdout.strip().splitlines()
     assert "Lufozen: 2L width=32" in lines[0]
     assert len([int(t) for t in lines[1].split(",")]) == 9
+
+
+def drawn_model(rng):
+    """A configuration drawn at random: layer kinds in any order, any loop, sizes from lists that hold the awkward ones (one
+    head, twelve query heads a key/value head, keys of 72, one tap, one state group or as many as heads)."""
+    ch = rng.choice
+    width, vocab = ch([24, 40, 64, 136]), rng.randint(50, 200)
+
+    def softmax(make, **kw):
+        kv, group, dim = ch([1, 2, 3]), ch([1, 1, 2, 3, 4, 12]), ch([8, 12, 16, 24, 32, 48, 64, 72, 128])
+        rot = None if rng.random() < 0.15 else ch([dim, 2 * rng.randint(1, dim // 2)])
+        scaling = (ch([2.0, 8.0]), ch([16, 64, 512]), ch([0.5, 1.0]), ch([2.0, 4.0])) if rng.random() < 0.7 else None
+        return make(kv * group, kv, dim, ch([4, 8, 24, 32, 48, 100, 128]), rot=rot, base=ch([500.0, 1e6]), scaling=scaling,
+                    scale=ch([dim ** -0.5, 0.1, 0.3]), **kw)
+
+    layers = []
+    for _ in range(rng.randint(2, 5)):
+        kind = ch(["attention", "gla", "parallel"])
+        if kind == "attention":
+            mixer = softmax(lt.attention, conv=ch([1, 2, 3, 4, 4, 6]))
+        elif kind == "gla":
+            mixer = lt.linear(ch([1, 2, 3]), ch([4, 8, 20, 32, 48, 64, 100]), ch([4, 12, 16, 32, 80]), ch([1.0, 4.0, 16.0, 64.0]))
+        else:
+            groups, per, vdim = ch([1, 2, 3]), ch([1, 2, 4]), ch([4, 8, 16, 20, 32, 64])
+            inner = groups * per * vdim
+            parts = ch([p for p in (1, 2, 3, groups, groups * per) if inner % p == 0])
+            mixer = lt.pair(softmax(lt.left), lt.right(groups * per, vdim, ch([4, 12, 16, 32, 50, 64, 128, 200]), groups,
+                                                       ch([1, 2, 3, 4, 4, 5]), parts), ch([0.6, 1.0, -0.4]), ch([0.5, 1.0, 1.7]))
+        layers.append((mixer, None if rng.random() < 0.3 else lt.dense(ch([16, 30, 64, 256]))))
+    loop = None
+    if rng.random() < 0.85:
+        start = rng.randint(0, len(layers) - 1)
+        loop = (start, rng.randint(start + 1, len(layers)), ch([1, 2, 3]))
+    raw = lt.config(layers, vocab, width, ch([1e-5, 1e-6]), loop, ch([None, 1, 97, 1000]), (rng.randint(0, 99), rng.randint(0, 99)),
+                    ch([1.0, 4.0, 12.0]), ch([0.5, 1.0, 2.0]))
+    return raw, ch([1, 3, 8, 33])
+
+
+@pytest.mark.parametrize("seed", [0, 1, 2, 3, 4, 5])
+def test_configurations_drawn_at_random(tmp_path, seed):
+    import random
+
+    rng = random.Random(seed)
+    raw, rank = drawn_model(rng)
+    w = lt.weights(raw, seed=seed, rank=rank)
+    requests = {f"q{i}": np.random.default_rng(seed + i).integers(0, raw["vocab"], size=n).tolist()
+                for i, n in enumerate([rng.randint(1, 45) for _ in range(3)])}
+    want = {rid: plain.forward(raw, w, toks).float() for rid, toks in requests.items()}
+    folder = lt.write(raw, w, tmp_path / "m")
+    steps = replay.mixed(requests, live=2, seed=seed, prefill_sizes=(9, 2, 17, 5), decode_tail=6)
+    top = max(float(v.abs().max()) for v in want.values())
+    got = replay.run_in_process(load(folder, "float32", page=8, tokens=replay.peak_tokens(steps, 8) + 8), steps)
+    assert worst(got, want) <= 2e-4 * max(1.0, top), raw
+    got = replay.run_in_process(load(folder, "bfloat16", page=8, tokens=replay.peak_tokens(steps, 8) + 8), steps)
+    errs = np.array([float((got[k] - want[k[0]][k[1]]).pow(2).mean().sqrt()) for k in got])
+    assert np.median(errs) <= 0.06 * float(torch.cat([v.flatten() for v in want.values()]).std()), raw
