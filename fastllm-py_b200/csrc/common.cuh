@@ -123,6 +123,8 @@ static inline bool fl_pdl_enabled() {
     return on == 1;
 }
 
+// overlap false: in plain stream order, for long kernels of no more CTAs than SMs.  Brought in while the predecessor still
+// runs, several of their CTAs end up on the first SMs that have room, and the kernel takes as long as the fullest SM.
 template <typename... KArgs, typename... Args>
 static inline int fl_launch_as(bool overlap, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
                                cudaStream_t stream, Args... args) {
@@ -143,12 +145,4 @@ template <typename... KArgs, typename... Args>
 static inline int fl_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
                             cudaStream_t stream, Args... args) {
     return fl_launch_as(true, kernel, grid, block, smem, stream, args...);
-}
-
-// In plain stream order, for long kernels of no more CTAs than SMs: brought in while the predecessor still runs, several
-// of their CTAs end up on the first SMs that have room, and the kernel takes as long as the fullest SM.
-template <typename... KArgs, typename... Args>
-static inline int fl_launch_spread(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
-                                   cudaStream_t stream, Args... args) {
-    return fl_launch_as(false, kernel, grid, block, smem, stream, args...);
 }
