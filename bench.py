@@ -1129,15 +1129,15 @@ def lufozen_config(size):
     rot = RotationConfig(500000.0, a["dim"], (8.0, 8192.0, 1.0, 4.0))
     lone = ("attention", AttentionConfig(*sizes, rot, a["conv"]))
     pair = ("parallel", PairConfig(AttentionConfig(*sizes, rot),
-                                   StateSpaceConfig(r["heads"], r["vdim"], r["state"], r["groups"], r["conv"], r["groups"]), 0.6, 0.5))
+                                   StateSpaceConfig(r["heads"], r["vdim"], r["state"], r["groups"], r["conv"], r["groups"]), 0.7, 0.4))
     linear = ("gla", GatedLinearAttentionConfig(g["heads"], g["dim"], g["vdim"], g["tau"]))
     if z["runs"] == 8:
         kinds, loop = [lone, pair, linear, pair, lone, linear], LoopConfig(1, 3, 2)
     else:
         kinds, loop = [lone, pair, linear], LoopConfig(1, 2, 2)
     layers = tuple(LufozenLayerConfig(*k, DenseConfig(z["ff"])) for k in kinds)
-    return LufozenConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, embedding_scale=16.0, bigram_buckets=65521,
-                         bigram_mul_prev=31, bigram_mul_cur=7, logit_scale=0.5, loop=loop, layers=layers)
+    return LufozenConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, embedding_scale=8.0, bigram_buckets=65521,
+                         bigram_mul_prev=17, bigram_mul_cur=5, logit_scale=0.5, loop=loop, layers=layers)
 
 
 def _lufozen_layer_sizes(layer, w):
