@@ -6,12 +6,14 @@ from .lasonex import LasonexConfig
 from .sakusun import SakusunConfig
 from .saberax import SaberaxConfig
 from .lufozen import LufozenConfig
+from .kerirax import KeriraxConfig
 from .registry import (Architecture, architecture_names, architecture_of, load_config,
                        register_architecture)
 
 __all__ = [
     "ConfigError", "read_raw_config", "EngineConfig", "canonical_dtype", "LinearRopeScaling",
     "LlamaConfig", "TigitarConfig", "LasonexConfig", "SakusunConfig", "SaberaxConfig", "LufozenConfig",
+    "KeriraxConfig",
     "Architecture", "architecture_names", "architecture_of", "load_config",
     "register_architecture",
 ]

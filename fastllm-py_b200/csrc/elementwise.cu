@@ -656,49 +656,161 @@ FL_API int fl_sandwich_norm_partial(float* x, long x_ld, const float* partial, i
 
 // ------------------------------------------------- two sums pending, two norms of one row
 // A layer whose mixer and feed-forward both read the same x leaves two outputs to add, and the
-// next such layer norms the sum twice, with two weights but one root mean square:
-//     x += d1 + d2;   r = (mean(x^2) + eps)^-1/2;   out1 = x r w1;   out2 = x r w2
-// d1, d2, w2 / out2 may each be absent.  x is the float residual stream (written back unless rows
-// are gathered).  The summed row waits in shared memory between the reduction and the last pass.
-template <typename TD, typename TW, typename TO>
-__global__ void norm_pair_kernel(float* __restrict__ x, long x_ld, const TD* __restrict__ d1, long d1_ld,
-                                 const TD* __restrict__ d2, long d2_ld, const TW* __restrict__ w1,
-                                 const TW* __restrict__ w2, TO* __restrict__ out1, long out1_ld, TO* __restrict__ out2,
-                                 long out2_ld, int dim, float eps, const int* __restrict__ rows) {
+// next such layer norms the sum once, or twice with two weights but one root mean square:
+//     x += d1 + d2 + the row vectors;   r = (mean(x^2) + eps)^-1/2;   out1 = x r w1;   out2 = x r w2
+// d1, d2, the vectors and w2 / out2 may each be absent.  d1 and d2 are rows of the activation type, or the split-K partial
+// sums of the product that made them (float slabs, added up in order while they are read).  x is the float residual stream
+// (written back unless rows are gathered).  The summed row waits in shared memory between the reduction and the last pass.
+struct Summand {
+    const void* p;
+    long ld;
+    int splits;                  // 0: rows of the activation type; else float slabs `stride` floats apart
+    long stride;
+};
+static inline bool summand_vec_ok(const Summand& d, int dim, size_t elem) {
+    return d.p == nullptr || (vec4_ok(dim, d.p, d.ld, d.splits > 0 ? 4 : elem) && (d.splits == 0 || d.stride % 4 == 0));
+}
+template <typename TD> __device__ __forceinline__ float summand1(const Summand& d, long r, int i) {
+    if (d.splits == 0) return to_f32<TD>(static_cast<const TD*>(d.p)[r * d.ld + i]);
+    const float* p = static_cast<const float*>(d.p) + r * d.ld + i;
+    float v = 0.0f;
+    for (int z = 0; z < d.splits; ++z) v += p[z * d.stride];
+    return v;
+}
+template <typename TD> __device__ __forceinline__ void add_summand4(float4& v, const Summand& d, long r, int i) {
+    float4 a;
+    if (d.splits == 0) {
+        load4(static_cast<const TD*>(d.p) + r * d.ld + i, a);
+    } else {
+        const float* p = static_cast<const float*>(d.p) + r * d.ld + i;
+        a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+        for (int z = 0; z < d.splits; ++z) {
+            const float4 q = *reinterpret_cast<const float4*>(p + z * d.stride);
+            a.x += q.x; a.y += q.y; a.z += q.z; a.w += q.w;
+        }
+    }
+    v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+}
+
+template <typename TD, typename TW, typename TO, bool VEC>
+__global__ void __launch_bounds__(1024) norm_pair_kernel(float* __restrict__ x, long x_ld, const Summand d1, const Summand d2,
+                                                         const RowAdd add, const TW* __restrict__ w1, const TW* __restrict__ w2,
+                                                         TO* __restrict__ out1, long out1_ld, TO* __restrict__ out2,
+                                                         long out2_ld, int dim, float eps, const int* __restrict__ rows) {
     pdl_wait();
     pdl_trigger();
-    extern __shared__ float pair_row[];                     // [dim]
+    extern __shared__ __align__(16) float pair_row[];       // [dim]
     __shared__ float scratch[32];
+    constexpr int STEP = VEC ? 4 : 1;
     const int r = blockIdx.x;
     const long src = rows ? (long)rows[r] : (long)r;
+    const bool write_back = !rows && (d1.p || d2.p || add.a || add.b);
     float* xr = x + src * x_ld;
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        float v = xr[i];
-        if (d1) v += to_f32<TD>(d1[src * d1_ld + i]);
-        if (d2) v += to_f32<TD>(d2[src * d2_ld + i]);
-        if ((d1 || d2) && !rows) xr[i] = v;
-        pair_row[i] = v;                                    // each thread re-reads what it wrote itself
-        ss += v * v;
+    for (int i = threadIdx.x * STEP; i < dim; i += blockDim.x * STEP) {
+        if (VEC) {
+            float4 v = *reinterpret_cast<const float4*>(xr + i);
+            if (d1.p) add_summand4<TD>(v, d1, src, i);
+            if (d2.p) add_summand4<TD>(v, d2, src, i);
+            add_rows4(v, add, i);
+            if (write_back) *reinterpret_cast<float4*>(xr + i) = v;
+            *reinterpret_cast<float4*>(pair_row + i) = v;
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        } else {
+            float v = xr[i];
+            if (d1.p) v += summand1<TD>(d1, src, i);
+            if (d2.p) v += summand1<TD>(d2, src, i);
+            add_rows1(v, add, i);
+            if (write_back) xr[i] = v;
+            pair_row[i] = v;                                // each thread re-reads what it wrote itself
+            ss += v * v;
+        }
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        const float v = pair_row[i] * inv;
-        out1[(long)r * out1_ld + i] = from_f32<TO>(v * to_f32<TW>(w1[i]));
-        if (out2) out2[(long)r * out2_ld + i] = from_f32<TO>(v * to_f32<TW>(w2[i]));
+    for (int i = threadIdx.x * STEP; i < dim; i += blockDim.x * STEP) {
+        if (VEC) {
+            const float4 v = *reinterpret_cast<const float4*>(pair_row + i);
+            float4 g;
+            load4(w1 + i, g);
+            store4(out1 + (long)r * out1_ld + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+            if (out2) {
+                load4(w2 + i, g);
+                store4(out2 + (long)r * out2_ld + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+            }
+        } else {
+            const float v = pair_row[i] * inv;
+            out1[(long)r * out1_ld + i] = from_f32<TO>(v * to_f32<TW>(w1[i]));
+            if (out2) out2[(long)r * out2_ld + i] = from_f32<TO>(v * to_f32<TW>(w2[i]));
+        }
     }
 }
 
-FL_API int fl_norm_pair(float* x, long x_ld, const void* d1, long d1_ld, const void* d2, long d2_ld, int d_dtype,
+FL_API int fl_norm_pair(float* x, long x_ld, const void* d1, long d1_ld, int d1_splits, long d1_stride, const void* d2, long d2_ld,
+                        int d2_splits, long d2_stride, int d_dtype, const float* add_a, const float* add_b,
                         const void* w1, const void* w2, int w_dtype, void* out1, long out1_ld, void* out2, long out2_ld,
                         int out_dtype, int n_rows, int dim, float eps, const int* rows, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if ((size_t)dim * sizeof(float) > 48 * 1024 || (out2 != nullptr) != (w2 != nullptr)) return (int)cudaErrorInvalidValue;
-    const int threads = norm_threads(dim, false);
-    FL_DISPATCH(d_dtype, TD, FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,
-        return fl_launch(norm_pair_kernel<TD, TW, TO>, dim3(n_rows), dim3(threads), (size_t)dim * sizeof(float), stream,
-                         x, x_ld, (const TD*)d1, d1_ld, (const TD*)d2, d2_ld, (const TW*)w1, (const TW*)w2, (TO*)out1,
-                         out1_ld, (TO*)out2, out2_ld, dim, eps, rows))));
+    const Summand s1{d1, d1_ld, d1_splits, d1_stride}, s2{d2, d2_ld, d2_splits, d2_stride};
+    const RowAdd add{add_a, add_b};
+    const size_t d_elem = d_dtype == FL_F32 ? 4 : 2, w_elem = w_dtype == FL_F32 ? 4 : 2, o_elem = out_dtype == FL_F32 ? 4 : 2;
+    const bool vec = row_add_vec_ok(add) && vec4_ok(dim, x, x_ld, 4) && summand_vec_ok(s1, dim, d_elem) && summand_vec_ok(s2, dim, d_elem) &&
+                     vec4_ok(dim, w1, 4, w_elem) && vec4_ok(dim, w2, 4, w_elem) && vec4_ok(dim, out1, out1_ld, o_elem) &&
+                     vec4_ok(dim, out2, out2_ld, o_elem);
+    const int threads = norm_threads(dim, vec);
+#define FL_PAIR_LAUNCH(VEC)                                                                                              \
+    FL_DISPATCH(d_dtype, TD, FL_DISPATCH(w_dtype, TW, FL_DISPATCH(out_dtype, TO,                                         \
+        return fl_launch(norm_pair_kernel<TD, TW, TO, VEC>, dim3(n_rows), dim3(threads), (size_t)dim * sizeof(float),    \
+                         stream, x, x_ld, s1, s2, add, (const TW*)w1, (const TW*)w2, (TO*)out1, out1_ld, (TO*)out2,      \
+                         out2_ld, dim, eps, rows))))
+    if (vec) { FL_PAIR_LAUNCH(true); } else { FL_PAIR_LAUNCH(false); }
+#undef FL_PAIR_LAUNCH
+    return 0;
+}
+
+// out[r] = x[r] + d1 + d2 + the row vectors in the output's type (each but x may be absent): the residual stream as the
+// operand of a product.  x stays as it is.
+template <typename TD, typename TO, bool VEC>
+__global__ void __launch_bounds__(256) sum_rows_kernel(const float* __restrict__ x, long x_ld, const Summand d1, const Summand d2,
+                                                       const RowAdd add, TO* __restrict__ out, long out_ld, int dim) {
+    pdl_wait();
+    pdl_trigger();
+    constexpr int STEP = VEC ? 4 : 1;
+    const long r = blockIdx.x;
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * STEP;
+    if (i >= dim) return;
+    if (VEC) {
+        float4 v = *reinterpret_cast<const float4*>(x + r * x_ld + i);
+        if (d1.p) add_summand4<TD>(v, d1, r, i);
+        if (d2.p) add_summand4<TD>(v, d2, r, i);
+        add_rows4(v, add, i);
+        store4(out + r * out_ld + i, v);
+    } else {
+        float v = x[r * x_ld + i];
+        if (d1.p) v += summand1<TD>(d1, r, i);
+        if (d2.p) v += summand1<TD>(d2, r, i);
+        add_rows1(v, add, i);
+        out[r * out_ld + i] = from_f32<TO>(v);
+    }
+}
+
+FL_API int fl_sum_rows(const float* x, long x_ld, const void* d1, long d1_ld, int d1_splits, long d1_stride, const void* d2, long d2_ld,
+                       int d2_splits, long d2_stride, int d_dtype, const float* add_a, const float* add_b, void* out, int out_dtype,
+                       long out_ld, int n_rows, int dim, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    const Summand s1{d1, d1_ld, d1_splits, d1_stride}, s2{d2, d2_ld, d2_splits, d2_stride};
+    const RowAdd add{add_a, add_b};
+    const size_t d_elem = d_dtype == FL_F32 ? 4 : 2;
+    const bool vec = row_add_vec_ok(add) && vec4_ok(dim, x, x_ld, 4) && summand_vec_ok(s1, dim, d_elem) && summand_vec_ok(s2, dim, d_elem) &&
+                     vec4_ok(dim, out, out_ld, out_dtype == FL_F32 ? 4 : 2);
+    const int per = 256 * (vec ? 4 : 1);
+#define FL_SUM_LAUNCH(VEC)                                                                                               \
+    FL_DISPATCH(d_dtype, TD, FL_DISPATCH(out_dtype, TO,                                                                  \
+        return fl_launch(sum_rows_kernel<TD, TO, VEC>, dim3(n_rows, (dim + per - 1) / per), dim3(256), 0, stream, x, x_ld, \
+                         s1, s2, add, (TO*)out, out_ld, dim)))
+    if (vec) { FL_SUM_LAUNCH(true); } else { FL_SUM_LAUNCH(false); }
+#undef FL_SUM_LAUNCH
     return 0;
 }

@@ -12,7 +12,8 @@
 //                     the token's cache row.  Rotary pairs are (i, i + rot/2), or with `interleaved`
 //                     (2i, 2i + 1); pair i turns by the table's column i either way
 //   latent_attention  per (token, head): softmax over the visible rows (a window, if the layer has one),
-//                     keys walked in tiles of 128 aligned to absolute positions
+//                     keys walked in tiles of 128 aligned to absolute positions; with a sink, exp(sink_h) is one more
+//                     term of the denominator
 //
 // Cache: [pages][page_size][rank + rot] in the activation type.  Scores, softmax and sums are float.
 #include "common.cuh"
@@ -71,7 +72,7 @@ template <typename T, typename TQ>
 __global__ void __launch_bounds__(LAT_TILE) latent_attention_kernel(
     const TQ* __restrict__ q, long q_ld, float* __restrict__ out, long out_ld, const T* __restrict__ cache,
     int page_size, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ tok_req,
-    const int* __restrict__ positions, int rank, int rot, int window, float scale) {
+    const int* __restrict__ positions, int rank, int rot, int window, float scale, const float* __restrict__ sink) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -87,7 +88,8 @@ __global__ void __launch_bounds__(LAT_TILE) latent_attention_kernel(
     const TQ* qr = q + (long)t * q_ld + (long)h * width;
     for (int d = tid; d < width; d += LAT_TILE) q_s[d] = to_f32<TQ>(qr[d]);
     __syncthreads();
-    float m = -CUDART_INF_F, l = 0.0f, acc[LAT_MAX_ACC];
+    // the sink is a term exp(sink) of the denominator without a value: the running maximum and sum start from it
+    float m = sink != nullptr ? sink[h] : -CUDART_INF_F, l = sink != nullptr ? 1.0f : 0.0f, acc[LAT_MAX_ACC];
 #pragma unroll
     for (int a = 0; a < LAT_MAX_ACC; ++a) acc[a] = 0.0f;
     for (int tile = (lo / LAT_TILE) * LAT_TILE; tile <= pos; tile += LAT_TILE) {
@@ -107,7 +109,7 @@ __global__ void __launch_bounds__(LAT_TILE) latent_attention_kernel(
         const float p = valid ? expf(s - m_new) : 0.0f;
         p_s[tid] = p;
         const float tile_sum = block_sum(p, scratch);     // its barriers also publish p_s / off_s
-        const float corr = expf(m - m_new);               // 0 at the first tile (m = -inf)
+        const float corr = expf(m - m_new);               // 0 at the first tile without a sink (m = -inf)
         l = l * corr + tile_sum;
         const int j_begin = max(0, lo - tile), j_end = min(LAT_TILE, pos - tile + 1);
 #pragma unroll
@@ -150,17 +152,17 @@ FL_API int fl_latent_prep(const void* proj, int dtype, long ld, const void* kv, 
     return 0;
 }
 
-// window <= 0: all earlier tokens.
+// window <= 0: all earlier tokens.  sink: [heads] float, or null.
 FL_API int fl_latent_attention(const void* q, int q_dtype, long q_ld, float* out, long out_ld, const void* cache, int cache_dtype,
                                int page_size, const int* block_table, int bt_stride, const int* tok_req,
                                const int* positions, int n_tokens, int heads, int rank, int rot, int window,
-                               float scale, cudaStream_t stream) {
+                               float scale, const float* sink, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank < 1 || rank > LAT_TILE * LAT_MAX_ACC || heads > 65535) return (int)cudaErrorInvalidValue;
     const size_t smem = LAT_TILE * (sizeof(long) + sizeof(float)) + (size_t)(rank + rot) * sizeof(float);
     FL_DISPATCH(cache_dtype, T, FL_DISPATCH(q_dtype, TQ,
         return fl_launch(latent_attention_kernel<T, TQ>, dim3(n_tokens, heads), dim3(LAT_TILE), smem, stream, (const TQ*)q,
                          q_ld, out, out_ld, (const T*)cache, page_size, block_table, bt_stride, tok_req, positions, rank, rot,
-                         window, scale)));
+                         window, scale, sink)));
     return 0;
 }

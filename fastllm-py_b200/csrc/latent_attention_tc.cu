@@ -35,7 +35,7 @@ template <typename TO>
 __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     const bf16* __restrict__ q, long q_ld, TO* __restrict__ out, long out_ld, const bf16* __restrict__ cache,
     int page_size, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ tok_req,
-    const int* __restrict__ positions, int heads, int window, float scale, int split_keys, float* __restrict__ partial) {
+    const int* __restrict__ positions, int heads, int window, float scale, int split_keys, float* __restrict__ partial, const float* __restrict__ sink) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char lt_smem[];
@@ -96,6 +96,14 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     for (int n = 0; n < LT_NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.0f;
     float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.0f, 0.0f};   // rows lane / 4 and lane / 4 + 8
     const int row0 = lane >> 2;
+    if (sink != nullptr && split_keys == 0) {                // the running maximum and sum start from the sink's term
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+            if (head0 + row0 + h * 8 < heads) {
+                m_run[h] = sink[head0 + row0 + h * 8];
+                l_run[h] = 1.0f;
+            }
+    }
     int buf = 0;
     for (int tile = first_tile; tile <= last; tile += LT_KEYS, buf ^= 1) {
         if (tile + LT_KEYS <= last) {
@@ -145,7 +153,7 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
             float m_new = m_run[h];
 #pragma unroll
             for (int w = 0; w < LT_WARPS; ++w) m_new = fmaxf(m_new, red_max[w * 16 + r]);
-            corr[h] = expf(m_run[h] - m_new);               // 0 at the first tile
+            corr[h] = expf(m_run[h] - m_new);               // 0 at the first tile without a sink
             m_run[h] = m_new;
             const float p0 = expf(s[h * 2] - m_new), p1 = expf(s[h * 2 + 1] - m_new);   // exp(-inf) = 0 out of sight
             float sum = p0 + p1;
@@ -219,17 +227,17 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     }
 }
 
-// out[t, head] = sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M), splits in order; one block per (token, head).
+// out[t, head] = sum_z acc_z e^(m_z - M) / ([e^(sink - M) +] sum_z l_z e^(m_z - M)), splits in order; one block per (token, head).
 template <typename TO>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ partial, TO* __restrict__ out,
-                                                           long out_ld, int heads, int n_splits) {
+                                                           long out_ld, int heads, int n_splits, const float* __restrict__ sink) {
     pdl_wait();
     pdl_trigger();
     const int t = blockIdx.x, head = blockIdx.y;
     const float* pr = partial + ((long)t * heads + head) * n_splits * (LAT_RANK + 2);
-    float mx = -CUDART_INF_F;
+    float mx = sink != nullptr ? sink[head] : -CUDART_INF_F;
     for (int z = 0; z < n_splits; ++z) mx = fmaxf(mx, pr[(long)z * (LAT_RANK + 2) + LAT_RANK]);
-    float l = 0.0f;
+    float l = sink != nullptr ? expf(sink[head] - mx) : 0.0f;
     for (int z = 0; z < n_splits; ++z) {
         const float* p = pr + (long)z * (LAT_RANK + 2);
         if (p[LAT_RANK + 1] > 0.0f) l += p[LAT_RANK + 1] * expf(p[LAT_RANK] - mx);
@@ -252,11 +260,12 @@ FL_API int fl_latent_attention_tc_rot() { return LAT_ROT; }
 // split_keys > 0 (a multiple of 32): the keys are shared out over n_splits blocks per token (decode steps,
 // where tokens are too few to fill the GPU); `partial` then holds n_tokens * heads * n_splits * (rank + 2)
 // floats and a merge kernel follows.  n_splits must reach the last key of every token:
-// (longest visible span - 1) / split_keys + 2 does.
+// (longest visible span - 1) / split_keys + 2 does.  sink: [heads] float, a term exp(sink) of each head's denominator, or
+// null.
 FL_API int fl_latent_attention_tc(const void* q, long q_ld, void* out, int out_dtype, long out_ld, const void* cache, int page_size,
                                   const int* block_table, int bt_stride, const int* tok_req, const int* positions,
                                   int n_tokens, int heads, int window, float scale, int split_keys, int n_splits,
-                                  float* partial, cudaStream_t stream) {
+                                  float* partial, const float* sink, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (split_keys < 0 || split_keys % LT_KEYS || (split_keys > 0 && (n_splits < 1 || n_splits > 65535 || partial == nullptr)))
         return (int)cudaErrorInvalidValue;
@@ -276,10 +285,10 @@ FL_API int fl_latent_attention_tc(const void* q, long q_ld, void* out, int out_d
     FL_DISPATCH(out_dtype, TO,
         rc = fl_launch(latent_attention_tc_kernel<TO>, dim3(n_tokens, (heads + 15) / 16, split_keys > 0 ? n_splits : 1),
                        dim3(LT_WARPS * 32), smem, stream, (const bf16*)q, q_ld, (TO*)out, out_ld, (const bf16*)cache,
-                       page_size, block_table, bt_stride, tok_req, positions, heads, window, scale, split_keys, partial));
+                       page_size, block_table, bt_stride, tok_req, positions, heads, window, scale, split_keys, partial, sink));
     if (rc || split_keys == 0) return rc;
     FL_DISPATCH(out_dtype, TO,
         return fl_launch(latent_merge_kernel<TO>, dim3(n_tokens, heads), dim3(128), 0, stream, (const float*)partial,
-                         (TO*)out, out_ld, heads, n_splits));
+                         (TO*)out, out_ld, heads, n_splits, sink));
     return 0;
 }

@@ -15,7 +15,8 @@
 //                 `accumulate` added to what `out` holds: a shared unit's result)
 //
 // The last two read an expert's matrices once per token that chose it: the right shape for decode
-// steps, where tokens are few and the matrices stream from memory.  All sums are float and depend only
+// steps, where tokens are few and the matrices stream from memory.  A token's weight multiplies its expert's output, or
+// (weight_on_input) what the expert reads: the gate and up sums then, which are linear in it, before the activation.  All sums are float and depend only
 // on the token itself.
 #include "common.cuh"
 
@@ -111,7 +112,8 @@ __global__ void __launch_bounds__(128) moe_pick_kernel(const float* __restrict__
 template <typename T, typename TW>
 __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ h, long h_ld, const TW* __restrict__ w_gu,
                                                           const int* __restrict__ chosen, float* __restrict__ a,
-                                                          int width, int ff, int top, FlGate act, int gated) {
+                                                          int width, int ff, int top, FlGate act, int gated,
+                                                          const float* __restrict__ in_weights) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ float moe_x[];                    // [width]
@@ -121,12 +123,13 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ 
     __syncthreads();
     const int f = blockIdx.y * 8 + warp;
     if (f >= ff) return;
+    const float win = in_weights != nullptr ? in_weights[pair] : 1.0f;      // what multiplies the expert's input
     if (!gated) {
         const TW* wx = w_gu + ((long)chosen[pair] * ff + f) * width;
         float x = 0.0f;
         for (int i = lane; i < width; i += 32) x += moe_x[i] * to_f32<TW>(wx[i]);
         x = warp_sum(x);
-        if (lane == 0) a[(long)pair * ff + f] = fl_gated(x, 1.0f, act);
+        if (lane == 0) a[(long)pair * ff + f] = fl_gated(x * win, 1.0f, act);
         return;
     }
     const TW* wg = w_gu + ((long)chosen[pair] * 2 * ff + f) * width;
@@ -138,7 +141,7 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ 
     }
     g = warp_sum(g);
     u = warp_sum(u);
-    if (lane == 0) a[(long)pair * ff + f] = fl_gated(g, u, act);
+    if (lane == 0) a[(long)pair * ff + f] = fl_gated(g * win, u * win, act);
 }
 
 // w_down: [experts][width][ff]
@@ -159,7 +162,7 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const float* __restrict__
         const float* ar = a + pair * ff;
         float y = 0.0f;
         for (int i = lane; i < ff; i += 32) y += ar[i] * to_f32<TW>(wd[i]);
-        sum += weights[pair] * warp_sum(y);
+        sum += (weights != nullptr ? weights[pair] : 1.0f) * warp_sum(y);
     }
     if (lane == 0) out[(long)t * out_ld + c] = from_f32<T>(accumulate ? to_f32<T>(out[(long)t * out_ld + c]) + sum : sum);
 }
@@ -183,7 +186,7 @@ FL_API int fl_moe_pick(const float* z, long z_ld, const void* bias, int bias_dty
 FL_API int fl_moe_experts(const void* h, int dtype, long h_ld, const void* w_gu, const void* w_down, int w_dtype,
                           const int* chosen, const float* weights, float* a, void* out, long out_ld, int n_tokens,
                           int width, int ff, int top, int act, float act_p0, float act_p1, int gated,
-                          int accumulate, cudaStream_t stream) {
+                          int accumulate, int weight_on_input, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if ((size_t)width * sizeof(float) > 48 * 1024 || (ff + 7) / 8 > 65535 || (width + 7) / 8 > 65535 || act < 0 || act >= FL_ACT_COUNT)
         return (int)cudaErrorInvalidValue;
@@ -191,11 +194,11 @@ FL_API int fl_moe_experts(const void* h, int dtype, long h_ld, const void* w_gu,
     FL_DISPATCH(dtype, T, FL_DISPATCH(w_dtype, TW,
         rc = fl_launch(moe_gate_up_kernel<T, TW>, dim3(n_tokens * top, (ff + 7) / 8), dim3(256),
                        (size_t)width * sizeof(float), stream, (const T*)h, h_ld, (const TW*)w_gu, chosen, a, width, ff,
-                       top, FlGate{act, act_p0, act_p1}, gated)));
+                       top, FlGate{act, act_p0, act_p1}, gated, weight_on_input ? weights : nullptr)));
     if (rc) return rc;
     FL_DISPATCH(dtype, T, FL_DISPATCH(w_dtype, TW,
         return fl_launch(moe_down_kernel<T, TW>, dim3(n_tokens, (width + 7) / 8), dim3(256), 0, stream, (const float*)a,
-                         (const TW*)w_down, chosen, weights, (T*)out, out_ld, width, ff, top, accumulate)));
+                         (const TW*)w_down, chosen, weight_on_input ? nullptr : weights, (T*)out, out_ld, width, ff, top, accumulate)));
     return 0;
 }
 
@@ -273,7 +276,7 @@ template <int MODE>
 __global__ void __launch_bounds__(256) moe_group_mma_kernel(
     const bf16* __restrict__ a, long a_ld, const bf16* __restrict__ w, int n_out, int K, const int* __restrict__ row_pair,
     const int* __restrict__ tile_expert, const int* __restrict__ n_tiles, int top, bf16* __restrict__ act_out,
-    float* __restrict__ y_out, long out_ld, FlGate act) {
+    float* __restrict__ y_out, long out_ld, FlGate act, const float* __restrict__ in_weights) {
     pdl_wait();
     pdl_trigger();
     constexpr bool GATED = MODE == MOE_GATED;
@@ -373,6 +376,8 @@ __global__ void __launch_bounds__(256) moe_group_mma_kernel(
         for (int half = 0; half < 2; ++half) {
             const int r = wm * 32 + i * 16 + (lane >> 2) + half * 8;
             const long row = (long)tile * MOE_TM + r;
+            float win = 1.0f;                                   // what multiplies the row's input
+            if (MODE != MOE_DOWN && in_weights != nullptr) win = pair_s[r] < 0 ? 0.0f : in_weights[pair_s[r]];
             if (GATED) {
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
@@ -380,8 +385,8 @@ __global__ void __launch_bounds__(256) moe_group_mma_kernel(
                     for (int c = 0; c < 2; ++c) {
                         const int f = blockIdx.y * 64 + wn * 16 + j * 8 + (lane & 3) * 2 + c;
                         if (f < n_out)
-                            act_out[row * out_ld + f] = __float2bfloat16_rn(fl_gated(acc[i][j][half * 2 + c],
-                                                                                     acc[i][j + 2][half * 2 + c], act));
+                            act_out[row * out_ld + f] = __float2bfloat16_rn(fl_gated(acc[i][j][half * 2 + c] * win,
+                                                                                     acc[i][j + 2][half * 2 + c] * win, act));
                     }
             } else {
 #pragma unroll
@@ -390,7 +395,7 @@ __global__ void __launch_bounds__(256) moe_group_mma_kernel(
                     for (int c = 0; c < 2; ++c) {
                         const int col = blockIdx.y * 128 + wn * 32 + j * 8 + (lane & 3) * 2 + c;
                         if (col >= n_out) continue;
-                        if (MODE == MOE_UP) act_out[row * out_ld + col] = __float2bfloat16_rn(fl_gated(acc[i][j][half * 2 + c], 1.0f, act));
+                        if (MODE == MOE_UP) act_out[row * out_ld + col] = __float2bfloat16_rn(fl_gated(acc[i][j][half * 2 + c] * win, 1.0f, act));
                         else y_out[row * out_ld + col] = acc[i][j][half * 2 + c];
                     }
             }
@@ -406,7 +411,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restric
     const int t = blockIdx.x;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
         float sum = 0.0f;
-        for (int k = 0; k < top; ++k) sum += weights[(long)t * top + k] * y[(long)pair_row[(long)t * top + k] * y_ld + c];
+        for (int k = 0; k < top; ++k) sum += (weights != nullptr ? weights[(long)t * top + k] : 1.0f) * y[(long)pair_row[(long)t * top + k] * y_ld + c];
         out[(long)t * out_ld + c] = from_f32<T>(accumulate ? to_f32<T>(out[(long)t * out_ld + c]) + sum : sum);
     }
 }
@@ -438,8 +443,9 @@ static int moe_group_smem_ready() {
 FL_API int fl_moe_experts_grouped(const void* h, long h_ld, const void* w_gu, const void* w_down, const int* chosen,
                                   const float* weights, int* ints, void* act, float* y, void* out, long out_ld,
                                   int n_tokens, int width, int ff, int top, int experts, int act_code, float act_p0, float act_p1,
-                                  int gated, int accumulate, cudaStream_t stream) {
+                                  int gated, int accumulate, int weight_on_input, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    const float* in_weights = weight_on_input ? weights : nullptr;
     if (act_code < 0 || act_code >= FL_ACT_COUNT) return (int)cudaErrorInvalidValue;
     const FlGate gate{act_code, act_p0, act_p1};
     const long rows = fl_moe_group_rows(n_tokens, top, experts);
@@ -457,18 +463,18 @@ FL_API int fl_moe_experts_grouped(const void* h, long h_ld, const void* w_gu, co
     if (gated)
         rc = fl_launch(moe_group_mma_kernel<MOE_GATED>, dim3(max_tiles, (ff + 63) / 64), dim3(256), MOE_SMEM, stream, (const bf16*)h, h_ld,
                        (const bf16*)w_gu, ff, width, (const int*)row_pair, (const int*)tile_expert, (const int*)n_tiles, top,
-                       (bf16*)act, (float*)nullptr, (long)ff, gate);
+                       (bf16*)act, (float*)nullptr, (long)ff, gate, in_weights);
     else
         rc = fl_launch(moe_group_mma_kernel<MOE_UP>, dim3(max_tiles, (ff + 127) / 128), dim3(256), MOE_SMEM, stream, (const bf16*)h, h_ld,
                        (const bf16*)w_gu, ff, width, (const int*)row_pair, (const int*)tile_expert, (const int*)n_tiles, top,
-                       (bf16*)act, (float*)nullptr, (long)ff, gate);
+                       (bf16*)act, (float*)nullptr, (long)ff, gate, in_weights);
     if (rc) return rc;
     rc = fl_launch(moe_group_mma_kernel<MOE_DOWN>, dim3(max_tiles, (width + 127) / 128), dim3(256), MOE_SMEM, stream,
                    (const bf16*)act, (long)ff, (const bf16*)w_down, width, ff, (const int*)row_pair,
-                   (const int*)tile_expert, (const int*)n_tiles, top, (bf16*)nullptr, y, (long)width, gate);
+                   (const int*)tile_expert, (const int*)n_tiles, top, (bf16*)nullptr, y, (long)width, gate, (const float*)nullptr);
     if (rc) return rc;
     int col_blocks = (width + 255) / 256;
     if (col_blocks > 8) col_blocks = 8;
     return fl_launch(moe_combine_kernel<bf16>, dim3(n_tokens, col_blocks), dim3(256), 0, stream, (const float*)y,
-                     (long)width, (const int*)pair_row, weights, (bf16*)out, out_ld, width, top, accumulate);
+                     (long)width, (const int*)pair_row, weight_on_input ? nullptr : weights, (bf16*)out, out_ld, width, top, accumulate);
 }

@@ -1,0 +1,569 @@
+// Selective scan: a recurrence per channel c and state element n whose decay is made from the token for every one of them
+// (the first form of a selective state space).
+//
+// Per token, from one product's row [u: inner | z: inner]:
+//     x <- silu(conv(u) + bias)                       one causal convolution per channel, `taps` taps
+//     low = W_x x                                     [dt: rank | B: state | C: state], a product the caller makes
+//     dt <- softplus(W_dt dt + bias)                  one number a channel
+//     S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,     y_c = sum_n S[c, n] C_n + D_c x_c       (A < 0)
+// then y * silu(z).  A request's state row is S [inner][state] float and behind it the convolution's last taps - 1 inputs,
+// [taps - 1][inner], oldest first; it is ignored when the request starts (context 0).
+//
+//   selective_conv      convolution and silu (in the activation type, which W_x reads); in steps of single tokens the
+//                       thread that owns a channel moves its kept inputs on
+//   selective_dt        dt of every token and channel: float sums on the CUDA cores, one order whatever the step
+//   selective_dt_mma    the same for bfloat16 models on mma.sync: the float row is split into two bfloat16 parts, so that
+//                       the product keeps about 16 bits of it; W_dt is bfloat16 as stored
+//   selective_scan      the recurrence over each request's tokens in order, read-out, skip and gate; its blocks also move
+//                       the kept inputs of requests on
+//   selective_step      steps of single tokens: dt, recurrence, read-out and gate of a request's channels in one kernel
+//
+// Everything but x, z and y (the activation type) is float.  The exponential is expf for 32-bit models; for bfloat16 ones
+// ex2.approx of a product with A log2(e).
+#include "short_conv.cuh"
+#include "state_scan.cuh"
+
+// ------------------------------------------------------------------ convolution
+// V channels a thread, `run` consecutive tokens; conv_w: [taps][inner].  move_tail: every request has one token (run is 1).
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) selective_conv_kernel(
+    const T* __restrict__ u, long ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b, int taps,
+    float* __restrict__ tail, long tail_stride, const StepTables st, T* __restrict__ x, long x_ld, int n_tokens, int run,
+    int inner, int move_tail) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    ShortConv<T, V, TAPS> conv;
+    ChanVec<V> b;
+    if (c < inner) {                                                  // (no kernel writes these: asked for before the wait)
+        conv.start(conv_w, taps, inner, c);
+        b = chan_load<float, V>(conv_b + c);
+    }
+    pdl_wait();
+    pdl_trigger();
+    if (c >= inner) return;
+    const int t0 = blockIdx.x * run, t1 = min(n_tokens, t0 + run);
+    const T* col = u + c;
+    for (int t = t0; t < t1; ++t) {
+        const ChanVec<V> in = chan_load<T, V>(col + (long)t * ld);
+        ChanVec<V> y = conv.at(t, in, col, ld, st, tail, tail_stride, taps, inner, c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
+        chan_store<T, V>(x + (long)t * x_ld + c, y);
+        if constexpr (TAPS > 1) {
+            if (move_tail) {                                          // kept row j: the input of position pos + 1 - (taps - 1) + j
+                float* kept = tail + (long)st.req_slot[st.tok_req[t]] * tail_stride + c;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) {
+                    const int j = k - (TAPS - taps);
+                    if (j >= 0) chan_store<float, V>(kept + (long)j * inner, conv.win[k]);
+                }
+            }
+        }
+    }
+}
+
+FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* conv_w, const float* conv_b, int taps, float* tail,
+                             long tail_stride, const int* tok_req, const int* positions, const int* req_start,
+                             const int* req_ctx, const int* req_qlen, const int* req_slot, void* x, long x_ld, int n_tokens,
+                             int inner, int move_tail, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (taps < 1 || taps > 16 || (taps > 1 && tail == nullptr)) return (int)cudaErrorInvalidValue;
+    const StepTables st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
+    const int run = move_tail ? 1 : n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : 1;
+    const int elem = dtype == FL_F32 ? 4 : 2;
+    const bool vec = inner % 4 == 0 && chan_aligned(u, ld, elem) && chan_aligned(x, x_ld, elem) && chan_aligned(conv_w, 4, 4) &&
+                     chan_aligned(conv_b, 4, 4) && (taps == 1 || chan_aligned(tail, tail_stride, 4));
+    const int per = 128 * (vec ? 4 : 1);
+    dim3 grid((n_tokens + run - 1) / run, (inner + per - 1) / per);
+    if (grid.y > 65535) return (int)cudaErrorInvalidValue;
+#define FL_SEL_CONV(V, TAPS)                                                                                              \
+    FL_DISPATCH(dtype, T, return fl_launch(selective_conv_kernel<T, V, TAPS>, grid, dim3(128), 0, stream, (const T*)u, ld, \
+                                           conv_w, conv_b, taps, tail, tail_stride, st, (T*)x, x_ld, n_tokens, run, inner, \
+                                           move_tail))
+    if (vec) { if (taps == 1) { FL_SEL_CONV(4, 1); } else if (taps <= 4) { FL_SEL_CONV(4, 4); } else { FL_SEL_CONV(4, 16); } }
+    else { if (taps == 1) { FL_SEL_CONV(1, 1); } else if (taps <= 4) { FL_SEL_CONV(1, 4); } else { FL_SEL_CONV(1, 16); } }
+#undef FL_SEL_CONV
+    return 0;
+}
+
+// ------------------------------------------------------------------ step sizes
+#define SEL_DT_TOKENS 8
+
+// dt[t, c] = softplus(sum_k low[t, k] w_t[k, c] + bias[c]); a thread takes one channel of SEL_DT_TOKENS tokens.
+__global__ void __launch_bounds__(128) selective_dt_kernel(const float* __restrict__ low, long low_ld, int rank,
+                                                           const float* __restrict__ w_t, const float* __restrict__ bias,
+                                                           float* __restrict__ dt, long dt_ld, int n_tokens, int inner) {
+    pdl_wait();
+    pdl_trigger();
+    extern __shared__ float sel_low[];                                // [rank][SEL_DT_TOKENS]
+    const int t0 = blockIdx.x * SEL_DT_TOKENS, here = min(SEL_DT_TOKENS, n_tokens - t0);
+    for (int i = threadIdx.x; i < rank * SEL_DT_TOKENS; i += blockDim.x) {
+        const int t = i / rank, k = i % rank;
+        sel_low[k * SEL_DT_TOKENS + t] = t < here ? low[(long)(t0 + t) * low_ld + k] : 0.0f;
+    }
+    __syncthreads();
+    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= inner) return;
+    float acc[SEL_DT_TOKENS];
+#pragma unroll
+    for (int t = 0; t < SEL_DT_TOKENS; ++t) acc[t] = 0.0f;
+    for (int k = 0; k < rank; ++k) {
+        const float w = w_t[(long)k * inner + c];
+#pragma unroll
+        for (int t = 0; t < SEL_DT_TOKENS; ++t) acc[t] = fmaf(sel_low[k * SEL_DT_TOKENS + t], w, acc[t]);
+    }
+    const float b = bias[c];
+#pragma unroll
+    for (int t = 0; t < SEL_DT_TOKENS; ++t)
+        if (t < here) dt[(long)(t0 + t) * dt_ld + c] = fl_softplus(acc[t] + b);
+}
+
+// low: float rows of which the first `rank` columns count; w_t: [rank][inner] float.
+FL_API int fl_selective_dt(const float* low, long low_ld, int rank, const float* w_t, const float* bias, float* dt, long dt_ld,
+                           int n_tokens, int inner, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    const size_t smem = (size_t)rank * SEL_DT_TOKENS * sizeof(float);
+    if (rank < 1 || smem > 160 * 1024 || (inner + 127) / 128 > 65535) return (int)cudaErrorInvalidValue;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(selective_dt_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    return fl_launch(selective_dt_kernel, dim3((n_tokens + SEL_DT_TOKENS - 1) / SEL_DT_TOKENS, (inner + 127) / 128), dim3(128),
+                     smem, stream, low, low_ld, rank, w_t, bias, dt, dt_ld, n_tokens, inner);
+}
+
+#define SEL_MM 64                    // tokens and channels of a block's tile
+#define SEL_MK 64                    // columns of a stage
+#define SEL_MP (SEL_MK + 8)          // bfloat16 elements between staged rows (ldmatrix without bank conflicts)
+
+__device__ __forceinline__ void sel_ldm4(unsigned (&r)[4], const bf16* p) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
+}
+__device__ __forceinline__ void sel_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// w: [inner][w_ld] bfloat16, w_ld a multiple of 8 and zero from column `rank` on.
+__global__ void __launch_bounds__(128) selective_dt_mma_kernel(const float* __restrict__ low, long low_ld, int rank,
+                                                               const bf16* __restrict__ w, int w_ld,
+                                                               const float* __restrict__ bias, float* __restrict__ dt,
+                                                               long dt_ld, int n_tokens, int inner) {
+    __shared__ __align__(16) bf16 hi_s[SEL_MM * SEL_MP], lo_s[SEL_MM * SEL_MP], w_s[SEL_MM * SEL_MP];
+    const int t0 = blockIdx.x * SEL_MM, c0 = blockIdx.y * SEL_MM, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    pdl_wait();
+    pdl_trigger();
+    float acc[SEL_MM / 8][4];
+#pragma unroll
+    for (int i = 0; i < SEL_MM / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    for (int k0 = 0; k0 < rank; k0 += SEL_MK) {
+        for (int i = tid; i < SEL_MM * SEL_MK; i += 128) {
+            const int r = i / SEL_MK, k = i % SEL_MK;
+            const float v = (t0 + r < n_tokens && k0 + k < rank) ? low[(long)(t0 + r) * low_ld + k0 + k] : 0.0f;
+            const bf16 hi = __float2bfloat16_rn(v);
+            hi_s[r * SEL_MP + k] = hi;
+            lo_s[r * SEL_MP + k] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        }
+        for (int i = tid; i < SEL_MM * (SEL_MK / 8); i += 128) {
+            const int r = i / (SEL_MK / 8), k = i % (SEL_MK / 8) * 8;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (c0 + r < inner && k0 + k < w_ld) v = *reinterpret_cast<const uint4*>(w + (long)(c0 + r) * w_ld + k0 + k);
+            *reinterpret_cast<uint4*>(w_s + r * SEL_MP + k) = v;
+        }
+        __syncthreads();
+        const int ks_end = min(SEL_MK, (rank - k0 + 15) / 16 * 16);
+        for (int ks = 0; ks < ks_end; ks += 16) {
+            unsigned hi[4], lo[4];
+            sel_ldm4(hi, hi_s + (warp * 16 + (lane & 15)) * SEL_MP + ks + (lane >> 4) * 8);
+            sel_ldm4(lo, lo_s + (warp * 16 + (lane & 15)) * SEL_MP + ks + (lane >> 4) * 8);
+#pragma unroll
+            for (int j = 0; j < SEL_MM / 16; ++j) {
+                unsigned b[4];
+                sel_ldm4(b, w_s + (j * 16 + (lane & 7) + (lane >> 4) * 8) * SEL_MP + ks + ((lane >> 3) & 1) * 8);
+                sel_mma(acc[2 * j], hi, b[0], b[1]);
+                sel_mma(acc[2 * j + 1], hi, b[2], b[3]);
+                sel_mma(acc[2 * j], lo, b[0], b[1]);
+                sel_mma(acc[2 * j + 1], lo, b[2], b[3]);
+            }
+        }
+        __syncthreads();
+    }
+    const bool pairs = inner % 2 == 0 && dt_ld % 2 == 0;
+#pragma unroll
+    for (int i = 0; i < SEL_MM / 8; ++i) {
+        const int c = c0 + i * 8 + (lane & 3) * 2;
+        if (c >= inner) continue;
+        const bool both = c + 1 < inner;
+        const float b0 = bias[c], b1 = both ? bias[c + 1] : 0.0f;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int t = t0 + warp * 16 + (lane >> 2) + h * 8;
+            if (t >= n_tokens) continue;
+            float* o = dt + (long)t * dt_ld + c;
+            const float d0 = fl_softplus(acc[i][2 * h] + b0), d1 = fl_softplus(acc[i][2 * h + 1] + b1);
+            if (pairs) *reinterpret_cast<float2*>(o) = make_float2(d0, d1);
+            else {
+                o[0] = d0;
+                if (both) o[1] = d1;
+            }
+        }
+    }
+}
+
+FL_API int fl_selective_dt_mma(const float* low, long low_ld, int rank, const void* w, int w_ld, const float* bias, float* dt,
+                               long dt_ld, int n_tokens, int inner, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (rank < 1 || w_ld < rank || w_ld % 8 || ((uintptr_t)w % 16) || ((uintptr_t)dt % 8) || (inner + SEL_MM - 1) / SEL_MM > 65535)
+        return (int)cudaErrorInvalidValue;
+    return fl_launch(selective_dt_mma_kernel, dim3((n_tokens + SEL_MM - 1) / SEL_MM, (inner + SEL_MM - 1) / SEL_MM), dim3(128), 0,
+                     stream, low, low_ld, rank, (const bf16*)w, w_ld, bias, dt, dt_ld, n_tokens, inner);
+}
+
+// ------------------------------------------------------------------ the recurrence
+// exp(v) for 32-bit models, 2^v (A comes multiplied by log2(e)) for bfloat16 ones.
+template <typename T> __device__ __forceinline__ float sel_exp(float v) {
+    if constexpr (sizeof(T) == 4) return expf(v);
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+
+// A lane's rows of a channel: the groups of four 4 (lane + LANES i).  Rows from n on are zero.
+template <int R, int LANES>
+__device__ __forceinline__ void sel_rows(scan_f2 (&out)[R / 2], const float* p, int lane, int n, bool there, int vec4) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int d = 4 * (lane + LANES * i);
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (there && vec4) {
+            if (d < n) v = *reinterpret_cast<const float4*>(p + d);
+        } else if (there) {
+            if (d < n) v.x = p[d];
+            if (d + 1 < n) v.y = p[d + 1];
+            if (d + 2 < n) v.z = p[d + 2];
+            if (d + 3 < n) v.w = p[d + 3];
+        }
+        out[2 * i] = scan_pack(v.x, v.y);
+        out[2 * i + 1] = scan_pack(v.z, v.w);
+    }
+}
+template <int R, int LANES>
+__device__ __forceinline__ void sel_rows_out(const scan_f2 (&in)[R / 2], float* p, int lane, int n, int vec4) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int d = 4 * (lane + LANES * i);
+        const float2 lo = scan_unpack(in[2 * i]), hi = scan_unpack(in[2 * i + 1]);
+        if (vec4) {
+            if (d < n) *reinterpret_cast<float4*>(p + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
+        } else {
+            if (d < n) p[d] = lo.x;
+            if (d + 1 < n) p[d + 1] = lo.y;
+            if (d + 2 < n) p[d + 2] = hi.x;
+            if (d + 3 < n) p[d + 3] = hi.y;
+        }
+    }
+}
+
+// One token of a lane's rows: S <- exp(dt A) S + (dt x) B; returns the rows' part of sum S C.
+template <typename T, int R, int LANES>
+__device__ __forceinline__ float sel_token(scan_f2 (&S)[R / 2], const scan_f2 (&A)[R / 2], const float* b, const float* c,
+                                           float dt, float x, int lane) {
+    const scan_f2 dt2 = scan_pack(dt, dt), dx = scan_pack(dt * x, dt * x);
+    scan_f2 sum = 0ULL;
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const ulonglong2 bb = reinterpret_cast<const ulonglong2*>(b)[lane + LANES * i];
+        const ulonglong2 cc = reinterpret_cast<const ulonglong2*>(c)[lane + LANES * i];
+        const float2 e0 = scan_unpack(scan_mul2(dt2, A[2 * i])), e1 = scan_unpack(scan_mul2(dt2, A[2 * i + 1]));
+        S[2 * i] = scan_fma2(scan_pack(sel_exp<T>(e0.x), sel_exp<T>(e0.y)), S[2 * i], scan_mul2(bb.x, dx));
+        S[2 * i + 1] = scan_fma2(scan_pack(sel_exp<T>(e1.x), sel_exp<T>(e1.y)), S[2 * i + 1], scan_mul2(bb.y, dx));
+        sum = i == 0 ? scan_mul2(S[0], cc.x) : scan_fma2(S[2 * i], cc.x, sum);
+        sum = scan_fma2(S[2 * i + 1], cc.y, sum);
+    }
+    const float2 v = scan_unpack(sum);
+    return v.x + v.y;
+}
+
+struct SelRows {                     // the step's rows: element type T, float, float
+    const void *x, *z, *u;           // convolved inputs, gates, inputs before the convolution
+    const float *dt, *low;
+    long x_ld, z_ld, u_ld, dt_ld, low_ld;
+    int b_at, c_at;                  // where low holds B and C
+};
+
+// A block takes one request and COLS channels, LANES lanes a channel; tokens come through four stages of shared memory
+// (cp.async, three chunks ahead of the one that is walked) and go four at a time, so that four read-out sums are added up
+// over the lanes together.  R and LANES follow from n alone: one order of sums whatever the cut.
+template <typename T, int R, int LANES, int COLS, int CHUNK>
+__global__ void __launch_bounds__(COLS * LANES) selective_scan_kernel(
+    const SelRows in, const float* __restrict__ a_log2, const float* __restrict__ skip, float scale, T* __restrict__ y, long y_ld,
+    float* __restrict__ state, long state_stride, long tail_off, int taps, const int* __restrict__ req_start,
+    const int* __restrict__ req_ctx, const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int inner, int n,
+    int vec_low, int vec_dt, int vec_x, int vec_z, int vec_y, int state_vec4) {
+    static_assert(CHUNK % 4 == 0 && R % 4 == 0 && (LANES == 4 || LANES == 8 || LANES == 16) && COLS % 8 == 0, "");
+    constexpr int DP = R * LANES, THREADS = COLS * LANES, TV = 16 / sizeof(T);
+    constexpr int STAGE = CHUNK * (2 * DP + COLS) * 4 + 2 * CHUNK * COLS * (int)sizeof(T);     // bytes
+    extern __shared__ __align__(16) unsigned char sel_s[];
+    T* y_s = reinterpret_cast<T*>(sel_s + SCAN_STAGES * STAGE);       // [CHUNK][COLS]
+    pdl_wait();
+    const int r = blockIdx.x, col0 = blockIdx.y * COLS;
+    const int tid = threadIdx.x, lane = tid & (LANES - 1), col = tid / LANES, c = col0 + col;
+    const int start = req_start[r], qlen = req_qlen[r], ctx = req_ctx[r];
+    const int cols = min(COLS, inner - col0);
+    const bool mine = c < inner;
+    for (int i = tid; i < SCAN_STAGES * STAGE / 16; i += THREADS)     // padding stays zero, stale places hold numbers
+        reinterpret_cast<float4*>(sel_s)[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float* base = state + (long)req_slot[r] * state_stride;
+    float* srow = base + (long)c * n;
+    scan_f2 S[R / 2], A[R / 2];
+    sel_rows<R, LANES>(S, srow, lane, n, mine && ctx != 0, state_vec4);
+    sel_rows<R, LANES>(A, a_log2 + (long)c * n, lane, n, mine, n % 4 == 0);
+    const float skip_c = mine ? skip[c] : 0.0f;
+    __syncthreads();
+    auto stage_bc = [&](int s) { return reinterpret_cast<float*>(sel_s + s * STAGE); };
+    auto stage_dt = [&](int s) { return stage_bc(s) + CHUNK * 2 * DP; };
+    auto stage_x = [&](int s) { return reinterpret_cast<T*>(stage_dt(s) + CHUNK * COLS); };
+    auto copy_floats = [&](float* dst, int d_step, const float* src, long s_step, int count, int here, int vec) {
+        if (vec) {
+            const int per = count / 4;
+            for (int i = tid; i < per * here; i += THREADS) scan_cp16(dst + i / per * d_step + i % per * 4, src + i / per * s_step + i % per * 4);
+        } else {
+            for (int i = tid; i < count * here; i += THREADS) scan_cp4(dst + i / count * d_step + i % count, src + i / count * s_step + i % count);
+        }
+    };
+    auto copy_rows = [&](T* dst, const T* src, long s_step, int here, int vec) {
+        if (vec) {
+            const int per = cols / TV;
+            for (int i = tid; i < per * here; i += THREADS) scan_cp16(dst + i / per * COLS + i % per * TV, src + i / per * s_step + i % per * TV);
+        } else {
+            for (int i = tid; i < cols * here; i += THREADS) dst[i / cols * COLS + i % cols] = src[i / cols * s_step + i % cols];
+        }
+    };
+    auto load = [&](int s, int c0) {
+        const int here = min(CHUNK, qlen - c0);
+        const long t = start + c0;
+        copy_floats(stage_bc(s), 2 * DP, in.low + t * in.low_ld + in.b_at, in.low_ld, n, here, vec_low);
+        copy_floats(stage_bc(s) + DP, 2 * DP, in.low + t * in.low_ld + in.c_at, in.low_ld, n, here, vec_low);
+        copy_floats(stage_dt(s), COLS, in.dt + t * in.dt_ld + col0, in.dt_ld, cols, here, vec_dt);
+        copy_rows(stage_x(s), (const T*)in.x + t * in.x_ld + col0, in.x_ld, here, vec_x);
+        copy_rows(stage_x(s) + CHUNK * COLS, (const T*)in.z + t * in.z_ld + col0, in.z_ld, here, vec_z);
+        asm volatile("cp.async.commit_group;");
+    };
+    // one group of copies per chunk, empty ones beyond the end: waiting for all but the last STAGES - 1 means this one landed
+#pragma unroll
+    for (int s = 0; s < SCAN_STAGES - 1; ++s) {
+        if (s * CHUNK < qlen) load(s, s * CHUNK); else asm volatile("cp.async.commit_group;");
+    }
+    const int my_u = ((lane & (LANES / 2)) ? 2 : 0) + ((lane & (LANES / 4)) ? 1 : 0);     // the token of four whose sum this lane gets
+    const bool writer = (lane & (LANES / 4 - 1)) == 0;
+    int stage = 0;
+    for (int c0 = 0; c0 < qlen; c0 += CHUNK, stage = (stage + 1) % SCAN_STAGES) {
+        const int here = min(CHUNK, qlen - c0), ahead = c0 + (SCAN_STAGES - 1) * CHUNK;
+        // (the stage copied into now was walked in the last round, behind that round's closing barrier)
+        if (ahead < qlen) load((stage + SCAN_STAGES - 1) % SCAN_STAGES, ahead); else asm volatile("cp.async.commit_group;");
+        asm volatile("cp.async.wait_group %0;" ::"n"(SCAN_STAGES - 1));
+        __syncthreads();                                              // this chunk has landed, y_s was written out
+        const float* bc = stage_bc(stage);
+        const float* dts = stage_dt(stage) + col;
+        const T* xs = stage_x(stage) + col;
+        const T* zs = xs + CHUNK * COLS;
+        auto group = [&](int t4, int left) {
+            float acc[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int t = t4 + u;
+                const float d = u < left ? dts[t * COLS] : 0.0f;      // (behind the end: decay one, nothing added)
+                acc[u] = sel_token<T, R, LANES>(S, A, bc + t * 2 * DP, bc + t * 2 * DP + DP, d, to_f32<T>(xs[t * COLS]), lane);
+            }
+            const bool up2 = lane & (LANES / 2), up1 = lane & (LANES / 4);
+            const float w0 = scan_fold(up2, acc[0], acc[2], LANES / 2), w1 = scan_fold(up2, acc[1], acc[3], LANES / 2);
+            float v = scan_fold(up1, w0, w1, LANES / 4);
+#pragma unroll
+            for (int off = LANES / 8; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+            const int t = t4 + my_u;
+            if (writer && my_u < left)
+                y_s[t * COLS + col] = from_f32<T>(fmaf(skip_c, to_f32<T>(xs[t * COLS]), v) * fl_silu(to_f32<T>(zs[t * COLS])) * scale);
+        };
+        if (here == CHUNK) {
+#pragma unroll
+            for (int t4 = 0; t4 < CHUNK; t4 += 4) group(t4, 4);
+        } else {
+#pragma unroll 1
+            for (int t4 = 0; t4 < here; t4 += 4) group(t4, here - t4);
+        }
+        __syncthreads();                                              // y_s is whole; the stage is copied into again in the next round
+        T* yo = y + (long)(start + c0) * y_ld + col0;
+        if (vec_y) {
+            const int per = cols / TV;
+            for (int i = tid; i < per * here; i += THREADS)
+                *reinterpret_cast<uint4*>(yo + i / per * y_ld + i % per * TV) = *reinterpret_cast<const uint4*>(y_s + i / per * COLS + i % per * TV);
+        } else {
+            for (int i = tid; i < cols * here; i += THREADS) yo[i / cols * y_ld + i % cols] = y_s[i / cols * COLS + i % cols];
+        }
+    }
+    pdl_trigger();                                                    // (not at the start: the successor's CTAs would only wait here)
+    if (mine) sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
+    // the kept inputs: entry j takes the input of position end - (taps - 1) + j (entries that stay move down)
+    const T* up = (const T*)in.u;
+    for (int i = tid; i < cols; i += THREADS) {
+        float* kept = base + tail_off + col0 + i;
+        for (int j = 0; j < taps - 1; ++j) {
+            const int at = ctx + qlen - (taps - 1) + j;
+            float v = 0.0f;
+            if (at >= ctx) v = to_f32<T>(up[(long)(start + at - ctx) * in.u_ld + col0 + i]);
+            else if (at >= 0) v = kept[(long)(j + qlen) * inner];
+            kept[(long)j * inner] = v;
+        }
+    }
+}
+
+template <typename T, int R, int LANES, int COLS>
+static int selective_scan_launch(const SelRows& in, const float* a, const float* skip, float scale, T* y, long y_ld, float* state,
+                                 long state_stride, long tail_off, int taps, const int* req_start, const int* req_ctx,
+                                 const int* req_qlen, const int* req_slot, int n_requests, int inner, int n, bool overlap,
+                                 cudaStream_t stream) {
+    constexpr int CHUNK = R * LANES <= 64 ? 16 : 8;
+    constexpr size_t smem = (size_t)SCAN_STAGES * CHUNK * ((2 * R * LANES + COLS) * 4 + 2 * COLS * sizeof(T)) + CHUNK * COLS * sizeof(T);
+    auto kernel = selective_scan_kernel<T, R, LANES, COLS, CHUNK>;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    constexpr int TV = 16 / (int)sizeof(T);
+    auto rows16 = [&](const void* p, long ld) { return inner % TV == 0 && ld % TV == 0 && ((uintptr_t)p % 16) == 0 ? 1 : 0; };
+    const int vec_low = n % 4 == 0 && in.b_at % 4 == 0 && in.c_at % 4 == 0 && in.low_ld % 4 == 0 && ((uintptr_t)in.low % 16) == 0;
+    const int vec_dt = inner % 4 == 0 && in.dt_ld % 4 == 0 && ((uintptr_t)in.dt % 16) == 0;
+    const int state_vec4 = n % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0;
+    return fl_launch_as(overlap, kernel, dim3(n_requests, (inner + COLS - 1) / COLS), dim3(COLS * LANES), smem, stream, in, a, skip,
+                        scale, y, y_ld, state, state_stride, tail_off, taps, req_start, req_ctx, req_qlen, req_slot, inner, n,
+                        vec_low, vec_dt, rows16(in.x, in.x_ld), rows16(in.z, in.z_ld), rows16(y, y_ld), state_vec4);
+}
+
+static inline bool selective_takes(int inner, int n, int taps) {
+    return n >= 1 && n <= 256 && inner >= 1 && (inner + 7) / 8 <= 65535 && taps >= 1 && taps <= 16;
+}
+
+// x, z, u, y: rows of the activation type; a: -exp(A_log) [inner][n], times log2(e) for bfloat16.  single_tokens: every
+// request of the step brings one token (a short kernel).
+FL_API int fl_selective_scan(const void* x, long x_ld, const void* z, long z_ld, const void* u, long u_ld, int dtype,
+                             const float* dt, long dt_ld, const float* low, long low_ld, int b_at, int c_at, const float* a,
+                             const float* skip, float scale, void* y, long y_ld, float* state, long state_stride, long tail_off,
+                             int taps, const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot,
+                             int n_requests, int inner, int n, int single_tokens, cudaStream_t stream) {
+    if (n_requests <= 0) return 0;
+    if (!selective_takes(inner, n, taps)) return (int)cudaErrorInvalidValue;
+    const SelRows in{x, z, u, dt, low, x_ld, z_ld, u_ld, dt_ld, low_ld, b_at, c_at};
+#define FL_SEL_SCAN(R, L, C)                                                                                                 \
+    FL_DISPATCH(dtype, T, return selective_scan_launch<T, R, L, C>(in, a, skip, scale, (T*)y, y_ld, state, state_stride, tail_off, \
+                                                                   taps, req_start, req_ctx, req_qlen, req_slot, n_requests, \
+                                                                   inner, n, single_tokens != 0, stream))
+    if (n <= 16) { FL_SEL_SCAN(4, 4, 32); }
+    else if (n <= 32) { FL_SEL_SCAN(4, 8, 16); }
+    else if (n <= 64) { FL_SEL_SCAN(8, 8, 16); }
+    else if (n <= 128) { FL_SEL_SCAN(8, 16, 8); }
+    else { FL_SEL_SCAN(16, 16, 8); }
+#undef FL_SEL_SCAN
+    return 0;
+}
+
+// ------------------------------------------------------------------ single tokens
+// A warp's eight values of a weight row.
+__device__ __forceinline__ void sel_load8(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void sel_load8(const bf16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        v[2 * i] = f.x;
+        v[2 * i + 1] = f.y;
+    }
+}
+
+// Row r of the step is request r's only token.  low: `splits` slabs of rows, added up in order while they are read (one
+// slab: the rows themselves); w_dt: [inner][w_ld], w_ld a multiple of 8 and zero from column `rank` on.
+template <typename T, typename TW, int R, int LANES, int COLS>
+__global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
+    const T* __restrict__ x, long x_ld, const T* __restrict__ z, long z_ld, const float* __restrict__ low, long low_ld, int splits,
+    long split_stride, int rank, const TW* __restrict__ w_dt, int w_ld, const float* __restrict__ dt_bias,
+    const float* __restrict__ a_log2, const float* __restrict__ skip, float scale, T* __restrict__ y, long y_ld,
+    float* __restrict__ state, long state_stride, const int* __restrict__ req_ctx, const int* __restrict__ req_slot, int inner,
+    int n, int state_vec4) {
+    constexpr int DP = R * LANES, THREADS = COLS * LANES;
+    extern __shared__ __align__(16) float step_s[];                   // B [DP] | C [DP] | dt's row [w_ld]
+    const int r = blockIdx.y, tid = threadIdx.x, lane = tid & (LANES - 1), c = blockIdx.x * COLS + tid / LANES;
+    const bool mine = c < inner;
+    scan_f2 S[R / 2], A[R / 2];
+    sel_rows<R, LANES>(A, a_log2 + (long)c * n, lane, n, mine, n % 4 == 0);
+    const float skip_c = mine ? skip[c] : 0.0f, bias_c = mine ? dt_bias[c] : 0.0f;
+    const int ctx = req_ctx[r];
+    float* srow = state + (long)req_slot[r] * state_stride + (long)c * n;
+    pdl_wait();
+    pdl_trigger();
+    sel_rows<R, LANES>(S, srow, lane, n, mine && ctx != 0, state_vec4);
+    for (int i = tid; i < 2 * DP + w_ld; i += THREADS) {
+        int from = -1;
+        if (i < DP) from = i < n ? rank + i : -1;
+        else if (i < 2 * DP) from = i - DP < n ? rank + n + (i - DP) : -1;
+        else from = i - 2 * DP < rank ? i - 2 * DP : -1;
+        float v = 0.0f;
+        if (from >= 0) {
+            const float* p = low + (long)r * low_ld + from;
+            v = p[0];
+            for (int s = 1; s < splits; ++s) v += p[s * split_stride];
+        }
+        step_s[i] = v;
+    }
+    __syncthreads();
+    const float* low_s = step_s + 2 * DP;
+    float dot = 0.0f;
+    if (mine)
+        for (int k = lane * 8; k < w_ld; k += LANES * 8) {
+            float w[8];
+            sel_load8(w_dt + (long)c * w_ld + k, w);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) dot = fmaf(w[e], low_s[k + e], dot);
+        }
+#pragma unroll
+    for (int off = LANES / 2; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
+    const float dt = fl_softplus(dot + bias_c);
+    const float xv = mine ? to_f32<T>(x[(long)r * x_ld + c]) : 0.0f;
+    float sum = sel_token<T, R, LANES>(S, A, step_s, step_s + DP, dt, xv, lane);
+#pragma unroll
+    for (int off = LANES / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+    if (!mine) return;
+    if (lane == 0)
+        y[(long)r * y_ld + c] = from_f32<T>(fmaf(skip_c, xv, sum) * fl_silu(to_f32<T>(z[(long)r * z_ld + c])) * scale);
+    sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
+}
+
+FL_API int fl_selective_step(const void* x, long x_ld, const void* z, long z_ld, int dtype, const float* low, long low_ld,
+                             int splits, long split_stride, int rank, const void* w_dt, int w_dtype, int w_ld,
+                             const float* dt_bias, const float* a, const float* skip, float scale, void* y, long y_ld,
+                             float* state, long state_stride, const int* req_ctx, const int* req_slot, int n_requests, int inner,
+                             int n, cudaStream_t stream) {
+    if (n_requests <= 0) return 0;
+    if (!selective_takes(inner, n, 1) || n_requests > 65535 || rank < 1 || w_ld < rank || w_ld % 8 || ((uintptr_t)w_dt % 16) ||
+        splits < 1 || w_ld > 8192)
+        return (int)cudaErrorInvalidValue;
+    const int state_vec4 = n % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0;
+#define FL_SEL_STEP(R, L, C)                                                                                                 \
+    FL_DISPATCH(dtype, T, FL_DISPATCH(w_dtype, TW,                                                                           \
+        return fl_launch(selective_step_kernel<T, TW, R, L, C>, dim3((inner + C - 1) / C, n_requests), dim3(C * L),          \
+                         (size_t)(2 * R * L + w_ld) * sizeof(float), stream, (const T*)x, x_ld, (const T*)z, z_ld, low, low_ld, \
+                         splits, split_stride, rank, (const TW*)w_dt, w_ld, dt_bias, a, skip, scale, (T*)y, y_ld, state,     \
+                         state_stride, req_ctx, req_slot, inner, n, state_vec4)))
+    if (n <= 16) { FL_SEL_STEP(4, 4, 32); }
+    else if (n <= 32) { FL_SEL_STEP(4, 8, 16); }
+    else if (n <= 64) { FL_SEL_STEP(8, 8, 16); }
+    else if (n <= 128) { FL_SEL_STEP(8, 16, 8); }
+    else { FL_SEL_STEP(16, 16, 8); }
+#undef FL_SEL_STEP
+    return 0;
+}

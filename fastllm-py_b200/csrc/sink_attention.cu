@@ -11,15 +11,16 @@
 //
 // A cache page is [kv_heads, page_size, dim + vdim]: a token's key, then its value (the blended one).
 //
-//   sink_prep             per token: biases, both norms, the blend; q to its buffer, k and v to the token's cache rows
+//   sink_prep             per token: biases, both norms, a rotation (for attention that has one), the blend; q to its
+//                         buffer, k and v to the token's cache rows
 //   head_prep             the per-head form of the preparation, for attention whose q and k are normed head by head and
-//                         rotated (see there); head_gate multiplies a head's result by a sigmoid
+//                         rotated (see there)
 //   sink_attention_simt   per (token, query head): CUDA cores, any sizes, bfloat16 or true 32-bit; key tiles start at
 //                         multiples of 128 of the absolute position and tiles without a visible key are skipped, so
 //                         every sum's order depends on the token's own position only
 //
-// The attention kernels may multiply their result, channel by channel, by the sigmoid of a gate row of the same token
-// ([heads x vdim], in the activation type) before it is rounded.
+// The attention kernels may multiply their result by the sigmoid of a gate row of the same token (one number a channel,
+// [heads x vdim], or one a head, [heads], in the activation type) before it is rounded.
 //
 // Scores, softmax, norms, gates and the blend are float.
 #include "common.cuh"
@@ -27,36 +28,103 @@
 #define SINK_TILE 128
 
 // proj row: heads x dim queries, kv_heads x dim keys, kv_heads x vdim values.  bias: the same layout, float, or null.
+// After the norms the first `rot` dimensions of every query and key head turn by the row `position` of cos / sin
+// ([positions, rot / 2]); pair i is (2i, 2i + 1) with `interleaved`, else (i, i + rot / 2).  Values are multiplied by v_scale.
 // v_mode 0: values as they are; 1: also kept in v_first (float, [n, kv_heads x vdim]); 2: blended with v_first.
-template <typename T, typename TQ>
+// Queries and keys pass through shared memory once: VEC elements a thread and access (16 bytes of bfloat16 with 8).
+template <typename T, int VEC> __device__ __forceinline__ void prep_load(const T* p, float (&v)[VEC]) {
+    if constexpr (VEC == 8 && sizeof(T) == 2) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(p);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(h[i]);
+            v[2 * i] = f.x;
+            v[2 * i + 1] = f.y;
+        }
+    } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = to_f32<T>(p[e]);
+    }
+}
+template <typename T, int VEC> __device__ __forceinline__ void prep_store(T* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 8 && sizeof(T) == 2) {
+        uint4 raw;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        *reinterpret_cast<uint4*>(p) = raw;
+    } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) p[e] = from_f32<T>(v[e]);
+    }
+}
+
+template <typename T, typename TQ, int VEC>
 __global__ void __launch_bounds__(256) sink_prep_kernel(
     const T* __restrict__ proj, long ld, const float* __restrict__ bias, const float* __restrict__ q_w,
-    const float* __restrict__ k_w, float eps, TQ* __restrict__ q_out, long q_ld, int heads, int kv_heads, int dim, int vdim,
-    int v_mode, float lambda, float* __restrict__ v_first, long vf_ld, const int* __restrict__ slots,
-    T* __restrict__ cache, long page_stride, int page_size) {
+    const float* __restrict__ k_w, float eps, int rot, int interleaved, const float* __restrict__ cos_t,
+    const float* __restrict__ sin_t, const int* __restrict__ positions, TQ* __restrict__ q_out, long q_ld, int heads,
+    int kv_heads, int dim, int vdim, int v_mode, float lambda, float v_scale, float* __restrict__ v_first, long vf_ld,
+    const int* __restrict__ slots, T* __restrict__ cache, long page_stride, int page_size) {
     pdl_wait();
     pdl_trigger();
+    extern __shared__ __align__(16) float sink_row[];                 // [heads x dim | kv_heads x dim]
     __shared__ float scratch[32];
     const int t = blockIdx.x, tid = threadIdx.x;
     const T* row = proj + (long)t * ld;
     const int nq = heads * dim, nk = kv_heads * dim, nv = kv_heads * vdim;
     float ssq = 0.0f, ssk = 0.0f;
-    for (int i = tid; i < nq; i += blockDim.x) {
-        const float a = to_f32<T>(row[i]) + (bias ? bias[i] : 0.0f);
-        ssq += a * a;
-    }
-    for (int i = tid; i < nk; i += blockDim.x) {
-        const float a = to_f32<T>(row[nq + i]) + (bias ? bias[nq + i] : 0.0f);
-        ssk += a * a;
+    for (int i = tid * VEC; i < nq + nk; i += blockDim.x * VEC) {
+        float a[VEC];
+        prep_load<T, VEC>(row + i, a);
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            if (bias) a[e] += bias[i + e];
+            ss += a[e] * a[e];
+            sink_row[i + e] = a[e];
+        }
+        if (i < nq) ssq += ss; else ssk += ss;                        // (dim is a multiple of VEC)
     }
     ssq = block_sum(ssq, scratch);
-    ssk = block_sum(ssk, scratch);
+    ssk = block_sum(ssk, scratch);                                    // (its barriers publish sink_row)
     const float inv_q = q_w != nullptr ? 1.0f / sqrtf(ssq / (float)nq + eps) : 1.0f;
     const float inv_k = k_w != nullptr ? 1.0f / sqrtf(ssk / (float)nk + eps) : 1.0f;
+    const int half = rot / 2;
+    const long table = rot > 0 ? (long)positions[t] * half : 0;
+    // elements i .. i + VEC - 1 (d .. of their head) of the queries or keys at src, normed and turned
+    auto finish = [&](const float* src, const float* w, float inv, int i, int d, float (&o)[VEC]) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) o[e] = src[i + e] * inv * (w != nullptr ? w[i + e] : 1.0f);
+        if (d >= rot) return;
+        if (VEC > 1 && interleaved) {                                 // pairs lie within the vector (rot may end inside it)
+#pragma unroll
+            for (int e = 0; e < VEC; e += 2) {
+                if (d + e >= rot) break;
+                const float c = cos_t[table + (d + e) / 2], sn = sin_t[table + (d + e) / 2], u = o[e], v = o[e + 1 < VEC ? e + 1 : e];
+                o[e] = u * c - v * sn;
+                if (e + 1 < VEC) o[e + 1] = v * c + u * sn;
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                const int de = d + e;
+                if (de >= rot) break;
+                const bool low = interleaved ? (de & 1) == 0 : de < half;
+                const int pair = interleaved ? de / 2 : (low ? de : de - half);
+                const int io = i + e + (interleaved ? (low ? 1 : -1) : (low ? half : -half));
+                const float other = src[io] * inv * (w != nullptr ? w[io] : 1.0f);
+                const float c = cos_t[table + pair], sn = sin_t[table + pair];
+                o[e] = low ? o[e] * c - other * sn : o[e] * c + other * sn;
+            }
+        }
+    };
     TQ* qo = q_out + (long)t * q_ld;
-    for (int i = tid; i < nq; i += blockDim.x) {
-        const float a = to_f32<T>(row[i]) + (bias ? bias[i] : 0.0f);
-        qo[i] = from_f32<TQ>(q_w != nullptr ? a * inv_q * q_w[i] : a);
+    for (int i = tid * VEC; i < nq; i += blockDim.x * VEC) {
+        float o[VEC];
+        finish(sink_row, q_w, inv_q, i, i % dim, o);
+        prep_store<TQ, VEC>(qo + i, o);
     }
     if (cache == nullptr) return;
     const int slot = slots[t];
@@ -65,30 +133,53 @@ __global__ void __launch_bounds__(256) sink_prep_kernel(
     const int row_w = dim + vdim;
     T* dst = cache + page * page_stride + (long)off * row_w;                  // head g's row: + g * page_size * row_w
     const long head_stride = (long)page_size * row_w;
-    for (int i = tid; i < nk; i += blockDim.x) {
+    for (int i = tid * VEC; i < nk; i += blockDim.x * VEC) {
         const int g = i / dim, d = i - g * dim;
-        const float a = to_f32<T>(row[nq + i]) + (bias ? bias[nq + i] : 0.0f);
-        dst[g * head_stride + d] = from_f32<T>(k_w != nullptr ? a * inv_k * k_w[i] : a);
+        float o[VEC];
+        finish(sink_row + nq, k_w, inv_k, i, d, o);
+        prep_store<T, VEC>(dst + g * head_stride + d, o);
     }
-    for (int i = tid; i < nv; i += blockDim.x) {
+    for (int i = tid * VEC; i < nv; i += blockDim.x * VEC) {
         const int g = i / vdim, d = i - g * vdim;
-        float a = to_f32<T>(row[nq + nk + i]) + (bias ? bias[nq + nk + i] : 0.0f);
-        if (v_mode == 1) v_first[(long)t * vf_ld + i] = a;
-        else if (v_mode == 2) a = (1.0f - lambda) * a + lambda * v_first[(long)t * vf_ld + i];
-        dst[g * head_stride + dim + d] = from_f32<T>(a);
+        float a[VEC];
+        prep_load<T, VEC>(row + nq + nk + i, a);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            if (bias) a[e] += bias[nq + nk + i + e];
+            if (v_mode == 1) v_first[(long)t * vf_ld + i + e] = a[e];
+            else if (v_mode == 2) a[e] = (1.0f - lambda) * a[e] + lambda * v_first[(long)t * vf_ld + i + e];
+            a[e] *= v_scale;
+        }
+        prep_store<T, VEC>(dst + g * head_stride + dim + d, a);
     }
 }
 
 FL_API int fl_sink_prep(const void* proj, int dtype, long ld, const float* bias, const float* q_w, const float* k_w, float eps,
+                        int rot, int interleaved, const float* cos_t, const float* sin_t, const int* positions,
                         void* q_out, int q_dtype, long q_ld, int n_tokens, int heads, int kv_heads, int dim, int vdim,
-                        int v_mode, float lambda, float* v_first, long vf_ld, const int* slots, void* cache,
+                        int v_mode, float lambda, float v_scale, float* v_first, long vf_ld, const int* slots, void* cache,
                         long page_stride, int page_size, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (v_mode < 0 || v_mode > 2 || (v_mode != 0 && v_first == nullptr)) return (int)cudaErrorInvalidValue;
-    FL_DISPATCH(dtype, T, FL_DISPATCH(q_dtype, TQ,
-        return fl_launch(sink_prep_kernel<T, TQ>, dim3(n_tokens), dim3(256), 0, stream, (const T*)proj, ld, bias, q_w, k_w,
-                         eps, (TQ*)q_out, q_ld, heads, kv_heads, dim, vdim, v_mode, lambda, v_first, vf_ld, slots, (T*)cache,
-                         page_stride, page_size)));
+    const size_t smem = (size_t)(heads + kv_heads) * dim * sizeof(float);
+    if (v_mode < 0 || v_mode > 2 || (v_mode != 0 && v_first == nullptr) || rot < 0 || rot > dim || (rot & 1) || smem > 200 * 1024 ||
+        (rot > 0 && (cos_t == nullptr || sin_t == nullptr || positions == nullptr)))
+        return (int)cudaErrorInvalidValue;
+    const bool vec = dtype == FL_BF16 && q_dtype == FL_BF16 && dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && q_ld % 8 == 0 &&
+                     page_stride % 8 == 0 && ((uintptr_t)proj % 16) == 0 && ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)cache % 16) == 0;
+#define FL_SINK_PREP(T, TQ, V)                                                                                            \
+    {                                                                                                                     \
+        auto kernel = sink_prep_kernel<T, TQ, V>;                                                                         \
+        if (smem > 40 * 1024) {                                                                                           \
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+            if (e != cudaSuccess) return (int)e;                                                                          \
+        }                                                                                                                 \
+        return fl_launch(kernel, dim3(n_tokens), dim3(256), smem, stream, (const T*)proj, ld, bias, q_w, k_w, eps, rot,   \
+                         interleaved, cos_t, sin_t, positions, (TQ*)q_out, q_ld, heads, kv_heads, dim, vdim, v_mode,      \
+                         lambda, v_scale, v_first, vf_ld, slots, (T*)cache, page_stride, page_size);                      \
+    }
+    if (vec) FL_SINK_PREP(bf16, bf16, 8)
+    FL_DISPATCH(dtype, T, FL_DISPATCH(q_dtype, TQ, FL_SINK_PREP(T, TQ, 1)));
+#undef FL_SINK_PREP
     return 0;
 }
 
@@ -194,30 +285,9 @@ FL_API int fl_head_prep(const void* proj, int dtype, long ld, const float* bias,
     return 0;
 }
 
-// x[t, h * vdim + d] *= sigmoid(gate[t, h]): one number per token and head on the head's whole result.
-template <typename T>
-__global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ x, long x_ld, const T* __restrict__ gate, long g_ld,
-                                                        int heads, int vdim) {
-    pdl_wait();
-    pdl_trigger();
-    const int t = blockIdx.x;
-    for (int i = threadIdx.x; i < heads * vdim; i += blockDim.x) {
-        const float g = to_f32<T>(gate[(long)t * g_ld + i / vdim]);
-        x[(long)t * x_ld + i] = from_f32<T>(to_f32<T>(x[(long)t * x_ld + i]) / (1.0f + expf(-g)));
-    }
-}
-
-FL_API int fl_head_gate(void* x, int dtype, long x_ld, const void* gate, long g_ld, int n_tokens, int heads, int vdim,
-                        cudaStream_t stream) {
-    if (n_tokens <= 0) return 0;
-    FL_DISPATCH(dtype, T, return fl_launch(head_gate_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, (T*)x, x_ld,
-                                           (const T*)gate, g_ld, heads, vdim));
-    return 0;
-}
-
-// v times the sigmoid of gate[at] (no gate: v).
-template <typename T> __device__ __forceinline__ float sink_gated(float v, const T* gate, long at) {
-    return gate != nullptr ? v / (1.0f + expf(-to_f32<T>(gate[at]))) : v;
+// v times the sigmoid of head h's gate: of its one number (gate_cols 1) or of the number of channel d (no gate: v).
+template <typename T> __device__ __forceinline__ float sink_gated(float v, const T* gate, long row, int h, int gate_cols, int d) {
+    return gate != nullptr ? v / (1.0f + expf(-to_f32<T>(gate[row + (long)h * gate_cols + (gate_cols > 1 ? d : 0)]))) : v;
 }
 
 // The score of key j for a query at `pos` from the dot product.
@@ -235,7 +305,7 @@ __global__ void __launch_bounds__(SINK_TILE) sink_attention_simt_kernel(
     int page_size, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ tok_req,
     const int* __restrict__ positions, int heads, int kv_heads, int dim, int vdim, int window, int keep_first, int chunk,
     float scale, float cap, const int* __restrict__ bucket_of, int n_dist, const float* __restrict__ rel,
-    const float* __restrict__ sink, const T* __restrict__ gate, long gate_ld) {
+    const float* __restrict__ sink, const T* __restrict__ gate, long gate_ld, int gate_cols) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char sink_smem[];
@@ -302,7 +372,7 @@ __global__ void __launch_bounds__(SINK_TILE) sink_attention_simt_kernel(
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
         const int d = tid + c * SINK_TILE;
-        if (d < vdim) dst[d] = from_f32<T>(sink_gated<T>(acc[c] / l, gate, (long)t * gate_ld + (long)h * vdim + d));
+        if (d < vdim) dst[d] = from_f32<T>(sink_gated<T>(acc[c] / l, gate, (long)t * gate_ld, h, gate_cols, d));
     }
 }
 
@@ -314,7 +384,7 @@ FL_API int fl_sink_attention_simt(const void* q, int q_dtype, long q_ld, void* o
                                   const int* tok_req, const int* positions, int n_tokens, int heads, int kv_heads, int dim,
                                   int vdim, int window, int keep_first, int chunk, float scale, float cap,
                                   const int* bucket_of, int n_dist, const float* rel, const float* sink, const void* gate,
-                                  long gate_ld, cudaStream_t stream) {
+                                  long gate_ld, int gate_cols, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (vdim < 1 || vdim > 2 * SINK_TILE || dim < 1 || dim > 4096 || heads > 65535 || heads % kv_heads ||
         (rel != nullptr && (bucket_of == nullptr || n_dist < 1)))
@@ -325,7 +395,7 @@ FL_API int fl_sink_attention_simt(const void* q, int q_dtype, long q_ld, void* o
         return fl_launch(sink_attention_simt_kernel<T, TQ>, grid, dim3(SINK_TILE), smem, stream, (const TQ*)q, q_ld, (T*)out,
                          out_ld, (const T*)cache, page_stride, page_size, block_table, bt_stride, tok_req, positions, heads,
                          kv_heads, dim, vdim, window, keep_first, chunk, scale, cap, bucket_of, n_dist, rel, sink,
-                         (const T*)gate, gate_ld)));
+                         (const T*)gate, gate_ld, gate_cols)));
     return 0;
 }
 
@@ -501,7 +571,7 @@ __global__ void __launch_bounds__(128) sink_decode_merge_kernel(const float* __r
                                                                 const int* __restrict__ decode_tokens, T* __restrict__ out,
                                                                 long out_ld, int heads, int vdim,
                                                                 const float* __restrict__ sink, const T* __restrict__ gate,
-                                                                long gate_ld) {
+                                                                long gate_ld, int gate_cols) {
     pdl_wait();
     pdl_trigger();
     const int h = blockIdx.y, tid = threadIdx.x;
@@ -520,7 +590,7 @@ __global__ void __launch_bounds__(128) sink_decode_merge_kernel(const float* __r
             const float ms = base[(long)s * (vdim + 2)];
             if (ms != -CUDART_INF_F) a += base[(long)s * (vdim + 2) + 2 + d] * expf(ms - top);
         }
-        dst[d] = from_f32<T>(sink_gated<T>(a / sum, gate, (long)decode_tokens[blockIdx.x] * gate_ld + (long)h * vdim + d));
+        dst[d] = from_f32<T>(sink_gated<T>(a / sum, gate, (long)decode_tokens[blockIdx.x] * gate_ld, h, gate_cols, d));
     }
 }
 
@@ -540,7 +610,7 @@ FL_API int fl_sink_decode(const void* q, int dtype, long q_ld, void* out, long o
                           const int* decode_tokens, int n_decode, float* partial, int n_splits, int kept_splits, int heads,
                           int kv_heads, int dim, int vdim, int window, int keep_first, int chunk, float scale, float cap,
                           const int* bucket_of, int n_dist, const float* rel, const float* sink, const void* gate, long gate_ld,
-                          cudaStream_t stream) {
+                          int gate_cols, cudaStream_t stream) {
     if (n_decode <= 0) return 0;
     if (!fl_sink_decode_takes(heads, kv_heads, dim, vdim) || n_splits < 1 || n_splits > 65535 || kv_heads > 65535 ||
         kept_splits < 0 || kept_splits >= n_splits || (rel != nullptr && (bucket_of == nullptr || n_dist < 1)))
@@ -565,6 +635,6 @@ FL_API int fl_sink_decode(const void* q, int dtype, long q_ld, void* out, long o
     if (rc) return rc;
     FL_DISPATCH(dtype, T, return fl_launch(sink_decode_merge_kernel<T>, dim3(n_decode, heads), dim3(128), 0, stream,
                                            (const float*)partial, n_splits, decode_tokens, (T*)out, out_ld, heads, vdim,
-                                           sink, (const T*)gate, gate_ld));
+                                           sink, (const T*)gate, gate_ld, gate_cols));
     return 0;
 }

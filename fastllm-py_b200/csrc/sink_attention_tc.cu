@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(STC_THREADS, 3) sink_attention_tc_kernel(
     const int* __restrict__ req_start, const int* __restrict__ req_ctx, const int* __restrict__ req_qlen,
     int n_requests, int include_single, int heads, int kv_heads, int window, int keep_first, int chunk, float scale, float cap,
     const int* __restrict__ row_of, int n_dist, const float* __restrict__ rel, const float* __restrict__ sink,
-    const bf16* __restrict__ gate, long gate_ld) {
+    const bf16* __restrict__ gate, long gate_ld, int gate_cols) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) unsigned char stc_raw[];
@@ -278,13 +278,14 @@ __global__ void __launch_bounds__(STC_THREADS, 3) sink_attention_tc_kernel(
         if (row >= rows_here) continue;
         const float inv = 1.0f / l_run[r];
         bf16* dst = out + (long)(tok0 + row) * out_ld + (long)h * SINK_VDIM + 2 * tq;
-        const bf16* gr = gate != nullptr ? gate + (long)(tok0 + row) * gate_ld + (long)h * SINK_VDIM + 2 * tq : nullptr;
+        const bool by_channel = gate_cols > 1;                // else one number for the head
+        const bf16* gr = gate != nullptr ? gate + (long)(tok0 + row) * gate_ld + (long)h * gate_cols + (by_channel ? 2 * tq : 0) : nullptr;
 #pragma unroll
         for (int i = 0; i < SINK_VDIM / 8; ++i) {
             float a = o_acc[i][2 * r] * inv, b = o_acc[i][2 * r + 1] * inv;
             if (gr != nullptr) {
-                a = a / (1.0f + expf(-__bfloat162float(gr[i * 8])));
-                b = b / (1.0f + expf(-__bfloat162float(gr[i * 8 + 1])));
+                a = a / (1.0f + expf(-__bfloat162float(gr[by_channel ? i * 8 : 0])));
+                b = b / (1.0f + expf(-__bfloat162float(gr[by_channel ? i * 8 + 1 : 0])));
             }
             *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(a, b);
         }
@@ -304,7 +305,7 @@ FL_API int fl_sink_attention_tc(const void* q, long q_ld, void* out, long out_ld
                                 int include_single, int heads,
                                 int kv_heads, int window, int keep_first, int chunk, float scale, float cap, const int* row_of,
                                 int n_dist, const float* rel, const float* sink, const void* gate, long gate_ld,
-                                cudaStream_t stream) {
+                                int gate_cols, cudaStream_t stream) {
     if (n_requests <= 0 || n_tokens <= 0) return 0;
     if (heads > 65535 || heads % kv_heads || (rel != nullptr && (row_of == nullptr || n_dist < 1)))
         return (int)cudaErrorInvalidValue;
@@ -327,5 +328,5 @@ FL_API int fl_sink_attention_tc(const void* q, long q_ld, void* out, long out_ld
     return fl_launch(sink_attention_tc_kernel, grid, dim3(STC_THREADS), smem, stream, (const bf16*)q, q_ld, (bf16*)out,
                      out_ld, (const bf16*)cache, page_stride, page_size, page_shift, block_table, bt_stride, req_start,
                      req_ctx, req_qlen, n_requests, include_single, heads, kv_heads, window, keep_first, chunk, scale, cap, row_of, n_dist, rel,
-                     sink, (const bf16*)gate, gate_ld);
+                     sink, (const bf16*)gate, gate_ld, gate_cols);
 }

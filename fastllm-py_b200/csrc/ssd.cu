@@ -18,11 +18,10 @@
 //
 // All arithmetic is float (dt and the decay, two numbers a head and token, in double and rounded once: the decay is
 // multiplied up over thousands of tokens).  Every sum's order depends on the sizes alone.
+#include "short_conv.cuh"
 #include "state_scan.cuh"
 
 #define SSD_CPT 4                // value columns of a thread of the single-token kernel
-
-__device__ __forceinline__ float ssd_silu(float v) { return v / (1.0f + expf(-v)); }
 
 // dt and decay from the raw dt: neg_a = -exp(A_log), in double.
 __device__ __forceinline__ void ssd_rates(float raw, float dt_bias, double neg_a, float& dt, float& decay) {
@@ -32,50 +31,15 @@ __device__ __forceinline__ void ssd_rates(float raw, float dt_bias, double neg_a
     decay = (float)exp(neg_a * soft);
 }
 
-template <int V> struct SsdVec { float v[V]; };
-template <typename T, int V> __device__ __forceinline__ SsdVec<V> ssd_load(const T* p) {
-    SsdVec<V> r;
-    if constexpr (V == 4 && sizeof(T) == 2) {
-        const uint2 q = *reinterpret_cast<const uint2*>(p);
-        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
-        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
-        r.v[0] = lo.x; r.v[1] = lo.y; r.v[2] = hi.x; r.v[3] = hi.y;
-    } else if constexpr (V == 4) {
-        const float4 q = *reinterpret_cast<const float4*>(p);
-        r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
-    } else {
-        r.v[0] = to_f32<T>(*p);
-    }
-    return r;
-}
-template <typename T, int V> __device__ __forceinline__ void ssd_store(T* p, const SsdVec<V>& r) {
-    if constexpr (V == 4 && sizeof(T) == 2) {
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(r.v[0], r.v[1]), hi = __floats2bfloat162_rn(r.v[2], r.v[3]);
-        uint2 q;
-        q.x = *reinterpret_cast<const unsigned*>(&lo);
-        q.y = *reinterpret_cast<const unsigned*>(&hi);
-        *reinterpret_cast<uint2*>(p) = q;
-    } else if constexpr (V == 4) {
-        *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-    } else {
-        *p = from_f32<T>(r.v[0]);
-    }
-}
-
-struct SsdStep {                 // the step's tables
-    const int *tok_req, *positions, *req_start, *req_ctx, *req_qlen, *req_slot;
-};
-
 // V channels a thread, `run` consecutive tokens; the last blockIdx.y does dt and decay.  conv_w: [taps][channels].
 // TAPS: the window's length (taps rounded up).
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(128) ssd_prep_kernel(
     const T* __restrict__ proj, long ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b, int taps,
     const float* __restrict__ dt_bias, const double* __restrict__ neg_a, const float* __restrict__ tail, long tail_stride,
-    const SsdStep st, float* __restrict__ work, long w_ld, int n_tokens, int run, int inner, int channels, int heads) {
+    const StepTables st, float* __restrict__ work, long w_ld, int n_tokens, int run, int inner, int channels, int heads) {
     pdl_wait();
     pdl_trigger();
-    constexpr int WIN = TAPS > 1 ? TAPS - 1 : 1;
     const int t0 = blockIdx.x * run, t1 = min(n_tokens, t0 + run);
     if (blockIdx.y == gridDim.y - 1) {
         for (int i = threadIdx.x; i < (t1 - t0) * heads; i += blockDim.x) {
@@ -89,50 +53,16 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(
     }
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
     if (c >= channels) return;
-    SsdVec<V> w[TAPS], win[WIN];
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) {
-        const int k = j - (TAPS - taps);
-        if (k >= 0) w[j] = ssd_load<float, V>(conv_w + (long)k * channels + c);
-        else
-#pragma unroll
-            for (int e = 0; e < V; ++e) w[j].v[e] = 0.0f;
-    }
-    const SsdVec<V> b = ssd_load<float, V>(conv_b + c);
+    ShortConv<T, V, TAPS> conv;
+    conv.start(conv_w, taps, channels, c);
+    const ChanVec<V> b = chan_load<float, V>(conv_b + c);
     const T* col = proj + inner + c;
-    int known = -1;
     for (int t = t0; t < t1; ++t) {
-        const SsdVec<V> x = ssd_load<T, V>(col + (long)t * ld);
-        SsdVec<V> y;
+        const ChanVec<V> x = chan_load<T, V>(col + (long)t * ld);
+        ChanVec<V> y = conv.at(t, x, col, ld, st, tail, tail_stride, taps, channels, c);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = 0.0f;
-        if constexpr (TAPS > 1) {
-            const int r = st.tok_req[t];
-            if (r != known) {
-                known = r;
-                const int pos = st.positions[t], ctx = st.req_ctx[r];
-                const float* kept = tail + (long)st.req_slot[r] * tail_stride + c;
-#pragma unroll
-                for (int k = 0; k < WIN; ++k) {
-                    const int back = WIN - k, at = pos - back;        // window entry k holds position pos - WIN + k
-#pragma unroll
-                    for (int e = 0; e < V; ++e) win[k].v[e] = 0.0f;
-                    if (at < 0 || back > taps - 1) continue;
-                    if (at >= ctx) win[k] = ssd_load<T, V>(col + (long)(t - back) * ld);
-                    else win[k] = ssd_load<float, V>(kept + (long)(at - ctx + taps - 1) * channels);
-                }
-            }
-#pragma unroll
-            for (int j = 0; j < WIN; ++j)
-#pragma unroll
-                for (int e = 0; e < V; ++e) y.v[e] = fmaf(w[j].v[e], win[j].v[e], y.v[e]);
-#pragma unroll
-            for (int j = 0; j + 1 < WIN; ++j) win[j] = win[j + 1];
-            win[WIN - 1] = x;
-        }
-#pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = ssd_silu(fmaf(w[TAPS - 1].v[e], x.v[e], y.v[e]) + b.v[e]);
-        ssd_store<float, V>(work + (long)t * w_ld + c, y);
+        for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
+        chan_store<float, V>(work + (long)t * w_ld + c, y);
     }
 }
 
@@ -215,7 +145,7 @@ __global__ void __launch_bounds__(COLS / SSD_CPT * LANES) ssd_step_kernel(
         if (c >= 0) {
             for (int j = 0; j < taps - 1; ++j)                        // tail entry j: position ctx - (taps - 1) + j
                 if (ctx - (taps - 1) + j >= 0) v = fmaf(conv_w[(long)j * channels + c], tail[(long)j * channels + c], v);
-            v = ssd_silu(fmaf(conv_w[(long)(taps - 1) * channels + c], to_f32<T>(row[c]), v) + conv_b[c]);
+            v = fl_silu(fmaf(conv_w[(long)(taps - 1) * channels + c], to_f32<T>(row[c]), v) + conv_b[c]);
         }
         tok[i] = v;
     }
@@ -300,27 +230,25 @@ __global__ void __launch_bounds__(512) ssd_norm_kernel(
     const T* zr = proj + t * ld + first;
     float ss = 0.0f;
     for (int i = threadIdx.x * V; i < part; i += blockDim.x * V) {
-        SsdVec<V> v = ssd_load<float, V>(yr + i);
-        const SsdVec<V> z = ssd_load<T, V>(zr + i);
+        ChanVec<V> v = chan_load<float, V>(yr + i);
+        const ChanVec<V> z = chan_load<T, V>(zr + i);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-            v.v[e] *= ssd_silu(z.v[e]);
+            v.v[e] *= fl_silu(z.v[e]);
             ss += v.v[e] * v.v[e];
         }
-        ssd_store<float, V>(ssd_row + i, v);
+        chan_store<float, V>(ssd_row + i, v);
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)part + eps);
     for (int i = threadIdx.x * V; i < part; i += blockDim.x * V) {    // each thread its own elements
-        SsdVec<V> v = ssd_load<float, V>(ssd_row + i);
-        const SsdVec<V> w = ssd_load<float, V>(weight + first + i);
+        ChanVec<V> v = chan_load<float, V>(ssd_row + i);
+        const ChanVec<V> w = chan_load<float, V>(weight + first + i);
 #pragma unroll
         for (int e = 0; e < V; ++e) v.v[e] = v.v[e] * inv * w.v[e];
-        ssd_store<T, V>(out + t * out_ld + first + i, v);
+        chan_store<T, V>(out + t * out_ld + first + i, v);
     }
 }
-
-static inline bool ssd_aligned(const void* p, long ld, int elem) { return ((uintptr_t)p % (4 * elem)) == 0 && ld % 4 == 0; }
 
 // proj: rows [z | x | B | C | dt] from the given column on; work: rows x | B | C | dt | a float; neg_a: -exp(A_log).
 FL_API int fl_ssd_prep(const void* proj, int dtype, long ld, const float* conv_w, const float* conv_b, int taps,
@@ -331,11 +259,11 @@ FL_API int fl_ssd_prep(const void* proj, int dtype, long ld, const float* conv_w
     if (n_tokens <= 0) return 0;
     const int inner = heads * vdim, channels = inner + 2 * groups * n;
     if (taps < 1 || taps > 16 || (taps > 1 && tail == nullptr) || groups < 1 || heads % groups) return (int)cudaErrorInvalidValue;
-    const SsdStep st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
+    const StepTables st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
     const int run = n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : 1;
-    const bool vec = channels % 4 == 0 && inner % 4 == 0 && ssd_aligned(proj, ld, dtype == FL_F32 ? 4 : 2) &&
-                     ssd_aligned(work, w_ld, 4) && ssd_aligned(conv_w, 4, 4) && ssd_aligned(conv_b, 4, 4) &&
-                     (taps == 1 || ssd_aligned(tail, tail_stride, 4));
+    const bool vec = channels % 4 == 0 && inner % 4 == 0 && chan_aligned(proj, ld, dtype == FL_F32 ? 4 : 2) &&
+                     chan_aligned(work, w_ld, 4) && chan_aligned(conv_w, 4, 4) && chan_aligned(conv_b, 4, 4) &&
+                     (taps == 1 || chan_aligned(tail, tail_stride, 4));
     const int per = 128 * (vec ? 4 : 1);
     dim3 grid((n_tokens + run - 1) / run, (channels + per - 1) / per + 1);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
@@ -405,8 +333,8 @@ FL_API int fl_ssd_norm(const float* y, long y_ld, const void* proj, int dtype, l
     const size_t smem = (size_t)part * sizeof(float);
     if (smem > 160 * 1024) return (int)cudaErrorInvalidValue;
     const int elem = dtype == FL_F32 ? 4 : 2;
-    const bool vec = part % 4 == 0 && ssd_aligned(y, y_ld, 4) && ssd_aligned(proj, ld, elem) && ssd_aligned(out, out_ld, elem) &&
-                     ssd_aligned(weight, 4, 4);
+    const bool vec = part % 4 == 0 && chan_aligned(y, y_ld, 4) && chan_aligned(proj, ld, elem) && chan_aligned(out, out_ld, elem) &&
+                     chan_aligned(weight, 4, 4);
     int threads = 32;
     while (threads < 512 && threads * (vec ? 8 : 2) < part) threads *= 2;
     const int share = (channels + threads * parts - 1) / (threads * parts);

@@ -318,23 +318,48 @@ def softcap(logits, cap: float):
     _check(fn(_ptr(logits), _ld(logits), logits.shape[0], logits.shape[1], float(cap), _stream()), "softcap")
 
 
-def norm_pair(resid, d1, d2, w1, w2, out1, out2, eps, rows=None):
-    """resid += d1 + d2 (each may be None; written back unless rows are gathered); r = rms of the row;
-    out1 = resid / r * w1 and, when given, out2 = resid / r * w2: two norms of one row in one pass."""
-    _require_cuda(resid, d1, d2, w1, w2, out1, out2, rows)
+def _two_summands(d1, d2, what):
+    """Arguments for two pending sums (tensors of one dtype, split-K partial sums, or None each) and that dtype."""
+    for d in (d1, d2):
+        if isinstance(d, torch.Tensor):
+            _require_cuda(d)
+    dense = [d.dtype for d in (d1, d2) if isinstance(d, torch.Tensor)]
+    if len(set(dense)) > 1:
+        raise KernelError(f"{what}: both sums share a dtype")
+    args = []
+    for d in (d1, d2):
+        ptr, ld, splits, stride, _ = _summand(d)
+        args += [ptr, ld, splits, stride]
+    return args + [_CODES[dense[0]] if dense else F32]
+
+
+def norm_pair(resid, d1, d2, w1, w2, out1, out2, eps, rows=None, vectors=()):
+    """resid += d1 + d2 + the row vectors (each may be None; written back unless rows are gathered); r = rms of the row;
+    out1 = resid / r * w1 and, when given, out2 = resid / r * w2: two norms of one row in one pass.  d1 and d2 may be
+    split-K partial sums, added up while they are read."""
+    _require_cuda(resid, w1, w2, out1, out2, rows)
     if resid.dtype != torch.float32:
         raise KernelError("norm_pair: the residual stream must be float32")
-    if (d1 is not None and d2 is not None and d1.dtype != d2.dtype) or (w2 is not None and w2.dtype != w1.dtype) or \
-            (out2 is not None and out2.dtype != out1.dtype) or (w2 is None) != (out2 is None):
-        raise KernelError("norm_pair: both sums, both weights and both outputs share a dtype each")
-    fn = _fn("elementwise", "fl_norm_pair", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p,
-                                             c_void_p, c_int, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
-                                             c_float, c_void_p, c_void_p])
-    d = d1 if d1 is not None else d2
-    _check(fn(_ptr(resid), _ld(resid), _ptr(d1), 0 if d1 is None else _ld(d1), _ptr(d2), 0 if d2 is None else _ld(d2),
-              F32 if d is None else dtype_code(d), _ptr(w1), _ptr(w2), dtype_code(w1), _ptr(out1), _ld(out1),
-              _ptr(out2), 0 if out2 is None else _ld(out2), dtype_code(out1), out1.shape[0], resid.shape[1],
-              float(eps), _ptr(rows), _stream()), "norm_pair")
+    if (w2 is not None and w2.dtype != w1.dtype) or (out2 is not None and out2.dtype != out1.dtype) or (w2 is None) != (out2 is None):
+        raise KernelError("norm_pair: both weights and both outputs share a dtype each")
+    fn = _fn("elementwise", "fl_norm_pair", [c_void_p, c_long, c_void_p, c_long, c_int, c_long, c_void_p, c_long, c_int, c_long,
+                                             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_long, c_void_p,
+                                             c_long, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+    _check(fn(_ptr(resid), _ld(resid), *_two_summands(d1, d2, "norm_pair"), *_row_vectors(vectors, resid.shape[1], "norm_pair"),
+              _ptr(w1), _ptr(w2), dtype_code(w1), _ptr(out1), _ld(out1), _ptr(out2), 0 if out2 is None else _ld(out2),
+              dtype_code(out1), out1.shape[0], resid.shape[1], float(eps), _ptr(rows), _stream()), "norm_pair")
+
+
+def sum_rows(resid, d1, d2, out, vectors=()):
+    """out = resid + d1 + d2 + the row vectors (each but resid may be absent; d1 and d2 as in `norm_pair`), in out's dtype;
+    resid (float32) stays as it is."""
+    _require_cuda(resid, out)
+    if resid.dtype != torch.float32 or out.shape != resid.shape:
+        raise KernelError("sum_rows: a float32 residual stream and an output of its shape")
+    fn = _fn("elementwise", "fl_sum_rows", [c_void_p, c_long, c_void_p, c_long, c_int, c_long, c_void_p, c_long, c_int, c_long,
+                                            c_int, c_void_p, c_void_p, c_void_p, c_int, c_long, c_int, c_int, c_void_p])
+    _check(fn(_ptr(resid), _ld(resid), *_two_summands(d1, d2, "sum_rows"), *_row_vectors(vectors, resid.shape[1], "sum_rows"),
+              _ptr(out), dtype_code(out), _ld(out), resid.shape[0], resid.shape[1], _stream()), "sum_rows")
 
 
 # ------------------------------------------------------ differential attention
@@ -548,18 +573,19 @@ def latent_prep(proj, q_out, heads, dim, rot, rank, norm_w, eps, cos, sin, posit
               _ptr(positions), _ptr(slots), _ptr(cache), 0 if cache is None else 1, _stream()), "latent_prep")
 
 
-def latent_attention(q, out, cache, block_table, tok_req, positions, heads, rank, rot, window, scale, page_size):
+def latent_attention(q, out, cache, block_table, tok_req, positions, heads, rank, rot, window, scale, page_size, sink=None):
     """Attention of every token over its request's cache rows; q [N, heads * (rank + rot)] (float32 or
-    bfloat16) and out [N, heads * rank] float32.  CUDA cores, any sizes, both number formats."""
-    _require_cuda(q, out, cache, block_table, tok_req, positions)
+    bfloat16) and out [N, heads * rank] float32; with `sink` (float32 [heads]) exp(sink) is one more term of a head's
+    denominator.  CUDA cores, any sizes, both number formats."""
+    _require_cuda(q, out, cache, block_table, tok_req, positions, sink)
     if out.dtype != torch.float32:
         raise KernelError("latent_attention: out must be float32")
     fn = _fn("latent_attention", "fl_latent_attention", [c_void_p, c_int, c_long, c_void_p, c_long, c_void_p, c_int, c_int,
                                                          c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                                         c_int, c_float, c_void_p])
+                                                         c_int, c_float, c_void_p, c_void_p])
     _check(fn(_ptr(q), dtype_code(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), dtype_code(cache), page_size,
               _ptr(block_table), block_table.stride(0), _ptr(tok_req), _ptr(positions), q.shape[0], heads, rank, rot,
-              int(window or 0), float(scale), _stream()), "latent_attention")
+              int(window or 0), float(scale), _ptr(sink), _stream()), "latent_attention")
 
 
 def latent_tc_takes(dtype, rank: int, rot: int) -> bool:
@@ -572,12 +598,12 @@ def latent_tc_library(rank: int, rot: int):
 
 
 def latent_attention_tc(q, out, cache, block_table, tok_req, positions, heads, rank, rot, window, scale, page_size,
-                        split_keys=0, n_splits=1, partial=None):
+                        split_keys=0, n_splits=1, partial=None, sink=None):
     """The same on tensor cores: q and cache bfloat16, out float32 or bfloat16; one build per (rank, rot).  With
     `split_keys` (a multiple of 32) each token's keys are shared out over `n_splits` blocks, which must reach
     every token's last key ((longest visible span - 1) // split_keys + 2 does), and merged from `partial`
     (float32, N * heads * n_splits * (rank + 2))."""
-    _require_cuda(q, out, cache, block_table, tok_req, positions)
+    _require_cuda(q, out, cache, block_table, tok_req, positions, sink)
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
         raise KernelError("latent_attention_tc: q and cache must be bfloat16")
     name, defines = latent_tc_library(rank, rot)
@@ -585,10 +611,10 @@ def latent_attention_tc(q, out, cache, block_table, tok_req, positions, heads, r
         raise KernelError("latent_attention_tc: the buffer for the splits' results is too small")
     fn = _fn(name, "fl_latent_attention_tc", [c_void_p, c_long, c_void_p, c_int, c_long, c_void_p, c_int, c_void_p, c_int,
                                               c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
-                                              c_void_p], defines)
+                                              c_void_p, c_void_p], defines)
     _check(fn(_ptr(q), _ld(q), _ptr(out), dtype_code(out), _ld(out), _ptr(cache), page_size, _ptr(block_table), block_table.stride(0),
               _ptr(tok_req), _ptr(positions), q.shape[0], heads, int(window or 0), float(scale), int(split_keys),
-              int(n_splits), _ptr(partial), _stream()), "latent_attention_tc", 2 if split_keys else 1)
+              int(n_splits), _ptr(partial), _ptr(sink), _stream()), "latent_attention_tc", 2 if split_keys else 1)
 
 
 def gemm_simt_batched(a, a_batch, w, out, out_batch):
@@ -708,28 +734,38 @@ def pair_embed(table, pairs, out, step, last_token, buckets, mul_prev, mul_cur, 
 
 # ------------------------------------------------- attention with soft cap, distance bias, kept first tokens, sink
 
-def sink_prep(proj, bias, q_w, k_w, eps, q_out, heads, kv_heads, dim, vdim, v_mode, lam, v_first, slots, cache, page_size):
-    """Biases, the whole-projection norms of q and k, the blend of v with `v_first` (v_mode 0: none, 1: v is kept in
-    v_first, 2: v <- (1 - lam) v + lam v_first); q to `q_out`, k and v into the tokens' rows of `cache`
+def sink_prep(proj, bias, q_w, k_w, eps, q_out, heads, kv_heads, dim, vdim, v_mode, lam, v_first, slots, cache, page_size,
+              rot=0, interleaved=False, cos=None, sin=None, positions=None, v_scale=1.0):
+    """Biases, the whole-projection norms of q and k, the rotation of every head's first `rot` dimensions (pairs (2i, 2i + 1)
+    with `interleaved`, else (i, i + rot / 2)), the blend of v with `v_first` (v_mode 0: none, 1: v is kept in v_first, 2:
+    v <- (1 - lam) v + lam v_first), v times `v_scale`; q to `q_out`, k and v into the tokens' rows of `cache`
     ([pages, kv_heads, page_size, dim + vdim])."""
-    _require_cuda(proj, bias, q_w, k_w, q_out, v_first, slots, cache)
+    _require_cuda(proj, bias, q_w, k_w, q_out, v_first, slots, cache, cos, sin)
     if cache.dtype != proj.dtype or not cache.is_contiguous():
         raise KernelError("sink_prep: the cache must be contiguous and of the activations' dtype")
-    for v in (bias, q_w, k_w, v_first):
+    for v in (bias, q_w, k_w, v_first, cos, sin):
         if v is not None and v.dtype != torch.float32:
-            raise KernelError("sink_prep: biases, norm weights and the first values are float32")
-    fn = _fn("sink_attention", "fl_sink_prep", [c_void_p, c_int, c_long, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
-                                                c_int, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
-                                                c_long, c_void_p, c_void_p, c_long, c_int, c_void_p])
-    _check(fn(_ptr(proj), dtype_code(proj), _ld(proj), _ptr(bias), _ptr(q_w), _ptr(k_w), float(eps), _ptr(q_out),
-              dtype_code(q_out), _ld(q_out), proj.shape[0], heads, kv_heads, dim, vdim, int(v_mode), float(lam),
-              _ptr(v_first), 0 if v_first is None else _ld(v_first), _ptr(slots), _ptr(cache), cache.stride(0), page_size,
-              _stream()), "sink_prep")
+            raise KernelError("sink_prep: biases, norm weights, the rotation's tables and the first values are float32")
+    if rot and cos.shape[1] != rot // 2:
+        raise KernelError("sink_prep: the rotation's tables do not fit the rotated dimensions")
+    fn = _fn("sink_attention", "fl_sink_prep", [c_void_p, c_int, c_long, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int,
+                                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_long, c_int, c_int, c_int,
+                                                c_int, c_int, c_int, c_float, c_float, c_void_p, c_long, c_void_p, c_void_p,
+                                                c_long, c_int, c_void_p])
+    _check(fn(_ptr(proj), dtype_code(proj), _ld(proj), _ptr(bias), _ptr(q_w), _ptr(k_w), float(eps), int(rot or 0),
+              int(bool(interleaved)), _ptr(cos) if rot else None, _ptr(sin) if rot else None, _ptr(positions) if rot else None,
+              _ptr(q_out), dtype_code(q_out), _ld(q_out), proj.shape[0], heads, kv_heads, dim, vdim, int(v_mode), float(lam),
+              float(v_scale), _ptr(v_first), 0 if v_first is None else _ld(v_first), _ptr(slots), _ptr(cache), cache.stride(0),
+              page_size, _stream()), "sink_prep")
 
 
-def _check_gate(gate, out):
-    if gate is not None and (gate.dtype != out.dtype or gate.shape != out.shape):
-        raise KernelError("attention: the output gate has the output's shape and dtype")
+def _gate_args(gate, out, heads, vdim):
+    """(pointer, row pitch, numbers a head has) of an attention's output gate."""
+    if gate is None:
+        return None, 0, 1
+    if gate.dtype != out.dtype or gate.shape[0] != out.shape[0] or gate.shape[1] not in (heads, heads * vdim):
+        raise KernelError("attention: the output gate has the output's dtype and a number a head or one a channel")
+    return _ptr(gate), _ld(gate), gate.shape[1] // heads
 
 
 def sink_attention_simt(q, out, cache, block_table, tok_req, positions, heads, kv_heads, dim, vdim, window, keep_first,
@@ -737,21 +773,21 @@ def sink_attention_simt(q, out, cache, block_table, tok_req, positions, heads, k
     """Attention of every token over its request's visible keys (the last `window` and the first `keep_first`), scores
     capped (`cap` None or 0: not), biased by `rel[bucket_of[distance]]` and with `sink` in the denominator (each may be
     None).  With `chunk` a query sees only keys at or after the last multiple of `chunk` at or below its own position.
-    With `gate` ([N, heads * vdim], typed like `out`) the result is multiplied by its sigmoid, channel by channel.
+    With `gate` (typed like `out`) the result is multiplied by its sigmoid: [N, heads * vdim] channel by channel,
+    [N, heads] head by head.
     CUDA cores, any sizes, both number formats."""
     _require_cuda(q, out, cache, block_table, tok_req, positions, bucket_of, rel, sink, gate)
-    _check_gate(gate, out)
     if vdim > 256:
         raise KernelError(f"sink_attention: value size {vdim} is beyond the kernel's limit of 256")
     fn = _fn("sink_attention", "fl_sink_attention_simt",
              [c_void_p, c_int, c_long, c_void_p, c_long, c_void_p, c_int, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p,
               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
-              c_void_p, c_long, c_void_p])
+              c_void_p, c_long, c_int, c_void_p])
     _check(fn(_ptr(q), dtype_code(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), dtype_code(cache), cache.stride(0), page_size,
               _ptr(block_table), block_table.stride(0), _ptr(tok_req), _ptr(positions), q.shape[0], heads, kv_heads, dim,
               vdim, int(window or 0), int(keep_first or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(bucket_of),
-              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _ptr(gate), 0 if gate is None else _ld(gate),
-              _stream()), "sink_attention_simt")
+              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink),
+              *_gate_args(gate, out, heads, vdim), _stream()), "sink_attention_simt")
 
 
 def sink_tc_takes(dtype, dim: int, vdim: int) -> bool:
@@ -768,19 +804,18 @@ def sink_attention_tc(q, out, cache, block_table, step, heads, kv_heads, dim, vd
     """`sink_attention_simt` on tensor cores: q, cache and out bfloat16; one build per (dim, vdim); 64 rows of a
     request and one head per block, single tokens as tiles of one row (left out with include_single=False)."""
     _require_cuda(q, out, cache, block_table, bucket_of, rel, sink, gate)
-    _check_gate(gate, out)
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("sink_attention_tc: q, cache and out must be bfloat16")
     name, defines = sink_tc_library(dim, vdim)
     fn = _fn(name, "fl_sink_attention_tc", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_int,
                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                             c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long,
-                                            c_void_p], defines)
+                                            c_int, c_void_p], defines)
     _check(fn(_ptr(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), cache.stride(0), page_size, _ptr(block_table),
               block_table.stride(0), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), step.n_requests,
               q.shape[0], int(include_single), heads, kv_heads, int(window or 0), int(keep_first or 0), int(chunk or 0),
               float(scale), float(cap or 0.0), _ptr(bucket_of), 0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink),
-              _ptr(gate), 0 if gate is None else _ld(gate), _stream()), "sink_attention_tc")
+              *_gate_args(gate, out, heads, vdim), _stream()), "sink_attention_tc")
 
 
 SINK_SPLIT = 128                 # keys of one split of the single-token kernel
@@ -807,7 +842,6 @@ def sink_decode(q, out, cache, block_table, tok_req, positions, decode_tokens, p
     blocks of 128, every query head of a key/value head served by the block that reads its rows, then a merge with
     the sink.  partial: float32, decode tokens * heads * n_splits * (vdim + 2)."""
     _require_cuda(q, out, cache, block_table, tok_req, positions, decode_tokens, partial, bucket_of, rel, sink, gate)
-    _check_gate(gate, out)
     n = decode_tokens.numel()
     if partial.dtype != torch.float32 or partial.numel() < n * heads * n_splits * (vdim + 2):
         raise KernelError("sink_decode: the buffer for the splits' results is too small")
@@ -816,13 +850,13 @@ def sink_decode(q, out, cache, block_table, tok_req, positions, decode_tokens, p
     fn = _fn("sink_attention", "fl_sink_decode",
              [c_void_p, c_int, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p,
               c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-              c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p])
+              c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
     _check(fn(_ptr(q), dtype_code(q), _ld(q), _ptr(out), _ld(out), _ptr(cache), cache.stride(0), page_size,
               _ptr(block_table), block_table.stride(0), _ptr(tok_req), _ptr(positions), _ptr(decode_tokens), n,
               _ptr(partial), int(n_splits), int(kept_splits), heads, kv_heads, dim, vdim, int(window or 0),
               int(keep_first or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(bucket_of),
-              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink), _ptr(gate), 0 if gate is None else _ld(gate),
-              _stream()), "sink_decode", 2)
+              0 if bucket_of is None else bucket_of.numel(), _ptr(rel), _ptr(sink),
+              *_gate_args(gate, out, heads, vdim), _stream()), "sink_decode", 2)
 
 
 def head_prep(proj, bias, q_w, k_w, norm_mode, eps, rot, interleaved, cos, sin, positions, temp, v_from_k, q_out, heads,
@@ -850,15 +884,6 @@ def head_prep(proj, bias, q_w, k_w, norm_mode, eps, rot, interleaved, cos, sin, 
               _ptr(positions), float(coef), int(every), int(bool(v_from_k)), _ptr(q_out), dtype_code(q_out), _ld(q_out),
               proj.shape[0], heads, kv_heads, dim, vdim, _ptr(slots), _ptr(cache), cache.stride(0), page_size, _stream()),
            "head_prep")
-
-
-def head_gate(x, gate, heads, vdim):
-    """x[t, h * vdim + d] *= sigmoid(gate[t, h])."""
-    _require_cuda(x, gate)
-    if x.dtype != gate.dtype:
-        raise KernelError("head_gate: x and the gate share a dtype")
-    fn = _fn("sink_attention", "fl_head_gate", [c_void_p, c_int, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(x), dtype_code(x), _ld(x), _ptr(gate), _ld(gate), x.shape[0], heads, vdim, _stream()), "head_gate")
 
 
 def conv_head_prep(proj, bias, conv_w, tail, q_w, k_w, norm_mode, eps, rot, interleaved, cos, sin, step, temp, v_scale, q_out,
@@ -962,6 +987,91 @@ def ssd_norm(y, proj, weight, out, parts, eps, tail, taps, channels, step):
               y.shape[1], int(parts), float(eps), _ptr(tail), 0 if tail is None else tail.stride(0), int(taps), int(channels),
               _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests, _stream()),
            "ssd_norm")
+
+
+# ------------------------------------------------------------- selective scan
+
+def selective_conv(u, conv_w, conv_b, tail, step, x, move_tail):
+    """x = silu(conv(u) + conv_b): a causal convolution per channel (`conv_w` [taps, inner] float32, the last row the current
+    token's), which takes the inputs before the step's first from `tail` ([slots, >= (taps - 1) * inner] float32; None
+    with one tap).  `move_tail`: every request of the step has one token, and its kept inputs move on here."""
+    _require_cuda(u, conv_w, conv_b, tail, x)
+    taps, inner = conv_w.shape
+    if x.dtype != u.dtype or conv_w.dtype != torch.float32 or conv_b.dtype != torch.float32 or not conv_w.is_contiguous() or \
+            u.shape[1] != inner or x.shape[1] != inner or (taps > 1 and (tail is None or tail.dtype != torch.float32)):
+        raise KernelError("selective_conv: u and x share a dtype; float32 taps [taps, inner], bias and kept inputs")
+    if move_tail and step.n_tokens != step.n_requests:
+        raise KernelError("selective_conv: kept inputs move on here in steps of single tokens only")
+    fn = _fn("selective_scan", "fl_selective_conv",
+             [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+              c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(u), dtype_code(u), _ld(u), _ptr(conv_w), _ptr(conv_b), taps, _ptr(tail), 0 if tail is None else tail.stride(0),
+              _ptr(step.tok_req), _ptr(step.positions), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen),
+              _ptr(step.req_slot), _ptr(x), _ld(x), u.shape[0], inner, int(bool(move_tail)), _stream()), "selective_conv")
+
+
+def selective_dt(low, rank, w, bias, dt):
+    """dt = softplus(low[:, :rank] @ w + bias), float32.  `w` float32 [rank, inner]: sums on the CUDA cores in one order; or
+    bfloat16 [inner, >= rank] (a row pitch that is a multiple of 8, zeros from column `rank` on): tensor cores, with low as
+    two bfloat16 parts."""
+    _require_cuda(low, w, bias, dt)
+    inner = dt.shape[1]
+    if low.dtype != torch.float32 or dt.dtype != torch.float32 or bias.dtype != torch.float32 or not w.is_contiguous():
+        raise KernelError("selective_dt: low, bias and dt are float32, w is contiguous")
+    if w.dtype == torch.float32:
+        if tuple(w.shape) != (rank, inner):
+            raise KernelError("selective_dt: a float32 matrix is [rank, inner]")
+        fn = _fn("selective_scan", "fl_selective_dt", [c_void_p, c_long, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int,
+                                                       c_void_p])
+        _check(fn(_ptr(low), _ld(low), rank, _ptr(w), _ptr(bias), _ptr(dt), _ld(dt), low.shape[0], inner, _stream()), "selective_dt")
+        return
+    if w.shape[0] != inner:
+        raise KernelError("selective_dt: a bfloat16 matrix is [inner, >= rank]")
+    fn = _fn("selective_scan", "fl_selective_dt_mma", [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int,
+                                                       c_int, c_void_p])
+    _check(fn(_ptr(low), _ld(low), rank, _ptr(w), w.shape[1], _ptr(bias), _ptr(dt), _ld(dt), low.shape[0], inner, _stream()),
+           "selective_dt_mma")
+
+
+def selective_scan(x, z, u, dt, low, rank, a, skip, scale, y, state_rows, tail_off, taps, step):
+    """S <- exp(dt a) S + dt x B, y = (S C + skip x) * silu(z) * scale per channel over the step's tokens; B and C are the
+    columns of `low` (float32) from `rank` on, `a` float32 [inner, state] (times log2(e) for bfloat16 rows).  State rows:
+    S [inner, state] float32, read unless the request starts and written, and from `tail_off` on the convolution's kept
+    inputs, which move on (u: the inputs)."""
+    _require_cuda(x, z, u, dt, low, a, skip, y, state_rows)
+    inner, n = a.shape
+    if len({x.dtype, z.dtype, u.dtype, y.dtype}) != 1 or not a.is_contiguous() or \
+            any(v.dtype != torch.float32 for v in (dt, low, a, skip, state_rows)) or low.shape[1] < rank + 2 * n:
+        raise KernelError("selective_scan: x, z, u and y share a dtype, everything else is float32")
+    fn = _fn("selective_scan", "fl_selective_scan",
+             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p, c_long, c_int, c_int,
+              c_void_p, c_void_p, c_float, c_void_p, c_long, c_void_p, c_long, c_long, c_int, c_void_p, c_void_p, c_void_p,
+              c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _ld(x), _ptr(z), _ld(z), _ptr(u), _ld(u), dtype_code(x), _ptr(dt), _ld(dt), _ptr(low), _ld(low), rank,
+              rank + n, _ptr(a), _ptr(skip), float(scale), _ptr(y), _ld(y), _ptr(state_rows), state_rows.stride(0), int(tail_off),
+              int(taps), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests,
+              inner, n, int(x.shape[0] == step.n_requests), _stream()), "selective_scan")
+
+
+def selective_step(x, z, low, rank, w_dt, dt_bias, a, skip, scale, y, state_rows, step):
+    """selective_dt and selective_scan in one kernel for a step in which every request brings one token (the kept inputs are
+    left as they are).  `low` may be split-K partial sums, added up while they are read; `w_dt` [inner, >= rank] as in
+    `selective_dt`, of either dtype."""
+    _require_cuda(x, z, w_dt, dt_bias, a, skip, y, state_rows)
+    inner, n = a.shape
+    if step.n_tokens != step.n_requests or len({x.dtype, z.dtype, y.dtype}) != 1 or not w_dt.is_contiguous() or \
+            w_dt.shape[0] != inner or any(v.dtype != torch.float32 for v in (dt_bias, a, skip, state_rows)) or not a.is_contiguous():
+        raise KernelError("selective_step: one token a request; x, z and y share a dtype; float32 parameters and state")
+    ptr, ld, splits, stride, code = _summand(low)
+    if code != F32:
+        raise KernelError("selective_step: low is float32")
+    fn = _fn("selective_scan", "fl_selective_step",
+             [c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_int, c_int, c_void_p,
+              c_void_p, c_void_p, c_float, c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _ld(x), _ptr(z), _ld(z), dtype_code(x), ptr, ld, max(splits, 1), stride, rank, _ptr(w_dt), dtype_code(w_dt),
+              w_dt.shape[1], _ptr(dt_bias), _ptr(a), _ptr(skip), float(scale), _ptr(y), _ld(y), _ptr(state_rows),
+              state_rows.stride(0), _ptr(step.req_ctx), _ptr(step.req_slot), step.n_requests, inner, n, _stream()),
+           "selective_step")
 
 
 # ----------------------------------------------- layer norm, mixes, activation
@@ -1125,21 +1235,22 @@ def moe_pick(logits, bias, chosen, weights, top, softmax_scores=False, renormali
 
 
 def moe_experts(h, w_gate_up, w_down, chosen, weights, act_buf, out, activation="silu", params=(0.0, 0.0), gated=True,
-                accumulate=False):
+                accumulate=False, weight_on_input=False):
     """out[t] = sum_k weights[t, k] * down[e](f(gate[e] h[t], up[e] h[t])), e = chosen[t, k], f as in ACTIVATIONS;
     w_gate_up [E, 2 ff, width], w_down [E, width, ff]; act_buf float32 [N * top, ff].  Without a gate
     (`gated=False`) w_gate_up is the up matrices alone, [E, ff, width], and the unit is f(up[e] h[t], 1).  With
-    `accumulate` the sum is added to what `out` holds."""
+    `accumulate` the sum is added to what `out` holds.  `weight_on_input`: a weight multiplies h[t] and not the result."""
     _require_cuda(h, w_gate_up, w_down, chosen, weights, act_buf, out)
     experts, ff2, width = w_gate_up.shape
     if not gated:
         ff2 *= 2
     fn = _fn("moe", "fl_moe_experts", [c_void_p, c_int, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                                       c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p])
+                                       c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int,
+                                       c_void_p])
     _check(fn(_ptr(h), dtype_code(h), _ld(h), _ptr(w_gate_up), _ptr(w_down), dtype_code(w_gate_up), _ptr(chosen),
               _ptr(weights), _ptr(act_buf), _ptr(out), _ld(out), h.shape[0], width, ff2 // 2, chosen.shape[1],
-              activation_code(activation), float(params[0]), float(params[1]), int(gated), int(accumulate), _stream()),
-           "moe_experts", 2)
+              activation_code(activation), float(params[0]), float(params[1]), int(gated), int(accumulate),
+              int(weight_on_input), _stream()), "moe_experts", 2)
 
 
 def moe_group_rows(n_tokens: int, top: int, experts: int) -> int:
@@ -1159,22 +1270,23 @@ def moe_group_takes(h_dtype, w_dtype, width: int, ff: int) -> bool:
 
 
 def moe_experts_grouped(h, w_gate_up, w_down, chosen, weights, ints, act, y, out, activation="silu", params=(0.0, 0.0),
-                        gated=True, accumulate=False):
+                        gated=True, accumulate=False, weight_on_input=False):
     """The same sum as `moe_experts` for many tokens: pairs ordered by expert, two tensor-core products
     over tiles of 64 rows, then the weighted sum per token.  All bfloat16; `ints` int32
     [rows + N * top + rows / 64 + 1], `act` bfloat16 [rows, ff], `y` float32 [rows, width] with
-    rows = moe_group_rows(N, top, experts).  `gated=False`: as in `moe_experts`."""
+    rows = moe_group_rows(N, top, experts).  `gated=False` and `weight_on_input`: as in
+    `moe_experts`."""
     _require_cuda(h, w_gate_up, w_down, chosen, weights, ints, act, y, out)
     experts, ff2, width = w_gate_up.shape
     if not gated:
         ff2 *= 2
     fn = _fn("moe", "fl_moe_experts_grouped", [c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                                c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int,
-                                               c_int, c_float, c_float, c_int, c_int, c_void_p])
+                                               c_int, c_float, c_float, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(h), _ld(h), _ptr(w_gate_up), _ptr(w_down), _ptr(chosen), _ptr(weights), _ptr(ints), _ptr(act),
               _ptr(y), _ptr(out), _ld(out), h.shape[0], width, ff2 // 2, chosen.shape[1], experts,
-              activation_code(activation), float(params[0]), float(params[1]), int(gated), int(accumulate), _stream()),
-           "moe_experts_grouped", 4)
+              activation_code(activation), float(params[0]), float(params[1]), int(gated), int(accumulate),
+              int(weight_on_input), _stream()), "moe_experts_grouped", 4)
 
 
 # -------------------------------------------------------------- rope + cache

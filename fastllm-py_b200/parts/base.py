@@ -17,6 +17,8 @@ engine's StepContext; buffers come from `step.workspace`):
   feed_forward  forward(h, out, step)
   block         forward(stream, step, cache)  the arrangement of mixer, feed-forward and norms
   head          forward(h, out)               h: [m, hidden] -> out: [m, vocab] float32
+  entry         keep(stream, step)            the stream as the embedding leaves it
+                forward(stream, step)         replaces the stream before a run of a layer
 
 What a part may declare beside its interface (all optional; absent means "no"):
 
@@ -33,7 +35,8 @@ What a part may declare beside its interface (all optional; absent means "no"):
                            (otherwise the stream adds them up into a tensor first)
   takes_post_norm = True   norm: `apply` understands `stream.pending_norm` (the pending sum is normed by
                            that part before it is added); such a norm also has `add_normed(stream)`
-  takes_extra = True       norm: `apply` adds `stream.extra` (a second tensor) along with a pending tensor; such a
+  takes_extra = True       norm: `apply` adds `stream.extra` (a second sum) along with the pending one, each a tensor
+                           or partial sums, also under gathered rows, and row vectors where nothing is pending; such a
                            norm also has `apply_pair(stream, other, out, out_other)`: its own norm and that of
                            `other` (same kind, size and eps) of the one row in one pass
   takes_vectors = True     norm: `apply` adds `stream.vectors` (row vectors) along with a pending sum
@@ -105,8 +108,8 @@ class ResidualStream:
         self.pending = None
         self.pending_norm = None     # a norm part the pending sum passes before it is added (blocks that norm
         self.spill = spill           # a sublayer's output); a norm with `takes_post_norm` does both in one kernel
-        self.extra = None            # a second tensor not yet added (a layer whose mixer and feed-forward run side by
-                                     # side leaves two); a norm with `takes_extra` adds both while it reads
+        self.extra = None            # a second sum not yet added (a layer whose mixer and feed-forward run side by
+                                     # side leaves two; a tensor, or partial sums); a norm with `takes_extra` adds both while it reads
         self.pending_scale = 1.0     # the pending sum is multiplied by this as it is added (a layer that scales its
                                      # sublayers' results); a norm with `takes_scale` does so while it reads
         self.vectors = ()            # float32 row vectors [hidden] not yet added, each to every row (a product's output
@@ -145,13 +148,24 @@ class ResidualStream:
             else:
                 ops.residual_add(self.x, self.pending)
                 self.pending = None
+        self._add_extra()
+
+    def _add_extra(self):
+        """x += extra, for whoever cannot take it itself."""
+        from ..native import ops
         if self.extra is not None:
+            if not isinstance(self.extra, torch.Tensor):
+                self.extra = self.extra.reduce_into(self.spill("delta_ff"))
             ops.residual_add(self.x, self.extra)
             self.extra = None
 
     def norm_into(self, norm, out, rows=None):
         """`norm.apply(self, out, rows)`, with a pending sum that the norm can take."""
         pending = self.pending
+        if getattr(norm, "takes_extra", False) and self.pending_scale == 1.0 and self.pending_norm is None and \
+                (self.extra is not None or (self.vectors and pending is None)):
+            norm.apply(self, out, rows)                  # everything that waits is added while the row is read
+            return
         if self.vectors and (pending is None or self.pending_scale != 1.0 or self.pending_norm is not None or
                              self.extra is not None or not getattr(norm, "takes_vectors", False)):
             self._add_vectors()
@@ -166,11 +180,7 @@ class ResidualStream:
             pending = None
         if pending is not None and self.pending_norm is not None and not getattr(norm, "takes_post_norm", False):
             self.pending_norm.add_normed(self)           # x += norm(pending), for a norm that cannot do it itself
-        if self.extra is not None and (not getattr(norm, "takes_extra", False) or self.pending_norm is not None
-                                       or not isinstance(self.pending, torch.Tensor)):
-            from ..native import ops
-            ops.residual_add(self.x, self.extra)         # x += extra, for a norm (or a pending sum) that cannot
-            self.extra = None
+        self._add_extra()
         norm.apply(self, out, rows)
 
 

@@ -13,8 +13,9 @@ its norm; the next norm of the stream does norm, add and norm in one kernel.
 
 "parallel" runs mixer and feed-forward side by side on the same x, each behind a norm of its own:
     x = x + mixer(norm_mixer(x)) + feed_forward(norm_ff(x))
-and may have no feed-forward.  Both outputs are left pending; the next layer's two norms share
-the row's root mean square, so one kernel adds both sums and writes both normed rows.
+or both behind the one norm: x = x + (mixer(h) + feed_forward(h)), h = norm_mixer(x); it may have no
+feed-forward.  Both outputs are left pending; the next layer's two norms share the row's root mean
+square, so one kernel adds both sums and writes both normed rows.
 """
 from __future__ import annotations
 
@@ -106,7 +107,7 @@ class SandwichBlock(Part):
 
 @register_part("block", "parallel")
 class ParallelBlock(Part):
-    """norm roles: "mixer" and, with a feed-forward, "feed_forward"."""
+    """norm roles: "mixer" and, for a feed-forward with a norm of its own, "feed_forward"."""
     category = "block"
 
     def __init__(self, layer_spec, ctx):
@@ -116,13 +117,17 @@ class ParallelBlock(Part):
         self.feed_forward = self.norm_ff = None
         if layer_spec.feed_forward is not None:
             self.feed_forward = build_part("feed_forward", layer_spec.feed_forward, ctx)
-            self.norm_ff = build_part("norm", layer_spec.norms["feed_forward"], ctx)
+            if "feed_forward" in layer_spec.norms:
+                self.norm_ff = build_part("norm", layer_spec.norms["feed_forward"], ctx)
+            # the mixer's last product may wait as partial sums while the feed-forward's products run
+            if getattr(self.mixer, "honours_partial_side", False):
+                self.mixer.partial_side = True
         self.hidden = self.norm_mixer.size
 
     def children(self):
         parts = [self.mixer, self.norm_mixer]
         if self.feed_forward is not None:
-            parts += [self.feed_forward, self.norm_ff]
+            parts += [self.feed_forward] + ([self.norm_ff] if self.norm_ff is not None else [])
         return parts
 
     def forward(self, stream, step, cache):
@@ -131,29 +136,25 @@ class ParallelBlock(Part):
         ws = step.workspace
         h = ws.rows("normed", n, self.hidden, dt)
         delta = ws.rows("delta", n, self.hidden, dt)
-        if self.feed_forward is None:
+        h_ff = h
+        if self.norm_ff is None:
             stream.norm_into(self.norm_mixer, h)
         else:
             h_ff = ws.rows("normed_ff", n, self.hidden, dt)
             pairs = getattr(self.norm_mixer, "pairs_with", None)
-            if pairs is not None and pairs(self.norm_ff) and stream.pending_norm is None:
-                if stream.pending is not None and not isinstance(stream.pending, torch.Tensor):
-                    stream.pending = stream.pending.reduce_into(stream.spill())
+            if pairs is not None and pairs(self.norm_ff) and stream.pending_norm is None and stream.pending_scale == 1.0:
                 self.norm_mixer.apply_pair(stream, self.norm_ff, h, h_ff)
             else:
                 stream.norm_into(self.norm_mixer, h)          # adds what was pending
                 stream.norm_into(self.norm_ff, h_ff)
-        # the split-K scratch is shared: partial sums are added up before the other sublayer's products run
         left = self.mixer.forward(h, delta, step, cache)
-        if left is not None:
-            left.reduce_into(delta)
-        stream.pending = delta
+        if left is not None and self.feed_forward is not None and not getattr(self.mixer, "partial_side", False):
+            left = left.reduce_into(delta)                    # the feed-forward's products use the same scratch
+        stream.pending = delta if left is None else left
         if self.feed_forward is not None:
             delta_ff = ws.rows("delta_ff", n, self.hidden, dt)
             left = self.feed_forward.forward(h_ff, delta_ff, step)
-            if left is not None:
-                left.reduce_into(delta_ff)
-            stream.extra = delta_ff
+            stream.extra = delta_ff if left is None else left
 
 
 @register_part("block", "gated_postnorm")

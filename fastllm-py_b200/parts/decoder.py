@@ -28,6 +28,7 @@ class Decoder:
         self.final_norm = build_part("norm", plan.final_norm, ctx)
         self.head = build_part("head", plan.head, ctx)
         self.vectors = build_part("vectors", plan.vectors, ctx) if plan.vectors is not None else None
+        self.entry = build_part("entry", plan.entry, ctx) if plan.entry is not None else None
         self.order = list(plan.order)
         # cache id of each run and, for a mixer with several needs, their names
         self._views_of = []
@@ -61,6 +62,8 @@ class Decoder:
         visit(self.embedding)
         if self.vectors is not None:
             visit(self.vectors)
+        if self.entry is not None:
+            visit(self.entry)
         for b in self.blocks:
             visit(b)
         visit(self.final_norm)
@@ -189,11 +192,13 @@ class Decoder:
         n = step.n_tokens
         ws = step.workspace
         stream = ResidualStream(ws.rows("residual", n, self.hidden, torch.float32),
-                                spill=lambda: ws.rows("delta", n, self.hidden, self.ctx.dtype))
+                                spill=lambda name="delta": ws.rows(name, n, self.hidden, self.ctx.dtype))
         if hasattr(self.embedding, "state_need"):
             self.embedding.forward(step, stream.x, step.cache_view(self.EMBEDDING_STATE, True))
         else:
             self.embedding.forward(step, stream.x)
+        if self.entry is not None:
+            self.entry.keep(stream, step)
         for i, run in enumerate(self.order):
             cache_id, names = self._views_of[i]
             block = self.blocks[run.layer]
@@ -201,6 +206,8 @@ class Decoder:
                 cache = {name: step.cache_view((cache_id, name), run.cache is None) for name in names}
             else:
                 cache = step.cache_view(cache_id, run.cache is None)
+            if run.entry:
+                self.entry.forward(stream, step)
             if run.vector is not None:
                 stream.add_vector(self.vectors.row(run.vector))
             if hasattr(block, "state_need"):

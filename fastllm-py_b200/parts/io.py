@@ -106,6 +106,43 @@ class VectorTable(Part):
         return self.table[i]
 
 
+@register_part("entry", "rejoin")
+class Rejoin(Part):
+    """x <- W [x; x0]: the residual stream replaced by a product of itself beside the embedding output.
+    params: hidden_size.  tensors: weight [hidden, 2 hidden] (x first)."""
+    category = "entry"
+
+    def __init__(self, spec, ctx):
+        super().__init__(spec, ctx)
+        self.hidden = int(spec.params["hidden_size"])
+        self.linear = None
+
+    def weight_shapes(self):
+        return {"weight": (self.hidden, 2 * self.hidden)}
+
+    def load(self, tensors):
+        self.linear = Linear([tensors["weight"]])
+
+    def reserve(self, limits):
+        if self.linear is not None:
+            self.linear.reserve(self.ctx.dtype, limits.max_tokens)
+
+    def _operand(self, stream, step):
+        return step.workspace.rows("entry_operand", stream.x.shape[0], 2 * self.hidden, self.ctx.dtype)
+
+    def keep(self, stream, step):
+        ops.sum_rows(stream.x, None, None, self._operand(stream, step)[:, self.hidden:])
+
+    def forward(self, stream, step):
+        operand = self._operand(stream, step)
+        if stream.pending_scale != 1.0 or stream.pending_norm is not None:
+            stream.settle()
+        ops.sum_rows(stream.x, stream.pending, stream.extra, operand[:, :self.hidden], stream.vectors)
+        stream.pending = stream.extra = None
+        stream.vectors = ()
+        self.linear.forward(operand, stream.x)               # (float accumulation, float result)
+
+
 @register_part("head", "linear")
 class LinearHead(Part):
     """params: vocab_size, hidden_size, softcap (None | c > 0).  tensors: weight [vocab, hidden]."""

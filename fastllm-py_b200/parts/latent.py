@@ -27,6 +27,7 @@ is then stacked with W_dkv (and the gate) into the layer's first product.
 `out_gate`: the concatenated heads are multiplied by sigmoid(W_g h) before W_o.
 `pairing` names the rotary pairs: "halves" (i, i + rot_dim/2) or "interleaved"
 (2i, 2i + 1); pair i turns by the position table's column i either way.
+`sink`: one learned number per head whose exponential is one more term of the softmax's denominator.
 """
 from __future__ import annotations
 
@@ -43,15 +44,17 @@ from .registry import build_part, register_part
 class LatentAttention(Part):
     """params: hidden_size, heads, dim, rot_dim, vdim, kv_rank, scale, window (None | int), keep (None | int: what the
     cache keeps; absent: `window`), norm_eps, position (PartSpec of rot_dim dims), shares_cache (bool),
-    q_rank (None | int), out_gate (bool), pairing ("halves" | "interleaved").
+    q_rank (None | int), out_gate (bool), pairing ("halves" | "interleaved"), sink (bool).
     tensors: q [heads * (dim + rot_dim), hidden] (with q_rank instead: dq [q_rank, hidden], dq_norm [q_rank],
     uq [heads * (dim + rot_dim), q_rank]), uk [heads * dim, kv_rank], uv [heads * vdim, kv_rank],
-    o [hidden, heads * vdim], with out_gate g [heads * vdim, hidden], and, unless shares_cache,
+    o [hidden, heads * vdim], with out_gate g [heads * vdim, hidden], with sink sink [heads], and, unless shares_cache,
     dkv [kv_rank + rot_dim, hidden], dkv_norm [kv_rank]."""
     category = "mixer"
     native_libraries = ("latent_attention", "gemm_mma", "gated_block")
     SPLIT_BELOW = 64                 # blocks (tokens x groups of 16 heads) under which a step's keys are split
     SCRATCH = "latent attention splits"
+    honours_partial_side = True      # with `partial_side` set, the last product's partial sums go to the second scratch
+    partial_side = False
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -66,6 +69,7 @@ class LatentAttention(Part):
         self.shares_cache = bool(p.get("shares_cache", False))
         self.q_rank = int(p["q_rank"]) if p.get("q_rank") else None
         self.out_gate = bool(p.get("out_gate", False))
+        self.has_sink = bool(p.get("sink", False))
         if p.get("pairing", "halves") not in ("halves", "interleaved"):
             raise ValueError(f"latent_attention: pairing {p.get('pairing')!r} is neither 'halves' nor 'interleaved'")
         self.interleaved = p.get("pairing", "halves") == "interleaved"
@@ -78,7 +82,7 @@ class LatentAttention(Part):
             raise ValueError("latent_attention: the position encoding must turn exactly rot_dim dimensions")
         self.q_cols = self.heads * (self.dim + self.rot)
         self.width = self.rank + self.rot                               # a cache row
-        self.proj = self.o = self.uq = self.dq_norm = None
+        self.proj = self.o = self.uq = self.dq_norm = self.sink = None
 
     def children(self):
         return [self.position]
@@ -96,6 +100,8 @@ class LatentAttention(Part):
                            "uq": (self.q_cols, self.q_rank)})
         if self.out_gate:
             shapes["g"] = (self.heads * self.vdim, self.hidden)
+        if self.has_sink:
+            shapes["sink"] = (self.heads,)
         if not self.shares_cache:
             shapes["dkv"] = (self.width, self.hidden)
             shapes["dkv_norm"] = (self.rank,)
@@ -118,6 +124,7 @@ class LatentAttention(Part):
         self.uk_t = tensors["uk"].view(self.heads, self.dim, self.rank).transpose(1, 2).contiguous()
         self.uv = tensors["uv"].view(self.heads, self.vdim, self.rank).contiguous()
         self.o = Linear([tensors["o"]])
+        self.sink = tensors["sink"].float().contiguous() if self.has_sink else None
 
     def native_builds(self):
         """(library, defines) pairs compiled for this part's sizes, so that a model's first load builds them beside
@@ -128,7 +135,7 @@ class LatentAttention(Part):
     def reserve(self, limits):
         for lin in (self.proj, self.o, self.uq):
             if lin is not None:
-                lin.reserve(self.ctx.dtype, limits.max_tokens)
+                lin.reserve(self.ctx.dtype, limits.max_tokens, side=lin is self.o and self.partial_side)
         if self.ctx.device.type == "cuda" and ops.latent_tc_takes(self.ctx.dtype, self.rank, self.rot):
             from ..native.build import load_library
             load_library(*ops.latent_tc_library(self.rank, self.rot))      # built now, not inside the first step
@@ -197,11 +204,11 @@ class LatentAttention(Part):
             keys, splits = step.plans[self.plan_key]
             ops.latent_attention_tc(q, mix, cache.tensor, cache.block_table, step.tok_req, step.positions, self.heads,
                                     self.rank, self.rot, self.window, self.scale, cache.page_size, keys, splits,
-                                    self._partials(n, splits) if keys else None)
+                                    self._partials(n, splits) if keys else None, self.sink)
         else:
             ops.latent_attention(q, mix, cache.tensor, cache.block_table, step.tok_req, step.positions, self.heads,
-                                 self.rank, self.rot, self.window, self.scale, cache.page_size)
+                                 self.rank, self.rot, self.window, self.scale, cache.page_size, self.sink)
         ctx = ws.rows("latent_ctx", n, self.heads * self.vdim, dt)
         ops.gemm_batched(mix, self.rank, self.uv, ctx, self.vdim,
                          gate=ws.rows("latent_proj", n, cols, dt)[:, first + kv_cols:] if self.out_gate else None)
-        return self.o.forward(ctx, out, defer=True)
+        return self.o.forward(ctx, out, defer=True, side=self.partial_side)

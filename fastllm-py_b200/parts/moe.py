@@ -8,7 +8,8 @@ the weights are the chosen experts' s, divided by their sum (+ `renormalise_eps`
 only if `renormalise` says so.  With `groups`, the experts form that many equal
 groups of neighbours, a group's score is the sum of the `group_top` largest s + bias
 in it (1: the largest), and only experts of the `keep_groups` best groups can be
-chosen.  The weights are multiplied by `weight_scale` at the end.  Expert e:
+chosen.  The weights are multiplied by `weight_scale` at the end.  A weight multiplies the
+expert's result, or with `weight_on` "input" what the expert reads (exactly: its gate and up sums, before the activation).  Expert e:
 W_down,e f(W_gate,e h, W_up,e h) with f = act(g) * u or the clamped swish unit
 (`native.ops.ACTIVATIONS`), no biases; without a gate (`gated` False) W_down,e f(W_up,e h, 1).
 The experts' matrices are stacked at load into [experts, 2 ff, hidden]
@@ -36,7 +37,7 @@ from .registry import build_part, register_part
 class RoutedExperts(Part):
     """params: hidden_size, experts, top, expert_ff, activation ("silu"), activation_params ((0, 0)), score ("sigmoid"),
     renormalise (False), renormalise_eps (0), groups (None), keep_groups (None: all), group_top (1),
-    weight_scale (1), gated (True), shared (None | PartSpec of a feed-forward),
+    weight_scale (1), weight_on ("output" | "input"), gated (True), shared (None | PartSpec of a feed-forward),
     choice_bias (True: a `correction` tensor is added to the scores for the choice).
     tensors: router [experts, hidden], correction [experts] (if choice_bias), and per expert i
     gate.i (if gated), up.i [ff, hidden], down.i [hidden, ff]."""
@@ -58,6 +59,9 @@ class RoutedExperts(Part):
         self.renormalise_eps = float(p.get("renormalise_eps", 0.0))
         self.group_top = int(p.get("group_top", 1))
         self.weight_scale = float(p.get("weight_scale", 1.0))
+        self.on_input = p.get("weight_on", "output") == "input"
+        if p.get("weight_on", "output") not in ("output", "input"):
+            raise ValueError(f"routed_experts: weight_on {p['weight_on']!r} is neither 'output' nor 'input'")
         self.gated = bool(p.get("gated", True))
         self.shared = build_part("feed_forward", p["shared"], ctx) if p.get("shared") is not None else None
         self.score = p.get("score", "sigmoid")
@@ -140,9 +144,9 @@ class RoutedExperts(Part):
         if n * self.top >= self.GROUP_FROM and self._grouped(h.dtype):
             ints, act, y = self._group_buffers(n, h.device)
             ops.moe_experts_grouped(h, self.gate_up, self.down, chosen, weights, ints, act, y, out, self.activation,
-                                    self.activation_params, self.gated, accumulate=shared)
+                                    self.activation_params, self.gated, accumulate=shared, weight_on_input=self.on_input)
         else:
             act = ws.rows("moe_act", n, self.top * self.ff, torch.float32)
             ops.moe_experts(h, self.gate_up, self.down, chosen, weights, act, out, self.activation, self.activation_params,
-                            self.gated, accumulate=shared)
+                            self.gated, accumulate=shared, weight_on_input=self.on_input)
         return None

@@ -19,7 +19,7 @@ class RMSNorm(Part):
     takes_vectors = True                 # row vectors are added while the row is read
     takes_partial = True                 # split-K partial sums are added while the row is read
     takes_post_norm = True               # a pending sum that passes another RMSNorm first: one kernel does both
-    takes_extra = True                   # two tensors pending: both are added while the row is read
+    takes_extra = True                   # two sums pending: both are added while the row is read
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -42,11 +42,13 @@ class RMSNorm(Part):
         With `rows` (int32 indices) only those rows are normed, into out[0..m), and the
         pending sum (a tensor then: `ResidualStream.norm_into` sees to it) stays pending."""
         post = getattr(stream, "pending_norm", None)
-        if getattr(stream, "extra", None) is not None:
-            # two sums pending (tensors; `ResidualStream.norm_into` sees to it): x += pending + extra; out = self(x)
-            ops.norm_pair(stream.x, stream.pending, stream.extra, self.weight, None, out, None, self.eps, rows)
+        vectors = getattr(stream, "vectors", ())
+        if getattr(stream, "extra", None) is not None or (vectors and stream.pending is None):
+            # two sums pending (tensors or partial sums), or row vectors alone: x += all of it; out = self(x)
+            ops.norm_pair(stream.x, stream.pending, stream.extra, self.weight, None, out, None, self.eps, rows, vectors)
             if rows is None:
                 stream.pending = stream.extra = None
+                stream.vectors = ()
             return
         if stream.pending is not None and post is not None:
             # x += post(pending); out = self(x): the layer norms the sublayer's output before adding it
@@ -81,10 +83,12 @@ class RMSNorm(Part):
             other.weight.dtype == self.weight.dtype
 
     def apply_pair(self, stream, other, out, out_other):
-        """x += pending (+ extra); out = self(x), out_other = other(x): the two norms share the row's root
-        mean square, so one pass serves both.  The pending sum must be a tensor (or none) without a norm of its own."""
-        ops.norm_pair(stream.x, stream.pending, stream.extra, self.weight, other.weight, out, out_other, self.eps)
+        """x += pending (+ extra, + row vectors); out = self(x), out_other = other(x): the two norms share the row's root
+        mean square, so one pass serves both.  The pending sum must be without a factor and a norm of its own."""
+        ops.norm_pair(stream.x, stream.pending, stream.extra, self.weight, other.weight, out, out_other, self.eps, None,
+                      stream.vectors)
         stream.pending = stream.extra = None
+        stream.vectors = ()
 
 
 @register_part("norm", "layernorm")

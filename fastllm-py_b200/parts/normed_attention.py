@@ -1,9 +1,10 @@
-"""Grouped-query softmax attention whose queries and keys are normed head by head.
+"""Grouped-query softmax attention whose queries and keys are normed, head by head or over the whole projection.
 
 Per token: q = W_q h (+ b_q), k = W_k h (+ b_k), v = W_v h (+ b_v), one stacked product; query head h reads
 key/value head h // (heads / kv_heads); keys have `dim`, values `vdim` elements.  Each query and key head passes an
 RMS norm over its `dim` elements: `qk_norm` "weighted" norms before the rotation with a weight [dim] that the heads
-share, "unit" after the rotation without a weight.  The rotation (a `position` part's tables) turns a head's first
+share, "unit" after the rotation without a weight; or, with "whole", all query heads of a token pass one RMS norm and all
+key heads another, with a weight per column, before the rotation.  The rotation (a `position` part's tables) turns a head's first
 `rot_dim` dimensions in pairs (2i, 2i + 1) (`pairing` "interleaved") or (i, i + rot_dim / 2) ("half").  With
 `q_temp` = (coef, every) a query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
 
@@ -13,8 +14,8 @@ share, "unit" after the rotation without a weight.  The rotation (a `position` p
 The sink is one learned number per head in the denominator, without key or value; `sink` "unit" is a sink whose number
 is 0 (one more unit in the denominator).  With `values_from_keys` there is no W_v: a token's value is its key as
 projected, before norm and rotation.  With `head_gate` head h's result is multiplied by sigmoid(W_g h)_h, one number per
-head and token; with `channel_gate` the concatenated heads by sigmoid(W_g h), one per channel (in the attention kernels,
-before they round).  W_g rides in the stacked product.  With `taps` every channel of q, k and v passes a causal
+head and token; with `channel_gate` the concatenated heads by sigmoid(W_g h), one per channel (both in the attention
+kernels, before they round).  W_g rides in the stacked product.  With `taps` every channel of q, k and v passes a causal
 convolution over time, directly after the projection and its bias; a request's last taps - 1 projected rows are state
 beside its cache.  With `out_bias` the output projection has a bias, which a block that can adds with the pending sum.
 
@@ -33,13 +34,14 @@ from .registry import build_part, register_part
 
 @register_part("mixer", "normed_attention")
 class NormedAttention(ProjectedMixer):
-    """params: hidden_size, heads, kv_heads, dim, vdim, scale, norm_eps, qk_norm (None | "weighted" | "unit"),
+    """params: hidden_size, heads, kv_heads, dim, vdim, scale, norm_eps, qk_norm (None | "weighted" | "unit" |
+    "whole"),
     position (PartSpec | None), pairing ("half" | "interleaved"), q_temp (None | (coef, every)), window (None | int),
     chunk (None | int), sink (False | True | "unit"), biases (bool), out_bias (bool), taps (None: no convolution),
     values_from_keys (bool), head_gate (bool), channel_gate (bool).
     tensors: q [heads * dim, hidden], k [kv_heads * dim, hidden], o [hidden, heads * vdim]; v [kv_heads * vdim, hidden]
     unless values_from_keys; with biases q_bias, k_bias (and v_bias); with out_bias o_bias [hidden]; for "weighted"
-    q_norm, k_norm [dim]; with taps q_conv, k_conv, v_conv [channels, taps]; with sink True sink [heads]; with a gate
+    q_norm, k_norm [dim], for "whole" [heads * dim], [kv_heads * dim]; with taps q_conv, k_conv, v_conv [channels, taps]; with sink True sink [heads]; with a gate
     gate [heads, hidden] or [heads * vdim, hidden]."""
     category = "mixer"
     SCRATCH = "sink attention splits"
@@ -70,8 +72,11 @@ class NormedAttention(ProjectedMixer):
         self.channel_gated = bool(p.get("channel_gate", False))
         if self.heads % self.kv_heads:
             raise ValueError(f"normed_attention: {self.heads} heads are not a multiple of {self.kv_heads} kv heads")
-        if self.qk_norm not in (None, "weighted", "unit"):
-            raise ValueError(f"normed_attention: qk_norm {self.qk_norm!r} is none of None, 'weighted', 'unit'")
+        if self.qk_norm not in (None, "weighted", "unit", "whole"):
+            raise ValueError(f"normed_attention: qk_norm {self.qk_norm!r} is none of None, 'weighted', 'unit', 'whole'")
+        if self.qk_norm == "whole" and (self.taps is not None or self.v_from_k or self.q_temp):
+            raise ValueError("normed_attention: norms over the whole projection do not go with a convolution, keys as values "
+                             "or scaled queries")
         if self.pairing not in ("half", "interleaved"):
             raise ValueError(f"normed_attention: pairing {self.pairing!r} is neither 'half' nor 'interleaved'")
         if self.sink_kind not in (False, True, "unit"):
@@ -101,7 +106,7 @@ class NormedAttention(ProjectedMixer):
 
     def _conv_prep(self) -> bool:
         """Whether the preparation with a convolution (or a factor on the values) serves this part."""
-        return (self.taps is not None or self.joint) and not self.v_from_k
+        return (self.taps is not None or self.joint) and not self.v_from_k and self.qk_norm != "whole"
 
     def children(self):
         return [self.position] if self.position is not None else []
@@ -133,6 +138,8 @@ class NormedAttention(ProjectedMixer):
             shapes["o_bias"] = (self.hidden,)
         if self.qk_norm == "weighted":
             shapes.update({"q_norm": (self.dim,), "k_norm": (self.dim,)})
+        elif self.qk_norm == "whole":
+            shapes.update({"q_norm": (self.q_cols,), "k_norm": (self.k_cols,)})
         if self.taps:
             shapes.update({f"{s}_conv": (n, self.taps) for s, n in cols.items()})
         if self.sink_kind is True:
@@ -143,13 +150,13 @@ class NormedAttention(ProjectedMixer):
         cols = ["q", "k"] + ([] if self.v_from_k else ["v"])
         if self.joint and (self.has_out_bias or self.v_from_k):
             raise ValueError("normed_attention: an output bias, or keys as values, do not go with shared products")
-        if self.result_scale != 1.0 and not self._conv_prep():
+        if self.result_scale != 1.0 and not self._conv_prep() and self.qk_norm != "whole":
             raise ValueError("normed_attention: a factor on the result needs values of their own")
         if self.biases:
             self.bias = torch.cat([tensors[f"{s}_bias"].float() for s in cols]).contiguous()
         if self.has_out_bias:
             self.out_bias = tensors["o_bias"].float().clone()
-        if self.qk_norm == "weighted":
+        if self.qk_norm in ("weighted", "whole"):
             self.q_w = tensors["q_norm"].float().contiguous()
             self.k_w = tensors["k_norm"].float().contiguous()
         if self.taps:                                         # [taps, channels]: the kernel reads along the channels
@@ -206,9 +213,13 @@ class NormedAttention(ProjectedMixer):
         """Queries to `q`, keys and values to the tokens' cache rows."""
         cos, sin = self.position.tables() if self.position is not None else (None, None)
         rot = self.position.rot_dim if self.position is not None else 0
-        mode = {None: 0, "weighted": 1, "unit": 2}[self.qk_norm]
+        mode = {"weighted": 1, "unit": 2}.get(self.qk_norm, 0)
         interleaved = self.pairing == "interleaved"
-        if self._conv_prep():
+        if self.qk_norm == "whole":
+            ops.sink_prep(proj, self.bias, self.q_w, self.k_w, self.norm_eps, q, self.heads, self.kv_heads, self.dim, self.vdim, 0,
+                          0.0, None, cache.slots, cache.tensor, cache.page_size, rot, interleaved, cos, sin, step.positions,
+                          self.result_scale)
+        elif self._conv_prep():
             ops.conv_head_prep(proj, self.bias, self.conv_w, tail, self.q_w, self.k_w, mode, self.norm_eps, rot, interleaved, cos,
                                sin, step, self.q_temp, self.result_scale, q, self.heads, self.kv_heads, self.dim, self.vdim,
                                cache.slots, cache.tensor, cache.page_size)
@@ -226,7 +237,6 @@ class NormedAttention(ProjectedMixer):
         q = step.workspace.rows("normed_attention_q", n, self.q_cols, dt)
         self._prepare(proj, q, step, cache, tail)
         gate = proj[:, self.channels:self.channels + self.gate_cols] if self.gate_cols else None
-        channel_gate = gate if self.channel_gated else None
         tc = self._tc()
         # (where only the CUDA-core kernel serves prompt rows, a mixed step gives it every row)
         single = step.n_decode_tokens if self._splits_single_tokens() and (tc or step.n_decode_tokens == n) else 0
@@ -237,19 +247,17 @@ class NormedAttention(ProjectedMixer):
             ops.sink_decode(q, ctx, cache.tensor, cache.block_table, step.tok_req, step.positions, step.decode_tokens,
                             self._partials(single, n_splits), n_splits, kept_splits, self.heads, self.kv_heads,
                             self.dim, self.vdim, self.window, 0, self.scale, None, None, None, self.sink, cache.page_size,
-                            chunk=self.chunk, gate=channel_gate)
+                            chunk=self.chunk, gate=gate)
         if single == n:
             pass
         elif tc:
             ops.sink_attention_tc(q, ctx, cache.tensor, cache.block_table, step, self.heads, self.kv_heads, self.dim,
                                   self.vdim, self.window, 0, self.scale, None, None, None, self.sink, cache.page_size,
-                                  include_single=not single, chunk=self.chunk, gate=channel_gate)
+                                  include_single=not single, chunk=self.chunk, gate=gate)
         else:
             ops.sink_attention_simt(q, ctx, cache.tensor, cache.block_table, step.tok_req, step.positions, self.heads,
                                     self.kv_heads, self.dim, self.vdim, self.window, 0, self.scale, None, None, None,
-                                    self.sink, cache.page_size, chunk=self.chunk, gate=channel_gate)
-        if self.gated:
-            ops.head_gate(ctx, gate, self.heads, self.vdim)
+                                    self.sink, cache.page_size, chunk=self.chunk, gate=gate)
 
     def forward(self, h, out, step, cache):
         left = super().forward(h, out, step, cache)

@@ -46,10 +46,12 @@ class LayerRun:
     `cache` names the cache (or state) this run uses: by default a cache of its
     own; the number of an earlier run to read that run's cache instead, in which
     case this run writes nothing to it.  `vector`: the row of ModelPlan.vectors that is
-    added to the residual stream before this run (None: none)."""
+    added to the residual stream before this run (None: none).  `entry`: before that, the
+    stream passes ModelPlan.entry."""
     layer: int
     cache: int | None = None
     vector: int | None = None
+    entry: bool = False
 
 
 @dataclass
@@ -63,6 +65,7 @@ class ModelPlan:
     final_norm: PartSpec
     head: PartSpec
     vectors: PartSpec | None = None      # a table [n, hidden] of vectors that runs start with (LayerRun.vector)
+    entry: PartSpec | None = None        # what the stream passes before runs that say so (LayerRun.entry)
     ignorable: tuple = ()      # fnmatch patterns of checkpoint names that may be present and are not used
 
     def validate(self):
@@ -72,6 +75,8 @@ class ModelPlan:
                 raise ValueError(f"order[{i}] names layer {run.layer}, plan has {n} layers")
             if run.vector is not None and self.vectors is None:
                 raise ValueError(f"order[{i}] starts with vector {run.vector}, but the plan has no vectors")
+            if run.entry and self.entry is None:
+                raise ValueError(f"order[{i}] starts with the plan's entry, but the plan has none")
             if run.cache is not None:
                 if not 0 <= run.cache < i:
                     raise ValueError(f"order[{i}] reads the cache of run {run.cache}, "
@@ -97,6 +102,8 @@ class ModelPlan:
         visit(self.embedding)
         if self.vectors is not None:
             visit(self.vectors)
+        if self.entry is not None:
+            visit(self.entry)
         for layer in self.layers:
             for name in layer.tensors.values():
                 if name not in seen:

@@ -7,7 +7,7 @@ change anywhere else; tests do exactly that with toy parts.
 """
 from __future__ import annotations
 
-CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "vectors")
+CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "vectors", "entry")
 _PARTS: dict = {c: {} for c in CATEGORIES}
 
 

@@ -126,9 +126,13 @@ class SumSideBySide(Sides):
     Both are mixers between two products (`ProjectedMixer`), so the pair needs two products and not four: their input
     matrices are stacked along the outputs (both read h), their output matrices along the inputs (the sum of two
     products is the product of the operands side by side).  Each core writes its columns of the one operand, its
-    scale applied before they are rounded.
+    scale applied before they are rounded.  (Zero rows between the two input matrices let the right mixer's columns start on
+    a multiple of eight, for its wide loads.)
     params: hidden_size, left (PartSpec), right (PartSpec), left_scale, right_scale.  tensors: none of its own (it
     holds the children's matrices)."""
+
+    honours_partial_side = True          # with `partial_side` set, the last product's partial sums go to the second scratch
+    partial_side = False
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -144,7 +148,8 @@ class SumSideBySide(Sides):
             setattr(self, side, part)
             tensors.update({f"{side}.{slot}": p[side].tensors[slot] for slot in part.product_shapes()})
         self.spec = PartSpec(spec.kind, spec.params, tensors)
-        self.in_cols = self.left.in_cols + self.right.in_cols
+        self.right_at = -(-self.left.in_cols // 8) * 8
+        self.in_cols = self.right_at + self.right.in_cols
         self.out_cols = self.left.out_cols + self.right.out_cols
         self.proj = self.o = None
 
@@ -153,7 +158,11 @@ class SumSideBySide(Sides):
                 for slot, shape in getattr(self, side).product_shapes().items()}
 
     def load(self, tensors):
-        mats = [tensors[f"{side}.{slot}"] for side in self.SIDES for slot in getattr(self, side).in_slots]
+        mats = {side: [tensors[f"{side}.{slot}"] for slot in getattr(self, side).in_slots] for side in self.SIDES}
+        gap = self.right_at - self.left.in_cols
+        if gap:
+            mats["left"].append(torch.zeros((gap, self.hidden), dtype=mats["left"][0].dtype, device=mats["left"][0].device))
+        mats = mats["left"] + mats["right"]
         outs = [tensors[f"{side}.{getattr(self, side).out_slot}"] for side in self.SIDES]
         if len({m.dtype for m in mats}) != 1 or len({m.dtype for m in outs}) != 1:
             raise ValueError("side_by_side_sum: the stacked matrices must be stored in one dtype")
@@ -161,20 +170,19 @@ class SumSideBySide(Sides):
         self.o = Linear([torch.cat(outs, dim=1)])
 
     def reserve(self, limits):
-        for lin in (self.proj, self.o):
-            if lin is not None:
-                lin.reserve(self.ctx.dtype, limits.max_tokens)
+        if self.proj is not None:
+            self.proj.reserve(self.ctx.dtype, limits.max_tokens)
+            self.o.reserve(self.ctx.dtype, limits.max_tokens, side=self.partial_side)
 
     def forward(self, h, out, step, cache):
         n, dt, ws = h.shape[0], self.ctx.dtype, step.workspace
         proj = ws.rows("sides_proj", n, self.in_cols, dt)
         self.proj.forward(h, proj)
         y = ws.rows("sides_y", n, self.out_cols, dt)
-        at_in = at_out = 0
-        for side in self.SIDES:
+        at_out = 0
+        for side, at_in in zip(self.SIDES, (0, self.right_at)):
             part = getattr(self, side)
             part.core(proj[:, at_in:at_in + part.in_cols], y[:, at_out:at_out + part.out_cols], step,
                       side_view(side, part, cache))
-            at_in += part.in_cols
             at_out += part.out_cols
-        return self.o.forward(y, out, defer=True)
+        return self.o.forward(y, out, defer=True, side=self.partial_side)
