@@ -18,21 +18,19 @@
 //                       the kept inputs of requests on
 //   selective_step      steps of single tokens: dt, recurrence, read-out and gate of a request's channels in one kernel
 //
-// Everything but x, z and y (the activation type) is float.  The exponential is expf for 32-bit models; for bfloat16 ones
-// ex2.approx of a product with A log2(e).
+// Everything but x, z and y (the activation type) is float.
 #include "short_conv.cuh"
 #include "state_scan.cuh"
 
 // ------------------------------------------------------------------ convolution
-// V channels a thread, `run` consecutive tokens; conv_w: [taps][inner].  move_tail: every request has one token (run is 1).
-template <typename T, int V, int TAPS>
+// V channels a thread, RUN consecutive tokens; conv_w: [taps][inner].  move_tail: every request has one token (RUN is 1).
+template <typename T, int V, int TAPS, int RUN>
 __global__ void __launch_bounds__(128) selective_conv_kernel(
     const T* __restrict__ u, long ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b, int taps,
-    float* __restrict__ tail, long tail_stride, const StepTables st, T* __restrict__ x, long x_ld, int n_tokens, int run,
-    int inner, int move_tail) {
+    float* tail, long tail_stride, const StepTables st, T* __restrict__ x, long x_ld, int n_tokens, int inner, int move_tail) {
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
-    ShortConv<T, V, TAPS> conv;
-    ChanVec<V> b;
+    ShortConv<T, V, TAPS, RUN> conv;
+    ChanVec<V> b = {};
     if (c < inner) {                                                  // (no kernel writes these: asked for before the wait)
         conv.start(conv_w, taps, inner, c);
         b = chan_load<float, V>(conv_b + c);
@@ -40,25 +38,20 @@ __global__ void __launch_bounds__(128) selective_conv_kernel(
     pdl_wait();
     pdl_trigger();
     if (c >= inner) return;
-    const int t0 = blockIdx.x * run, t1 = min(n_tokens, t0 + run);
-    const T* col = u + c;
-    for (int t = t0; t < t1; ++t) {
-        const ChanVec<V> in = chan_load<T, V>(col + (long)t * ld);
-        ChanVec<V> y = conv.at(t, in, col, ld, st, tail, tail_stride, taps, inner, c);
+    const int t0 = blockIdx.x * RUN, t1 = min(n_tokens, t0 + RUN);
+    conv.run(t0, t1, u + c, ld, st, tail, tail_stride, taps, inner, c, [&](int t, ChanVec<V> y, const ChanVec<V>* in) {
 #pragma unroll
         for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
         chan_store<T, V>(x + (long)t * x_ld + c, y);
-        if constexpr (TAPS > 1) {
-            if (move_tail) {                                          // kept row j: the input of position pos + 1 - (taps - 1) + j
-                float* kept = tail + (long)st.req_slot[st.tok_req[t]] * tail_stride + c;
+        if (RUN == 1 && TAPS > 1 && move_tail) {                      // kept row j: the input of position pos - (taps - 2) + j
+            float* kept = tail + (long)st.req_slot[st.tok_req[t]] * tail_stride + c;
 #pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k) {
-                    const int j = k - (TAPS - taps);
-                    if (j >= 0) chan_store<float, V>(kept + (long)j * inner, conv.win[k]);
-                }
+            for (int k = 1; k < TAPS; ++k) {
+                const int j = k - 1 - (TAPS - taps);
+                if (j >= 0) chan_store<float, V>(kept + (long)j * inner, in[k]);
             }
         }
-    }
+    });
 }
 
 FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* conv_w, const float* conv_b, int taps, float* tail,
@@ -68,19 +61,20 @@ FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* con
     if (n_tokens <= 0) return 0;
     if (taps < 1 || taps > 16 || (taps > 1 && tail == nullptr)) return (int)cudaErrorInvalidValue;
     const StepTables st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
-    const int run = move_tail ? 1 : n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : 1;
+    const int run = !move_tail && n_tokens >= 256 ? 4 : 1;
     const int elem = dtype == FL_F32 ? 4 : 2;
     const bool vec = inner % 4 == 0 && chan_aligned(u, ld, elem) && chan_aligned(x, x_ld, elem) && chan_aligned(conv_w, 4, 4) &&
                      chan_aligned(conv_b, 4, 4) && (taps == 1 || chan_aligned(tail, tail_stride, 4));
     const int per = 128 * (vec ? 4 : 1);
     dim3 grid((n_tokens + run - 1) / run, (inner + per - 1) / per);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-#define FL_SEL_CONV(V, TAPS)                                                                                              \
-    FL_DISPATCH(dtype, T, return fl_launch(selective_conv_kernel<T, V, TAPS>, grid, dim3(128), 0, stream, (const T*)u, ld, \
-                                           conv_w, conv_b, taps, tail, tail_stride, st, (T*)x, x_ld, n_tokens, run, inner, \
-                                           move_tail))
-    if (vec) { if (taps == 1) { FL_SEL_CONV(4, 1); } else if (taps <= 4) { FL_SEL_CONV(4, 4); } else { FL_SEL_CONV(4, 16); } }
-    else { if (taps == 1) { FL_SEL_CONV(1, 1); } else if (taps <= 4) { FL_SEL_CONV(1, 4); } else { FL_SEL_CONV(1, 16); } }
+#define FL_SEL_CONV(V, TAPS, RUN)                                                                                         \
+    FL_DISPATCH(dtype, T, return fl_launch(selective_conv_kernel<T, V, TAPS, RUN>, grid, dim3(128), 0, stream, (const T*)u, ld, \
+                                           conv_w, conv_b, taps, tail, tail_stride, st, (T*)x, x_ld, n_tokens, inner, move_tail))
+#define FL_SEL_CONV_RUN(V, TAPS) { if (run == 4) { FL_SEL_CONV(V, TAPS, 4); } else { FL_SEL_CONV(V, TAPS, 1); } }
+    if (vec) { if (taps == 1) FL_SEL_CONV_RUN(4, 1) else if (taps <= 4) FL_SEL_CONV_RUN(4, 4) else FL_SEL_CONV_RUN(4, 16) }
+    else { if (taps == 1) FL_SEL_CONV_RUN(1, 1) else if (taps <= 4) FL_SEL_CONV_RUN(1, 4) else FL_SEL_CONV_RUN(1, 16) }
+#undef FL_SEL_CONV_RUN
 #undef FL_SEL_CONV
     return 0;
 }
@@ -221,12 +215,19 @@ FL_API int fl_selective_dt_mma(const float* low, long low_ld, int rank, const vo
 }
 
 // ------------------------------------------------------------------ the recurrence
-// exp(v) for 32-bit models, 2^v (A comes multiplied by log2(e)) for bfloat16 ones.
-template <typename T> __device__ __forceinline__ float sel_exp(float v) {
-    if constexpr (sizeof(T) == 4) return expf(v);
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
-    return r;
+// exp(v) S + add for a pair of rows, v = dt A.  For 32-bit models as S + expm1(v) S: near 1 a float exponential is off by a
+// like part of itself token after token, which adds up along a sequence, where expm1's error is a part of the small v.  For
+// bfloat16 models 2^v (A comes multiplied by log2(e)).
+template <typename T> __device__ __forceinline__ scan_f2 sel_decay(scan_f2 S, scan_f2 v, scan_f2 b, scan_f2 dx) {
+    const float2 e = scan_unpack(v);
+    if constexpr (sizeof(T) == 4) {
+        return scan_fma2(b, dx, scan_fma2(scan_pack(expm1f(e.x), expm1f(e.y)), S, S));
+    } else {
+        float p, q;
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(p) : "f"(e.x));
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(q) : "f"(e.y));
+        return scan_fma2(scan_pack(p, q), S, scan_mul2(b, dx));
+    }
 }
 
 // A lane's rows of a channel: the groups of four 4 (lane + LANES i).  Rows from n on are zero.
@@ -275,9 +276,8 @@ __device__ __forceinline__ float sel_token(scan_f2 (&S)[R / 2], const scan_f2 (&
     for (int i = 0; i < R / 4; ++i) {
         const ulonglong2 bb = reinterpret_cast<const ulonglong2*>(b)[lane + LANES * i];
         const ulonglong2 cc = reinterpret_cast<const ulonglong2*>(c)[lane + LANES * i];
-        const float2 e0 = scan_unpack(scan_mul2(dt2, A[2 * i])), e1 = scan_unpack(scan_mul2(dt2, A[2 * i + 1]));
-        S[2 * i] = scan_fma2(scan_pack(sel_exp<T>(e0.x), sel_exp<T>(e0.y)), S[2 * i], scan_mul2(bb.x, dx));
-        S[2 * i + 1] = scan_fma2(scan_pack(sel_exp<T>(e1.x), sel_exp<T>(e1.y)), S[2 * i + 1], scan_mul2(bb.y, dx));
+        S[2 * i] = sel_decay<T>(S[2 * i], scan_mul2(dt2, A[2 * i]), bb.x, dx);
+        S[2 * i + 1] = sel_decay<T>(S[2 * i + 1], scan_mul2(dt2, A[2 * i + 1]), bb.y, dx);
         sum = i == 0 ? scan_mul2(S[0], cc.x) : scan_fma2(S[2 * i], cc.x, sum);
         sum = scan_fma2(S[2 * i + 1], cc.y, sum);
     }

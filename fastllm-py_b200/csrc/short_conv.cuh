@@ -1,5 +1,5 @@
 // What the recurrent mixers' short convolutions share: vectors of neighbouring channels, the step's tables, and a causal
-// convolution per channel whose window slides along a request's tokens in registers.
+// convolution per channel over a request's tokens.
 #pragma once
 
 #include "common.cuh"
@@ -43,57 +43,76 @@ struct StepTables {              // per token: its request and position; per req
     const int *tok_req, *positions, *req_start, *req_ctx, *req_qlen, *req_slot;
 };
 
-// V channels from `c` on; TAPS: the window's length (the convolution's taps rounded up).  The taps - 1 inputs before a
-// request's first token of the step come from its kept rows [taps - 1][channels] float, oldest first; inputs before the
-// sequence's start are zeros.
-template <typename T, int V, int TAPS> struct ShortConv {
-    static constexpr int WIN = TAPS > 1 ? TAPS - 1 : 1;
-    ChanVec<V> w[TAPS], win[WIN];
-    int known;
-    // conv_w: [taps][channels], the last row the current token's
+// A causal convolution on V channels from `c` on, at the RUN (at most) consecutive tokens t0 .. t1 - 1 of the step; TAPS: the
+// window's length (the convolution's taps rounded up).  col: the channels' column of the step's rows; conv_w: [taps][channels]
+// float, the last row the current token's.  The taps - 1 inputs before a request's first token of the step come from its kept
+// rows [taps - 1][channels] float, oldest first; inputs before the sequence's start are zeros.
+//   emit(t, y, in)    y: the convolution at token t (no bias); in[k]: the input of position pos - (TAPS - 1) + k, in[TAPS - 1]
+//                     being the token's own
+// All inputs of a run within one request are asked for before the first is used.
+template <typename T, int V, int TAPS, int RUN> struct ShortConv {
+    static constexpr int WIN = TAPS - 1;
+    float w[TAPS][V];
+
     __device__ __forceinline__ void start(const float* conv_w, int taps, int channels, int c) {
-        known = -1;
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
             const int k = j - (TAPS - taps);
-            if (k >= 0) w[j] = chan_load<float, V>(conv_w + (long)k * channels + c);
-            else
+            ChanVec<V> tap = {};
+            if (k >= 0) tap = chan_load<float, V>(conv_w + (long)k * channels + c);
 #pragma unroll
-                for (int e = 0; e < V; ++e) w[j].v[e] = 0.0f;
+            for (int e = 0; e < V; ++e) w[j][e] = tap.v[e];
         }
     }
-    // The convolution at token t, whose input is x (tokens come in order); col: the channels' column of the step's rows.
-    __device__ __forceinline__ ChanVec<V> at(int t, const ChanVec<V>& x, const T* col, long ld, const StepTables& st,
-                                             const float* tail, long tail_stride, int taps, int channels, int c) {
-        ChanVec<V> y;
+    // The input `back` tokens before the one of row t, at position pos, whose request has `ctx` tokens before the step.
+    __device__ __forceinline__ ChanVec<V> before(const T* col, long ld, int t, int back, int pos, int ctx, const float* kept,
+                                                 int taps, int channels) const {
+        const int p = pos - back;
+        ChanVec<V> in = {};
+        if (p >= 0 && back <= taps - 1) {
+            if (p >= ctx) in = chan_load<T, V>(col + (long)(t - back) * ld);
+            else in = chan_load<float, V>(kept + (long)(p - ctx + taps - 1) * channels);
+        }
+        return in;
+    }
+    __device__ __forceinline__ ChanVec<V> sum(const ChanVec<V>* in) const {
+        ChanVec<V> y = {};
 #pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = 0.0f;
-        if constexpr (TAPS > 1) {
-            const int r = st.tok_req[t];
-            if (r != known) {
-                known = r;
-                const int pos = st.positions[t], ctx = st.req_ctx[r];
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int e = 0; e < V; ++e) y.v[e] = fmaf(w[j][e], in[j].v[e], y.v[e]);
+        return y;
+    }
+    template <typename F>
+    __device__ __forceinline__ void run(int t0, int t1, const T* col, long ld, const StepTables& st, const float* tail,
+                                        long tail_stride, int taps, int channels, int c, F emit) const {
+        const int r = WIN > 0 ? st.tok_req[t0] : 0;
+        if (RUN == 1 || WIN == 0 || (t1 - t0 == RUN && st.tok_req[t1 - 1] == r)) {
+            ChanVec<V> in[WIN + RUN];
+            if (WIN > 0) {
+                const int pos = st.positions[t0], ctx = st.req_ctx[r];
                 const float* kept = tail + (long)st.req_slot[r] * tail_stride + c;
 #pragma unroll
-                for (int k = 0; k < WIN; ++k) {
-                    const int back = WIN - k, p = pos - back;         // window entry k holds position pos - WIN + k
-#pragma unroll
-                    for (int e = 0; e < V; ++e) win[k].v[e] = 0.0f;
-                    if (p < 0 || back > taps - 1) continue;
-                    if (p >= ctx) win[k] = chan_load<T, V>(col + (long)(t - back) * ld);
-                    else win[k] = chan_load<float, V>(kept + (long)(p - ctx + taps - 1) * channels);
-                }
+                for (int k = 0; k < WIN; ++k) in[k] = before(col, ld, t0, WIN - k, pos, ctx, kept, taps, channels);
             }
 #pragma unroll
-            for (int j = 0; j < WIN; ++j)
+            for (int i = 0; i < RUN; ++i)
+                if (RUN == 1 || t0 + i < t1) in[WIN + i] = chan_load<T, V>(col + (long)(t0 + i) * ld);
 #pragma unroll
-                for (int e = 0; e < V; ++e) y.v[e] = fmaf(w[j].v[e], win[j].v[e], y.v[e]);
-#pragma unroll
-            for (int j = 0; j + 1 < WIN; ++j) win[j] = win[j + 1];
-            win[WIN - 1] = x;
+            for (int i = 0; i < RUN; ++i)
+                if (RUN == 1 || t0 + i < t1) emit(t0 + i, sum(in + i), in + i);
+            return;
         }
+        if constexpr (RUN > 1 && WIN > 0) {
+            for (int t = t0; t < t1; ++t) {                               // a run across requests, or at the step's end
+                const int rt = st.tok_req[t], pos = st.positions[t], ctx = st.req_ctx[rt];
+                const float* kept = tail + (long)st.req_slot[rt] * tail_stride + c;
+                ChanVec<V> in[TAPS];
 #pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = fmaf(w[TAPS - 1].v[e], x.v[e], y.v[e]);
-        return y;
+                for (int k = 0; k < WIN; ++k) in[k] = before(col, ld, t, WIN - k, pos, ctx, kept, taps, channels);
+                in[WIN] = chan_load<T, V>(col + (long)t * ld);
+                emit(t, sum(in), in);
+            }
+        }
     }
 };

@@ -31,16 +31,16 @@ __device__ __forceinline__ void ssd_rates(float raw, float dt_bias, double neg_a
     decay = (float)exp(neg_a * soft);
 }
 
-// V channels a thread, `run` consecutive tokens; the last blockIdx.y does dt and decay.  conv_w: [taps][channels].
+// V channels a thread, RUN consecutive tokens; the last blockIdx.y does dt and decay.  conv_w: [taps][channels].
 // TAPS: the window's length (taps rounded up).
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, int RUN>
 __global__ void __launch_bounds__(128) ssd_prep_kernel(
     const T* __restrict__ proj, long ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b, int taps,
     const float* __restrict__ dt_bias, const double* __restrict__ neg_a, const float* __restrict__ tail, long tail_stride,
-    const StepTables st, float* __restrict__ work, long w_ld, int n_tokens, int run, int inner, int channels, int heads) {
+    const StepTables st, float* __restrict__ work, long w_ld, int n_tokens, int inner, int channels, int heads) {
     pdl_wait();
     pdl_trigger();
-    const int t0 = blockIdx.x * run, t1 = min(n_tokens, t0 + run);
+    const int t0 = blockIdx.x * RUN, t1 = min(n_tokens, t0 + RUN);
     if (blockIdx.y == gridDim.y - 1) {
         for (int i = threadIdx.x; i < (t1 - t0) * heads; i += blockDim.x) {
             const int t = t0 + i / heads, h = i % heads;
@@ -53,17 +53,15 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(
     }
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
     if (c >= channels) return;
-    ShortConv<T, V, TAPS> conv;
+    ShortConv<T, V, TAPS, RUN> conv;
     conv.start(conv_w, taps, channels, c);
     const ChanVec<V> b = chan_load<float, V>(conv_b + c);
-    const T* col = proj + inner + c;
-    for (int t = t0; t < t1; ++t) {
-        const ChanVec<V> x = chan_load<T, V>(col + (long)t * ld);
-        ChanVec<V> y = conv.at(t, x, col, ld, st, tail, tail_stride, taps, channels, c);
+    conv.run(t0, t1, proj + inner + c, ld, st, tail, tail_stride, taps, channels, c,
+             [&](int t, ChanVec<V> y, const ChanVec<V>*) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
-        chan_store<float, V>(work + (long)t * w_ld + c, y);
-    }
+                 for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
+                 chan_store<float, V>(work + (long)t * w_ld + c, y);
+             });
 }
 
 // The four column sums of a group of LANES lanes, each lane holding its rows' part of all four.  After the exchange a
@@ -260,19 +258,21 @@ FL_API int fl_ssd_prep(const void* proj, int dtype, long ld, const float* conv_w
     const int inner = heads * vdim, channels = inner + 2 * groups * n;
     if (taps < 1 || taps > 16 || (taps > 1 && tail == nullptr) || groups < 1 || heads % groups) return (int)cudaErrorInvalidValue;
     const StepTables st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
-    const int run = n_tokens >= 1024 ? 8 : n_tokens >= 256 ? 4 : 1;
+    const int run = n_tokens >= 256 ? 4 : 1;
     const bool vec = channels % 4 == 0 && inner % 4 == 0 && chan_aligned(proj, ld, dtype == FL_F32 ? 4 : 2) &&
                      chan_aligned(work, w_ld, 4) && chan_aligned(conv_w, 4, 4) && chan_aligned(conv_b, 4, 4) &&
                      (taps == 1 || chan_aligned(tail, tail_stride, 4));
     const int per = 128 * (vec ? 4 : 1);
     dim3 grid((n_tokens + run - 1) / run, (channels + per - 1) / per + 1);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-#define FL_SSD_PREP(V, TAPS)                                                                                             \
-    FL_DISPATCH(dtype, T, return fl_launch(ssd_prep_kernel<T, V, TAPS>, grid, dim3(128), 0, stream, (const T*)proj, ld, conv_w, \
-                                           conv_b, taps, dt_bias, neg_a, tail, tail_stride, st, work, w_ld, n_tokens, run, inner, \
-                                           channels, heads))
-    if (vec) { if (taps == 1) { FL_SSD_PREP(4, 1); } else if (taps <= 4) { FL_SSD_PREP(4, 4); } else { FL_SSD_PREP(4, 16); } }
-    else { if (taps == 1) { FL_SSD_PREP(1, 1); } else if (taps <= 4) { FL_SSD_PREP(1, 4); } else { FL_SSD_PREP(1, 16); } }
+#define FL_SSD_PREP(V, TAPS, RUN)                                                                                        \
+    FL_DISPATCH(dtype, T, return fl_launch(ssd_prep_kernel<T, V, TAPS, RUN>, grid, dim3(128), 0, stream, (const T*)proj, ld, \
+                                           conv_w, conv_b, taps, dt_bias, neg_a, tail, tail_stride, st, work, w_ld, n_tokens, \
+                                           inner, channels, heads))
+#define FL_SSD_PREP_RUN(V, TAPS) { if (run == 4) { FL_SSD_PREP(V, TAPS, 4); } else { FL_SSD_PREP(V, TAPS, 1); } }
+    if (vec) { if (taps == 1) FL_SSD_PREP_RUN(4, 1) else if (taps <= 4) FL_SSD_PREP_RUN(4, 4) else FL_SSD_PREP_RUN(4, 16) }
+    else { if (taps == 1) FL_SSD_PREP_RUN(1, 1) else if (taps <= 4) FL_SSD_PREP_RUN(1, 4) else FL_SSD_PREP_RUN(1, 16) }
+#undef FL_SSD_PREP_RUN
 #undef FL_SSD_PREP
     return 0;
 }
