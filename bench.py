@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--workload decode|serve|67b|tables|hybrid|lasonex|sakusun|saberax|lufozen]
+                    [--workload decode|serve|67b|tables|hybrid|lasonex|sakusun|saberax|lufozen|kerirax]
 
 The default run is the DeepSeek-LLM-7B sized model (30 layers, hidden 4096,
 32 heads, head size 128, feed-forward 11008, vocabulary 102400) with random
@@ -50,6 +50,8 @@ Two more workloads, each printing one line of its own:
                      chunked attention, experts without a gate) beside the Lasonex design and the dense decoder
   --workload lufozen the Lufozen design (attention behind a short convolution, gated linear attention, attention beside a
                      state-space recurrence, layers that run twice) beside the Saberax design and the dense decoder
+  --workload kerirax the Kerirax design (attention beside a selective scan, latent attention with a sink, experts, parallel
+                     layers of which some run twice) beside the Lufozen design, the Tigitar hybrid and the dense decoder
   --workload 67b     deepseek-llm-67b size (95 layers, hidden 8192, 64 heads over 8 key/value
              heads; 135 GB of weights on the one GPU): a 2048-token prompt step and decode
              steps at batch 1, 8 and 16 with 4000-token contexts, with their roofline fractions.
@@ -1251,6 +1253,155 @@ def run_lufozen(args, warmup):
     return 0
 
 
+KERIRAX_SIZES = {
+    # parallel layers at the widths of HYBRID_SIZES with its latent attention, unit and experts, so many runs as the other
+    # designs have layers (some layers run twice).  The Lufozen design (attention beside a state-space recurrence in looped
+    # layers), the Tigitar hybrid (latent attention and experts) and the dense decoder are timed beside it
+    "w2048": dict(width=2048, vocab=32256, attention=dict(heads=16, kv_heads=4, dim=128, vdim=128),
+                  scan=dict(inner=4096, state=16, dt_rank=128, conv=4), q_rank=1024, runs=8),
+    "w4096": dict(width=4096, vocab=32256, attention=dict(heads=32, kv_heads=8, dim=128, vdim=128),
+                  scan=dict(inner=8192, state=16, dt_rank=256, conv=4), q_rank=1536, runs=4),
+}
+
+
+def kerirax_config(size):
+    from fastllm_py_b200.config.kerirax import (AttentionConfig, DenseConfig, ExpertsConfig, KeriraxConfig, KeriraxLayerConfig,
+                                                LatentConfig, LoopConfig, PairConfig, RotationConfig, SelectiveScanConfig)
+
+    z, hz = KERIRAX_SIZES[size], HYBRID_SIZES[size]
+    a, r, m = z["attention"], z["scan"], hz["latent"]
+    pair = PairConfig(AttentionConfig(a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["dim"] ** -0.5,
+                                      RotationConfig(500000.0, a["dim"], 4.0)),
+                      SelectiveScanConfig(r["inner"], r["state"], r["dt_rank"], r["conv"]), 0.7, 0.4)
+    latent = LatentConfig(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], z["q_rank"],
+                          (m["dim"] + m["rot_dim"]) ** -0.5, RotationConfig(10000.0, m["rot_dim"], None))
+    dense, experts = DenseConfig(hz["dense_ff"]), ExpertsConfig(hz["experts"], hz["top"], hz["expert_ff"], 7.0)
+    if z["runs"] == 8:
+        kinds = [(pair, dense), (latent, experts), (pair, dense), (pair, experts), (latent, dense), (pair, dense)]
+        loop = LoopConfig(1, 3, 2)
+    else:
+        kinds, loop = [(pair, dense), (latent, experts), (pair, dense)], LoopConfig(1, 2, 2)
+    layers = tuple(KeriraxLayerConfig("parallel" if m is pair else "latent_attention", m, f) for m, f in kinds)
+    return KeriraxConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, embedding_scale=8.0, logit_softcap=30.0, loop=loop,
+                         layers=layers)
+
+
+def _kerirax_run_sizes(layer, w):
+    """(weight elements a token's mixer products touch, state floats per request, cache elements per token, attention FLOPs
+    per query and key, state elements)."""
+    from fastllm_py_b200.config.kerirax import LatentConfig
+
+    m = layer.mixer
+    if isinstance(m, LatentConfig):
+        weights = w * (m.q_rank + m.kv_rank + m.rot_dim + m.heads * m.vdim) + m.q_rank * m.heads * (m.dim + m.rot_dim) + \
+            m.kv_rank * m.heads * (m.dim + m.vdim)
+        return weights, 0, m.kv_rank + m.rot_dim, 2 * m.heads * (2 * m.kv_rank + m.rot_dim), 0
+    a, r = m.left, m.right
+    weights = w * (a.heads * (a.dim + a.vdim + 1) + a.kv_heads * (a.dim + a.vdim) + 3 * r.inner) + \
+        r.inner * (2 * r.dt_rank + 2 * r.state)
+    return (weights, r.inner * (r.state + r.conv - 1), a.kv_heads * (a.dim + a.vdim), 2 * a.heads * (a.dim + a.vdim),
+            r.inner * r.state)
+
+
+def kerirax_decode_bytes(cfg, batch, context):
+    """Bytes a decode step has to move: every run's weights in bfloat16 (of the experts those that the batch's tokens can
+    reach), every request's states read and written in float, the cache rows that the attentions see."""
+    from fastllm_py_b200.config.kerirax import ExpertsConfig
+
+    w, total = cfg.width, 0
+    for i, started in cfg.running_order():
+        layer = cfg.layers[i]
+        weights, state, cached, _, _ = _kerirax_run_sizes(layer, w)
+        total += 2 * weights + batch * (2 * 4 * state + 2 * context * cached)
+        if started is not None:
+            total += 2 * 2 * w * w
+        f = layer.mlp
+        if isinstance(f, ExpertsConfig):
+            total += 2 * (w * f.experts + min(f.experts, batch * f.top) * 3 * w * f.ff)
+        elif f is not None:
+            total += 2 * 3 * w * f.ff
+    return total + 2 * w * cfg.vocab + 2 * batch * w
+
+
+def kerirax_prefill_flops(cfg, tokens):
+    """Matrix-product FLOPs of a prompt step (projections, feed-forwards, attention in latent space where it runs there, head)
+    and 6 per state element and token of the recurrence."""
+    from fastllm_py_b200.config.kerirax import ExpertsConfig
+
+    w, total = cfg.width, 0
+    for i, started in cfg.running_order():
+        layer = cfg.layers[i]
+        weights, _, _, attention, states = _kerirax_run_sizes(layer, w)
+        total += 2 * tokens * weights + attention * (tokens * (tokens + 1) // 2) + 6 * tokens * states
+        if started is not None:
+            total += 2 * tokens * 2 * w * w
+        f = layer.mlp
+        if isinstance(f, ExpertsConfig):
+            total += 2 * tokens * (w * f.experts + f.top * 3 * w * f.ff)
+        elif f is not None:
+            total += 2 * tokens * 3 * w * f.ff
+    return total + 2 * w * cfg.vocab
+
+
+def run_kerirax(args, warmup):
+    """The Kerirax design beside the Lufozen design, the Tigitar hybrid and the dense decoder of equal width and number of layer
+    runs, one JSON line: prompt steps of 512 and 2048 tokens and decode steps at batch 1 and 8 over 2048-token contexts, with
+    each model's fraction of its own roofline (measured tensor peak for prompts, measured copy bandwidth for decode steps)."""
+    import gc
+
+    import torch
+
+    from fastllm_py_b200 import LlamaConfig, Model
+
+    pk = peaks()
+    steps = max(8, min(args.steps, 32))
+    out = {}
+    sampler = ClockSampler().start()
+    sampler.__enter__()
+    for size in (args.size.split(",") if args.size else list(KERIRAX_SIZES)):
+        z, hz = KERIRAX_SIZES[size], HYBRID_SIZES[size]
+        llama = LlamaConfig(architecture="LlamaForCausalLM", rope_scaling=None, tie_word_embeddings=False,
+                            num_layers=z["runs"], hidden_size=z["width"], vocab_size=z["vocab"], rope_theta=10000.0,
+                            rms_norm_eps=1e-6, max_position_embeddings=4096, **hz["llama"])
+        models = [("kerirax", kerirax_config(size), kerirax_prefill_flops, kerirax_decode_bytes),
+                  ("lufozen", lufozen_config(size), lufozen_prefill_flops, lufozen_decode_bytes),
+                  ("hybrid", hybrid_config(size), hybrid_prefill_flops, hybrid_decode_bytes),
+                  ("dense", llama, prefill_flops, decode_bytes)]
+        res = {}
+        for name, cfg, flops_of, bytes_of in models:
+            if args.only and name not in args.only.split(","):
+                continue
+            model = Model.from_config(cfg, seed=0, dtype="bfloat16", page_size=16, max_tokens=8 * (CONTEXT + 256),
+                                      max_requests=8, max_batched_tokens=2048, max_model_len=4096,
+                                      cuda_graph=not args.no_graph)
+            r = {"prompt_step": {}, "decode": {}}
+            for t in (512, 2048):
+                ms, _ = time_prefill(model, t, 8, 3)
+                r["prompt_step"][str(t)] = {"ms": round(ms, 3), "value": round(t * 1000.0 / ms, 1),
+                                            "frac": round(flops_of(cfg, t) / (ms * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
+            for b in (1, 8):
+                v, ms, launches, _ = time_decode(model, b, steps, warmup, CONTEXT)
+                ctx = CONTEXT + warmup + (steps + 1) / 2
+                r["decode"][f"{b}x{CONTEXT}"] = {"ms_per_step": round(ms, 3), "value": round(v, 1),
+                                                 "launches_per_step": launches // steps,
+                                                 "frac": round(bytes_of(cfg, b, ctx) / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+            res[name] = r
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        out[size] = res
+    sampler.__exit__()
+    print(json.dumps({
+        "metric": "prompt and decode steps of the Kerirax design beside the Lufozen design, the Tigitar hybrid and the dense "
+                  "decoder of equal size, bf16",
+        "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours", "steps": steps, "warmup": warmup,
+        "config": {"sizes": {k: dict(KERIRAX_SIZES[k]) for k in out}, "page_size": 16,
+                   "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"],
+                   "cuda_graph": not args.no_graph},
+        "sizes": out, "clocks": sampler.summary()}))
+    return 0
+
+
 def reference_cpu_path(ref_root, layers=1, context=256, decode_tokens=8):
     """fastllm-py's own NumPy model code (its CPU device, float32) timed at DeepSeek-LLM-7B layer
     sizes: `layers` of the 30 layers, one sequence (that path has no batch), a `context`-token
@@ -1387,11 +1538,12 @@ def main():
                     help="run fewer layers of the same sizes (the line names both numbers)")
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64 and the prefill")
     ap.add_argument("--no-graph", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "67b", "tables", "hybrid", "lasonex", "sakusun", "saberax", "lufozen"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "67b", "tables", "hybrid", "lasonex", "sakusun", "saberax", "lufozen",
+                                                              "kerirax"],
                     help="decode: the headline line (DeepSeek-LLM-7B size); serve: continuous batching at "
                          "deepseek-coder-1.3b size; 67b: prompt and decode steps at deepseek-llm-67b size")
-    ap.add_argument("--size", default="", help="hybrid, lasonex, sakusun, saberax, lufozen: which sizes (w2048,w4096; default both)")
-    ap.add_argument("--only", default="", help="lasonex, sakusun, saberax, lufozen: which of the models timed side by side (the design itself, hybrid, lasonex or saberax, dense)")
+    ap.add_argument("--size", default="", help="hybrid, lasonex, sakusun, saberax, lufozen, kerirax: which sizes (w2048,w4096; default both)")
+    ap.add_argument("--only", default="", help="lasonex, sakusun, saberax, lufozen, kerirax: which of the models timed side by side (the design's name, hybrid, dense, ...)")
     ap.add_argument("--requests", type=int, default=128, help="serve: how many requests")
     ap.add_argument("--rate", type=float, default=16.0, help="serve: mean arrivals a second")
     ap.add_argument("--reference-cpu", action="store_true",
@@ -1418,6 +1570,8 @@ def main():
         return run_saberax(args, warmup)
     if args.workload == "lufozen":
         return run_lufozen(args, warmup)
+    if args.workload == "kerirax":
+        return run_kerirax(args, warmup)
     if args.workload == "hybrid":
         return run_hybrid(args, warmup)
     args.layers = args.layers or MODEL_7B["num_layers"]

@@ -128,6 +128,7 @@ FL_API int fl_selective_dt(const float* low, long low_ld, int rank, const float*
 #define SEL_MM 64                    // tokens and channels of a block's tile
 #define SEL_MK 64                    // columns of a stage
 #define SEL_MP (SEL_MK + 8)          // bfloat16 elements between staged rows (ldmatrix without bank conflicts)
+#define SEL_MC 4                     // tiles of channels that a block walks with the same tokens
 
 __device__ __forceinline__ void sel_ldm4(unsigned (&r)[4], const bf16* p) {
     const unsigned s = (unsigned)__cvta_generic_to_shared(p);
@@ -143,63 +144,87 @@ __device__ __forceinline__ void sel_mma(float (&d)[4], const unsigned (&a)[4], u
 __global__ void __launch_bounds__(128) selective_dt_mma_kernel(const float* __restrict__ low, long low_ld, int rank,
                                                                const bf16* __restrict__ w, int w_ld,
                                                                const float* __restrict__ bias, float* __restrict__ dt,
-                                                               long dt_ld, int n_tokens, int inner) {
-    __shared__ __align__(16) bf16 hi_s[SEL_MM * SEL_MP], lo_s[SEL_MM * SEL_MP], w_s[SEL_MM * SEL_MP];
-    const int t0 = blockIdx.x * SEL_MM, c0 = blockIdx.y * SEL_MM, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+                                                               long dt_ld, int n_tokens, int inner, int low_vec) {
+    // all of low's columns for 64 tokens stay staged (as two parts) while the block walks its tiles of channels
+    extern __shared__ __align__(16) unsigned char sel_mma_s[];
+    const int k_end = (rank + 15) / 16 * 16, pitch = k_end + 8;
+    bf16* hi_s = reinterpret_cast<bf16*>(sel_mma_s);                  // [SEL_MM][pitch]
+    bf16* lo_s = hi_s + SEL_MM * pitch;
+    bf16* w_s = lo_s + SEL_MM * pitch;                                // [SEL_MM][SEL_MP]
+    const int t0 = blockIdx.x * SEL_MM, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     pdl_wait();
     pdl_trigger();
-    float acc[SEL_MM / 8][4];
+    for (int i = tid; i < SEL_MM * k_end / 4; i += 128) {
+        const int r = i / (k_end / 4), k = i % (k_end / 4) * 4;
+        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        if (t0 + r < n_tokens) {
+            const float* p = low + (long)(t0 + r) * low_ld + k;
+            if (low_vec && k + 4 <= rank) {
+                const float4 q = *reinterpret_cast<const float4*>(p);
+                v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+            } else {
 #pragma unroll
-    for (int i = 0; i < SEL_MM / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
-    for (int k0 = 0; k0 < rank; k0 += SEL_MK) {
-        for (int i = tid; i < SEL_MM * SEL_MK; i += 128) {
-            const int r = i / SEL_MK, k = i % SEL_MK;
-            const float v = (t0 + r < n_tokens && k0 + k < rank) ? low[(long)(t0 + r) * low_ld + k0 + k] : 0.0f;
-            const bf16 hi = __float2bfloat16_rn(v);
-            hi_s[r * SEL_MP + k] = hi;
-            lo_s[r * SEL_MP + k] = __float2bfloat16_rn(v - __bfloat162float(hi));
-        }
-        for (int i = tid; i < SEL_MM * (SEL_MK / 8); i += 128) {
-            const int r = i / (SEL_MK / 8), k = i % (SEL_MK / 8) * 8;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (c0 + r < inner && k0 + k < w_ld) v = *reinterpret_cast<const uint4*>(w + (long)(c0 + r) * w_ld + k0 + k);
-            *reinterpret_cast<uint4*>(w_s + r * SEL_MP + k) = v;
-        }
-        __syncthreads();
-        const int ks_end = min(SEL_MK, (rank - k0 + 15) / 16 * 16);
-        for (int ks = 0; ks < ks_end; ks += 16) {
-            unsigned hi[4], lo[4];
-            sel_ldm4(hi, hi_s + (warp * 16 + (lane & 15)) * SEL_MP + ks + (lane >> 4) * 8);
-            sel_ldm4(lo, lo_s + (warp * 16 + (lane & 15)) * SEL_MP + ks + (lane >> 4) * 8);
-#pragma unroll
-            for (int j = 0; j < SEL_MM / 16; ++j) {
-                unsigned b[4];
-                sel_ldm4(b, w_s + (j * 16 + (lane & 7) + (lane >> 4) * 8) * SEL_MP + ks + ((lane >> 3) & 1) * 8);
-                sel_mma(acc[2 * j], hi, b[0], b[1]);
-                sel_mma(acc[2 * j + 1], hi, b[2], b[3]);
-                sel_mma(acc[2 * j], lo, b[0], b[1]);
-                sel_mma(acc[2 * j + 1], lo, b[2], b[3]);
+                for (int e = 0; e < 4; ++e)
+                    if (k + e < rank) v[e] = p[e];
             }
         }
-        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+            const __nv_bfloat162 hi = __floats2bfloat162_rn(v[e], v[e + 1]);
+            const float2 f = __bfloat1622float2(hi);
+            *reinterpret_cast<__nv_bfloat162*>(hi_s + r * pitch + k + e) = hi;
+            *reinterpret_cast<__nv_bfloat162*>(lo_s + r * pitch + k + e) = __floats2bfloat162_rn(v[e] - f.x, v[e + 1] - f.y);
+        }
     }
-    const bool pairs = inner % 2 == 0 && dt_ld % 2 == 0;
+    for (int tile = 0; tile < SEL_MC; ++tile) {
+        const int c0 = (blockIdx.y * SEL_MC + tile) * SEL_MM;
+        if (c0 >= inner) break;
+        float acc[SEL_MM / 8][4];
 #pragma unroll
-    for (int i = 0; i < SEL_MM / 8; ++i) {
-        const int c = c0 + i * 8 + (lane & 3) * 2;
-        if (c >= inner) continue;
-        const bool both = c + 1 < inner;
-        const float b0 = bias[c], b1 = both ? bias[c + 1] : 0.0f;
+        for (int i = 0; i < SEL_MM / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+        for (int k0 = 0; k0 < rank; k0 += SEL_MK) {
+            __syncthreads();                                              // low is staged; w_s was read
+            for (int i = tid; i < SEL_MM * (SEL_MK / 8); i += 128) {
+                const int r = i / (SEL_MK / 8), k = i % (SEL_MK / 8) * 8;
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (c0 + r < inner && k0 + k < w_ld) v = *reinterpret_cast<const uint4*>(w + (long)(c0 + r) * w_ld + k0 + k);
+                *reinterpret_cast<uint4*>(w_s + r * SEL_MP + k) = v;
+            }
+            __syncthreads();
+            const int ks_end = min(SEL_MK, k_end - k0);
+            for (int ks = 0; ks < ks_end; ks += 16) {
+                unsigned hi[4], lo[4];
+                sel_ldm4(hi, hi_s + (warp * 16 + (lane & 15)) * pitch + k0 + ks + (lane >> 4) * 8);
+                sel_ldm4(lo, lo_s + (warp * 16 + (lane & 15)) * pitch + k0 + ks + (lane >> 4) * 8);
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const int t = t0 + warp * 16 + (lane >> 2) + h * 8;
-            if (t >= n_tokens) continue;
-            float* o = dt + (long)t * dt_ld + c;
-            const float d0 = fl_softplus(acc[i][2 * h] + b0), d1 = fl_softplus(acc[i][2 * h + 1] + b1);
-            if (pairs) *reinterpret_cast<float2*>(o) = make_float2(d0, d1);
-            else {
-                o[0] = d0;
-                if (both) o[1] = d1;
+                for (int j = 0; j < SEL_MM / 16; ++j) {
+                    unsigned b[4];
+                    sel_ldm4(b, w_s + (j * 16 + (lane & 7) + (lane >> 4) * 8) * SEL_MP + ks + ((lane >> 3) & 1) * 8);
+                    sel_mma(acc[2 * j], hi, b[0], b[1]);
+                    sel_mma(acc[2 * j + 1], hi, b[2], b[3]);
+                    sel_mma(acc[2 * j], lo, b[0], b[1]);
+                    sel_mma(acc[2 * j + 1], lo, b[2], b[3]);
+                }
+            }
+        }
+        const bool pairs = inner % 2 == 0 && dt_ld % 2 == 0;
+#pragma unroll
+        for (int i = 0; i < SEL_MM / 8; ++i) {
+            const int c = c0 + i * 8 + (lane & 3) * 2;
+            if (c >= inner) continue;
+            const bool both = c + 1 < inner;
+            const float b0 = bias[c], b1 = both ? bias[c + 1] : 0.0f;
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int t = t0 + warp * 16 + (lane >> 2) + h * 8;
+                if (t >= n_tokens) continue;
+                float* o = dt + (long)t * dt_ld + c;
+                const float d0 = fl_softplus(acc[i][2 * h] + b0), d1 = fl_softplus(acc[i][2 * h + 1] + b1);
+                if (pairs) *reinterpret_cast<float2*>(o) = make_float2(d0, d1);
+                else {
+                    o[0] = d0;
+                    if (both) o[1] = d1;
+                }
             }
         }
     }
@@ -208,10 +233,18 @@ __global__ void __launch_bounds__(128) selective_dt_mma_kernel(const float* __re
 FL_API int fl_selective_dt_mma(const float* low, long low_ld, int rank, const void* w, int w_ld, const float* bias, float* dt,
                                long dt_ld, int n_tokens, int inner, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (rank < 1 || w_ld < rank || w_ld % 8 || ((uintptr_t)w % 16) || ((uintptr_t)dt % 8) || (inner + SEL_MM - 1) / SEL_MM > 65535)
+    const int per = SEL_MM * SEL_MC, k_end = (rank + 15) / 16 * 16;
+    const size_t smem = ((size_t)2 * SEL_MM * (k_end + 8) + SEL_MM * SEL_MP) * sizeof(bf16);
+    if (rank < 1 || smem > 220 * 1024 || w_ld < rank || w_ld % 8 || ((uintptr_t)w % 16) || ((uintptr_t)dt % 8) ||
+        (inner + per - 1) / per > 65535)
         return (int)cudaErrorInvalidValue;
-    return fl_launch(selective_dt_mma_kernel, dim3((n_tokens + SEL_MM - 1) / SEL_MM, (inner + SEL_MM - 1) / SEL_MM), dim3(128), 0,
-                     stream, low, low_ld, rank, (const bf16*)w, w_ld, bias, dt, dt_ld, n_tokens, inner);
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(selective_dt_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    const int low_vec = low_ld % 4 == 0 && ((uintptr_t)low % 16) == 0;
+    return fl_launch(selective_dt_mma_kernel, dim3((n_tokens + SEL_MM - 1) / SEL_MM, (inner + per - 1) / per), dim3(128), smem,
+                     stream, low, low_ld, rank, (const bf16*)w, w_ld, bias, dt, dt_ld, n_tokens, inner, low_vec);
 }
 
 // ------------------------------------------------------------------ the recurrence
@@ -368,6 +401,7 @@ __global__ void __launch_bounds__(COLS * LANES) selective_scan_kernel(
         const float* dts = stage_dt(stage) + col;
         const T* xs = stage_x(stage) + col;
         const T* zs = xs + CHUNK * COLS;
+        float sums[CHUNK / 4];                                        // of this lane's token of each group
         auto group = [&](int t4, int left) {
             float acc[4];
 #pragma unroll
@@ -381,16 +415,22 @@ __global__ void __launch_bounds__(COLS * LANES) selective_scan_kernel(
             float v = scan_fold(up1, w0, w1, LANES / 4);
 #pragma unroll
             for (int off = LANES / 8; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-            const int t = t4 + my_u;
-            if (writer && my_u < left)
-                y_s[t * COLS + col] = from_f32<T>(fmaf(skip_c, to_f32<T>(xs[t * COLS]), v) * fl_silu(to_f32<T>(zs[t * COLS])) * scale);
+            return v;
         };
+        // a whole chunk is straight-line code without a store in it, so that a group's reads overlap the sums before it
         if (here == CHUNK) {
 #pragma unroll
-            for (int t4 = 0; t4 < CHUNK; t4 += 4) group(t4, 4);
+            for (int g = 0; g < CHUNK / 4; ++g) sums[g] = group(4 * g, 4);
         } else {
-#pragma unroll 1
-            for (int t4 = 0; t4 < here; t4 += 4) group(t4, here - t4);
+#pragma unroll
+            for (int g = 0; g < CHUNK / 4; ++g)
+                if (4 * g < here) sums[g] = group(4 * g, here - 4 * g);
+        }
+#pragma unroll
+        for (int g = 0; g < CHUNK / 4; ++g) {
+            const int t = 4 * g + my_u;
+            if (writer && t < here)
+                y_s[t * COLS + col] = from_f32<T>(fmaf(skip_c, to_f32<T>(xs[t * COLS]), sums[g]) * fl_silu(to_f32<T>(zs[t * COLS])) * scale);
         }
         __syncthreads();                                              // y_s is whole; the stage is copied into again in the next round
         T* yo = y + (long)(start + c0) * y_ld + col0;
@@ -504,8 +544,16 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
     const float skip_c = mine ? skip[c] : 0.0f, bias_c = mine ? dt_bias[c] : 0.0f;
     const int ctx = req_ctx[r];
     float* srow = state + (long)req_slot[r] * state_stride + (long)c * n;
+    constexpr int KEEP = 4;                                           // of the weight row: vectors that wait in registers
+    float w_keep[KEEP][8];
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int k = (lane + i * LANES) * 8;
+        if (mine && k < w_ld) sel_load8(w_dt + (long)c * w_ld + k, w_keep[i]);
+    }
     pdl_wait();
     pdl_trigger();
+    const float xv = mine ? to_f32<T>(x[(long)r * x_ld + c]) : 0.0f, zv = mine ? to_f32<T>(z[(long)r * z_ld + c]) : 0.0f;
     sel_rows<R, LANES>(S, srow, lane, n, mine && ctx != 0, state_vec4);
     for (int i = tid; i < 2 * DP + w_ld; i += THREADS) {
         int from = -1;
@@ -515,16 +563,23 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
         float v = 0.0f;
         if (from >= 0) {
             const float* p = low + (long)r * low_ld + from;
-            v = p[0];
-            for (int s = 1; s < splits; ++s) v += p[s * split_stride];
+#pragma unroll 8
+            for (int s = 0; s < splits; ++s) v += p[s * split_stride];
         }
         step_s[i] = v;
     }
     __syncthreads();
     const float* low_s = step_s + 2 * DP;
     float dot = 0.0f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int k = (lane + i * LANES) * 8;
+        if (mine && k < w_ld)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) dot = fmaf(w_keep[i][e], low_s[k + e], dot);
+    }
     if (mine)
-        for (int k = lane * 8; k < w_ld; k += LANES * 8) {
+        for (int k = (lane + KEEP * LANES) * 8; k < w_ld; k += LANES * 8) {
             float w[8];
             sel_load8(w_dt + (long)c * w_ld + k, w);
 #pragma unroll
@@ -533,13 +588,12 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
 #pragma unroll
     for (int off = LANES / 2; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
     const float dt = fl_softplus(dot + bias_c);
-    const float xv = mine ? to_f32<T>(x[(long)r * x_ld + c]) : 0.0f;
     float sum = sel_token<T, R, LANES>(S, A, step_s, step_s + DP, dt, xv, lane);
 #pragma unroll
     for (int off = LANES / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
     if (!mine) return;
     if (lane == 0)
-        y[(long)r * y_ld + c] = from_f32<T>(fmaf(skip_c, xv, sum) * fl_silu(to_f32<T>(z[(long)r * z_ld + c])) * scale);
+        y[(long)r * y_ld + c] = from_f32<T>(fmaf(skip_c, xv, sum) * fl_silu(zv) * scale);
     sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
 }
 

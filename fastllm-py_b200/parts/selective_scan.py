@@ -35,6 +35,7 @@ class SelectiveScan(ProjectedMixer):
     native_libraries = ("selective_scan",)
     in_slots = ("in",)
     workspace_name = "selective"
+    TENSOR_CORE_RANK = 768
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -72,8 +73,8 @@ class SelectiveScan(ProjectedMixer):
         pitch = -(-self.rank // 8) * 8
         self.dt_w = torch.zeros((self.inner, pitch), dtype=w.dtype, device=w.device)      # rows that start on 16 bytes
         self.dt_w[:, :self.rank] = w
-        # the 32-bit path sums on the CUDA cores, along the channels
-        exact = self.ctx.dtype == torch.float32 or w.dtype == torch.float32
+        # the 32-bit path (and a rank beyond the tensor-core kernel's shared memory) sums on the CUDA cores, along the channels
+        exact = self.ctx.dtype == torch.float32 or w.dtype == torch.float32 or self.rank > self.TENSOR_CORE_RANK
         self.dt_t = w.float().t().contiguous() if exact else None
         self.dt_bias = tensors["dt_bias"].float().contiguous()
         a = -torch.exp(tensors["A_log"].double())
