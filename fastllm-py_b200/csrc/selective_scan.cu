@@ -248,21 +248,6 @@ FL_API int fl_selective_dt_mma(const float* low, long low_ld, int rank, const vo
 }
 
 // ------------------------------------------------------------------ the recurrence
-// exp(v) S + add for a pair of rows, v = dt A.  For 32-bit models as S + expm1(v) S: near 1 a float exponential is off by a
-// like part of itself token after token, which adds up along a sequence, where expm1's error is a part of the small v.  For
-// bfloat16 models 2^v (A comes multiplied by log2(e)).
-template <typename T> __device__ __forceinline__ scan_f2 sel_decay(scan_f2 S, scan_f2 v, scan_f2 b, scan_f2 dx) {
-    const float2 e = scan_unpack(v);
-    if constexpr (sizeof(T) == 4) {
-        return scan_fma2(b, dx, scan_fma2(scan_pack(expm1f(e.x), expm1f(e.y)), S, S));
-    } else {
-        float p, q;
-        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(p) : "f"(e.x));
-        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(q) : "f"(e.y));
-        return scan_fma2(scan_pack(p, q), S, scan_mul2(b, dx));
-    }
-}
-
 // A lane's rows of a channel: the groups of four 4 (lane + LANES i).  Rows from n on are zero.
 template <int R, int LANES>
 __device__ __forceinline__ void sel_rows(scan_f2 (&out)[R / 2], const float* p, int lane, int n, bool there, int vec4) {
@@ -299,24 +284,57 @@ __device__ __forceinline__ void sel_rows_out(const scan_f2 (&in)[R / 2], float* 
     }
 }
 
-// One token of a lane's rows: S <- exp(dt A) S + (dt x) B; returns the rows' part of sum S C.
+// What one token does to a lane's rows, formed before S is needed: S <- p S + bx, sum += S c.
+template <int R> struct SelToken {
+    scan_f2 p[R / 2], bx[R / 2], c[R / 2];
+};
+// The decay exp(v), v = dt A, of a pair of rows.  For 32-bit models p is expm1(v), applied as S + p S: near 1 a float exponential
+// is off by a like part of itself token after token, which adds up along a sequence, where expm1's error is a part of the
+// small v.  For bfloat16 models p is 2^v (A comes multiplied by log2(e)).
+template <typename T> __device__ __forceinline__ scan_f2 sel_decay(scan_f2 v) {
+    const float2 e = scan_unpack(v);
+    float p, q;
+    if constexpr (sizeof(T) == 4) {
+        p = expm1f(e.x);
+        q = expm1f(e.y);
+    } else {
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(p) : "f"(e.x));
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(q) : "f"(e.y));
+    }
+    return scan_pack(p, q);
+}
 template <typename T, int R, int LANES>
-__device__ __forceinline__ float sel_token(scan_f2 (&S)[R / 2], const scan_f2 (&A)[R / 2], const float* b, const float* c,
-                                           float dt, float x, int lane) {
+__device__ __forceinline__ void sel_prepare(SelToken<R>& t, const scan_f2 (&A)[R / 2], const float* b, const float* c, float dt,
+                                            float x, int lane) {
     const scan_f2 dt2 = scan_pack(dt, dt), dx = scan_pack(dt * x, dt * x);
-    scan_f2 sum = 0ULL;
 #pragma unroll
     for (int i = 0; i < R / 4; ++i) {
         const ulonglong2 bb = reinterpret_cast<const ulonglong2*>(b)[lane + LANES * i];
         const ulonglong2 cc = reinterpret_cast<const ulonglong2*>(c)[lane + LANES * i];
-        S[2 * i] = sel_decay<T>(S[2 * i], scan_mul2(dt2, A[2 * i]), bb.x, dx);
-        S[2 * i + 1] = sel_decay<T>(S[2 * i + 1], scan_mul2(dt2, A[2 * i + 1]), bb.y, dx);
-        sum = i == 0 ? scan_mul2(S[0], cc.x) : scan_fma2(S[2 * i], cc.x, sum);
-        sum = scan_fma2(S[2 * i + 1], cc.y, sum);
+        t.p[2 * i] = sel_decay<T>(scan_mul2(dt2, A[2 * i]));
+        t.p[2 * i + 1] = sel_decay<T>(scan_mul2(dt2, A[2 * i + 1]));
+        t.bx[2 * i] = scan_mul2(bb.x, dx);
+        t.bx[2 * i + 1] = scan_mul2(bb.y, dx);
+        t.c[2 * i] = cc.x;
+        t.c[2 * i + 1] = cc.y;
+    }
+}
+// The rows' part of sum S c after the token.
+template <typename T, int R>
+__device__ __forceinline__ float sel_apply(scan_f2 (&S)[R / 2], const SelToken<R>& t) {
+    const scan_f2 one = scan_pack(1.0f, 1.0f);
+    scan_f2 sum = 0ULL;
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+        if constexpr (sizeof(T) == 4) S[i] = scan_fma2(t.bx[i], one, scan_fma2(t.p[i], S[i], S[i]));
+        else S[i] = scan_fma2(t.p[i], S[i], t.bx[i]);
+        sum = i == 0 ? scan_mul2(S[0], t.c[0]) : scan_fma2(S[i], t.c[i], sum);
     }
     const float2 v = scan_unpack(sum);
     return v.x + v.y;
 }
+
+template <int N> struct ScanCount { static constexpr int value = N; };
 
 struct SelRows {                     // the step's rows: element type T, float, float
     const void *x, *z, *u;           // convolved inputs, gates, inputs before the convolution
@@ -325,128 +343,182 @@ struct SelRows {                     // the step's rows: element type T, float, 
     int b_at, c_at;                  // where low holds B and C
 };
 
-// A block takes one request and COLS channels, LANES lanes a channel; tokens come through four stages of shared memory
-// (cp.async, three chunks ahead of the one that is walked) and go four at a time, so that four read-out sums are added up
-// over the lanes together.  R and LANES follow from n alone: one order of sums whatever the cut.
+// A block takes one request and COLS channels.  Half of its threads walk the tokens, LANES lanes a channel, and do nothing
+// else: a chunk of tokens is straight-line code that reads shared memory and leaves the read-out sums there.  The other
+// half copies the chunks two ahead (cp.async, four stages) and turns the sums of the chunk before into outputs (skip, gate,
+// store).  Tokens go four at a time, so that four sums are added up over the lanes together.  R and LANES follow from n alone:
+// one order of sums whatever the cut.
 template <typename T, int R, int LANES, int COLS, int CHUNK>
-__global__ void __launch_bounds__(COLS * LANES) selective_scan_kernel(
+__global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
     const SelRows in, const float* __restrict__ a_log2, const float* __restrict__ skip, float scale, T* __restrict__ y, long y_ld,
     float* __restrict__ state, long state_stride, long tail_off, int taps, const int* __restrict__ req_start,
     const int* __restrict__ req_ctx, const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int inner, int n,
     int vec_low, int vec_dt, int vec_x, int vec_z, int vec_y, int state_vec4) {
-    static_assert(CHUNK % 4 == 0 && R % 4 == 0 && (LANES == 4 || LANES == 8 || LANES == 16) && COLS % 8 == 0, "");
-    constexpr int DP = R * LANES, THREADS = COLS * LANES, TV = 16 / sizeof(T);
+    static_assert(CHUNK % 4 == 0 && R % 4 == 0 && (LANES == 4 || LANES == 8 || LANES == 16) && COLS % 8 == 0 && SCAN_STAGES == 4, "");
+    constexpr int DP = R * LANES, HALF = COLS * LANES, TV = 16 / sizeof(T);
     constexpr int STAGE = CHUNK * (2 * DP + COLS) * 4 + 2 * CHUNK * COLS * (int)sizeof(T);     // bytes
     extern __shared__ __align__(16) unsigned char sel_s[];
-    T* y_s = reinterpret_cast<T*>(sel_s + SCAN_STAGES * STAGE);       // [CHUNK][COLS]
+    float* sum_s = reinterpret_cast<float*>(sel_s + SCAN_STAGES * STAGE);                      // [2][CHUNK][COLS]
     pdl_wait();
-    const int r = blockIdx.x, col0 = blockIdx.y * COLS;
-    const int tid = threadIdx.x, lane = tid & (LANES - 1), col = tid / LANES, c = col0 + col;
+    const int r = blockIdx.x, col0 = blockIdx.y * COLS, tid = threadIdx.x;
     const int start = req_start[r], qlen = req_qlen[r], ctx = req_ctx[r];
-    const int cols = min(COLS, inner - col0);
-    const bool mine = c < inner;
-    for (int i = tid; i < SCAN_STAGES * STAGE / 16; i += THREADS)     // padding stays zero, stale places hold numbers
+    const int cols = min(COLS, inner - col0), chunks = (qlen + CHUNK - 1) / CHUNK;
+    for (int i = tid; i < SCAN_STAGES * STAGE / 16; i += 2 * HALF)    // padding stays zero, stale places hold numbers
         reinterpret_cast<float4*>(sel_s)[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     float* base = state + (long)req_slot[r] * state_stride;
-    float* srow = base + (long)c * n;
-    scan_f2 S[R / 2], A[R / 2];
-    sel_rows<R, LANES>(S, srow, lane, n, mine && ctx != 0, state_vec4);
-    sel_rows<R, LANES>(A, a_log2 + (long)c * n, lane, n, mine, n % 4 == 0);
-    const float skip_c = mine ? skip[c] : 0.0f;
-    __syncthreads();
     auto stage_bc = [&](int s) { return reinterpret_cast<float*>(sel_s + s * STAGE); };
     auto stage_dt = [&](int s) { return stage_bc(s) + CHUNK * 2 * DP; };
     auto stage_x = [&](int s) { return reinterpret_cast<T*>(stage_dt(s) + CHUNK * COLS); };
-    auto copy_floats = [&](float* dst, int d_step, const float* src, long s_step, int count, int here, int vec) {
+    __syncthreads();
+    if (tid < HALF) {
+        const int lane = tid & (LANES - 1), col = tid / LANES, c = col0 + col;
+        const bool mine = c < inner;
+        float* srow = base + (long)c * n;
+        scan_f2 S[R / 2], A[R / 2];
+        sel_rows<R, LANES>(S, srow, lane, n, mine && ctx != 0, state_vec4);
+        sel_rows<R, LANES>(A, a_log2 + (long)c * n, lane, n, mine, n % 4 == 0);
+        const int my_u = ((lane & (LANES / 2)) ? 2 : 0) + ((lane & (LANES / 4)) ? 1 : 0);     // whose sum of four this lane gets
+        const bool writer = (lane & (LANES / 4 - 1)) == 0;
+        for (int k = 0; k <= chunks; ++k) {
+            __syncthreads();                                          // chunk k has landed
+            if (k == chunks) break;
+            const int here = min(CHUNK, qlen - k * CHUNK), stage = k & 3;
+            const float* bc = stage_bc(stage);
+            const float* dts = stage_dt(stage) + col;
+            const T* xs = stage_x(stage) + col;
+            float sums[CHUNK / 4];                                    // of this lane's token of each four
+            auto prepare = [&](SelToken<R>& tok, int t, bool real) {
+                const float d = real ? dts[t * COLS] : 0.0f;          // (behind the end: decay one, nothing added)
+                sel_prepare<T, R, LANES>(tok, A, bc + t * 2 * DP, bc + t * 2 * DP + DP, d, to_f32<T>(xs[t * COLS]), lane);
+            };
+            auto fold = [&](const float (&acc)[4]) {
+                const bool up2 = lane & (LANES / 2), up1 = lane & (LANES / 4);
+                const float w0 = scan_fold(up2, acc[0], acc[2], LANES / 2), w1 = scan_fold(up2, acc[1], acc[3], LANES / 2);
+                float v = scan_fold(up1, w0, w1, LANES / 4);
+#pragma unroll
+                for (int off = LANES / 8; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
+                return v;
+            };
+            if (here == CHUNK) {
+                float acc[CHUNK];
+#pragma unroll
+                for (int t = 0; t < CHUNK; ++t) {
+                    SelToken<R> tok;
+                    prepare(tok, t, true);
+                    acc[t] = sel_apply<T, R>(S, tok);
+                }
+#pragma unroll
+                for (int g = 0; g < CHUNK / 4; ++g) {
+                    const float four[4] = {acc[4 * g], acc[4 * g + 1], acc[4 * g + 2], acc[4 * g + 3]};
+                    sums[g] = fold(four);
+                }
+            } else {
+#pragma unroll
+                for (int g = 0; g < CHUNK / 4; ++g) {
+                    if (4 * g >= here) break;
+                    float acc[4];
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        SelToken<R> tok;
+                        prepare(tok, 4 * g + u, 4 * g + u < here);
+                        acc[u] = sel_apply<T, R>(S, tok);
+                    }
+                    sums[g] = fold(acc);
+                }
+            }
+            float* out = sum_s + (k & 1) * CHUNK * COLS + my_u * COLS + col;
+#pragma unroll
+            for (int g = 0; g < CHUNK / 4; ++g)
+                if (writer && 4 * g < here) out[4 * g * COLS] = sums[g];
+        }
+        pdl_trigger();                                                // (not at the start: the successor's CTAs would only wait here)
+        if (mine) sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
+        return;
+    }
+    const int ht = tid - HALF;
+    // rows of `count` (at most PER vectors of) elements: the loops' bounds and divisors are the tile's, not the layer's
+    auto copy_floats = [&](auto per, float* dst, int d_step, const float* src, long s_step, int count, int here, int vec) {
+        constexpr int PER = decltype(per)::value;                     // (vectors of four)
         if (vec) {
-            const int per = count / 4;
-            for (int i = tid; i < per * here; i += THREADS) scan_cp16(dst + i / per * d_step + i % per * 4, src + i / per * s_step + i % per * 4);
+#pragma unroll
+            for (int i = ht; i < PER * CHUNK; i += HALF) {
+                const int t = i / PER, e = i % PER * 4;
+                if (t < here && e < count) scan_cp16(dst + t * d_step + e, src + t * s_step + e);
+            }
         } else {
-            for (int i = tid; i < count * here; i += THREADS) scan_cp4(dst + i / count * d_step + i % count, src + i / count * s_step + i % count);
+            for (int i = ht; i < PER * 4 * CHUNK; i += HALF) {
+                const int t = i / (PER * 4), e = i % (PER * 4);
+                if (t < here && e < count) scan_cp4(dst + t * d_step + e, src + t * s_step + e);
+            }
         }
     };
     auto copy_rows = [&](T* dst, const T* src, long s_step, int here, int vec) {
         if (vec) {
-            const int per = cols / TV;
-            for (int i = tid; i < per * here; i += THREADS) scan_cp16(dst + i / per * COLS + i % per * TV, src + i / per * s_step + i % per * TV);
+#pragma unroll
+            for (int i = ht; i < COLS / TV * CHUNK; i += HALF) {
+                const int t = i / (COLS / TV), e = i % (COLS / TV) * TV;
+                if (t < here && e < cols) scan_cp16(dst + t * COLS + e, src + t * s_step + e);
+            }
         } else {
-            for (int i = tid; i < cols * here; i += THREADS) dst[i / cols * COLS + i % cols] = src[i / cols * s_step + i % cols];
+            for (int i = ht; i < COLS * CHUNK; i += HALF) {
+                const int t = i / COLS, e = i % COLS;
+                if (t < here && e < cols) dst[t * COLS + e] = src[t * s_step + e];
+            }
         }
     };
-    auto load = [&](int s, int c0) {
-        const int here = min(CHUNK, qlen - c0);
-        const long t = start + c0;
-        copy_floats(stage_bc(s), 2 * DP, in.low + t * in.low_ld + in.b_at, in.low_ld, n, here, vec_low);
-        copy_floats(stage_bc(s) + DP, 2 * DP, in.low + t * in.low_ld + in.c_at, in.low_ld, n, here, vec_low);
-        copy_floats(stage_dt(s), COLS, in.dt + t * in.dt_ld + col0, in.dt_ld, cols, here, vec_dt);
-        copy_rows(stage_x(s), (const T*)in.x + t * in.x_ld + col0, in.x_ld, here, vec_x);
-        copy_rows(stage_x(s) + CHUNK * COLS, (const T*)in.z + t * in.z_ld + col0, in.z_ld, here, vec_z);
+    auto load = [&](int k) {                                          // (one group of copies a chunk, empty ones beyond the end)
+        if (k < chunks) {
+            const int here = min(CHUNK, qlen - k * CHUNK), s = k & 3;
+            const long t = start + k * CHUNK;
+            copy_floats(ScanCount<DP / 4>(), stage_bc(s), 2 * DP, in.low + t * in.low_ld + in.b_at, in.low_ld, n, here, vec_low);
+            copy_floats(ScanCount<DP / 4>(), stage_bc(s) + DP, 2 * DP, in.low + t * in.low_ld + in.c_at, in.low_ld, n, here, vec_low);
+            copy_floats(ScanCount<COLS / 4>(), stage_dt(s), COLS, in.dt + t * in.dt_ld + col0, in.dt_ld, cols, here, vec_dt);
+            copy_rows(stage_x(s), (const T*)in.x + t * in.x_ld + col0, in.x_ld, here, vec_x);
+            copy_rows(stage_x(s) + CHUNK * COLS, (const T*)in.z + t * in.z_ld + col0, in.z_ld, here, vec_z);
+        }
         asm volatile("cp.async.commit_group;");
     };
-    // one group of copies per chunk, empty ones beyond the end: waiting for all but the last STAGES - 1 means this one landed
+    // outputs of a chunk, four channels a thread (always the same four: HALF is a multiple of COLS / 4)
+    constexpr int QUADS = COLS / 4;
+    const int e0 = ht % QUADS * 4;
+    float skip_e[4];
 #pragma unroll
-    for (int s = 0; s < SCAN_STAGES - 1; ++s) {
-        if (s * CHUNK < qlen) load(s, s * CHUNK); else asm volatile("cp.async.commit_group;");
-    }
-    const int my_u = ((lane & (LANES / 2)) ? 2 : 0) + ((lane & (LANES / 4)) ? 1 : 0);     // the token of four whose sum this lane gets
-    const bool writer = (lane & (LANES / 4 - 1)) == 0;
-    int stage = 0;
-    for (int c0 = 0; c0 < qlen; c0 += CHUNK, stage = (stage + 1) % SCAN_STAGES) {
-        const int here = min(CHUNK, qlen - c0), ahead = c0 + (SCAN_STAGES - 1) * CHUNK;
-        // (the stage copied into now was walked in the last round, behind that round's closing barrier)
-        if (ahead < qlen) load((stage + SCAN_STAGES - 1) % SCAN_STAGES, ahead); else asm volatile("cp.async.commit_group;");
-        asm volatile("cp.async.wait_group %0;" ::"n"(SCAN_STAGES - 1));
-        __syncthreads();                                              // this chunk has landed, y_s was written out
-        const float* bc = stage_bc(stage);
-        const float* dts = stage_dt(stage) + col;
-        const T* xs = stage_x(stage) + col;
+    for (int e = 0; e < 4; ++e) skip_e[e] = e0 + e < cols ? skip[col0 + e0 + e] : 0.0f;
+    auto finish = [&](int k) {
+        const int here = min(CHUNK, qlen - k * CHUNK);
+        const float* sums = sum_s + (k & 1) * CHUNK * COLS;
+        const T* xs = stage_x(k & 3);
         const T* zs = xs + CHUNK * COLS;
-        float sums[CHUNK / 4];                                        // of this lane's token of each group
-        auto group = [&](int t4, int left) {
-            float acc[4];
+        T* yo = y + (long)(start + k * CHUNK) * y_ld + col0 + e0;
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const int t = t4 + u;
-                const float d = u < left ? dts[t * COLS] : 0.0f;      // (behind the end: decay one, nothing added)
-                acc[u] = sel_token<T, R, LANES>(S, A, bc + t * 2 * DP, bc + t * 2 * DP + DP, d, to_f32<T>(xs[t * COLS]), lane);
+        for (int t = ht / QUADS; t < CHUNK; t += HALF / QUADS) {
+            if (t >= here || e0 >= cols) continue;
+            const ChanVec<4> v = chan_load<float, 4>(sums + t * COLS + e0), x = chan_load<T, 4>(xs + t * COLS + e0),
+                             z = chan_load<T, 4>(zs + t * COLS + e0);
+            ChanVec<4> o;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o.v[e] = fmaf(skip_e[e], x.v[e], v.v[e]) * fl_silu(z.v[e]) * scale;
+            if (vec_y) {
+                chan_store<T, 4>(yo + t * y_ld, o);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (e0 + e < cols) yo[t * y_ld + e] = from_f32<T>(o.v[e]);
             }
-            const bool up2 = lane & (LANES / 2), up1 = lane & (LANES / 4);
-            const float w0 = scan_fold(up2, acc[0], acc[2], LANES / 2), w1 = scan_fold(up2, acc[1], acc[3], LANES / 2);
-            float v = scan_fold(up1, w0, w1, LANES / 4);
-#pragma unroll
-            for (int off = LANES / 8; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-            return v;
-        };
-        // a whole chunk is straight-line code without a store in it, so that a group's reads overlap the sums before it
-        if (here == CHUNK) {
-#pragma unroll
-            for (int g = 0; g < CHUNK / 4; ++g) sums[g] = group(4 * g, 4);
-        } else {
-#pragma unroll
-            for (int g = 0; g < CHUNK / 4; ++g)
-                if (4 * g < here) sums[g] = group(4 * g, here - 4 * g);
         }
-#pragma unroll
-        for (int g = 0; g < CHUNK / 4; ++g) {
-            const int t = 4 * g + my_u;
-            if (writer && t < here)
-                y_s[t * COLS + col] = from_f32<T>(fmaf(skip_c, to_f32<T>(xs[t * COLS]), sums[g]) * fl_silu(to_f32<T>(zs[t * COLS])) * scale);
-        }
-        __syncthreads();                                              // y_s is whole; the stage is copied into again in the next round
-        T* yo = y + (long)(start + c0) * y_ld + col0;
-        if (vec_y) {
-            const int per = cols / TV;
-            for (int i = tid; i < per * here; i += THREADS)
-                *reinterpret_cast<uint4*>(yo + i / per * y_ld + i % per * TV) = *reinterpret_cast<const uint4*>(y_s + i / per * COLS + i % per * TV);
-        } else {
-            for (int i = tid; i < cols * here; i += THREADS) yo[i / cols * y_ld + i % cols] = y_s[i / cols * COLS + i % cols];
-        }
+    };
+    load(0);
+    load(1);
+    asm volatile("cp.async.wait_group 1;");
+    for (int k = 0; k <= chunks; ++k) {
+        __syncthreads();                                              // chunk k has landed, the sums of k - 1 are there
+        load(k + 2);                                                  // (into the stage of chunk k - 2, which no one reads any more)
+        if (k > 0) finish(k - 1);
+        asm volatile("cp.async.wait_group 1;");
     }
-    pdl_trigger();                                                    // (not at the start: the successor's CTAs would only wait here)
-    if (mine) sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
     // the kept inputs: entry j takes the input of position end - (taps - 1) + j (entries that stay move down)
     const T* up = (const T*)in.u;
-    for (int i = tid; i < cols; i += THREADS) {
+    for (int i = ht; i < cols; i += HALF) {
         float* kept = base + tail_off + col0 + i;
         for (int j = 0; j < taps - 1; ++j) {
             const int at = ctx + qlen - (taps - 1) + j;
@@ -464,7 +536,7 @@ static int selective_scan_launch(const SelRows& in, const float* a, const float*
                                  const int* req_qlen, const int* req_slot, int n_requests, int inner, int n, bool overlap,
                                  cudaStream_t stream) {
     constexpr int CHUNK = R * LANES <= 64 ? 16 : 8;
-    constexpr size_t smem = (size_t)SCAN_STAGES * CHUNK * ((2 * R * LANES + COLS) * 4 + 2 * COLS * sizeof(T)) + CHUNK * COLS * sizeof(T);
+    constexpr size_t smem = (size_t)SCAN_STAGES * CHUNK * ((2 * R * LANES + COLS) * 4 + 2 * COLS * sizeof(T)) + 2 * CHUNK * COLS * 4;
     auto kernel = selective_scan_kernel<T, R, LANES, COLS, CHUNK>;
     static bool configured = false;
     if (!configured) {
@@ -477,9 +549,10 @@ static int selective_scan_launch(const SelRows& in, const float* a, const float*
     const int vec_low = n % 4 == 0 && in.b_at % 4 == 0 && in.c_at % 4 == 0 && in.low_ld % 4 == 0 && ((uintptr_t)in.low % 16) == 0;
     const int vec_dt = inner % 4 == 0 && in.dt_ld % 4 == 0 && ((uintptr_t)in.dt % 16) == 0;
     const int state_vec4 = n % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0;
-    return fl_launch_as(overlap, kernel, dim3(n_requests, (inner + COLS - 1) / COLS), dim3(COLS * LANES), smem, stream, in, a, skip,
+    return fl_launch_as(overlap, kernel, dim3(n_requests, (inner + COLS - 1) / COLS), dim3(2 * COLS * LANES), smem, stream, in, a, skip,
                         scale, y, y_ld, state, state_stride, tail_off, taps, req_start, req_ctx, req_qlen, req_slot, inner, n,
-                        vec_low, vec_dt, rows16(in.x, in.x_ld), rows16(in.z, in.z_ld), rows16(y, y_ld), state_vec4);
+                        vec_low, vec_dt, rows16(in.x, in.x_ld), rows16(in.z, in.z_ld),
+                        inner % 4 == 0 && chan_aligned(y, y_ld, sizeof(T)) ? 1 : 0, state_vec4);
 }
 
 static inline bool selective_takes(int inner, int n, int taps) {
@@ -588,7 +661,9 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
 #pragma unroll
     for (int off = LANES / 2; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
     const float dt = fl_softplus(dot + bias_c);
-    float sum = sel_token<T, R, LANES>(S, A, step_s, step_s + DP, dt, xv, lane);
+    SelToken<R> tok;
+    sel_prepare<T, R, LANES>(tok, A, step_s, step_s + DP, dt, xv, lane);
+    float sum = sel_apply<T, R>(S, tok);
 #pragma unroll
     for (int off = LANES / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
     if (!mine) return;
