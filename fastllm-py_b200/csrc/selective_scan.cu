@@ -11,9 +11,8 @@
 //
 //   selective_conv      convolution and silu (in the activation type, which W_x reads); in steps of single tokens the
 //                       thread that owns a channel moves its kept inputs on
-//   selective_dt        dt of every token and channel: float sums on the CUDA cores, one order whatever the step
-//   selective_dt_mma    the same for bfloat16 models on mma.sync: the float row is split into two bfloat16 parts, so that
-//                       the product keeps about 16 bits of it; W_dt is bfloat16 as stored
+//   selective_split     the product W_dt dt (the caller's) reads dt's float row as two bfloat16 parts, which keep about 16
+//                       bits of it, against W_dt twice over
 //   selective_scan      the recurrence over each request's tokens in order, read-out, skip and gate; its blocks also move
 //                       the kept inputs of requests on
 //   selective_step      steps of single tokens: dt, recurrence, read-out and gate of a request's channels in one kernel
@@ -80,171 +79,25 @@ FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* con
 }
 
 // ------------------------------------------------------------------ step sizes
-#define SEL_DT_TOKENS 8
-
-// dt[t, c] = softplus(sum_k low[t, k] w_t[k, c] + bias[c]); a thread takes one channel of SEL_DT_TOKENS tokens.
-__global__ void __launch_bounds__(128) selective_dt_kernel(const float* __restrict__ low, long low_ld, int rank,
-                                                           const float* __restrict__ w_t, const float* __restrict__ bias,
-                                                           float* __restrict__ dt, long dt_ld, int n_tokens, int inner) {
+// out[t] = [hi | lo], two bfloat16 parts of the first `rank` columns of low[t]: lo is what rounding to hi leaves.
+__global__ void __launch_bounds__(256) selective_split_kernel(const float* __restrict__ low, long low_ld, int rank,
+                                                              bf16* __restrict__ out, long out_ld) {
     pdl_wait();
     pdl_trigger();
-    extern __shared__ float sel_low[];                                // [rank][SEL_DT_TOKENS]
-    const int t0 = blockIdx.x * SEL_DT_TOKENS, here = min(SEL_DT_TOKENS, n_tokens - t0);
-    for (int i = threadIdx.x; i < rank * SEL_DT_TOKENS; i += blockDim.x) {
-        const int t = i / rank, k = i % rank;
-        sel_low[k * SEL_DT_TOKENS + t] = t < here ? low[(long)(t0 + t) * low_ld + k] : 0.0f;
+    const float* row = low + (long)blockIdx.x * low_ld;
+    bf16* o = out + (long)blockIdx.x * out_ld;
+    for (int k = threadIdx.x; k < rank; k += blockDim.x) {
+        const bf16 hi = __float2bfloat16_rn(row[k]);
+        o[k] = hi;
+        o[rank + k] = __float2bfloat16_rn(row[k] - __bfloat162float(hi));
     }
-    __syncthreads();
-    const int c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c >= inner) return;
-    float acc[SEL_DT_TOKENS];
-#pragma unroll
-    for (int t = 0; t < SEL_DT_TOKENS; ++t) acc[t] = 0.0f;
-    for (int k = 0; k < rank; ++k) {
-        const float w = w_t[(long)k * inner + c];
-#pragma unroll
-        for (int t = 0; t < SEL_DT_TOKENS; ++t) acc[t] = fmaf(sel_low[k * SEL_DT_TOKENS + t], w, acc[t]);
-    }
-    const float b = bias[c];
-#pragma unroll
-    for (int t = 0; t < SEL_DT_TOKENS; ++t)
-        if (t < here) dt[(long)(t0 + t) * dt_ld + c] = fl_softplus(acc[t] + b);
 }
 
-// low: float rows of which the first `rank` columns count; w_t: [rank][inner] float.
-FL_API int fl_selective_dt(const float* low, long low_ld, int rank, const float* w_t, const float* bias, float* dt, long dt_ld,
-                           int n_tokens, int inner, cudaStream_t stream) {
+FL_API int fl_selective_split(const float* low, long low_ld, int rank, void* out, long out_ld, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    const size_t smem = (size_t)rank * SEL_DT_TOKENS * sizeof(float);
-    if (rank < 1 || smem > 160 * 1024 || (inner + 127) / 128 > 65535) return (int)cudaErrorInvalidValue;
-    if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(selective_dt_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return (int)e;
-    }
-    return fl_launch(selective_dt_kernel, dim3((n_tokens + SEL_DT_TOKENS - 1) / SEL_DT_TOKENS, (inner + 127) / 128), dim3(128),
-                     smem, stream, low, low_ld, rank, w_t, bias, dt, dt_ld, n_tokens, inner);
-}
-
-#define SEL_MM 64                    // tokens and channels of a block's tile
-#define SEL_MK 64                    // columns of a stage
-#define SEL_MP (SEL_MK + 8)          // bfloat16 elements between staged rows (ldmatrix without bank conflicts)
-#define SEL_MC 4                     // tiles of channels that a block walks with the same tokens
-
-__device__ __forceinline__ void sel_ldm4(unsigned (&r)[4], const bf16* p) {
-    const unsigned s = (unsigned)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void sel_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-// w: [inner][w_ld] bfloat16, w_ld a multiple of 8 and zero from column `rank` on.
-__global__ void __launch_bounds__(128) selective_dt_mma_kernel(const float* __restrict__ low, long low_ld, int rank,
-                                                               const bf16* __restrict__ w, int w_ld,
-                                                               const float* __restrict__ bias, float* __restrict__ dt,
-                                                               long dt_ld, int n_tokens, int inner, int low_vec) {
-    // all of low's columns for 64 tokens stay staged (as two parts) while the block walks its tiles of channels
-    extern __shared__ __align__(16) unsigned char sel_mma_s[];
-    const int k_end = (rank + 15) / 16 * 16, pitch = k_end + 8;
-    bf16* hi_s = reinterpret_cast<bf16*>(sel_mma_s);                  // [SEL_MM][pitch]
-    bf16* lo_s = hi_s + SEL_MM * pitch;
-    bf16* w_s = lo_s + SEL_MM * pitch;                                // [SEL_MM][SEL_MP]
-    const int t0 = blockIdx.x * SEL_MM, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    pdl_wait();
-    pdl_trigger();
-    for (int i = tid; i < SEL_MM * k_end / 4; i += 128) {
-        const int r = i / (k_end / 4), k = i % (k_end / 4) * 4;
-        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        if (t0 + r < n_tokens) {
-            const float* p = low + (long)(t0 + r) * low_ld + k;
-            if (low_vec && k + 4 <= rank) {
-                const float4 q = *reinterpret_cast<const float4*>(p);
-                v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
-            } else {
-#pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    if (k + e < rank) v[e] = p[e];
-            }
-        }
-#pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-            const __nv_bfloat162 hi = __floats2bfloat162_rn(v[e], v[e + 1]);
-            const float2 f = __bfloat1622float2(hi);
-            *reinterpret_cast<__nv_bfloat162*>(hi_s + r * pitch + k + e) = hi;
-            *reinterpret_cast<__nv_bfloat162*>(lo_s + r * pitch + k + e) = __floats2bfloat162_rn(v[e] - f.x, v[e + 1] - f.y);
-        }
-    }
-    for (int tile = 0; tile < SEL_MC; ++tile) {
-        const int c0 = (blockIdx.y * SEL_MC + tile) * SEL_MM;
-        if (c0 >= inner) break;
-        float acc[SEL_MM / 8][4];
-#pragma unroll
-        for (int i = 0; i < SEL_MM / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
-        for (int k0 = 0; k0 < rank; k0 += SEL_MK) {
-            __syncthreads();                                              // low is staged; w_s was read
-            for (int i = tid; i < SEL_MM * (SEL_MK / 8); i += 128) {
-                const int r = i / (SEL_MK / 8), k = i % (SEL_MK / 8) * 8;
-                uint4 v = make_uint4(0, 0, 0, 0);
-                if (c0 + r < inner && k0 + k < w_ld) v = *reinterpret_cast<const uint4*>(w + (long)(c0 + r) * w_ld + k0 + k);
-                *reinterpret_cast<uint4*>(w_s + r * SEL_MP + k) = v;
-            }
-            __syncthreads();
-            const int ks_end = min(SEL_MK, k_end - k0);
-            for (int ks = 0; ks < ks_end; ks += 16) {
-                unsigned hi[4], lo[4];
-                sel_ldm4(hi, hi_s + (warp * 16 + (lane & 15)) * pitch + k0 + ks + (lane >> 4) * 8);
-                sel_ldm4(lo, lo_s + (warp * 16 + (lane & 15)) * pitch + k0 + ks + (lane >> 4) * 8);
-#pragma unroll
-                for (int j = 0; j < SEL_MM / 16; ++j) {
-                    unsigned b[4];
-                    sel_ldm4(b, w_s + (j * 16 + (lane & 7) + (lane >> 4) * 8) * SEL_MP + ks + ((lane >> 3) & 1) * 8);
-                    sel_mma(acc[2 * j], hi, b[0], b[1]);
-                    sel_mma(acc[2 * j + 1], hi, b[2], b[3]);
-                    sel_mma(acc[2 * j], lo, b[0], b[1]);
-                    sel_mma(acc[2 * j + 1], lo, b[2], b[3]);
-                }
-            }
-        }
-        const bool pairs = inner % 2 == 0 && dt_ld % 2 == 0;
-#pragma unroll
-        for (int i = 0; i < SEL_MM / 8; ++i) {
-            const int c = c0 + i * 8 + (lane & 3) * 2;
-            if (c >= inner) continue;
-            const bool both = c + 1 < inner;
-            const float b0 = bias[c], b1 = both ? bias[c + 1] : 0.0f;
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int t = t0 + warp * 16 + (lane >> 2) + h * 8;
-                if (t >= n_tokens) continue;
-                float* o = dt + (long)t * dt_ld + c;
-                const float d0 = fl_softplus(acc[i][2 * h] + b0), d1 = fl_softplus(acc[i][2 * h + 1] + b1);
-                if (pairs) *reinterpret_cast<float2*>(o) = make_float2(d0, d1);
-                else {
-                    o[0] = d0;
-                    if (both) o[1] = d1;
-                }
-            }
-        }
-    }
-}
-
-FL_API int fl_selective_dt_mma(const float* low, long low_ld, int rank, const void* w, int w_ld, const float* bias, float* dt,
-                               long dt_ld, int n_tokens, int inner, cudaStream_t stream) {
-    if (n_tokens <= 0) return 0;
-    const int per = SEL_MM * SEL_MC, k_end = (rank + 15) / 16 * 16;
-    const size_t smem = ((size_t)2 * SEL_MM * (k_end + 8) + SEL_MM * SEL_MP) * sizeof(bf16);
-    if (rank < 1 || smem > 220 * 1024 || w_ld < rank || w_ld % 8 || ((uintptr_t)w % 16) || ((uintptr_t)dt % 8) ||
-        (inner + per - 1) / per > 65535)
-        return (int)cudaErrorInvalidValue;
-    if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(selective_dt_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return (int)e;
-    }
-    const int low_vec = low_ld % 4 == 0 && ((uintptr_t)low % 16) == 0;
-    return fl_launch(selective_dt_mma_kernel, dim3((n_tokens + SEL_MM - 1) / SEL_MM, (inner + per - 1) / per), dim3(128), smem,
-                     stream, low, low_ld, rank, (const bf16*)w, w_ld, bias, dt, dt_ld, n_tokens, inner, low_vec);
+    if (rank < 1 || out_ld < 2L * rank) return (int)cudaErrorInvalidValue;
+    const int threads = rank >= 256 ? 256 : (rank + 31) / 32 * 32;
+    return fl_launch(selective_split_kernel, dim3(n_tokens), dim3(threads), 0, stream, low, low_ld, rank, (bf16*)out, out_ld);
 }
 
 // ------------------------------------------------------------------ the recurrence
@@ -336,21 +189,42 @@ __device__ __forceinline__ float sel_apply(scan_f2 (&S)[R / 2], const SelToken<R
 
 template <int N> struct ScanCount { static constexpr int value = N; };
 
+// softplus(v) = max(v, 0) + log(1 + u), u = exp(-|v|); log(1 + u) = 2 artanh(s) with s = u / (2 + u) <= 1/3, as its power
+// series in s^2 (eight terms leave 3e-9 of the sum).  No branch, and exact relative to the result also where it is small.
+template <typename T> __device__ __forceinline__ float sel_softplus(float v) {
+    const float u = sizeof(T) == 4 ? expf(-fabsf(v)) : __expf(-fabsf(v));
+    const float s = sizeof(T) == 4 ? u / (2.0f + u) : __fdividef(u, 2.0f + u);
+    const float q = s * s;
+    float p = 1.0f / 15.0f;
+    p = fmaf(p, q, 1.0f / 13.0f);
+    p = fmaf(p, q, 1.0f / 11.0f);
+    p = fmaf(p, q, 1.0f / 9.0f);
+    p = fmaf(p, q, 1.0f / 7.0f);
+    p = fmaf(p, q, 1.0f / 5.0f);
+    p = fmaf(p, q, 1.0f / 3.0f);
+    return fmaxf(v, 0.0f) + fmaf(2.0f * s * q, p, 2.0f * s);
+}
+// silu with the fast exponential and division where the result is rounded to bfloat16.
+template <typename T> __device__ __forceinline__ float sel_silu(float v) {
+    return sizeof(T) == 4 ? fl_silu(v) : __fdividef(v, 1.0f + __expf(-v));
+}
+
 struct SelRows {                     // the step's rows: element type T, float, float
     const void *x, *z, *u;           // convolved inputs, gates, inputs before the convolution
-    const float *dt, *low;
+    const float *dt, *low;           // (dt before bias and softplus)
     long x_ld, z_ld, u_ld, dt_ld, low_ld;
     int b_at, c_at;                  // where low holds B and C
 };
 
 // A block takes one request and COLS channels.  Half of its threads walk the tokens, LANES lanes a channel, and do nothing
 // else: a chunk of tokens is straight-line code that reads shared memory and leaves the read-out sums there.  The other
-// half copies the chunks two ahead (cp.async, four stages) and turns the sums of the chunk before into outputs (skip, gate,
-// store).  Tokens go four at a time, so that four sums are added up over the lanes together.  R and LANES follow from n alone:
+// half copies the chunks two ahead (cp.async, four stages), makes the step sizes of the next one (softplus of W_dt dt + bias)
+// and turns the sums of the chunk before into outputs (skip, gate, store).  Tokens go four at a time, so that four sums are added up over the lanes together.  R and LANES follow from n alone:
 // one order of sums whatever the cut.
 template <typename T, int R, int LANES, int COLS, int CHUNK>
 __global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
-    const SelRows in, const float* __restrict__ a_log2, const float* __restrict__ skip, float scale, T* __restrict__ y, long y_ld,
+    const SelRows in, const float* __restrict__ dt_bias, const float* __restrict__ a_log2, const float* __restrict__ skip, float scale,
+    T* __restrict__ y, long y_ld,
     float* __restrict__ state, long state_stride, long tail_off, int taps, const int* __restrict__ req_start,
     const int* __restrict__ req_ctx, const int* __restrict__ req_qlen, const int* __restrict__ req_slot, int inner, int n,
     int vec_low, int vec_dt, int vec_x, int vec_z, int vec_y, int state_vec4) {
@@ -481,9 +355,37 @@ __global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
     // outputs of a chunk, four channels a thread (always the same four: HALF is a multiple of COLS / 4)
     constexpr int QUADS = COLS / 4;
     const int e0 = ht % QUADS * 4;
-    float skip_e[4];
+    float skip_e[4], bias_e[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) skip_e[e] = e0 + e < cols ? skip[col0 + e0 + e] : 0.0f;
+    for (int e = 0; e < 4; ++e) {
+        skip_e[e] = e0 + e < cols ? skip[col0 + e0 + e] : 0.0f;
+        bias_e[e] = e0 + e < cols ? dt_bias[col0 + e0 + e] : 0.0f;
+    }
+    const float bias_1 = ht % COLS < cols ? dt_bias[col0 + ht % COLS] : 0.0f;
+    // step sizes of a chunk, in place: a thread takes the places it copied, which its own wait has made visible to it
+    auto rates = [&](int k) {
+        if (k >= chunks) return;
+        const int here = min(CHUNK, qlen - k * CHUNK);
+        float* d = stage_dt(k & 3);
+        if (vec_dt) {
+#pragma unroll
+            for (int t = ht / QUADS; t < CHUNK; t += HALF / QUADS) {
+                if (t >= here || e0 >= cols) continue;
+                float4* p = reinterpret_cast<float4*>(d + t * COLS + e0);
+                float4 v = *p;
+                v.x = sel_softplus<T>(v.x + bias_e[0]);
+                v.y = sel_softplus<T>(v.y + bias_e[1]);
+                v.z = sel_softplus<T>(v.z + bias_e[2]);
+                v.w = sel_softplus<T>(v.w + bias_e[3]);
+                *p = v;
+            }
+        } else {
+            for (int t = ht / COLS; t < CHUNK; t += HALF / COLS) {
+                float* p = d + t * COLS + ht % COLS;
+                if (t < here && ht % COLS < cols) *p = sel_softplus<T>(*p + bias_1);
+            }
+        }
+    };
     auto finish = [&](int k) {
         const int here = min(CHUNK, qlen - k * CHUNK);
         const float* sums = sum_s + (k & 1) * CHUNK * COLS;
@@ -497,7 +399,7 @@ __global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
                              z = chan_load<T, 4>(zs + t * COLS + e0);
             ChanVec<4> o;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) o.v[e] = fmaf(skip_e[e], x.v[e], v.v[e]) * fl_silu(z.v[e]) * scale;
+            for (int e = 0; e < 4; ++e) o.v[e] = fmaf(skip_e[e], x.v[e], v.v[e]) * sel_silu<T>(z.v[e]) * scale;
             if (vec_y) {
                 chan_store<T, 4>(yo + t * y_ld, o);
             } else {
@@ -509,12 +411,14 @@ __global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
     };
     load(0);
     load(1);
-    asm volatile("cp.async.wait_group 1;");
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    rates(0);
     for (int k = 0; k <= chunks; ++k) {
         __syncthreads();                                              // chunk k has landed, the sums of k - 1 are there
         load(k + 2);                                                  // (into the stage of chunk k - 2, which no one reads any more)
         if (k > 0) finish(k - 1);
-        asm volatile("cp.async.wait_group 1;");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        rates(k + 1);
     }
     // the kept inputs: entry j takes the input of position end - (taps - 1) + j (entries that stay move down)
     const T* up = (const T*)in.u;
@@ -531,7 +435,7 @@ __global__ void __launch_bounds__(2 * COLS * LANES, 1) selective_scan_kernel(
 }
 
 template <typename T, int R, int LANES, int COLS>
-static int selective_scan_launch(const SelRows& in, const float* a, const float* skip, float scale, T* y, long y_ld, float* state,
+static int selective_scan_launch(const SelRows& in, const float* dt_bias, const float* a, const float* skip, float scale, T* y, long y_ld, float* state,
                                  long state_stride, long tail_off, int taps, const int* req_start, const int* req_ctx,
                                  const int* req_qlen, const int* req_slot, int n_requests, int inner, int n, bool overlap,
                                  cudaStream_t stream) {
@@ -549,7 +453,7 @@ static int selective_scan_launch(const SelRows& in, const float* a, const float*
     const int vec_low = n % 4 == 0 && in.b_at % 4 == 0 && in.c_at % 4 == 0 && in.low_ld % 4 == 0 && ((uintptr_t)in.low % 16) == 0;
     const int vec_dt = inner % 4 == 0 && in.dt_ld % 4 == 0 && ((uintptr_t)in.dt % 16) == 0;
     const int state_vec4 = n % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state % 16) == 0;
-    return fl_launch_as(overlap, kernel, dim3(n_requests, (inner + COLS - 1) / COLS), dim3(2 * COLS * LANES), smem, stream, in, a, skip,
+    return fl_launch_as(overlap, kernel, dim3(n_requests, (inner + COLS - 1) / COLS), dim3(2 * COLS * LANES), smem, stream, in, dt_bias, a, skip,
                         scale, y, y_ld, state, state_stride, tail_off, taps, req_start, req_ctx, req_qlen, req_slot, inner, n,
                         vec_low, vec_dt, rows16(in.x, in.x_ld), rows16(in.z, in.z_ld),
                         inner % 4 == 0 && chan_aligned(y, y_ld, sizeof(T)) ? 1 : 0, state_vec4);
@@ -559,10 +463,10 @@ static inline bool selective_takes(int inner, int n, int taps) {
     return n >= 1 && n <= 256 && inner >= 1 && (inner + 7) / 8 <= 65535 && taps >= 1 && taps <= 16;
 }
 
-// x, z, u, y: rows of the activation type; a: -exp(A_log) [inner][n], times log2(e) for bfloat16.  single_tokens: every
+// x, z, u, y: rows of the activation type; dt: W_dt dt without its bias; a: -exp(A_log) [inner][n], times log2(e) for bfloat16.  single_tokens: every
 // request of the step brings one token (a short kernel).
 FL_API int fl_selective_scan(const void* x, long x_ld, const void* z, long z_ld, const void* u, long u_ld, int dtype,
-                             const float* dt, long dt_ld, const float* low, long low_ld, int b_at, int c_at, const float* a,
+                             const float* dt, long dt_ld, const float* dt_bias, const float* low, long low_ld, int b_at, int c_at, const float* a,
                              const float* skip, float scale, void* y, long y_ld, float* state, long state_stride, long tail_off,
                              int taps, const int* req_start, const int* req_ctx, const int* req_qlen, const int* req_slot,
                              int n_requests, int inner, int n, int single_tokens, cudaStream_t stream) {
@@ -570,7 +474,7 @@ FL_API int fl_selective_scan(const void* x, long x_ld, const void* z, long z_ld,
     if (!selective_takes(inner, n, taps)) return (int)cudaErrorInvalidValue;
     const SelRows in{x, z, u, dt, low, x_ld, z_ld, u_ld, dt_ld, low_ld, b_at, c_at};
 #define FL_SEL_SCAN(R, L, C)                                                                                                 \
-    FL_DISPATCH(dtype, T, return selective_scan_launch<T, R, L, C>(in, a, skip, scale, (T*)y, y_ld, state, state_stride, tail_off, \
+    FL_DISPATCH(dtype, T, return selective_scan_launch<T, R, L, C>(in, dt_bias, a, skip, scale, (T*)y, y_ld, state, state_stride, tail_off, \
                                                                    taps, req_start, req_ctx, req_qlen, req_slot, n_requests, \
                                                                    inner, n, single_tokens != 0, stream))
     if (n <= 16) { FL_SEL_SCAN(4, 4, 32); }
@@ -660,7 +564,7 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
         }
 #pragma unroll
     for (int off = LANES / 2; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
-    const float dt = fl_softplus(dot + bias_c);
+    const float dt = sel_softplus<T>(dot + bias_c);
     SelToken<R> tok;
     sel_prepare<T, R, LANES>(tok, A, step_s, step_s + DP, dt, xv, lane);
     float sum = sel_apply<T, R>(S, tok);
@@ -668,7 +572,7 @@ __global__ void __launch_bounds__(COLS * LANES) selective_step_kernel(
     for (int off = LANES / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
     if (!mine) return;
     if (lane == 0)
-        y[(long)r * y_ld + c] = from_f32<T>(fmaf(skip_c, xv, sum) * fl_silu(zv) * scale);
+        y[(long)r * y_ld + c] = from_f32<T>(fmaf(skip_c, xv, sum) * sel_silu<T>(zv) * scale);
     sel_rows_out<R, LANES>(S, srow, lane, n, state_vec4);
 }
 

@@ -37,7 +37,6 @@ template <typename T, int V> __device__ __forceinline__ void chan_store(T* p, co
 static inline bool chan_aligned(const void* p, long ld, int elem) { return ((uintptr_t)p % (4 * elem)) == 0 && ld % 4 == 0; }
 
 __device__ __forceinline__ float fl_silu(float v) { return v / (1.0f + expf(-v)); }
-__device__ __forceinline__ float fl_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
 struct StepTables {              // per token: its request and position; per request: first row, context, tokens, slot
     const int *tok_req, *positions, *req_start, *req_ctx, *req_qlen, *req_slot;

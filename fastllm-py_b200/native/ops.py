@@ -1010,53 +1010,40 @@ def selective_conv(u, conv_w, conv_b, tail, step, x, move_tail):
               _ptr(step.req_slot), _ptr(x), _ld(x), u.shape[0], inner, int(bool(move_tail)), _stream()), "selective_conv")
 
 
-def selective_dt(low, rank, w, bias, dt):
-    """dt = softplus(low[:, :rank] @ w + bias), float32.  `w` float32 [rank, inner]: sums on the CUDA cores in one order; or
-    bfloat16 [inner, >= rank] (a row pitch that is a multiple of 8, zeros from column `rank` on): tensor cores, with low as
-    two bfloat16 parts."""
-    _require_cuda(low, w, bias, dt)
-    inner = dt.shape[1]
-    if low.dtype != torch.float32 or dt.dtype != torch.float32 or bias.dtype != torch.float32 or not w.is_contiguous():
-        raise KernelError("selective_dt: low, bias and dt are float32, w is contiguous")
-    if w.dtype == torch.float32:
-        if tuple(w.shape) != (rank, inner):
-            raise KernelError("selective_dt: a float32 matrix is [rank, inner]")
-        fn = _fn("selective_scan", "fl_selective_dt", [c_void_p, c_long, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int,
-                                                       c_void_p])
-        _check(fn(_ptr(low), _ld(low), rank, _ptr(w), _ptr(bias), _ptr(dt), _ld(dt), low.shape[0], inner, _stream()), "selective_dt")
-        return
-    if w.shape[0] != inner:
-        raise KernelError("selective_dt: a bfloat16 matrix is [inner, >= rank]")
-    fn = _fn("selective_scan", "fl_selective_dt_mma", [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int,
-                                                       c_int, c_void_p])
-    _check(fn(_ptr(low), _ld(low), rank, _ptr(w), w.shape[1], _ptr(bias), _ptr(dt), _ld(dt), low.shape[0], inner, _stream()),
-           "selective_dt_mma")
+def selective_split(low, rank, out):
+    """out = [hi | lo]: the first `rank` columns of `low` (float32) as two bfloat16 parts, lo being what rounding to hi leaves."""
+    _require_cuda(low, out)
+    if low.dtype != torch.float32 or out.dtype != torch.bfloat16 or out.shape[1] != 2 * rank or out.shape[0] != low.shape[0]:
+        raise KernelError("selective_split: low is float32, out bfloat16 [N, 2 rank]")
+    fn = _fn("selective_scan", "fl_selective_split", [c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_void_p])
+    _check(fn(_ptr(low), _ld(low), rank, _ptr(out), _ld(out), low.shape[0], _stream()), "selective_split")
 
 
-def selective_scan(x, z, u, dt, low, rank, a, skip, scale, y, state_rows, tail_off, taps, step):
-    """S <- exp(dt a) S + dt x B, y = (S C + skip x) * silu(z) * scale per channel over the step's tokens; B and C are the
+def selective_scan(x, z, u, dt, dt_bias, low, rank, a, skip, scale, y, state_rows, tail_off, taps, step):
+    """With d = softplus(dt + dt_bias): S <- exp(d a) S + d x B, y = (S C + skip x) * silu(z) * scale per channel over the step's
+    tokens; B and C are the
     columns of `low` (float32) from `rank` on, `a` float32 [inner, state] (times log2(e) for bfloat16 rows).  State rows:
     S [inner, state] float32, read unless the request starts and written, and from `tail_off` on the convolution's kept
     inputs, which move on (u: the inputs)."""
-    _require_cuda(x, z, u, dt, low, a, skip, y, state_rows)
+    _require_cuda(x, z, u, dt, dt_bias, low, a, skip, y, state_rows)
     inner, n = a.shape
     if len({x.dtype, z.dtype, u.dtype, y.dtype}) != 1 or not a.is_contiguous() or \
-            any(v.dtype != torch.float32 for v in (dt, low, a, skip, state_rows)) or low.shape[1] < rank + 2 * n:
+            any(v.dtype != torch.float32 for v in (dt, dt_bias, low, a, skip, state_rows)) or low.shape[1] < rank + 2 * n:
         raise KernelError("selective_scan: x, z, u and y share a dtype, everything else is float32")
     fn = _fn("selective_scan", "fl_selective_scan",
-             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p, c_long, c_int, c_int,
-              c_void_p, c_void_p, c_float, c_void_p, c_long, c_void_p, c_long, c_long, c_int, c_void_p, c_void_p, c_void_p,
+             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_void_p, c_void_p, c_long, c_int,
+              c_int, c_void_p, c_void_p, c_float, c_void_p, c_long, c_void_p, c_long, c_long, c_int, c_void_p, c_void_p, c_void_p,
               c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(x), _ld(x), _ptr(z), _ld(z), _ptr(u), _ld(u), dtype_code(x), _ptr(dt), _ld(dt), _ptr(low), _ld(low), rank,
+    _check(fn(_ptr(x), _ld(x), _ptr(z), _ld(z), _ptr(u), _ld(u), dtype_code(x), _ptr(dt), _ld(dt), _ptr(dt_bias), _ptr(low), _ld(low), rank,
               rank + n, _ptr(a), _ptr(skip), float(scale), _ptr(y), _ld(y), _ptr(state_rows), state_rows.stride(0), int(tail_off),
               int(taps), _ptr(step.req_start), _ptr(step.req_ctx), _ptr(step.req_qlen), _ptr(step.req_slot), step.n_requests,
               inner, n, int(x.shape[0] == step.n_requests), _stream()), "selective_scan")
 
 
 def selective_step(x, z, low, rank, w_dt, dt_bias, a, skip, scale, y, state_rows, step):
-    """selective_dt and selective_scan in one kernel for a step in which every request brings one token (the kept inputs are
-    left as they are).  `low` may be split-K partial sums, added up while they are read; `w_dt` [inner, >= rank] as in
-    `selective_dt`, of either dtype."""
+    """W_dt's product and selective_scan in one kernel for a step in which every request brings one token (the kept inputs are
+    left as they are).  `low` may be split-K partial sums, added up while they are read; `w_dt` [inner, >= rank] of either
+    dtype, with a row pitch that is a multiple of 8 and zeros from column `rank` on."""
     _require_cuda(x, z, w_dt, dt_bias, a, skip, y, state_rows)
     inner, n = a.shape
     if step.n_tokens != step.n_requests or len({x.dtype, z.dtype, y.dtype}) != 1 or not w_dt.is_contiguous() or \

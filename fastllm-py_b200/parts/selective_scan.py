@@ -35,7 +35,6 @@ class SelectiveScan(ProjectedMixer):
     native_libraries = ("selective_scan",)
     in_slots = ("in",)
     workspace_name = "selective"
-    TENSOR_CORE_RANK = 768
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -46,12 +45,12 @@ class SelectiveScan(ProjectedMixer):
             raise ValueError(f"selective_scan: state {self.state} is beyond the kernels' limit of 256")
         if not 1 <= self.taps <= 16:
             raise ValueError(f"selective_scan: {self.taps} taps are beyond the kernels' 16")
-        if self.rank > 4096:
-            raise ValueError(f"selective_scan: rank {self.rank} is beyond the kernels' limit of 4096")
+        if self.rank > 8192:
+            raise ValueError(f"selective_scan: rank {self.rank} is beyond the kernels' limit of 8192")
         self.low_cols = self.rank + 2 * self.state
         self.in_cols, self.out_cols = 2 * self.inner, self.inner
         self.state_floats = -(-self.inner * self.state // 4) * 4              # (the kept inputs start on 16 bytes)
-        self.low = None
+        self.low = self.dt = None
 
     def cache_need(self):
         floats = self.state_floats + (self.taps - 1) * self.inner
@@ -73,9 +72,9 @@ class SelectiveScan(ProjectedMixer):
         pitch = -(-self.rank // 8) * 8
         self.dt_w = torch.zeros((self.inner, pitch), dtype=w.dtype, device=w.device)      # rows that start on 16 bytes
         self.dt_w[:, :self.rank] = w
-        # the 32-bit path (and a rank beyond the tensor-core kernel's shared memory) sums on the CUDA cores, along the channels
-        exact = self.ctx.dtype == torch.float32 or w.dtype == torch.float32 or self.rank > self.TENSOR_CORE_RANK
-        self.dt_t = w.float().t().contiguous() if exact else None
+        # prompt portions: W_dt twice over, against the two bfloat16 parts of a float row, where the product is bfloat16
+        self.split = self.ctx.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
+        self.dt = Linear([torch.cat([w, w], dim=1) if self.split else w])
         self.dt_bias = tensors["dt_bias"].float().contiguous()
         a = -torch.exp(tensors["A_log"].double())
         self.a = (a * math.log2(math.e) if self.ctx.dtype == torch.bfloat16 else a).float().contiguous()
@@ -84,6 +83,8 @@ class SelectiveScan(ProjectedMixer):
     def reserve(self, limits):
         super().reserve(limits)
         self.low.reserve(self.ctx.dtype, limits.max_tokens)
+        if self.split:
+            self.dt.reserve(self.ctx.dtype, limits.max_tokens)
 
     def core(self, proj, y, step, cache):
         n = proj.shape[0]
@@ -101,6 +102,11 @@ class SelectiveScan(ProjectedMixer):
                                self.result_scale, y, rows, step)
             return
         dt = ws.rows("selective_dt", n, self.inner, torch.float32)
-        ops.selective_dt(low, self.rank, self.dt_w if self.dt_t is None else self.dt_t, self.dt_bias, dt)
-        ops.selective_scan(x, z, u, dt, low, self.rank, self.a, self.skip, self.result_scale, y, rows, self.state_floats,
-                           self.taps, step)
+        if self.split:
+            parts = ws.rows("selective_parts", n, 2 * self.rank, torch.bfloat16)
+            ops.selective_split(low, self.rank, parts)
+            self.dt.forward(parts, dt)
+        else:
+            self.dt.forward(low[:, :self.rank], dt)
+        ops.selective_scan(x, z, u, dt, self.dt_bias, low, self.rank, self.a, self.skip, self.result_scale, y, rows,
+                           self.state_floats, self.taps, step)
