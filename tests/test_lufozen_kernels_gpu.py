@@ -41,9 +41,11 @@ LENS = [328, 275]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("sizes", [(4, 8, 12, 2, 4, 2), (6, 5, 7, 3, 1, 1), (2, 64, 128, 1, 3, 2), (3, 20, 33, 3, 6, 4), (1, 7, 200, 1, 2, 1)])
-def test_state_space_kernels_over_steps(dtype, sizes):
-    """heads, vdim, state, groups, taps, norm parts; a step of single tokens also through the one-kernel form."""
+@pytest.mark.parametrize("sizes,pad", [((4, 8, 12, 2, 4, 2), 1), ((4, 8, 12, 2, 4, 2), 4), ((6, 5, 7, 3, 1, 1), 1), ((2, 64, 128, 1, 3, 2), 4),
+                                       ((3, 20, 33, 3, 6, 4), 1), ((4, 12, 16, 1, 6, 4), 4), ((1, 7, 200, 1, 2, 1), 1)])
+def test_state_space_kernels_over_steps(dtype, sizes, pad):
+    """heads, vdim, state, groups, taps, norm parts; a step of single tokens also through the one-kernel form.  `pad`: floats
+    behind a state row (four: rows stay on 16 bytes, for the kernels' wide loads)."""
     from fastllm_py_b200.native import ops
 
     H, P, N, G, taps, parts = sizes
@@ -62,7 +64,7 @@ def test_state_space_kernels_over_steps(dtype, sizes):
     neg_a = dev(-torch.exp(t["A_log"]))
     floats = inner * N
     for fused in (False, True):
-        state = torch.full((3, floats + (taps - 1) * ch + 1), 1e4, device="cuda")
+        state = torch.full((3, floats + (taps - 1) * ch + pad), 1e4, device="cuda")
         tail = state[:, floats:] if taps > 1 else None
         for entries in SCHEDULE:
             step, starts = step_of(entries, {0: 2, 1: 0})
