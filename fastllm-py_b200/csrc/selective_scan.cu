@@ -21,6 +21,11 @@
 #include "short_conv.cuh"
 #include "state_scan.cuh"
 
+// silu with the fast exponential and division where the result is rounded to bfloat16.
+template <typename T> __device__ __forceinline__ float sel_silu(float v) {
+    return sizeof(T) == 4 ? fl_silu(v) : __fdividef(v, 1.0f + __expf(-v));
+}
+
 // ------------------------------------------------------------------ convolution
 // V channels a thread, RUN consecutive tokens; conv_w: [taps][inner].  move_tail: every request has one token (RUN is 1).
 template <typename T, int V, int TAPS, int RUN>
@@ -40,7 +45,7 @@ __global__ void __launch_bounds__(128) selective_conv_kernel(
     const int t0 = blockIdx.x * RUN, t1 = min(n_tokens, t0 + RUN);
     conv.run(t0, t1, u + c, ld, st, tail, tail_stride, taps, inner, c, [&](int t, ChanVec<V> y, const ChanVec<V>* in) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) y.v[e] = fl_silu(y.v[e] + b.v[e]);
+        for (int e = 0; e < V; ++e) y.v[e] = sel_silu<T>(y.v[e] + b.v[e]);
         chan_store<T, V>(x + (long)t * x_ld + c, y);
         if (RUN == 1 && TAPS > 1 && move_tail) {                      // kept row j: the input of position pos - (taps - 2) + j
             float* kept = tail + (long)st.req_slot[st.tok_req[t]] * tail_stride + c;
@@ -60,7 +65,7 @@ FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* con
     if (n_tokens <= 0) return 0;
     if (taps < 1 || taps > 16 || (taps > 1 && tail == nullptr)) return (int)cudaErrorInvalidValue;
     const StepTables st{tok_req, positions, req_start, req_ctx, req_qlen, req_slot};
-    const int run = !move_tail && n_tokens >= 256 ? 4 : 1;
+    const int run = move_tail || n_tokens < 256 ? 1 : n_tokens >= 1024 ? 8 : 4;
     const int elem = dtype == FL_F32 ? 4 : 2;
     const bool vec = inner % 4 == 0 && chan_aligned(u, ld, elem) && chan_aligned(x, x_ld, elem) && chan_aligned(conv_w, 4, 4) &&
                      chan_aligned(conv_b, 4, 4) && (taps == 1 || chan_aligned(tail, tail_stride, 4));
@@ -70,7 +75,8 @@ FL_API int fl_selective_conv(const void* u, int dtype, long ld, const float* con
 #define FL_SEL_CONV(V, TAPS, RUN)                                                                                         \
     FL_DISPATCH(dtype, T, return fl_launch(selective_conv_kernel<T, V, TAPS, RUN>, grid, dim3(128), 0, stream, (const T*)u, ld, \
                                            conv_w, conv_b, taps, tail, tail_stride, st, (T*)x, x_ld, n_tokens, inner, move_tail))
-#define FL_SEL_CONV_RUN(V, TAPS) { if (run == 4) { FL_SEL_CONV(V, TAPS, 4); } else { FL_SEL_CONV(V, TAPS, 1); } }
+#define FL_SEL_CONV_RUN(V, TAPS)                                                                                          \
+    { if (run == 8) { FL_SEL_CONV(V, TAPS, 8); } else if (run == 4) { FL_SEL_CONV(V, TAPS, 4); } else { FL_SEL_CONV(V, TAPS, 1); } }
     if (vec) { if (taps == 1) FL_SEL_CONV_RUN(4, 1) else if (taps <= 4) FL_SEL_CONV_RUN(4, 4) else FL_SEL_CONV_RUN(4, 16) }
     else { if (taps == 1) FL_SEL_CONV_RUN(1, 1) else if (taps <= 4) FL_SEL_CONV_RUN(1, 4) else FL_SEL_CONV_RUN(1, 16) }
 #undef FL_SEL_CONV_RUN
@@ -204,11 +210,6 @@ template <typename T> __device__ __forceinline__ float sel_softplus(float v) {
     p = fmaf(p, q, 1.0f / 3.0f);
     return fmaxf(v, 0.0f) + fmaf(2.0f * s * q, p, 2.0f * s);
 }
-// silu with the fast exponential and division where the result is rounded to bfloat16.
-template <typename T> __device__ __forceinline__ float sel_silu(float v) {
-    return sizeof(T) == 4 ? fl_silu(v) : __fdividef(v, 1.0f + __expf(-v));
-}
-
 struct SelRows {                     // the step's rows: element type T, float, float
     const void *x, *z, *u;           // convolved inputs, gates, inputs before the convolution
     const float *dt, *low;           // (dt before bias and softplus)
