@@ -71,6 +71,29 @@ def test_selective_scan_kernels_over_steps(dtype, sizes, pad):
         assert float(state[1].min()) == 1e4                                  # a slot of no request is left alone
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 7])
+def test_convolution_of_long_steps(dtype, taps):
+    """Steps in which a thread takes several tokens, runs that end with a request or with the step among them."""
+    from fastllm_py_b200.native import ops
+
+    inner = 20
+    gen = torch.Generator().manual_seed(taps)
+    w, b = torch.randn(inner, taps, generator=gen) * 0.6, torch.randn(inner, generator=gen) * 0.3
+    for lengths in ((300,), (259, 6), (1101,), (3, 1030, 2)):
+        u = [torch.randn(n, inner, generator=gen).to(dtype) for n in lengths]
+        tails = torch.randn(len(lengths), (taps - 1) * inner, generator=gen)
+        ctx = [0 if i % 2 else 50 for i in range(len(lengths))]
+        step, starts = step_of([(i, ctx[i], n) for i, n in enumerate(lengths)], {i: i for i in range(len(lengths))})
+        kept = dev(tails) if taps > 1 else None
+        x = torch.empty(sum(lengths), inner, dtype=dtype, device="cuda")
+        ops.selective_conv(dev(torch.cat(u)), dev(w.T.contiguous()), dev(b), kept, step, x, False)
+        for i, n in enumerate(lengths):
+            tail = tails[i].view(taps - 1, inner).double() * (1.0 if ctx[i] else 0.0)
+            want = plain.silu(plain.short_conv(u[i].double(), w.double(), b.double(), tail))
+            near(x[starts[i]:starts[i + 1]], want, 1e-5 if dtype == torch.float32 else 0.01, (lengths, i))
+
+
 def test_the_scan_is_the_same_whatever_the_cut_and_the_batch():
     """32-bit: one order of sums, bit for bit, alone and beside seven other requests, whole and in portions."""
     from fastllm_py_b200.native import ops
